@@ -59,7 +59,8 @@ class PositionSpec:
 
 @dataclass(frozen=True)
 class NormSpec:
-    """kind "rmsnorm": a gain per coordinate; "rmsnorm_scalar": one gain for all coordinates."""
+    """kind "rmsnorm": a gain per coordinate; "rmsnorm_scalar": one gain for all coordinates; "dynamic_tanh":
+    tanh(alpha x) * w + b, without statistics (eps is not read)."""
     kind: str = "rmsnorm"
     eps: float = 1e-5
 
@@ -138,6 +139,9 @@ class LayerSpec:
     the feed-forward with its two norms may be absent.
     arrangement "output_norm":  h += norm1(mixer(h)); h += norm2(ffn(h)) - the sublayers read the stream itself and
     ``mixer_norm`` / ``ffn_norm`` are the norms on their OUTPUTS.
+    arrangement "hyper_connections":  the model carries several residual streams (``ModelConfig.streams``; the
+    layer's extra repeats the number as "streams"); a sublayer reads a weighted sum of them through its norm, and then
+    every stream is made anew from all of them and the sublayer's output.
     ``extra`` carries the arrangement's own constants (for instance the width of a per-layer token
     input that it adds after the feed-forward).
 
@@ -194,6 +198,7 @@ class ModelConfig:
     head: HeadSpec = field(default_factory=HeadSpec)
     stream_inputs: int = 0      # rows of the table that ``LayerRun.stream_input`` names (0: the model has none)
     stream_input_kind: str = "row"      # "row": a table row is added; "project_with_embedding": x <- W [x; x0]
+    streams: int = 0            # residual streams side by side (arrangement "hyper_connections"; 0: the ordinary single one)
 
     @property
     def num_layers(self) -> int:
@@ -217,6 +222,11 @@ class ModelConfig:
             raise ConfigError("a model needs at least one layer")
         if not self.schedule:
             raise ConfigError("the schedule is empty")
+        hyper = [layer.arrangement == "hyper_connections" for layer in self.layers]
+        if self.streams < 0 or any(h != (self.streams > 0) for h in hyper):
+            raise ConfigError("a model with residual streams side by side has hyper_connections layers and no others")
+        if self.streams > 0 and self.stream_inputs > 0:
+            raise ConfigError("stream inputs join a single residual stream, not several")
         if self.stream_input_kind not in ("row", "project_with_embedding"):
             raise ConfigError(f"stream_input_kind '{self.stream_input_kind}' is not known (row, project_with_embedding)")
         for r, run in enumerate(self.schedule):

@@ -2,12 +2,14 @@
 //
 //   route     z = W_router x, s = softmax(z) over all experts - or s = sigmoid(z), each expert on its own -, all FP32;
 //             the `top` experts with the largest s + bias are chosen (ties: the lower index), their weights are s
-//             (optionally divided by their sum).  Experts numbered n_real and above are identity experts: their
-//             output is x itself.
+//             (optionally divided by their sum + 1e-20), times a factor.  Experts numbered n_real and above are identity
+//             experts: their output is x itself.  With groups > 1 the experts form that many equal groups of neighbours, a
+//             group counts as much as its best expert, and only experts of the best `keep` groups can be chosen.
 //   unit      an expert is W_down act(W_gate x, W_up x) with act(g, u) = g' * sigmoid(slope * g') * (u' + shift),
 //             g' = min(r g, limit), u' = clamp(r u, -limit, limit): limit = infinity, slope = 1, shift = 0, r = 1 is
 //             silu(g) * u; r is a number per row - the token's weight where a design multiplies the expert's INPUT by
-//             it (both products are linear in the input, so the factor is applied to their results, in FP32)
+//             it (both products are linear in the input, so the factor is applied to their results, in FP32).  Or an
+//             ungated unit: W_down relu(r W_up x)^2 (act code 2)
 //   layout    the (token, choice) pairs are laid out expert by expert (layout + scatter; where a pair lands
 //             inside its expert's stretch is decided by an atomic counter and changes no result, since every
 //             row is computed on its own)
@@ -33,10 +35,11 @@ __global__ void __launch_bounds__(RT_ROUTE_WARPS * 32)
 route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
              const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights,
              int* __restrict__ counts, int n_tokens, int d, int n_all, int n_real, int top,
-             int renormalize, int sigmoid_scores, float* __restrict__ all_scores) {
+             int renormalize, int sigmoid_scores, float* __restrict__ all_scores, int groups, int keep, float weight_scale) {
     extern __shared__ __align__(16) float xs[];          // [d]
     __shared__ float choice[RT_MAX_EXPERTS];
     __shared__ float score[RT_MAX_EXPERTS];
+    __shared__ float group_best[RT_MAX_EXPERTS];
     const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
     const T* xr = x + (size_t)t * d;
@@ -84,6 +87,23 @@ route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
         if (all_scores && e < n_real) all_scores[(size_t)t * n_real + e] = s;      // every real expert's score, chosen or not
     }
     __syncwarp();
+    if (groups > 1) {
+        const int per = n_all / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float b = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, choice[e]);
+            group_best[g] = b;
+        }
+        __syncwarp();
+        // a group stays if fewer than `keep` others are better (ties: the lower index is)
+        for (int e = lane; e < n_all; e += 32) {
+            const int g = e / per;
+            int better = 0;
+            for (int o = 0; o < groups; ++o) better += (group_best[o] > group_best[g] || (group_best[o] == group_best[g] && o < g));
+            if (better >= keep) choice[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float wsum = 0.f;
     for (int j = 0; j < top; ++j) {
         float best = -INFINITY;
@@ -109,7 +129,10 @@ route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
         }
         __syncwarp();
     }
-    if (renormalize && lane < top) weights[(size_t)t * top + lane] /= wsum;   // top <= 32 when this is asked
+    if (renormalize || weight_scale != 1.0f) {
+        const float factor = renormalize ? weight_scale / (wsum + 1e-20f) : weight_scale;
+        for (int j = lane; j < top; j += 32) weights[(size_t)t * top + j] *= factor;
+    }
 }
 
 // offsets[e] = first row of expert e's stretch, tile_first[e] = first row tile (tiles of `tile_rows` rows);
@@ -161,18 +184,24 @@ __device__ __forceinline__ float rt_act(float g, float u, const RtAct a, float r
     return g / (1.0f + expf(-a.slope * g)) * (u + a.shift);
 }
 
+// ACT codes of the products below: 0 none, 1 the gated unit (the matrix holds gate rows, then up rows), 2 relu(.)^2
+__device__ __forceinline__ float rt_relu2(float u, float r) {
+    u = fmaxf(u * r, 0.f);
+    return u * u;
+}
+
 #define RT_BM 64
 #define RT_BN 64
 #define RT_BK 16
 
-template <typename T, bool ACT>
+template <typename T, int ACT>
 __global__ void __launch_bounds__(256)
 expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row, const T* __restrict__ w,
                    T* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tile_first,
                    int n_real, int N, int K, RtAct act, const float* __restrict__ row_scale) {
     __shared__ float as[RT_BK][RT_BM + 4];
     __shared__ float ws[RT_BK][RT_BN + 4];
-    __shared__ float us[ACT ? RT_BK : 1][RT_BN + 4];
+    __shared__ float us[ACT == 1 ? RT_BK : 1][RT_BN + 4];
     __shared__ int src_row[RT_BM];
     __shared__ int s_expert;
     const int tile = blockIdx.y;
@@ -190,16 +219,16 @@ expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row
         src_row[threadIdx.x] = r < row_hi ? (token_of_row ? token_of_row[r] : r) : -1;
     }
     __syncthreads();
-    const T* we = w + (size_t)e * (ACT ? 2 : 1) * N * K;
+    const T* we = w + (size_t)e * (ACT == 1 ? 2 : 1) * N * K;
     const int n0 = blockIdx.x * RT_BN;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    float acc[4][4], acu[ACT ? 4 : 1][4];
+    float acc[4][4], acu[ACT == 1 ? 4 : 1][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             acc[i][j] = 0.f;
-            if (ACT) acu[i][j] = 0.f;
+            if (ACT == 1) acu[i][j] = 0.f;
         }
     for (int k0 = 0; k0 < K; k0 += RT_BK) {
 #pragma unroll
@@ -210,7 +239,7 @@ expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row
             const int sr = src_row[r];
             as[kk][r] = (sr >= 0 && k < K) ? ni_to_float(a[(size_t)sr * K + k]) : 0.f;
             ws[kk][r] = (n0 + r < N && k < K) ? ni_to_float(we[(size_t)(n0 + r) * K + k]) : 0.f;
-            if (ACT) us[kk][r] = (n0 + r < N && k < K) ? ni_to_float(we[(size_t)(N + n0 + r) * K + k]) : 0.f;
+            if (ACT == 1) us[kk][r] = (n0 + r < N && k < K) ? ni_to_float(we[(size_t)(N + n0 + r) * K + k]) : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -221,14 +250,14 @@ expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 bv[j] = ws[kk][tx * 4 + j];
-                if (ACT) uv[j] = us[kk][tx * 4 + j];
+                if (ACT == 1) uv[j] = us[kk][tx * 4 + j];
             }
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
-                    if (ACT) acu[i][j] = fmaf(av[i], uv[j], acu[i][j]);
+                    if (ACT == 1) acu[i][j] = fmaf(av[i], uv[j], acu[i][j]);
                 }
         }
         __syncthreads();
@@ -242,10 +271,12 @@ expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if (ACT) {
+            if (ACT == 1) {
                 // the products are rounded to the activations' type first, as a separate product would leave them
                 const float g = ni_to_float(ni_from_float<T>(v)), u = ni_to_float(ni_from_float<T>(acu[i][j]));
                 v = rt_act(g, u, act, row_scale ? row_scale[r] : 1.0f);
+            } else if (ACT == 2) {
+                v = rt_relu2(ni_to_float(ni_from_float<T>(v)), row_scale ? row_scale[r] : 1.0f);
             }
             out[(size_t)r * N + n] = ni_from_float<T>(v);
         }
@@ -254,7 +285,7 @@ expert_gemm_kernel(const T* __restrict__ a, const int* __restrict__ token_of_row
 
 // Few rows, bfloat16: one warp per (pair, output).  a: the tokens' rows [T, K] (GATHER: pair p reads row
 // p / top) or the pairs' own rows [P, K]; K a multiple of 8.
-template <bool ACT>
+template <int ACT>
 __global__ void expert_rows_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w,
                                    __nv_bfloat16* __restrict__ out, const int* __restrict__ ids, int n_pairs, int top,
                                    int gather, int n_real, int N, int K, RtAct act, const float* __restrict__ row_scale) {
@@ -264,7 +295,7 @@ __global__ void expert_rows_kernel(const __nv_bfloat16* __restrict__ a, const __
     const int e = ids[p];
     if (e >= n_real) return;
     const __nv_bfloat16* ar = a + (size_t)(gather ? p / top : p) * K;
-    const __nv_bfloat16* wg = w + ((size_t)e * (ACT ? 2 : 1) * N + warp) * K;
+    const __nv_bfloat16* wg = w + ((size_t)e * (ACT == 1 ? 2 : 1) * N + warp) * K;
     const __nv_bfloat16* wu = wg + (size_t)N * K;
     float g = 0.f, u = 0.f;
     for (int k = lane * 8; k < K; k += 256) {
@@ -278,7 +309,7 @@ __global__ void expert_rows_kernel(const __nv_bfloat16* __restrict__ a, const __
             g = fmaf(af.x, gf.x, g);
             g = fmaf(af.y, gf.y, g);
         }
-        if (ACT) {
+        if (ACT == 1) {
             const uint4 uv = *reinterpret_cast<const uint4*>(wu + k);
             const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
 #pragma unroll
@@ -290,11 +321,13 @@ __global__ void expert_rows_kernel(const __nv_bfloat16* __restrict__ a, const __
         }
     }
     g = ni_warp_sum(g);
-    if (ACT) {
+    if (ACT == 1) {
         u = ni_warp_sum(u);
         g = __bfloat162float(__float2bfloat16_rn(g));
         u = __bfloat162float(__float2bfloat16_rn(u));
         g = rt_act(g, u, act, row_scale ? row_scale[p] : 1.0f);
+    } else if (ACT == 2) {
+        g = rt_relu2(__bfloat162float(__float2bfloat16_rn(g)), row_scale ? row_scale[p] : 1.0f);
     }
     if (lane == 0) out[(size_t)p * N + warp] = __float2bfloat16_rn(g);
 }
@@ -401,21 +434,22 @@ __global__ void combine_add_normed_vec_kernel(const T* __restrict__ z, const T* 
 
 NI_EXPORT int ni_route(const void* x, int dtype, const float* w_router, const float* bias, int* ids, float* weights,
                        int* counts, int n_tokens, int d, int n_all, int n_real, int top, int renormalize,
-                       int sigmoid_scores, float* all_scores, cudaStream_t stream) {
+                       int sigmoid_scores, float* all_scores, int groups, int keep, float weight_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return NI_OK;
     if (d <= 0 || n_all <= 0 || n_real < 0 || n_real > n_all || top <= 0 || top > n_all) return NI_ERR_BAD_ARGUMENT;
-    if (n_all > RT_MAX_EXPERTS || (renormalize && top > 32)) return NI_ERR_UNSUPPORTED_SIZE;
+    if (groups > 1 && (n_all % groups || keep <= 0 || (long long)keep * (n_all / groups) < top)) return NI_ERR_BAD_ARGUMENT;
+    if (n_all > RT_MAX_EXPERTS) return NI_ERR_UNSUPPORTED_SIZE;
     if (d > 12000) return NI_ERR_UNSUPPORTED_SIZE;                    // the row lies in shared memory as FP32
     const size_t smem = (size_t)d * sizeof(float);
     if (dtype == NI_DTYPE_F32)
         route_kernel<float><<<n_tokens, RT_ROUTE_WARPS * 32, smem, stream>>>((const float*)x, w_router, bias, ids, weights,
                                                                            counts, n_tokens, d, n_all, n_real, top, renormalize,
-                                                                           sigmoid_scores, all_scores);
+                                                                           sigmoid_scores, all_scores, groups, keep, weight_scale);
     else if (dtype == NI_DTYPE_BF16)
         route_kernel<__nv_bfloat16><<<n_tokens, RT_ROUTE_WARPS * 32, smem, stream>>>((const __nv_bfloat16*)x, w_router, bias,
                                                                                    ids, weights, counts, n_tokens, d, n_all,
                                                                                    n_real, top, renormalize, sigmoid_scores,
-                                                                                   all_scores);
+                                                                                   all_scores, groups, keep, weight_scale);
     else
         return NI_ERR_BAD_ARGUMENT;
     NI_RETURN_LAUNCH_STATUS();
@@ -434,12 +468,12 @@ NI_EXPORT int ni_route_layout(const int* ids, int* counts, int* offsets, int* ti
     NI_RETURN_LAUNCH_STATUS();
 }
 
-// act != 0: w is [n_real, 2 N, K] (gate rows, then up rows) and out = silu(gate) * up
+// act 1: w is [n_real, 2 N, K] (gate rows, then up rows) and out = the gated unit's activation; act 2: out = relu(.)^2
 NI_EXPORT int ni_expert_gemm(const void* a, int dtype, const int* token_of_row, const void* w, void* out,
                              const int* offsets, const int* tile_first, int n_pairs, int n_real, int N, int K, int act,
                              float limit, float slope, float shift, const float* row_scale, cudaStream_t stream) {
     if (n_pairs <= 0 || n_real <= 0 || N <= 0) return NI_OK;
-    if (K <= 0) return NI_ERR_BAD_ARGUMENT;
+    if (K <= 0 || act < 0 || act > 2) return NI_ERR_BAD_ARGUMENT;
     const int max_tiles = (n_pairs + RT_BM - 1) / RT_BM + (n_real < n_pairs ? n_real : n_pairs);
     dim3 grid((N + RT_BN - 1) / RT_BN, max_tiles);
     if (grid.y > 65535) return NI_ERR_UNSUPPORTED_SIZE;
@@ -447,8 +481,8 @@ NI_EXPORT int ni_expert_gemm(const void* a, int dtype, const int* token_of_row, 
 #define LAUNCH(T, ACT)                                                                                             \
     expert_gemm_kernel<T, ACT><<<grid, 256, 0, stream>>>((const T*)a, token_of_row, (const T*)w, (T*)out, offsets, \
                                                          tile_first, n_real, N, K, ra, row_scale)
-    if (dtype == NI_DTYPE_F32) { if (act) LAUNCH(float, true); else LAUNCH(float, false); }
-    else if (dtype == NI_DTYPE_BF16) { if (act) LAUNCH(__nv_bfloat16, true); else LAUNCH(__nv_bfloat16, false); }
+    if (dtype == NI_DTYPE_F32) { if (act == 1) LAUNCH(float, 1); else if (act == 2) LAUNCH(float, 2); else LAUNCH(float, 0); }
+    else if (dtype == NI_DTYPE_BF16) { if (act == 1) LAUNCH(__nv_bfloat16, 1); else if (act == 2) LAUNCH(__nv_bfloat16, 2); else LAUNCH(__nv_bfloat16, 0); }
     else return NI_ERR_BAD_ARGUMENT;
 #undef LAUNCH
     NI_RETURN_LAUNCH_STATUS();
@@ -458,16 +492,17 @@ NI_EXPORT int ni_expert_rows(const void* a, const void* w, void* out, const int*
                              int n_real, int N, int K, int act, float limit, float slope, float shift,
                              const float* row_scale, cudaStream_t stream) {
     if (n_pairs <= 0 || n_real <= 0 || N <= 0) return NI_OK;
-    if (K <= 0 || top <= 0) return NI_ERR_BAD_ARGUMENT;
+    if (K <= 0 || top <= 0 || act < 0 || act > 2) return NI_ERR_BAD_ARGUMENT;
     if (K % 8 || n_pairs > 65535) return NI_ERR_UNSUPPORTED_SIZE;
     dim3 grid((N + 7) / 8, n_pairs);
     const RtAct ra = {limit, slope, shift};
-    if (act)
-        expert_rows_kernel<true><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w,
-                                                           (__nv_bfloat16*)out, ids, n_pairs, top, gather, n_real, N, K, ra, row_scale);
-    else
-        expert_rows_kernel<false><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w,
-                                                            (__nv_bfloat16*)out, ids, n_pairs, top, gather, n_real, N, K, ra, row_scale);
+#define LAUNCH(ACT)                                                                                                      \
+    expert_rows_kernel<ACT><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ids, \
+                                                      n_pairs, top, gather, n_real, N, K, ra, row_scale)
+    if (act == 1) LAUNCH(1);
+    else if (act == 2) LAUNCH(2);
+    else LAUNCH(0);
+#undef LAUNCH
     NI_RETURN_LAUNCH_STATUS();
 }
 

@@ -95,6 +95,8 @@ class DecoderModel:
             self.embedding.forward(ctx.tokens, h)
         delta = None
         h0 = None
+        if cfg.streams > 0:
+            h = ops.ResidualStreams(h, cfg.streams)       # several streams, all equal to the embedding's output so far
         if self.projects_stream:
             h0 = h                   # what the embedding produced stays as it is: the runs go on in a stream of their own
             h = None

@@ -171,22 +171,26 @@ class Runtime:
         return y
 
     def experts_linear(self, a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, tile_first: torch.Tensor,
-                       n_rows: int, token_of_row: Optional[torch.Tensor] = None, act: bool = False,
+                       n_rows: int, token_of_row: Optional[torch.Tensor] = None, act: int = ops.NO_ACT,
                        glu=ops.PLAIN_GLU, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
         """One product per expert over rows laid out expert by expert: y[r] = a[r] . w[e]^T for the rows r of
         expert e's stretch [offsets[e], offsets[e + 1]) (int32 on the device; nothing is read on the host).
-        ``token_of_row``: row r reads a[token_of_row[r]] instead.  ``act``: w is [E, 2N, K], gate rows then up
-        rows, and y = the gated unit's activation (``glu`` = (limit, slope, shift), ``row_scale`` float32 [rows]: see
+        ``token_of_row``: row r reads a[token_of_row[r]] instead.  ``act`` RELU2_ACT: y = the square of the product's
+        positive part; GATED_ACT: w is [E, 2N, K], gate rows then up rows, and y = the gated unit's activation (``glu`` = (limit, slope, shift), ``row_scale`` float32 [rows]: see
         ops.capped_glu; the default is silu(gate) * up).  float32: the package's FFMA kernel, one ascending chain per element;
         bfloat16 with sizes that are multiples of 8: a library grouped product (FP32 accumulation), as the
         other projections of prompt portions are library products; rows beyond the last stretch are undefined."""
         n_experts, wn, k = w.shape
-        n = wn // 2 if act else wn
+        gated = act == ops.GATED_ACT
+        n = wn // 2 if gated else wn
         if self.dtype == torch.bfloat16 and k % 8 == 0 and wn % 8 == 0 and n % 8 == 0:
             if token_of_row is not None:
                 a = torch.index_select(a, 0, token_of_row[:n_rows])
             y = torch.nn.functional.grouped_mm(a[:n_rows], w.transpose(1, 2), offs=offsets[1:n_experts + 1])
-            if not act:
+            if act == ops.NO_ACT:
+                return y
+            if not gated:
+                ops.relu_squared(y, y)
                 return y
             out = self.empty(n_rows, n)
             ops.capped_glu(y, out, *glu, row_scale=row_scale)      # 16 bytes per thread

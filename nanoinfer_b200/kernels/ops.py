@@ -34,7 +34,7 @@ _SIGNATURES = {
         "ni_rope_kv_write": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "attention_generic": {
-        "ni_attention_generic": [_P, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _F, _I, _I, _I, _P],
+        "ni_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _F, _I, _I, _I, _I, _P],
     },
     "gemm_f32": {
         "ni_gemm_f32": [_P, _P, _P, _I, _I, _I, _P],
@@ -66,12 +66,24 @@ _SIGNATURES = {
         "ni_lightning_max_chunks": [_I, _I],
         "ni_lightning_gated_norm": [_P, _P, _I, _I, _I, _P, _F, _P, _I, _I, _P],
     },
+    "mlstm": {
+        "ni_mlstm_token_step": [_P, _I, _P, _I, _I, _I, _P, _P, _F, _P, _LL, _P, _P, _I, _F, _P, _F, _P, _I, _I, _I, _I, _P],
+        "ni_mlstm_chunk_step": [_P, _I, _I, _P, _I, _I, _I, _P, _P, _F, _P, _LL, _P, _P, _I, _I, _I, _F, _P, _F, _P, _LL, _P, _P, _P,
+                                _I, _I, _I, _P],
+    },
+    "hyper": {
+        "ni_hyper_step": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P],
+        "ni_hyper_max_streams": [],
+    },
+    "difference": {
+        "ni_difference_norm": [_P, _P, _I, _P, _I, _I, _I, _F, _F, _F, _P],
+    },
     "conv_attention": {
         "ni_conv_qk_prepare": [_P, _I, _I, _P, _P, _P, _F, _P, _LL, _P, _P, _P, _P, _P, _I, _P, _P, _P, _P,
                                _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "routed": {
-        "ni_route": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+        "ni_route": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P],
         "ni_route_layout": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _P],
         "ni_expert_gemm": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
         "ni_expert_rows": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
@@ -178,6 +190,8 @@ def load(module: str) -> ctypes.CDLL:
             lib.ni_attention_decode_set_cluster_merge(0)
         if module == "attention_decode" and lib.ni_attention_decode_fresh_keys() != DECODE_FRESH_KEYS:
             raise KernelError("attention_decode: DEC_FRESH_KEYS of the built kernel differs from ops.DECODE_FRESH_KEYS")
+        if module == "hyper" and lib.ni_hyper_max_streams() != HYPER_MAX_STREAMS:
+            raise KernelError("hyper: HY_MAX_STREAMS of the built kernel differs from ops.HYPER_MAX_STREAMS")
         _libs[module] = lib
     return lib
 
@@ -350,34 +364,36 @@ def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                       page_size: int, window: Optional[int], scale: float,
                       token_list: Optional[torch.Tensor] = None, head_slopes: Optional[torch.Tensor] = None,
                       score_cap: float = 0.0, value_dim: Optional[int] = None, chunk: int = 0,
-                      sink: bool = False) -> None:
+                      sink: bool = False, maps: int = 1) -> None:
     """The plain attention kernel (any dtype, any head size up to 1,024).  ``token_list``
     int32 [n] restricts it to those tokens of the step.  ``head_slopes`` float32 [Hq] adds
     slope[h] * (key position - query position) to the scaled scores of head h.  ``score_cap`` c > 0
     bounds the scaled scores: s <- c * tanh(s / c).  ``value_dim``: the size of a value where it differs
     from the keys' (value pages [P, Hkv, page_size, value_dim], out [T, Hq * value_dim]).  ``chunk`` c > 0: a token at
-    position p sees only the keys from p - p % c on.  ``sink``: one is added to the softmax's denominator."""
+    position p sees only the keys from p - p % c on.  ``sink``: one is added to the softmax's denominator.  ``maps`` = m >
+    1: every head has m attention maps over the same values; ``n_q_heads`` counts maps (head h's map i is row h m + i of
+    q), and a key row holds m parts of ``head_dim`` side by side.  ``out`` may be float32 where the rest is bfloat16."""
     if head_slopes is not None and head_slopes.numel() != n_q_heads:
         raise KernelError("attention: one slope per query head")
     n = q.shape[0]
     v_dim = head_dim if value_dim is None else int(value_dim)
     if q.shape != (n, n_q_heads * head_dim) or out.shape != (n, n_q_heads * v_dim):
         raise KernelError("attention: q must be [T, Hq * head_dim] and out [T, Hq * value_dim]")
-    if not (q.dtype == out.dtype == k_pages.dtype == v_pages.dtype):
-        raise KernelError("attention: all operands must share one dtype")
+    if not (q.dtype == k_pages.dtype == v_pages.dtype) or out.dtype not in (q.dtype, torch.float32):
+        raise KernelError("attention: all operands must share one dtype (the output may be float32)")
     if head_dim > 1024 or v_dim > 1024 or v_dim <= 0:
         raise KernelError(f"attention: head_dim {head_dim} or value_dim {v_dim} beyond 1,024 is not supported")
-    if k_pages.shape[-1] != head_dim or v_pages.shape[-1] != v_dim:
+    if k_pages.shape[-1] != maps * head_dim or v_pages.shape[-1] != v_dim:
         raise KernelError("attention: the pages' rows must have the keys' and the values' sizes")
     _check(load("attention_generic").ni_attention_generic(
         _dev(q, "q"), _code(q, "q"), _dev(k_pages, "k_pages"), _dev(v_pages, "v_pages"),
-        _dev(out, "out"), _dev(token_list, "token_list", torch.int32) if token_list is not None else None,
+        _dev(out, "out"), _code(out, "out"), _dev(token_list, "token_list", torch.int32) if token_list is not None else None,
         _dev(positions, "positions", torch.int32),
         _dev(seq_of_token, "seq_of_token", torch.int32), _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], n if token_list is None else token_list.numel(), n_q_heads, n_kv_heads, head_dim, page_size,
         int(window) if window else 0, float(scale),
         _dev(head_slopes, "head_slopes", torch.float32) if head_slopes is not None else None, float(score_cap),
-        v_dim, int(chunk or 0), 1 if sink else 0, _stream()), "attention_generic")
+        v_dim, int(chunk or 0), 1 if sink else 0, int(maps), _stream()), "attention_generic")
 
 
 def gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -756,6 +772,185 @@ def lightning_gated_norm(o, proj, col0, weight, eps, y) -> None:
         _dev(weight, "weight", torch.float32), float(eps), _dev(y, "y"), n, width, _stream()), "lightning_gated_norm")
 
 
+class ResidualStreams:
+    """The residual stream of a model that carries several of them side by side: ``x`` float32 [T, S, d], written from
+    the first sublayer's end on; before that all streams equal the one row per token in ``base`` [T, d].  What the last
+    sublayer left - its output and how the streams are made anew from it - stays pending (``leave``) and is applied by
+    the pass that reads the streams for the next sublayer (``read``)."""
+
+    def __init__(self, base: torch.Tensor, streams: int) -> None:
+        self.base, self.streams = base, int(streams)
+        self.x: Optional[torch.Tensor] = None
+        self.pending = None
+
+    def leave(self, y, mix: torch.Tensor, out: torch.Tensor) -> None:
+        """``y``: float32 [T, d], or the RoutedRows of experts not yet summed.  mix [S, S] (from, to), out [S]."""
+        if self.pending is not None:
+            raise KernelError("residual streams: an output is pending already")
+        self.pending = (y, mix, out)
+
+    def read(self, coef, tanh_norm=None, out_dtype=torch.float32, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """sum_s coef[s] x_s (``coef`` None: the plain sum) of the streams after the pending update; with ``tanh_norm`` =
+        (alpha, weight, bias) float32: tanh(alpha u) * weight + bias in ``out_dtype``, else u itself, float32.  ``rows``
+        int32: those rows only, and the streams stay as they are."""
+        t, d = self.base.shape
+        n = t if rows is None else rows.numel()
+        h = torch.empty(n, d, dtype=out_dtype if tanh_norm is not None else torch.float32, device=self.base.device)
+        source, target = (self.base if self.x is None else None), self.x
+        keep = rows is None and self.pending is not None
+        if keep and target is None:
+            target = torch.empty(t, self.streams, d, dtype=torch.float32, device=self.base.device)
+        hyper_step(target, source, self.streams, self.pending, coef, tanh_norm, h, rows, keep)
+        if keep:
+            self.x, self.pending = target, None
+        return h
+
+
+class RoutedRows:
+    """What a step's routed experts left, not yet summed: y[t] = sum_j weights[t, j] * z[row of pair (t, j)], pair (t, j)'s
+    row being row_of_pair[t top + j], t top + j itself (``row_of_pair`` None), or t E + ids[t, j] (``all_experts`` = E)."""
+
+    def __init__(self, z, ids, weights, row_of_pair, all_experts: int = 0) -> None:
+        self.z, self.ids, self.weights, self.row_of_pair, self.all_experts = z, ids, weights, row_of_pair, int(all_experts)
+
+
+def hyper_step(x, base, streams: int, pending, coef, tanh_norm, h, rows, write_back: bool) -> None:
+    """One pass over residual streams (see ResidualStreams): apply ``pending`` = (y or RoutedRows, mix, out) or None,
+    write the streams back if asked, read them with ``coef`` and norm the sum into h."""
+    f32, i32 = torch.float32, torch.int32
+    d = h.shape[1]
+    s = int(streams)
+    if (x is not None and tuple(x.shape[1:]) != (s, d)) or (base is not None and base.shape[1] != d) or \
+            (coef is not None and coef.numel() != s) or (rows is not None and rows.numel() != h.shape[0]):
+        raise KernelError("hyper_step: shapes do not agree")
+    n_tokens = base.shape[0] if base is not None else x.shape[0]
+    if rows is None and h.shape[0] != n_tokens:
+        raise KernelError("hyper_step: one output row per token")
+    kind, y, r = 0, None, None
+    mix = out = None
+    if pending is not None:
+        y, mix, out = pending
+        if mix.shape != (s, s) or out.numel() != s:
+            raise KernelError("hyper_step: the mixing coefficients do not fit the streams")
+        kind = 1
+        if isinstance(y, RoutedRows):
+            kind, r, y = 2, y, None
+            if r.z.shape[1] != d or r.ids.shape[0] != n_tokens:
+                raise KernelError("hyper_step: the experts' rows do not fit the streams")
+        elif y.shape != (n_tokens, d):
+            raise KernelError("hyper_step: the sublayer's output does not fit the streams")
+    if tanh_norm is not None and (tanh_norm[0].numel() != 1 or tanh_norm[1].numel() != d or tanh_norm[2].numel() != d):
+        raise KernelError("hyper_step: the norm has another width")
+    act = _code(r.z, "z") if r is not None else _code(h, "h")
+    if r is not None and tanh_norm is not None and r.z.dtype != h.dtype:
+        raise KernelError("hyper_step: the experts' rows and the normed output must share one dtype")
+    if tanh_norm is None and h.dtype != f32:
+        raise KernelError("hyper_step: without a norm the output is float32")
+
+    def opt(t, name, dtype):
+        return _dev(t, name, dtype) if t is not None else None
+
+    _check(load("hyper").ni_hyper_step(
+        opt(x, "x", f32), opt(base, "base", f32), s, d, h.shape[0], 1 if write_back else 0, kind, opt(y, "y", f32),
+        _dev(r.z, "z") if r is not None else None, act, opt(r.ids if r else None, "ids", i32), opt(r.weights if r else None, "weights", f32),
+        opt(r.row_of_pair if r else None, "row_of_pair", i32), r.ids.shape[1] if r is not None else 0,
+        r.all_experts if r is not None else 0, opt(mix, "mix", f32), opt(out, "out", f32), opt(coef, "coef", f32),
+        *((opt(v, "norm", f32) for v in tanh_norm) if tanh_norm is not None else (None, None, None)), _dev(h, "h"),
+        opt(rows, "rows", i32), _stream()), "hyper_step")
+
+
+HYPER_MAX_STREAMS = 32      # what the kernel keeps of a column in registers (checked against the built library)
+
+
+def tanh_norm(h, delta, alpha, weight, bias, out, rows=None) -> None:
+    """Residual add fused with the norm tanh(alpha h) * weight + bias: as add_rmsnorm, h float32 [T, d], delta float32
+    or None (added into h unless ``rows`` is given)."""
+    one = _unit_coefficients(h.device) if delta is not None else None
+    hyper_step(h.view(h.shape[0], 1, h.shape[1]), None, 1, (delta, one.view(1, 1), one) if delta is not None else None, None,
+               (alpha, weight, bias), out, rows, delta is not None and rows is None)
+
+
+_units: Dict[torch.device, torch.Tensor] = {}
+
+
+def _unit_coefficients(device) -> torch.Tensor:
+    t = _units.get(device)
+    if t is None:
+        t = _units[device] = torch.ones(1, dtype=torch.float32, device=device)
+    return t
+
+
+def difference_norm(a, out, lam: float, eps: float, factor: float, token_list=None) -> None:
+    """out[t, h, :] = u / sqrt(mean(u^2) + eps) * factor with u = a[t, 2h, :] - lam * a[t, 2h + 1, :]; a float32
+    [T, 2 H V] (two maps per head), out [T, H V]; ``token_list`` int32: those tokens only."""
+    n = a.shape[0] if token_list is None else token_list.numel()
+    if a.dim() != 3 or out.shape != (a.shape[0], (a.shape[1] // 2) * a.shape[2]) or a.shape[1] % 2:
+        raise KernelError("difference_norm: a must be [T, 2 H, V] and out [T, H V]")
+    _check(load("difference").ni_difference_norm(
+        _dev(a, "a", torch.float32), _dev(out, "out"), _code(out, "out"),
+        _dev(token_list, "token_list", torch.int32) if token_list is not None else None, n, a.shape[1] // 2, a.shape[2],
+        float(lam), float(eps), float(factor), _stream()), "difference_norm")
+
+
+MLSTM_MAX_DIM = 256      # the largest key size whose chunk buffers fit a block's shared memory
+
+
+def mlstm_state_floats(n_heads: int, dim: int, vdim: int) -> int:
+    """Floats of one request's state: per head a record (matrix, normaliser, padded to 4), then every head's maximum."""
+    record = -(-(dim * vdim + dim) // 4) * 4
+    return n_heads * record + -(-n_heads // 4) * 4
+
+
+def mlstm_buffer_floats(n_tokens: int, n_seqs: int, n_heads: int, dim: int, vdim: int) -> int:
+    """Floats of scratch that mlstm_chunk_step needs."""
+    f = load("mlstm").ni_mlstm_buffer_floats
+    f.restype, f.argtypes = _LL, [_I] * 5
+    return int(f(n_tokens, n_seqs, n_heads, dim, vdim))
+
+
+def _mlstm_check(proj, gates, bias_i, bias_f, state, weight, y, n_heads, dim, vdim, what) -> None:
+    n = proj.shape[0]
+    if proj.shape[1] < 2 * n_heads * (dim + vdim) or gates.shape[0] != n or bias_i.numel() != n_heads or bias_f.numel() != n_heads \
+            or state.shape[1] != mlstm_state_floats(n_heads, dim, vdim) or weight.numel() != n_heads * vdim or y.shape != (n, n_heads * vdim):
+        raise KernelError(f"{what}: shapes do not agree")
+
+
+def mlstm_token_step(proj, gates, col_i, col_f, bias_i, bias_f, cap, state, cu_q, slots, n_seqs, q_scale, weight, eps, y,
+                     n_heads, dim, vdim) -> None:
+    """A step in which every request brings ONE token, for a matrix-memory layer, in one launch: gates, state update,
+    read-out, the norm per head and the output gate.  proj float32 [n_seqs, ld] with columns q | k | v | gate | ...; gates
+    float32 [n_seqs, ldg] (it may be proj), the input gates' logits in columns col_i .. col_i + H, the forget gates' in
+    col_f .. col_f + H; state float32 [slots, mlstm_state_floats]; y [n_seqs, H vdim]."""
+    _mlstm_check(proj, gates, bias_i, bias_f, state, weight, y, n_heads, dim, vdim, "mlstm_token_step")
+    f32, i32 = torch.float32, torch.int32
+    _check(load("mlstm").ni_mlstm_token_step(
+        _dev(proj, "proj", f32), proj.shape[1], _dev(gates, "gates", f32), gates.shape[1], int(col_i), int(col_f),
+        _dev(bias_i, "bias_i", f32), _dev(bias_f, "bias_f", f32), float(cap), _dev(state, "state", f32), state.shape[1],
+        _dev(cu_q, "cu_q", i32), _dev(slots, "slots", i32), n_seqs, float(q_scale), _dev(weight, "weight", f32), float(eps),
+        _dev(y, "y"), _code(y, "y"), n_heads, dim, vdim, _stream()), "mlstm_token_step")
+
+
+def mlstm_chunk_step(proj, gates, col_i, col_f, bias_i, bias_f, cap, state, cu_q, slots, n_seqs, max_q_len, q_scale, weight,
+                     eps, buf, out, y, n_heads, dim, vdim) -> None:
+    """Any step of a matrix-memory layer, chunk by chunk; arguments as mlstm_token_step, proj in the activations' type
+    (y's too), buf float32 with mlstm_buffer_floats(...) entries, out float32 [T, H vdim] scratch.  Where the read-out
+    kernel has a head's whole values it norms and gates them itself; otherwise group_gated_norm follows."""
+    n = proj.shape[0]
+    _mlstm_check(proj, gates, bias_i, bias_f, state, weight, y, n_heads, dim, vdim, "mlstm_chunk_step")
+    if out.shape != y.shape or y.dtype != proj.dtype:
+        raise KernelError("mlstm_chunk_step: out and y must be [T, H vdim], y of proj's dtype")
+    f32, i32 = torch.float32, torch.int32
+    finished = ctypes.c_int(0)
+    _check(load("mlstm").ni_mlstm_chunk_step(
+        _dev(proj, "proj"), _code(proj, "proj"), proj.shape[1], _dev(gates, "gates", f32), gates.shape[1], int(col_i), int(col_f),
+        _dev(bias_i, "bias_i", f32), _dev(bias_f, "bias_f", f32), float(cap), _dev(state, "state", f32), state.shape[1],
+        _dev(cu_q, "cu_q", i32), _dev(slots, "slots", i32), n, n_seqs, int(max_q_len), float(q_scale),
+        _dev(weight, "weight", f32), float(eps), _dev(buf, "buf", f32), buf.numel(), _dev(out, "out", f32), _dev(y, "y"),
+        ctypes.byref(finished), n_heads, dim, vdim, _stream()), "mlstm_chunk_step")
+    if not finished.value:
+        group_gated_norm(out, proj, 2 * n_heads * dim + n_heads * vdim, weight, eps, y, vdim, gate="sigmoid")
+
+
 def conv_qk_prepare(proj, conv_w, q_gain, k_gain, eps, state, positions, seq_of_token, cu_q, slots, n_seqs, block_table,
                     inv_freq, q_out, k_pages, v_pages, n_heads, n_kv_heads, head_dim, rotary_dim, taps, page_size) -> None:
     """From the fused projection ``proj`` [T, ld] (columns: the queries' channels, the keys' channels, then whatever
@@ -792,12 +987,14 @@ ROUTE_MAX_EXPERTS = 256      # what the routing kernel keeps in shared memory pe
 
 
 def route(x, w_router, bias, ids, weights, counts, n_real, top, renormalize=False, sigmoid_scores=False,
-          all_scores=None) -> None:
+          all_scores=None, groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0) -> None:
     """Per token: scores = softmax(w_router x), or with ``sigmoid_scores`` sigmoid(w_router x), each expert on its own
     (float32; w_router float32 [E, d]); ``all_scores`` float32 [T, n_real] (or None) receives every real expert's score;
     the ``top`` experts with the
     largest score + bias (``bias`` float32 [E] or None) -> ids int32 [T, top], their scores -> weights float32
-    [T, top] (divided by their sum if ``renormalize``).  ``counts`` int32 [n_real] (or None) receives how many
+    [T, top] (divided by their sum if ``renormalize``, then times ``weight_scale``).  ``groups`` > 1: the experts form that
+    many equal groups of neighbours, and only experts of the ``keep_groups`` groups with the best single experts can be
+    chosen.  ``counts`` int32 [n_real] (or None) receives how many
     tokens chose each of the first ``n_real`` experts (added to what it holds)."""
     n, d = x.shape
     e = w_router.shape[0]
@@ -811,7 +1008,7 @@ def route(x, w_router, bias, ids, weights, counts, n_real, top, renormalize=Fals
                                    _dev(counts, "counts", torch.int32) if counts is not None else None, n, d, e, n_real, top,
                                    1 if renormalize else 0, 1 if sigmoid_scores else 0,
                                    _dev(all_scores, "all_scores", torch.float32) if all_scores is not None else None,
-                                   _stream()), "route")
+                                   int(groups), int(keep_groups), float(weight_scale), _stream()), "route")
 
 
 def route_layout(ids, counts, offsets, tile_first, cursor, row_of_pair, token_of_row, n_real, weights=None,
@@ -836,19 +1033,23 @@ def route_layout(ids, counts, offsets, tile_first, cursor, row_of_pair, token_of
 PLAIN_GLU = (float("inf"), 1.0, 0.0)      # (limit, slope, shift) of silu(gate) * up
 
 
-def expert_gemm(a, token_of_row, w, out, offsets, tile_first, n_pairs, act: bool, glu=PLAIN_GLU, row_scale=None) -> None:
+NO_ACT, GATED_ACT, RELU2_ACT = 0, 1, 2     # what an expert's first product ends with
+
+
+def expert_gemm(a, token_of_row, w, out, offsets, tile_first, n_pairs, act: int, glu=PLAIN_GLU, row_scale=None) -> None:
     """out[row] = a[row] . w[e]^T for the rows of every expert e's stretch (``token_of_row`` given: a[token of the
-    row]); w [E, N, K], or with ``act`` [E, 2N, K] (gate rows, then up rows) and out = the gated unit's activation
-    with ``glu`` = (limit, slope, shift) and ``row_scale`` float32 [rows] (see capped_glu; the default is silu(gate) *
+    row]); w [E, N, K] (``act`` RELU2_ACT: out = the square of the product's positive part), or with GATED_ACT [E, 2N, K]
+    (gate rows, then up rows) and out = the gated unit's activation with ``glu`` = (limit, slope, shift) and ``row_scale`` float32 [rows] (see capped_glu; the default is silu(gate) *
     up).  Each output element is one ascending chain of FP32 fused multiply-adds."""
     e, wn, k = w.shape
-    n = wn // 2 if act else wn
+    act = int(act)
+    n = wn // 2 if act == GATED_ACT else wn
     if a.shape[1] != k or out.shape[1] != n or out.shape[0] < n_pairs or a.dtype != w.dtype or out.dtype != w.dtype:
         raise KernelError("expert_gemm: shapes or dtypes do not agree")
     _check(load("routed").ni_expert_gemm(_dev(a, "a"), _code(a, "a"),
                                          _dev(token_of_row, "token_of_row", torch.int32) if token_of_row is not None else None,
                                          _dev(w, "w"), _dev(out, "out"), _dev(offsets, "offsets", torch.int32),
-                                         _dev(tile_first, "tile_first", torch.int32), n_pairs, e, n, k, 1 if act else 0,
+                                         _dev(tile_first, "tile_first", torch.int32), n_pairs, e, n, k, act,
                                          float(glu[0]), float(glu[1]), float(glu[2]),
                                          _dev(row_scale, "row_scale", torch.float32) if row_scale is not None else None,
                                          _stream()), "expert_gemm")
@@ -857,17 +1058,18 @@ def expert_gemm(a, token_of_row, w, out, offsets, tile_first, n_pairs, act: bool
 EXPERT_ROWS_MAX_PAIRS = 64      # (token, choice) pairs up to which a step takes the kernel with one warp per output
 
 
-def expert_rows(a, w, out, ids, gather: bool, act: bool, glu=PLAIN_GLU, row_scale=None) -> None:
+def expert_rows(a, w, out, ids, gather: bool, act: int, glu=PLAIN_GLU, row_scale=None) -> None:
     """A few rows, bfloat16: out[p] = a[p or p / top] . w[ids[p]]^T for every pair p of a real expert (others are
     skipped), one warp per output; ``act`` as in expert_gemm.  K must be a multiple of 8."""
     e, wn, k = w.shape
-    n = wn // 2 if act else wn
+    act = int(act)
+    n = wn // 2 if act == GATED_ACT else wn
     n_pairs, top = ids.numel(), ids.shape[1]
     bf = torch.bfloat16
     if a.shape[1] != k or out.shape != (n_pairs, n) or a.shape[0] != (n_pairs // top if gather else n_pairs):
         raise KernelError("expert_rows: shapes do not agree")
     _check(load("routed").ni_expert_rows(_dev(a, "a", bf), _dev(w, "w", bf), _dev(out, "out", bf), _dev(ids, "ids", torch.int32),
-                                         n_pairs, top, 1 if gather else 0, e, n, k, 1 if act else 0,
+                                         n_pairs, top, 1 if gather else 0, e, n, k, act,
                                          float(glu[0]), float(glu[1]), float(glu[2]),
                                          _dev(row_scale, "row_scale", torch.float32) if row_scale is not None else None,
                                          _stream()), "expert_rows")

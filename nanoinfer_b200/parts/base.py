@@ -63,7 +63,7 @@ from typing import Dict, Optional, Tuple
 class WeightSlot:
     """Shape and initialisation rule of one weight of a part.
 
-    init "normal": N(0, std) in random-weights mode; "ones": 1.0 (norm gains).
+    init "normal": N(0, std) in random-weights mode; "ones": 1.0 (norm gains); "zeros"; "eye": the identity matrix.
     """
     shape: Tuple[int, ...]
     init: str = "normal"

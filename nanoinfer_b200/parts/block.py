@@ -344,6 +344,90 @@ class OutputNormBlock:
         return StreamCopy(h, x) if bf16 else None
 
 
+class HyperConnectionBlock:
+    """Pre-norm sublayers over several residual streams x_1 .. x_S (``ModelConfig.streams``).  For each of the two
+    sublayers, with its own coefficients in [S], mix [S, S] (from, to) and out [S]:
+
+        u = sum_s in[s] x_s;   y = sublayer(norm(u));   x_t <- sum_s mix[s, t] x_s + out[t] y   for all t at once
+
+    (a layer may have no feed-forward, then only the first).  The streams come as an ``ops.ResidualStreams``, which
+    carries a sublayer's output along until the next reader's pass applies it: one kernel per sublayer makes the
+    streams anew, sums them for the next input and - with a norm that needs no statistics - norms it.  Other norms read
+    the FP32 sum.  Streams, sums and coefficients are FP32; a sublayer hands its output over in FP32, routed experts as
+    rows that the same pass sums up (``leaves_rows``)."""
+
+    kernel_modules = ("hyper",)       # libraries of csrc that this part's kernels live in
+    takes_streams = True
+
+    @staticmethod
+    def weight_slots(layer_spec, hidden_size: int):
+        s = int(layer_spec.extra_dict()["streams"])
+        slots = {}
+        for q in (1,) if layer_spec.feed_forward is None else (1, 2):
+            slots.update({f"hc{q}.in": WeightSlot((s,), init="ones"), f"hc{q}.out": WeightSlot((s,), init="ones"),
+                          f"hc{q}.mix": WeightSlot((s, s), init="eye")})
+        return slots
+
+    def __init__(self, layer_spec, hidden_size: int, weights_of, rt) -> None:
+        self.rt, self.hidden_size = rt, hidden_size
+        s = int(layer_spec.extra_dict()["streams"])
+        if not 0 < s <= ops.HYPER_MAX_STREAMS:
+            raise ValueError(f"hyper-connections: {s} streams are not supported (1 to {ops.HYPER_MAX_STREAMS})")
+
+        def norm(spec, what):
+            return part("norm", spec.kind)(spec, hidden_size, weights_of(what), rt)
+
+        self.mixer_norm = norm(layer_spec.mixer_norm, "mixer_norm")
+        self.mixer = part("mixer", layer_spec.mixer.kind)(layer_spec.mixer, hidden_size, weights_of("mixer"), rt)
+        self.ffn_norm = self.feed_forward = None
+        if layer_spec.feed_forward is not None:
+            if layer_spec.ffn_norm is None:
+                raise ValueError("a hyper-connection layer's feed-forward needs its norm")
+            self.ffn_norm = norm(layer_spec.ffn_norm, "ffn_norm")
+            self.feed_forward = part("feed_forward", layer_spec.feed_forward.kind)(
+                layer_spec.feed_forward, hidden_size, weights_of("feed_forward"), rt)
+        w = weights_of("block")
+        self.coef = [tuple(rt.gain(w[f"hc{q}.{what}"]) for what in ("in", "mix", "out"))
+                     for q in ((1,) if self.feed_forward is None else (1, 2))]
+
+    def weights_in_order(self) -> tuple:
+        ffn = self.feed_forward
+        return tuple(getattr(self.mixer, "weights_in_order", tuple)()) + \
+            (tuple(getattr(ffn, "weights_in_order", tuple)()) if ffn is not None else ())
+
+    def first_norm(self):
+        return None
+
+    def _input(self, streams, coef, norm):
+        fused = getattr(norm, "tanh_norm", None)
+        if fused is not None:
+            return streams.read(coef, fused, self.rt.dtype)
+        return norm.forward(streams.read(coef), None)
+
+    @staticmethod
+    def _leave(streams, y, mix, out) -> None:
+        if isinstance(y, torch.Tensor) and y.dtype != torch.float32:
+            y = y.float()
+        streams.leave(y, mix, out)
+
+    def forward(self, streams, delta, ctx, cache):
+        (c_in, c_mix, c_out), ffn = self.coef[0], self.feed_forward
+        after = ctx.read_after                       # what runs after this block
+        ctx.read_after = (tuple(getattr(ffn, "weights_in_order", tuple)()) if ffn is not None else ()) + tuple(after)
+        try:
+            y = self.mixer.forward(self._input(streams, c_in, self.mixer_norm), ctx, cache)
+        finally:
+            ctx.read_after = after
+        self._leave(streams, y, c_mix, c_out)
+        if ffn is not None:
+            c_in, c_mix, c_out = self.coef[1]
+            x = self._input(streams, c_in, self.ffn_norm)
+            y = ffn.forward(x, ctx, leave_rows=True) if getattr(ffn, "leaves_rows", False) else ffn.forward(x, ctx)
+            self._leave(streams, y, c_mix, c_out)
+        return None
+
+
+register_part("arrangement", "hyper_connections", HyperConnectionBlock, replace=True)
 register_part("arrangement", "pre_norm", PreNormBlock, replace=True)
 register_part("arrangement", "output_norm", OutputNormBlock, replace=True)
 register_part("arrangement", "sandwich_norm", SandwichNormBlock, replace=True)

@@ -246,10 +246,16 @@ class RoutedExperts(Part):
     The unit's activation is act(g, u) = g' sigmoid(slope g') (u' + shift) with g' = min(g, limit) and
     u' = clamp(u, -limit, limit); ``limit`` (default: none), ``gate_slope`` (1) and ``up_shift`` (0) come in the
     spec's extra, and their defaults make it silu(g) u.  With ``weight_on_input`` a chosen expert reads the token's
-    input MULTIPLIED by its weight and its output counts once: sum_e unit_e(s_e x).  Both first products are linear
+    input MULTIPLIED by its weight and its output counts once: sum_e unit_e(s_e x).  The first products are linear
     in the input, so the weight multiplies their results, in FP32, before the limits - no scaled copy of the
     input is made.  ``shared_ff`` > 0 adds one more unit of that size (limit ``shared_limit``, same slope and
     shift) that every token runs on its plain input; its output is added.
+
+    ``unit`` "relu2" instead of the default "gated": an expert is W_down relu(W_up x)^2, with no gate.  ``weight_scale``
+    multiplies the weights (after the division by their sum, if any).  ``groups`` = n > 1: the experts form n equal groups
+    of neighbours, a group counts as much as its best expert, and only experts of the ``keep_groups`` best groups can be
+    chosen.  With ``leave_rows`` forward hands the chosen experts' rows over unsummed (ops.RoutedRows), for an
+    arrangement whose next kernel sums them on its way (no identity experts, no shared unit).
 
     The experts' matrices are stacked ([E, 2F, d] gate rows then up rows, and [E, d, F]).  In bfloat16, steps of a
     few tokens with at least as many (token, choice) pairs as experts multiply with ALL experts' matrices (one
@@ -275,8 +281,10 @@ class RoutedExperts(Part):
         slots = {"router": WeightSlot((n_real + n_id, hidden_size))}
         if spec.extra_dict().get("choice_bias", False):
             slots["correction"] = WeightSlot((n_real + n_id,))
+        gated = spec.extra_dict().get("unit", "gated") == "gated"
         for j in range(n_real):
-            slots[f"e{j}.gate"] = WeightSlot((f, hidden_size))
+            if gated:
+                slots[f"e{j}.gate"] = WeightSlot((f, hidden_size))
             slots[f"e{j}.up"] = WeightSlot((f, hidden_size))
             slots[f"e{j}.down"] = WeightSlot((hidden_size, f))
         sf = int(spec.extra_dict().get("shared_ff", 0))
@@ -300,6 +308,17 @@ class RoutedExperts(Part):
             raise ConfigError(f"routed experts: scores '{scores}' is not known (softmax, sigmoid)")
         self.sigmoid_scores = scores == "sigmoid"
         self.weight_on_input = bool(e.get("weight_on_input", False))
+        unit = e.get("unit", "gated")
+        if unit not in ("gated", "relu2"):
+            raise ConfigError(f"routed experts: unit '{unit}' is not known (gated, relu2)")
+        self.gated = unit == "gated"
+        self.first_act = ops.GATED_ACT if self.gated else ops.RELU2_ACT
+        self.weight_scale = float(e.get("weight_scale", 1.0))
+        self.groups, self.keep_groups = int(e.get("groups", 1)), int(e.get("keep_groups", 1))
+        if self.groups < 1 or self.n_all % self.groups or not 0 < self.keep_groups <= self.groups or \
+                self.keep_groups * (self.n_all // self.groups) < top:
+            raise ConfigError(f"routed experts: {self.groups} groups (of which {self.keep_groups} stay) do not fit {self.n_all} "
+                              f"experts with top {top}")
         slope, shift = float(e.get("gate_slope", 1.0)), float(e.get("up_shift", 0.0))
         limit = e.get("limit")
         self.glu = (float("inf") if limit is None else float(limit), slope, shift)
@@ -308,8 +327,9 @@ class RoutedExperts(Part):
         self.w_router = rt.gain(weights["router"])                  # the router runs in FP32
         self.bias = rt.gain(weights["correction"]) if "correction" in weights else None
         if n_real > 0:
-            self.w_gate_up = rt.weight(torch.stack([torch.cat([weights[f"e{j}.gate"], weights[f"e{j}.up"]], dim=0)
-                                                    for j in range(n_real)]))
+            # [E, 2F, d] gate rows, then up rows (an ungated unit: [E, F, d], its up rows)
+            self.w_gate_up = rt.weight(torch.stack([torch.cat([weights[f"e{j}.gate"], weights[f"e{j}.up"]], dim=0) if self.gated
+                                                    else weights[f"e{j}.up"] for j in range(n_real)]))
             self.w_down = rt.weight(torch.stack([weights[f"e{j}.down"] for j in range(n_real)]))
         else:
             self.w_gate_up = self.w_down = None
@@ -327,6 +347,9 @@ class RoutedExperts(Part):
         routed = (self.w_gate_up, self.w_down) if self.n_real > 0 else ()
         return routed + ((self.w_shared_gate_up, self.w_shared_down) if self.shared_inter > 0 else ())
 
+        # forward accepts leave_rows=True and hands the chosen experts' rows over (a hook for arrangements that sum them)
+        self.leaves_rows = n_real == self.n_all and self.shared_inter <= 0 and not self.weight_on_input
+
     adds_normed = True          # forward accepts normed_into=(h, gain, eps): h += RMSNorm(output) * gain, returns None
 
     def _shared(self, x):
@@ -339,7 +362,16 @@ class RoutedExperts(Part):
         ops.capped_glu(gate_up, act, *self.shared_glu)
         return rt.linear(act, self.w_shared_down, out_dtype=torch.float32)
 
+    def _activate(self, first, act, row_scale=None) -> None:
+        """The first products' results ([rows, 2F] gate | up, or [rows, F]) through the unit's activation."""
+        if self.gated:
+            ops.capped_glu(first, act, *self.glu, row_scale=row_scale)
+        else:
+            ops.relu_squared(first, act)
+
     def _combine(self, z, x, ids, weights, row_of_pair, n_real, normed_into, all_experts=0):
+        if normed_into is _LEAVE_ROWS:
+            return ops.RoutedRows(z, ids, weights, row_of_pair, all_experts)
         unit = self.weight_on_input            # real experts' rows count once: their weight went into their input
         y = self._shared(x)
         if y is None and normed_into is not None and x.shape[1] <= 12000:
@@ -356,8 +388,8 @@ class RoutedExperts(Part):
             return None
         return y
 
-    def forward(self, x: torch.Tensor, ctx, normed_into=None):
-        return self.finish(self._first(x, None, None), ctx, normed_into=normed_into)
+    def forward(self, x: torch.Tensor, ctx, normed_into=None, leave_rows: bool = False):
+        return self.finish(self._first(x, None, None), ctx, normed_into=_LEAVE_ROWS if leave_rows else normed_into)
 
     def project(self, h: torch.Tensor, norm):
         """A few rows (bfloat16): the norm of the stream, and - where the step has at least as many (token, choice)
@@ -370,12 +402,13 @@ class RoutedExperts(Part):
         n = (x if x is not None else h).shape[0]
         dense = (rt.dtype == torch.bfloat16 and self.n_real > 0 and rt.skinny(n, self.hidden_size)
                  and n * self.top >= self.n_real and self.inter % 8 == 0
-                 and not (self.weight_on_input and self.renormalize))     # that path scales by the plain scores
+                 and not (self.weight_on_input and (self.renormalize or self.weight_scale != 1.0 or not self.gated)))
+        # (with the weight on the input that path scales by the plain scores)
         if x is None:
             x = norm.forward(h, None)                 # the router and the identity experts read the normed rows
         gate_up_all = None
         if dense:
-            w_all = self.w_gate_up.view(self.n_real * 2 * self.inter, self.hidden_size)
+            w_all = self.w_gate_up.view(-1, self.hidden_size)
             gate_up_all = rt.empty(n, w_all.shape[0])
             if h is not None:
                 ops.gemv_norm_bf16(h, norm.gain, norm.eps, None, w_all, gate_up_all, ops.STORE_BF16)
@@ -385,7 +418,8 @@ class RoutedExperts(Part):
 
     def _route(self, x, ids, weights, counts, all_scores=None):
         ops.route(x, self.w_router, self.bias, ids, weights, counts, self.n_real, self.top, self.renormalize,
-                  sigmoid_scores=self.sigmoid_scores, all_scores=all_scores)
+                  sigmoid_scores=self.sigmoid_scores, all_scores=all_scores, groups=self.groups, keep_groups=self.keep_groups,
+                  weight_scale=self.weight_scale)
 
     def finish(self, first, ctx, normed_into=None):
         x, gate_up_all = first
@@ -405,18 +439,17 @@ class RoutedExperts(Part):
             scores = rt.empty(n, n_real, dtype=f32) if on_input else None
             self._route(x, ids, weights, None, all_scores=scores)
             act = rt.empty(n * n_real, f)
-            ops.capped_glu(gate_up_all.view(n * n_real, 2 * f), act, *self.glu,
-                           row_scale=scores.view(-1) if on_input else None)
+            self._activate(gate_up_all.view(n * n_real, -1), act, row_scale=scores.view(-1) if on_input else None)
             z = rt.heads_linear(act.view(n, n_real * f), self.w_down)                           # [T, E d]
             return self._combine(z.view(n * n_real, d), x, ids, weights, None, n_real, normed_into, all_experts=n_real)
         few = (rt.dtype == torch.bfloat16 and pairs <= ops.EXPERT_ROWS_MAX_PAIRS and d % 8 == 0 and f % 8 == 0)
         if few:
             self._route(x, ids, weights, None)
             act = rt.empty(pairs, f)
-            ops.expert_rows(x, self.w_gate_up, act, ids, gather=True, act=True, glu=self.glu,
+            ops.expert_rows(x, self.w_gate_up, act, ids, gather=True, act=self.first_act, glu=self.glu,
                             row_scale=weights.view(-1) if on_input else None)
             z = rt.empty(pairs, d)
-            ops.expert_rows(act, self.w_down, z, ids, gather=False, act=False)
+            ops.expert_rows(act, self.w_down, z, ids, gather=False, act=ops.NO_ACT)
             return self._combine(z, x, ids, weights, None, n_real, normed_into)
         counts = rt.workspace("routed_counts", ops.ROUTE_MAX_EXPERTS, i32, zero=True)
         self._route(x, ids, weights, counts)
@@ -427,11 +460,13 @@ class RoutedExperts(Part):
         weight_of_row = torch.zeros(pairs, dtype=f32, device=rt.device) if on_input else None
         ops.route_layout(ids, counts, offsets, tile_first, cursor, row_of_pair, token_of_row, n_real,
                          weights=weights if on_input else None, weight_of_row=weight_of_row)
-        act = rt.experts_linear(x, self.w_gate_up, offsets, tile_first, pairs, token_of_row=token_of_row, act=True,
+        act = rt.experts_linear(x, self.w_gate_up, offsets, tile_first, pairs, token_of_row=token_of_row, act=self.first_act,
                                 glu=self.glu, row_scale=weight_of_row)
         z = rt.experts_linear(act, self.w_down, offsets, tile_first, pairs)
         return self._combine(z, x, ids, weights, row_of_pair, n_real, normed_into)
 
+
+_LEAVE_ROWS = object()       # in the place of normed_into: the rows are handed over unsummed
 
 register_part("feed_forward", "swiglu", SwiGLU, replace=True)
 register_part("feed_forward", "capped_glu", CappedGLU, replace=True)

@@ -44,6 +44,12 @@ class LinearHead(Part):
         rt = self.rt
         if ctx.n_logit_rows == 0:
             return rt.empty(0, self.vocab_size, dtype=torch.float32)
+        if isinstance(h, ops.ResidualStreams):        # several streams: their sum at the wanted rows, then the norm
+            fused = getattr(norm, "tanh_norm", None)
+            x = h.read(None, fused, rt.dtype, rows=ctx.logit_rows)
+            if fused is None:
+                x = norm.forward(x, None)
+            return rt.linear(x, self.weight, out_dtype=torch.float32)
         if delta is None and rt.skinny(ctx.n_logit_rows, self.hidden_size) and rt.fuses_norm(norm):
             # few rows: final norm, row selection and output projection in one launch
             logits = rt.empty(ctx.n_logit_rows, self.vocab_size, dtype=torch.float32)

@@ -618,6 +618,124 @@ class NormedQKAttention(PagedAttendMixin, Part):
         return rt.linear(att, self.w_o, out_dtype=torch.float32, residual=residual)
 
 
+class DifferentialAttention(PagedAttendMixin, Part):
+    """Differential attention: every head has TWO softmax maps over the same values, and the second is taken off the first.
+    With x the mixer's input, H = ``num_heads``, G = ``num_kv_heads``, D = ``head_dim`` and V = ``value_dim``:
+
+        q = W_q x  [H, 2, D],  k = W_k x  [G, 2, D],  v = W_v x  [G, V]        (head by head: map 1, map 2; no positions)
+        a_m = softmax over the earlier keys of (q_m . k_m softmax_scale), times v          for each map m
+        lambda = exp(sum lq1 lk1) - exp(sum lq2 lk2) + ``diff``                            one number for the layer
+        o = a_1 - lambda a_2;   o / sqrt(mean(o^2) + ``norm_eps``) * (1 - diff) per head;  then W_o on the heads side by side
+
+    ``own_kv`` false in the extra: no W_k and W_v; the layer reads the pages of the run whose cache it shares
+    (``LayerRun.cache_of``) with its own queries.
+
+    The cache holds a token's key heads 2 D wide, the two maps side by side, and its value heads.  Where V = 2 D (heads
+    of 64 or 128 in the cache) the layer is ordinary attention of that head size up to the scores: projection and cache
+    write are the ones of grouped-query attention without rotation, and the tensor-core attention kernels run both maps of
+    a head in one block over one fetch of the keys and values (tcgen05 for prompt portions: the two maps are its two
+    streams; split-K for single tokens: they are two rows of its tile), take the difference and norm it.  Other sizes
+    and FP32 go through the plain kernel, FP32 out, and ``difference_norm``."""
+
+    kernel_modules = ("rope_kv", "qk_norm_rope", "difference")       # libraries of csrc that this part's kernels live in
+    kernel_modules_bf16 = ("attention_prefill_tc",)
+
+    adds_into_residual = True
+    graph_safe = "all"
+
+    @staticmethod
+    def _dims(spec):
+        e = spec.extra_dict()
+        return spec.num_heads, spec.num_kv_heads, spec.head_dim, int(e.get("value_dim", 2 * spec.head_dim)), bool(e.get("own_kv", True))
+
+    @staticmethod
+    def weight_slots(spec, hidden_size: int) -> Dict[str, WeightSlot]:
+        h, g, d, v, own = DifferentialAttention._dims(spec)
+        slots = {"q": WeightSlot((h * 2 * d, hidden_size))}
+        if own:
+            slots.update({"k": WeightSlot((g * 2 * d, hidden_size)), "v": WeightSlot((g * v, hidden_size))})
+        slots.update({name: WeightSlot((d,)) for name in ("lq1", "lk1", "lq2", "lk2")})
+        slots["o"] = WeightSlot((hidden_size, h * v))
+        return slots
+
+    def __init__(self, spec, hidden_size, weights, rt) -> None:
+        Part.__init__(self, spec, hidden_size, weights, rt)
+        h, g, d, v, own = self._dims(spec)
+        if h <= 0 or g <= 0 or h % g:
+            raise ConfigError("differential attention: heads must be a positive multiple of kv_heads")
+        if not 0 < d <= 256 or not 0 < v <= 512:
+            raise ConfigError(f"differential attention: key size {d} (1 to 256) or value size {v} (1 to 512) is not supported")
+        if spec.window is not None:
+            raise ConfigError("differential attention sees every earlier key (no window)")
+        if spec.position.kind != "none":
+            raise ConfigError("differential attention takes no position encoding")
+        e = spec.extra_dict()
+        self.n_heads, self.n_kv, self.map_dim, self.value_dim, self.own_kv = h, g, d, v, own
+        self.head_dim = 2 * d                        # a key head as the cache holds it
+        self.window = None
+        self.scale = float(spec.softmax_scale)
+        self.eps, self.diff = float(e.get("norm_eps", 1e-6)), float(e["diff"])
+        self.position = part("position", "none")(spec.position, hidden_size, {}, rt)
+        lam = {n: weights[n].double() for n in ("lq1", "lk1", "lq2", "lk2")}
+        self.lam = float(torch.exp((lam["lq1"] * lam["lk1"]).sum()) - torch.exp((lam["lq2"] * lam["lk2"]).sum())) + self.diff
+        rows = [weights["q"]] + ([weights["k"], weights["v"]] if own else [])
+        # ... as whole heads of one size where values are as wide as a key head (what the fused projection kernels take)
+        self.uniform = v == 2 * d
+        pad = 0 if self.uniform else -sum(r.shape[0] for r in rows) % 8      # zero rows: every result row starts on 16 bytes
+        if pad:
+            rows.append(torch.zeros(pad, hidden_size, dtype=weights["q"].dtype, device=weights["q"].device))
+        self.w_in = rt.weight(torch.cat(rows, dim=0))
+        self.w_o = rt.weight(weights["o"])
+
+    def cache_need(self):
+        if not self.own_kv:
+            return None
+        if self.uniform:
+            return PagedKVNeed(self.n_kv, self.head_dim, None)
+        return PagedNeed((("k", (self.n_kv, self.head_dim)), ("v", (self.n_kv, self.value_dim))), None)
+
+    def weights_in_order(self) -> tuple:
+        return (self.w_in, self.w_o)
+
+    def _project(self, x, ctx, cache, table):
+        """The queries [T, H 2 D]; a layer with keys and values of its own leaves this step's in the pages."""
+        rt = self.rt
+        n, h, g, hd, v = x.shape[0], self.n_heads, self.n_kv, self.head_dim, self.value_dim
+        if not self.own_kv:
+            return rt.linear(x, self.w_in)[:, :h * hd].contiguous()
+        if not cache.writable:
+            raise ConfigError("differential attention: a layer with keys of its own needs a cache of its own")
+        q = rt.empty(n, h * hd)
+        pages = (cache.k_pages, cache.v_pages)
+        if self.uniform and rt.skinny(n, self.hidden_size) and hd % 16 == 0:
+            ops.gemv_qkv_rope(x, None, 0.0, self.w_in, q, *pages, ctx.positions, ctx.seq_of_token, table, self.position.inv_freq,
+                              h, g, hd, 0, rt.page_size)
+        elif self.uniform:
+            ops.rope_kv_write(rt.linear(x, self.w_in), q, *pages, ctx.positions, ctx.seq_of_token, table, self.position.inv_freq,
+                              h, g, hd, 0, True, rt.page_size)
+        else:
+            ops.qk_norm_rope(rt.linear(x, self.w_in), None, None, None, self.eps, ctx.positions, ctx.seq_of_token, table,
+                             self.position.inv_freq, 1.0, q, *pages, h, g, hd, v, 0, rt.page_size)
+        return q
+
+    def _plain(self, q, cache, out, ctx, table, token_list=None) -> None:
+        """Both maps of every head through the plain kernel (FP32 out), then their normed difference."""
+        n, h, v = q.shape[0], self.n_heads, self.value_dim
+        maps = self.rt.empty(n, 2 * h, v, dtype=torch.float32)
+        ops.attention_generic(q, cache.k_pages, cache.v_pages, maps.view(n, 2 * h * v), ctx.positions, ctx.seq_of_token, table,
+                              2 * h, self.n_kv, self.map_dim, self.rt.page_size, None, self.scale, token_list=token_list,
+                              value_dim=v, maps=2)
+        ops.difference_norm(maps, out, self.lam, self.eps, 1.0 - self.diff, token_list=token_list)
+
+    def forward(self, x: torch.Tensor, ctx, cache, residual=None):
+        rt = self.rt
+        table = ctx.block_tables[cache.group]
+        q = self._project(x, ctx, cache, table)
+        att = rt.empty(x.shape[0], self.n_heads * self.value_dim)
+        self._plain(q, cache, att, ctx, table)
+        return rt.linear(att, self.w_o, out_dtype=torch.float32, residual=residual)
+
+
 class ParallelMixers(Part):
     """Two mixers side by side that read the same input: y = left_scale * left(x) + right_scale * right(x).  The two
     specs (``left``, ``right``: MixerSpec of any registered kinds) and the two scales come in the spec's extra; the
@@ -704,4 +822,5 @@ register_part("mixer", "attention", PagedAttention, replace=True)
 register_part("mixer", "latent_attention", LatentAttention, replace=True)
 register_part("mixer", "conv_key_attention", ConvKeyAttention, replace=True)
 register_part("mixer", "normed_qk_attention", NormedQKAttention, replace=True)
+register_part("mixer", "differential_attention", DifferentialAttention, replace=True)
 register_part("mixer", "parallel_mixers", ParallelMixers, replace=True)

@@ -64,6 +64,33 @@ class RMSNormOnePlus(RMSNorm):
         self.gain = rt.gain(weights["weight"]) + 1.0
 
 
+class DynamicTanh(Part):
+    """y = tanh(alpha x) * w + b, coordinate by coordinate: one learned scalar ``alpha``, a weight and a bias ("weight",
+    "alpha", "b").  It has no statistics (the spec's eps is not read), so whatever forms x in registers can norm it on
+    the spot: ``tanh_norm`` is the triple (alpha, weight, bias), FP32 on the device."""
+
+    kernel_modules = ("hyper",)       # libraries of csrc that this part's kernels live in
+
+    @staticmethod
+    def weight_slots(spec, hidden_size: int) -> Dict[str, WeightSlot]:
+        return {"weight": WeightSlot((hidden_size,), init="ones"), "b": WeightSlot((hidden_size,), init="zeros"),
+                "alpha": WeightSlot((), init="ones")}
+
+    def __init__(self, spec, hidden_size, weights, rt) -> None:
+        super().__init__(spec, hidden_size, weights, rt)
+        self.tanh_norm = (rt.gain(weights["alpha"]).reshape(1), rt.gain(weights["weight"]), rt.gain(weights["b"]))
+
+    def forward(self, h: torch.Tensor, delta: Optional[torch.Tensor],
+                rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if delta is not None and delta.dtype != torch.float32:
+            ops.residual_add(h, delta)
+            delta = None
+        out = self.rt.empty(h.shape[0] if rows is None else rows.numel(), self.hidden_size)
+        ops.tanh_norm(h, delta, *self.tanh_norm, out, rows)
+        return out
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh, replace=True)
 register_part("norm", "rmsnorm", RMSNorm, replace=True)
 register_part("norm", "rmsnorm_one_plus", RMSNormOnePlus, replace=True)
 register_part("norm", "rmsnorm_scalar", ScalarRMSNorm, replace=True)

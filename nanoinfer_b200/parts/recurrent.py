@@ -287,6 +287,96 @@ class Retention(Part):
         return rt.linear(y, self.w_o, out_dtype=f32, residual=residual)
 
 
+class MatrixMemory(Part):
+    """A matrix memory with exponential gates (the mLSTM cell of xLSTM).  Per head, with a matrix S [head_dim, value_dim], a
+    normaliser n [head_dim] and a running maximum m, all FP32 and zero at a sequence's start:
+
+        q = W_q x * head_dim^-1/2, k = W_k x, v = W_v x
+        i = cap tanh((W_i x + b_i) / cap),  f = logsigmoid(cap tanh((W_f x + b_f) / cap))       (one number per head each)
+        m' = max(f + m, i);   S <- e^(f + m - m') S + e^(i - m') k v^T;   n <- e^(f + m - m') n + e^(i - m') k;   m <- m'
+        o = S^T q / (max(|n . q|, e^-m) + 1e-6)
+
+    Each head's o is divided by its own root mean square (``norm_eps``), multiplied by a weight over all heads ("norm") and
+    by sigmoid(W_g x), and leaves through W_o.  ``value_dim`` and ``gate_cap`` come in the spec's extra.
+
+    A step of single tokens is one FP32-out product for everything the layer projects and ONE launch for the rest
+    (csrc/mlstm.cu).  Other steps run in chunks: the queries, keys, values and output gates in the compute type, the
+    logits of i and f as a product of their own that leaves in FP32; every chunk's own sum, a scan, every chunk's
+    read-out.  The state is a slot of the runner's state pool."""
+
+    kernel_modules = ("mlstm", "lightning")       # libraries of csrc that this part's kernels live in
+
+    adds_into_residual = True
+    graph_safe = "all"
+
+    @staticmethod
+    def _dims(spec):
+        e = spec.extra_dict()
+        return spec.num_heads, spec.head_dim, int(e.get("value_dim", spec.head_dim))
+
+    @staticmethod
+    def weight_slots(spec, hidden_size: int) -> Dict[str, WeightSlot]:
+        h, d, v = MatrixMemory._dims(spec)
+        return {"q": WeightSlot((h * d, hidden_size)), "k": WeightSlot((h * d, hidden_size)),
+                "v": WeightSlot((h * v, hidden_size)), "g": WeightSlot((h * v, hidden_size)),
+                "o": WeightSlot((hidden_size, h * v)), "norm": WeightSlot((h * v,), init="ones"),
+                "i": WeightSlot((h, hidden_size)), "i.b": WeightSlot((h,)),
+                "f": WeightSlot((h, hidden_size)), "f.b": WeightSlot((h,))}
+
+    def __init__(self, spec, hidden_size, weights, rt) -> None:
+        super().__init__(spec, hidden_size, weights, rt)
+        h, d, v = self._dims(spec)
+        e = spec.extra_dict()
+        if h <= 0 or v <= 0:
+            raise ConfigError("matrix memory: heads and value size must be positive")
+        if not 0 < d <= ops.MLSTM_MAX_DIM:
+            raise ConfigError(f"matrix memory: a key size of {d} is not supported (1 to {ops.MLSTM_MAX_DIM})")
+        self.H, self.D, self.V = h, d, v
+        self.eps, self.cap = float(e.get("norm_eps", 1e-6)), float(e["gate_cap"])
+        if not self.cap > 0.0:
+            raise ConfigError("matrix memory: gate_cap must be positive")
+        self.q_scale = float(d) ** -0.5
+
+        def padded(names):
+            rows = [weights[s] for s in names]
+            pad = -sum(r.shape[0] for r in rows) % 8         # zero rows, so that every row of the result starts on 16 bytes
+            if pad:
+                rows.append(torch.zeros(pad, hidden_size, dtype=weights["q"].dtype, device=weights["q"].device))
+            return rows
+
+        wide, narrow = padded(("q", "k", "v", "g")), padded(("i", "f"))
+        self.n_wide = sum(r.shape[0] for r in wide)
+        self.w_in = rt.weight(torch.cat(wide + narrow, dim=0))          # q | k | v | gate | pad | i | f | pad
+        self.w_o = rt.weight(weights["o"])
+        self.norm_w = rt.gain(weights["norm"])
+        self.bias_i, self.bias_f = rt.gain(weights["i.b"]), rt.gain(weights["f.b"])
+
+    def cache_need(self):
+        return StateNeed((ops.mlstm_state_floats(self.H, self.D, self.V),), "float32")
+
+    def weights_in_order(self) -> tuple:
+        return (self.w_in, self.w_o)
+
+    def forward(self, x: torch.Tensor, ctx, cache, residual=None):
+        rt = self.rt
+        n = x.shape[0]
+        h, d, v = self.H, self.D, self.V
+        f32 = torch.float32
+        y = rt.empty(n, h * v)
+        gates = (self.bias_i, self.bias_f, self.cap, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs)
+        if ctx.max_q_len == 1:
+            proj = rt.linear(x, self.w_in, out_dtype=f32)
+            ops.mlstm_token_step(proj, proj, self.n_wide, self.n_wide + h, *gates, self.q_scale, self.norm_w, self.eps, y, h, d, v)
+        else:
+            proj = rt.linear(x, self.w_in[:self.n_wide])
+            z = rt.linear(x, self.w_in[self.n_wide:], out_dtype=f32)
+            buf = rt.workspace("mlstm_chunks", ops.mlstm_buffer_floats(n, ctx.n_seqs, h, d, v), f32)     # one for all layers
+            out = rt.empty(n, h * v, dtype=f32)
+            ops.mlstm_chunk_step(proj, z, 0, h, *gates, ctx.max_q_len, self.q_scale, self.norm_w, self.eps, buf, out, y, h, d, v)
+        return rt.linear(y, self.w_o, out_dtype=f32, residual=residual)
+
+
+register_part("mixer", "matrix_memory", MatrixMemory, replace=True)
 register_part("mixer", "gated_delta", GatedDeltaRule, replace=True)
 register_part("mixer", "retention", Retention, replace=True)
 register_part("mixer", "lightning", LightningAttention, replace=True)

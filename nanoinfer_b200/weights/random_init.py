@@ -36,6 +36,8 @@ def random_tensors(config, seed: int, std: float = 0.02, dtype: torch.dtype = to
             yield p.name, torch.ones(p.shape, dtype=dtype)
         elif p.init == "zeros":
             yield p.name, torch.zeros(p.shape, dtype=dtype)
+        elif p.init == "eye":
+            yield p.name, torch.eye(*p.shape, dtype=dtype)
         else:
             g = torch.Generator(device="cpu")
             g.manual_seed(_tensor_seed(seed, p.name))
