@@ -109,11 +109,16 @@ __device__ __forceinline__ void dec_warm(const unsigned char* p, unsigned long l
 // cluster barrier, and that block merges them in split order - no scratch in global memory, no
 // fence, no ticket.
 // chunk > 0: the token at position p sees only the keys from p - p % chunk on; flags bit 0 (sink): one is added to the
-// softmax's denominator; flags bit 1: all kv heads of the launch read the pages' one head.
+// softmax's denominator; flags >> 1 = n > 1: n neighbouring kv heads of the launch read one head of the pages.
+// DIFF (differential attention): a query head has two maps, which are two rows of the tile; a query row has HD / 2 numbers
+// and stands in the half of the tile's row that its map's keys stand in (a key row holds both maps side by side), zeros in
+// the other half.  The result of a head is u = a_0 - lambda a_1 of its two rows, u / sqrt(mean(u^2) + eps) * factor.
 // CAP: the scaled scores are bounded smoothly, s <- cap * tanh(s / cap), before the softmax.  The kernel is then
 // handed scale_log2e = 2 log2(e) scale / cap and cap_l2 = cap log2(e): with x = exp2(raw * scale_log2e),
 // cap_l2 - 2 cap_l2 / (x + 1) is the capped score in the exponent's base.
-template <int HD, int SEG, bool CL, bool CAP>
+struct DecDiff { float lambda, eps, factor; };
+
+template <int HD, int SEG, bool CL, bool CAP, bool DIFF>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                         const __nv_bfloat16* __restrict__ v_pages, __nv_bfloat16* __restrict__ out,
@@ -122,11 +127,12 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                         int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                         float scale_log2e, float cap_l2, int n_splits, float* __restrict__ scratch,
                         int* __restrict__ tickets, const unsigned char* __restrict__ warm_a, unsigned long long warm_a_bytes,
-                        const unsigned char* __restrict__ warm_b, unsigned long long warm_b_bytes, int chunk, int flags) {
-    // flags: bit 0 - the sink; bit 1 - the pages hold ONE head that all the launch's kv heads share (a compressed cache
-    // whose many query heads are dealt over several "kv heads" of at most 16 rows each)
+                        const unsigned char* __restrict__ warm_b, unsigned long long warm_b_bytes, int chunk, int flags,
+                        const DecDiff diff) {
+    // flags: bit 0 - the sink; the rest - how many of the launch's kv heads share one head of the pages (0: each has its
+    // own): more than 16 query rows over one page head are dealt over several "kv heads" of at most 16 rows each
     const int sink = flags & 1;
-    const bool shared_pages = (flags & 2) != 0;
+    const int share = flags >> 1 > 1 ? flags >> 1 : 1;
     // Weights that the kernels after this one will read (the caller's hint, up to two regions): asked
     // into L2 now, in pieces dealt over the blocks, while this kernel - which waits on latencies
     // more than on bandwidth - leaves the memory system room.  Nothing here depends on the kernel before.
@@ -144,6 +150,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
 
     const int item = blockIdx.x;             // index into token_list
     const int kvh = blockIdx.y;
+    const int page_head = kvh / share, page_heads = n_kv_heads / share;
     const int split = blockIdx.z;
     const int t_idx = token_list ? token_list[item] : item;
     const int pos = positions[t_idx];
@@ -207,8 +214,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
             key = key < k_end ? key : k_end - 1;
             const int pi = page_shift >= 0 ? key >> page_shift : key / page_size;
             const int slot = page_shift >= 0 ? key & (page_size - 1) : key - pi * page_size;
-            const size_t off = shared_pages ? ((size_t)page[it] * page_size + slot) * HD + c * 8
-                                            : (((size_t)page[it] * n_kv_heads + kvh) * page_size + slot) * HD + c * 8;
+            const size_t off = (((size_t)page[it] * page_heads + page_head) * page_size + slot) * HD + c * 8;
             dec_cp_async16(sK + dec_sw<HD>(r, c), k_pages + off);
             dec_cp_async16(sV + dec_sw<HD>(r, c), v_pages + off);
         }
@@ -224,7 +230,13 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
         for (int idx = threadIdx.x; idx < 16 * CH; idx += blockDim.x) {
             const int r = idx / CH, c = idx - r * CH;
             __nv_bfloat16* dst = sQ + dec_sw<HD>(r, c);
-            if (r < G)
+            if (DIFF) {
+                const int cc = c - (r & 1) * (CH / 2);              // the chunk of the map's own half row
+                if (r < G && cc >= 0 && cc < CH / 2)
+                    dec_cp_async16(dst, q + ((size_t)t_idx * n_q_heads + (size_t)kvh * G + r) * (HD / 2) + cc * 8);
+                else
+                    *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+            } else if (r < G)
                 dec_cp_async16(dst, q + ((size_t)t_idx * n_q_heads + (size_t)kvh * G + r) * HD + c * 8);
             else
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
@@ -358,6 +370,10 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
             acc += sm_o[w][row][d] * f;
             ll += sm_l[w][row] * f;
         }
+        if (n_splits == 1 && DIFF) {      // a map's finished row; its head's other map follows
+            sm_o[0][row][d] = acc / ll;
+            continue;
+        }
         if (n_splits == 1) {   // nothing to merge with: this is the result
             out[((size_t)t_idx * n_q_heads + (size_t)kvh * G + row) * HD + d] = __float2bfloat16_rn(acc / ll);
             continue;
@@ -372,7 +388,27 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
         dst[2 + d] = acc;
         if (d == 0) { dst[0] = mm; dst[1] = ll; }
     }
-    if (n_splits == 1) return;
+    // DIFF: both maps of every head lie finished in sm_o[0]; a warp takes a head at a time
+    auto difference = [&]() {
+        __syncthreads();
+        for (int h = warp; h < G / 2; h += DEC_WARPS) {
+            float u[HD / 32], ss = 0.f;
+#pragma unroll
+            for (int k = 0; k < HD / 32; ++k) {
+                u[k] = fmaf(-diff.lambda, sm_o[0][2 * h + 1][lane + 32 * k], sm_o[0][2 * h][lane + 32 * k]);
+                ss = fmaf(u[k], u[k], ss);
+            }
+            ss = ni_warp_sum(ss);
+            const float f = diff.factor / sqrtf(ss / (float)HD + diff.eps);
+            __nv_bfloat16* orow = out + ((size_t)t_idx * (n_q_heads / 2) + (size_t)kvh * (G / 2) + h) * HD;
+#pragma unroll
+            for (int k = 0; k < HD / 32; ++k) orow[lane + 32 * k] = __float2bfloat16_rn(u[k] * f);
+        }
+    };
+    if (n_splits == 1) {
+        if (DIFF) difference();
+        return;
+    }
     if (CL) {
         // ---- the cluster's first block merges the splits, from its own shared memory ----
         dec_cluster_arrive();   // this block's partial results are written
@@ -427,8 +463,10 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                 ll += ls[j] * f;
             }
         }
-        out[((size_t)t_idx * n_q_heads + (size_t)kvh * G + row) * HD + d] = __float2bfloat16_rn(acc / ll);
+        if (DIFF) sm_o[0][row][d] = acc / ll;
+        else out[((size_t)t_idx * n_q_heads + (size_t)kvh * G + row) * HD + d] = __float2bfloat16_rn(acc / ll);
     }
+    if (DIFF) difference();
 }
 
 // ---- the balanced variant: keys dealt evenly over a fixed set of blocks ---------------------------
@@ -830,22 +868,22 @@ NI_EXPORT int ni_attention_decode_balanced(const void* q, const void* k_pages, c
     }
 }
 
-template <int HD, int SEG, bool CL, bool CAP>
+template <int HD, int SEG, bool CL, bool CAP, bool DIFF>
 static int launch_decode_cl(const void* q, const void* k_pages, const void* v_pages, void* out, const int* token_list,
                          int n_items, const int* positions, const int* seq_of_token, const int* block_table,
                          int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                          float scale_log2e, float cap_l2, int n_splits, float* scratch, int* tickets, const void* warm_a,
                          unsigned long long warm_a_bytes, const void* warm_b, unsigned long long warm_b_bytes,
-                         int chunk, int flags, cudaStream_t stream) {
+                         int chunk, int flags, const DecDiff& diff, cudaStream_t stream) {
     const size_t kv_smem = (size_t)(16 + 4 * SEG) * HD * sizeof(__nv_bfloat16);
     const size_t smem = kv_smem + (CL ? (size_t)n_splits * (n_q_heads / n_kv_heads) * (HD + 2) * sizeof(float) : 0);
     static size_t configured = 0;
     if (configured < smem) {
-        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<HD, SEG, CL, CAP>,
+        cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<HD, SEG, CL, CAP, DIFF>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         if (CL) {   // clusters of 9 to 16 blocks (a lone request's many splits) are beyond the portable size
-            e = cudaFuncSetAttribute(attention_decode_kernel<HD, SEG, CL, CAP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+            e = cudaFuncSetAttribute(attention_decode_kernel<HD, SEG, CL, CAP, DIFF>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
             if (e != cudaSuccess) return (int)e;
         }
         configured = smem;
@@ -868,12 +906,12 @@ static int launch_decode_cl(const void* q, const void* k_pages, const void* v_pa
     // 1.13).  Started after its predecessor, the cluster variant wins (0.804; batch 4: 0.801 -> 0.773).
     cfg.attrs = CL ? attr + 1 : attr;
     cfg.numAttrs = 1;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_decode_kernel<HD, SEG, CL, CAP>, (const __nv_bfloat16*)q,
+    cudaError_t e = cudaLaunchKernelEx(&cfg, attention_decode_kernel<HD, SEG, CL, CAP, DIFF>, (const __nv_bfloat16*)q,
                                        (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
                                        (__nv_bfloat16*)out, token_list, positions, seq_of_token, block_table,
                                        bt_stride, n_q_heads, n_kv_heads, page_size, window, scale_log2e, cap_l2, n_splits,
                                        scratch, tickets, (const unsigned char*)warm_a, warm_a_bytes,
-                                       (const unsigned char*)warm_b, warm_b_bytes, chunk, flags);
+                                       (const unsigned char*)warm_b, warm_b_bytes, chunk, flags, diff);
     return e == cudaSuccess ? NI_OK : (int)e;
 }
 
@@ -891,16 +929,18 @@ static int launch_decode(const void* q, const void* k_pages, const void* v_pages
                          int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                          float scale_log2e, float cap_l2, int n_splits, float* scratch, int* tickets, const void* warm_a,
                          unsigned long long warm_a_bytes, const void* warm_b, unsigned long long warm_b_bytes,
-                         int chunk, int flags, cudaStream_t stream) {
+                         int chunk, int flags, const DecDiff* diff, cudaStream_t stream) {
+    const DecDiff none = {0.f, 0.f, 0.f};
     const size_t slot_bytes = (size_t)n_splits * (n_q_heads / n_kv_heads) * (HD + 2) * sizeof(float);
     const bool few_blocks = (long long)n_items * n_kv_heads * n_splits <= 2LL * ni_sm_count() && slot_bytes <= 65536;
     if (dec_cluster_merge && n_splits >= 2 && ((n_splits <= 8 && slot_bytes <= DEC_CLUSTER_SLOT_BYTES) || (n_splits <= 16 && few_blocks)))
-#define NI_DEC_GO(CL, CAP)                                                                                          \
-    launch_decode_cl<HD, SEG, CL, CAP>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,          \
-                                       block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window, scale_log2e,   \
-                                       cap_l2, n_splits, scratch, tickets, warm_a, warm_a_bytes, warm_b, warm_b_bytes, chunk, flags, stream)
-        return cap_l2 > 0.f ? NI_DEC_GO(true, true) : NI_DEC_GO(true, false);
-    return cap_l2 > 0.f ? NI_DEC_GO(false, true) : NI_DEC_GO(false, false);
+#define NI_DEC_GO(CL, CAP, DIFF)                                                                                    \
+    launch_decode_cl<HD, SEG, CL, CAP, DIFF>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,    \
+                                             block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,          \
+                                             scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, warm_a_bytes,     \
+                                             warm_b, warm_b_bytes, chunk, flags, diff ? *diff : none, stream)
+        return diff ? NI_DEC_GO(true, false, true) : (cap_l2 > 0.f ? NI_DEC_GO(true, true, false) : NI_DEC_GO(true, false, false));
+    return diff ? NI_DEC_GO(false, false, true) : (cap_l2 > 0.f ? NI_DEC_GO(false, true, false) : NI_DEC_GO(false, false, false));
 #undef NI_DEC_GO
 }
 
@@ -914,9 +954,9 @@ static int decode_dispatch(const void* q, const void* k_pages, const void* v_pag
                                   int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                   float scale, float score_cap, int n_splits, float* scratch, int* tickets,
                                   const void* warm_a, long long warm_a_bytes, const void* warm_b,
-                                  long long warm_b_bytes, int chunk, int flags, cudaStream_t stream) {
+                                  long long warm_b_bytes, int chunk, int flags, const DecDiff* diff, cudaStream_t stream) {
     if (n_items <= 0) return NI_OK;
-    if (chunk < 0) return NI_ERR_BAD_ARGUMENT;
+    if (chunk < 0 || (flags >> 1 > 1 && n_kv_heads % (flags >> 1))) return NI_ERR_BAD_ARGUMENT;
     if (warm_a_bytes < 0 || (warm_a_bytes & 15) || (warm_a_bytes && (!warm_a || ((uintptr_t)warm_a & 15)))) return NI_ERR_BAD_ARGUMENT;
     if (warm_b_bytes < 0 || (warm_b_bytes & 15) || (warm_b_bytes && (!warm_b || ((uintptr_t)warm_b & 15)))) return NI_ERR_BAD_ARGUMENT;
     if (n_q_heads <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads || page_size <= 0 || n_splits <= 0 ||
@@ -935,16 +975,16 @@ static int decode_dispatch(const void* q, const void* k_pages, const void* v_pag
                 return launch_decode<64, 128>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                               block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                               scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
             return launch_decode<64, 64>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                           block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                           scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
         case 128:
             return launch_decode<128, 64>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                            block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                            scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
         default: return NI_ERR_UNSUPPORTED_SIZE;
     }
 }
@@ -958,12 +998,12 @@ NI_EXPORT int ni_attention_decode(const void* q, const void* k_pages, const void
                                   long long warm_b_bytes, cudaStream_t stream) {
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, 0.f, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, nullptr, stream);
 }
 
 // The same with a chunk mask (chunk > 0: the token at position p sees only the keys from p - p % chunk on) and flags:
-// bit 0 - one is added to the softmax's denominator (a sink); bit 1 - k_pages / v_pages hold ONE head
-// ([P, 1, page_size, hd]) that all n_kv_heads of the call read, so that more than 16 query heads over one shared head
+// bit 0 - one is added to the softmax's denominator (a sink); flags >> 1 = n > 1 - n neighbouring kv heads of the call read
+// one head of k_pages / v_pages ([P, n_kv_heads / n, page_size, hd]), so that more than 16 query heads over one page head
 // can be dealt over several groups of at most 16.  score_cap 0: scores are not bounded.
 NI_EXPORT int ni_attention_decode_masked(const void* q, const void* k_pages, const void* v_pages, void* out,
                                          const int* token_list, int n_items, const int* positions,
@@ -975,7 +1015,25 @@ NI_EXPORT int ni_attention_decode_masked(const void* q, const void* k_pages, con
     if (score_cap < 0.f) return NI_ERR_BAD_ARGUMENT;
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, score_cap, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, chunk, flags & 3, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, chunk, flags, nullptr, stream);
+}
+
+// Differential attention: two maps per head.  q [n_tokens, Hm, head_dim / 2], Hm = n_map_heads counting maps (a head's two
+// follow one another); key rows hold both maps side by side, value rows head_dim numbers; out [n_tokens, Hm / 2, head_dim] =
+// (a_0 - lambda a_1) / sqrt(mean(.^2) + eps) * factor.  The group n_map_heads / n_kv_heads is even and at most 16; share > 1:
+// that many neighbouring kv heads of the call read one head of the pages.
+NI_EXPORT int ni_attention_decode_difference(const void* q, const void* k_pages, const void* v_pages, void* out,
+                                             const int* token_list, int n_items, const int* positions,
+                                             const int* seq_of_token, const int* block_table, int bt_stride,
+                                             int n_map_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                             float lambda, float eps, float factor, int share, int n_splits, float* scratch,
+                                             int* tickets, const void* warm_a, long long warm_a_bytes, const void* warm_b,
+                                             long long warm_b_bytes, cudaStream_t stream) {
+    if (n_kv_heads <= 0 || n_map_heads % n_kv_heads || (n_map_heads / n_kv_heads) % 2 || share < 0) return NI_ERR_BAD_ARGUMENT;
+    const DecDiff d = {lambda, eps, factor};
+    return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
+                           n_map_heads, n_kv_heads, head_dim, page_size, 0, scale, 0.f, n_splits, scratch, tickets,
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, share << 1, &d, stream);
 }
 
 // The same with the scaled scores bounded by score_cap * tanh(s / score_cap) (score_cap > 0).
@@ -989,7 +1047,7 @@ NI_EXPORT int ni_attention_decode_capped(const void* q, const void* k_pages, con
     if (!(score_cap > 0.f)) return NI_ERR_BAD_ARGUMENT;
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, score_cap, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, nullptr, stream);
 }
 
 // ---- the variant that allocates nothing (see attention_decode_noalloc.h) ----------------------

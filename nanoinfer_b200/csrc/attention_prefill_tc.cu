@@ -35,6 +35,11 @@
 // a wait that runs out records a code in the error word, and the block frees its tensor memory
 // and returns.
 //
+// Differential attention (DIFF) is the same kernel with the two streams given to ONE head: a head's query and key rows
+// are two maps side by side (HD / 2 numbers each) over the same values, stream s multiplies the s-th halves, and at the
+// end out = (a_0 - lambda a_1) / sqrt(mean(.^2) + eps) * factor over the head's HD values - four threads per row, each with
+// a quarter of the columns of both accumulators.
+//
 // Takes head sizes 64 and 128, two or more query heads per kv head, and page sizes 8 to
 // 128 that divide 128; everything else is the business of attention_prefill.cu.
 //
@@ -172,6 +177,15 @@ __device__ __forceinline__ void at_ld32(uint32_t taddr, uint32_t r[32]) {
         : "r"(taddr));
     asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 }
+__device__ __forceinline__ void at_ld16(uint32_t taddr, uint32_t r[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];\n"
+        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+          "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+        : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+}
 __device__ __forceinline__ void at_st32(uint32_t taddr, const uint32_t r[32]) {
     asm volatile(
         "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
@@ -223,9 +237,10 @@ struct AtParams {
     int* error;
     int chunk;                     // > 0: a query at position p sees only the keys from p - p % chunk on
     int sink;                      // != 0: one is added to every row's softmax denominator (a key of score 0 without a value)
+    float lambda, eps, factor;     // DIFF
 };
 
-template <int HD, int STAGES>
+template <int HD, int STAGES, bool DIFF>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const AtParams p) {
@@ -268,7 +283,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // "longest job first" over the whole launch (with the tiles on the grid's fast axis every head
     // pair's light tiles came before the next pair's heavy ones: 2,048 tokens took 25 tile-times
     // of the heaviest block's 16, against 16 to 18 this way).
-    const int pairs = p.n_kv_heads * ((p.n_q_heads / p.n_kv_heads + 1) / 2);
+    const int pairs = DIFF ? p.n_q_heads : p.n_kv_heads * ((p.n_q_heads / p.n_kv_heads + 1) / 2);
     const int tile_index = blockIdx.x / pairs, pair_index = blockIdx.x - tile_index * pairs;
     const int seq = p.tile_seq[tile_index];
     const int row0 = p.tile_row0[tile_index];
@@ -288,10 +303,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     // block of an odd group has one head left: its second stream runs that head again, so that
     // the streams' hand-offs stay as they are, and stores nothing.
     const int blocks_per_kv = (G + 1) / 2;
-    const int kvh = pair_index / blocks_per_kv;
+    const int kvh = DIFF ? pair_index / G : pair_index / blocks_per_kv;
     const int first = 2 * (pair_index - kvh * blocks_per_kv);
-    const int head0 = kvh * G + first;
-    const int head1 = first + 1 < G ? head0 + 1 : head0;
+    const int head0 = DIFF ? pair_index : kvh * G + first;
+    const int head1 = DIFF ? head0 : (first + 1 < G ? head0 + 1 : head0);
 
     if (threadIdx.x == 0) {
         at_mbar_init(q_full, 1);
@@ -322,8 +337,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (warp == 0) {
         // ---- TMA producer: lane 0 waits and announces the bytes, lane g copies page g of a tile ----
         if (lane == 0) {
-            at_mbar_expect_tx(q_full, 2 * TILE_BYTES);
-            for (int s = 0; s < 2; ++s)
+            at_mbar_expect_tx(q_full, (DIFF ? 1 : 2) * TILE_BYTES);
+            for (int s = 0; s < (DIFF ? 1 : 2); ++s)         // (DIFF: both streams read one head's row)
                 for (int h = 0; h < HALVES; ++h)
                     at_tma_2d(sQ + s * TILE_BYTES + h * HALF_BYTES, &map_q, (s ? head1 : head0) * HD + h * 64, q_begin + row0, q_full);
         }
@@ -387,9 +402,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const uint64_t dq0 = at_desc(sQ, 1024), dk0 = at_desc(sK, 1024);
             const uint64_t dv0 = at_desc(sV, HALVES > 1 ? HALF_BYTES : 1024);
             auto scores = [&](int s, int i) {      // S_s = Q_s K_i^T
-                const uint64_t dq = dq0 + (uint64_t)((s * TILE_BYTES) >> 4);
-                const uint64_t dk = dk0 + (uint64_t)(((i % STAGES) * TILE_BYTES) >> 4);
-                if (leader) {
+                // DIFF: stream s contracts over the s-th half of the rows only (a 64-column half, or 2 of its 4 steps)
+                const uint64_t dq = dq0 + (uint64_t)((DIFF ? s * (HALVES > 1 ? HALF_BYTES : 64) : s * TILE_BYTES) >> 4);
+                const uint64_t dk = dk0 + (uint64_t)(((i % STAGES) * TILE_BYTES + (DIFF ? s * (HALVES > 1 ? HALF_BYTES : 64) : 0)) >> 4);
+                if (DIFF) {
+                    if (leader) {
+#pragma unroll
+                        for (int kk = 0; kk < (HALVES > 1 ? 4 : 2); ++kk)
+                            at_mma_ss(tmem_base + s * AT_BN, dq + (uint64_t)((kk * 32) >> 4), dk + (uint64_t)((kk * 32) >> 4), idesc_s,
+                                      kk != 0 ? 1u : 0u);
+                        at_commit(&s_full[s]);
+                    }
+                } else if (leader) {
 #pragma unroll
                     for (int h = 0; h < HALVES; ++h)
 #pragma unroll
@@ -603,12 +627,57 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         // ---- the finished rows: O / l -> bfloat16; the row's sum is the two halves' together ----
         if (p.sink && half == 0) l += at_exp2(-(m_used == -INFINITY ? 0.f : m_used));      // the sink's weight, counted once per row
-        row_max[0][s][half][r] = l;                        // (the buffer of an even tile; see below)
-        if (ok && n_tiles > 0 &&
-            __all_sync(0xffffffffu, at_wait(&o_done[s], (uint32_t)(n_tiles - 1) & 1u, abort_flag, p.error, AT_ERR_SOFTMAX))) {
+        const bool finished = ok && n_tiles > 0 &&
+                              __all_sync(0xffffffffu, at_wait(&o_done[s], (uint32_t)(n_tiles - 1) & 1u, abort_flag, p.error, AT_ERR_SOFTMAX));
+        if (DIFF) {
+            // The four threads of a row (two streams, two halves) meet twice: when both streams' products are done - the
+            // row sums go through the maxima's buffer 0, whose last reader has passed the product just waited for - and
+            // with their sums of squares.  Every warp comes here, whatever happened to its waits.
+            if (finished) at_fence_after();
+            row_max[0][s][half][r] = l;
+            at_fence_before();
+            asm volatile("bar.sync %0, 128;\n" ::"r"(10 + quarter) : "memory");
             at_fence_after();
-            // Both warps of the pair pass this barrier after their last tile's exchange, whichever
-            // buffer that used; the sums go through buffer 0, written above after the last read of it.
+            const float inv0 = 1.0f / (row_max[0][0][0][r] + row_max[0][0][1][r]);
+            const float inv1 = p.lambda / (row_max[0][1][0][r] + row_max[0][1][1][r]);
+            constexpr int COLS = HD / 4;
+            const int part = 2 * s + half;
+            const uint32_t t_a = lane_base + O_COL + COLS * part;
+            float u[COLS];
+            float ss = 0.f;
+#pragma unroll
+            for (int c = 0; c < COLS / 16; ++c) {
+                uint32_t a0[16], a1[16];
+                at_ld16(t_a + 16 * c, a0);
+                at_ld16(t_a + HD + 16 * c, a1);
+#pragma unroll
+                for (int e = 0; e < 16; ++e) {
+                    const float d = fmaf(-inv1, __uint_as_float(a1[e]), __uint_as_float(a0[e]) * inv0);
+                    u[16 * c + e] = d;
+                    ss = fmaf(d, d, ss);
+                }
+            }
+            row_max[1][s][half][r] = ss;
+            asm volatile("bar.sync %0, 128;\n" ::"r"(10 + quarter) : "memory");
+            ss = (row_max[1][0][0][r] + row_max[1][0][1][r]) + (row_max[1][1][0][r] + row_max[1][1][1][r]);
+            const float f = p.factor / sqrtf(ss / (float)HD + p.eps);
+            if (finished && r < rows) {
+                __nv_bfloat16* orow = p.out + (size_t)(q_begin + row0 + r) * ((size_t)p.n_q_heads * HD) + (size_t)head0 * HD + COLS * part;
+#pragma unroll
+                for (int e = 0; e < COLS; e += 8) {
+                    uint4 w;
+                    w.x = at_pack(u[e] * f, u[e + 1] * f);
+                    w.y = at_pack(u[e + 2] * f, u[e + 3] * f);
+                    w.z = at_pack(u[e + 4] * f, u[e + 5] * f);
+                    w.w = at_pack(u[e + 6] * f, u[e + 7] * f);
+                    *reinterpret_cast<uint4*>(orow + e) = w;
+                }
+            }
+        } else if (finished) {
+            at_fence_after();
+            // The row sums go through the maxima's buffer 0: its last reader, the other warp of the pair, has read it before
+            // it handed over the probabilities of the product just waited for.
+            row_max[0][s][half][r] = l;
             asm volatile("bar.sync %0, 64;\n" ::"r"(pair_bar) : "memory");
             const float inv = 1.0f / (l + row_max[0][s][half ^ 1][r]);
             __nv_bfloat16* orow = p.out + (size_t)(q_begin + row0 + r) * ((size_t)p.n_q_heads * HD) +
@@ -684,22 +753,22 @@ static int at_make_map(CUtensorMap* map, const void* ptr, long long rows, long l
     return r == CUDA_SUCCESS ? NI_OK : NI_ERR_BAD_ARGUMENT;
 }
 
-template <int HD, int STAGES>
+template <int HD, int STAGES, bool DIFF>
 static int launch_at(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AtParams& p,
                      int n_tiles, cudaStream_t stream) {
     constexpr size_t tile = (size_t)(HD / 64) * AT_BN * 128;
     constexpr size_t smem = 1024 + (2 + 2 * STAGES) * tile + 512 + 2 * 2 * 2 * AT_BM * sizeof(float);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, STAGES>,
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, STAGES, DIFF>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    const long long blocks = (long long)n_tiles * p.n_kv_heads * ((p.n_q_heads / p.n_kv_heads + 1) / 2);
+    const long long blocks = (long long)n_tiles * (DIFF ? p.n_q_heads : p.n_kv_heads * ((p.n_q_heads / p.n_kv_heads + 1) / 2));
     if (blocks > 0x7fffffffLL) return NI_ERR_UNSUPPORTED_SIZE;
     dim3 grid((unsigned)blocks);
-    attention_prefill_tc_kernel<HD, STAGES><<<grid, AT_THREADS, smem, stream>>>(mq, mk, mv, p);
+    attention_prefill_tc_kernel<HD, STAGES, DIFF><<<grid, AT_THREADS, smem, stream>>>(mq, mk, mv, p);
     NI_RETURN_LAUNCH_STATUS();
 }
 
@@ -713,19 +782,12 @@ NI_EXPORT int ni_attention_prefill_tc_supports(int n_q_heads, int n_kv_heads, in
     return 1;
 }
 
-// q, out: bf16 [n_tokens, Hq * hd]; k_pages, v_pages: bf16 [n_pages, Hkv, page_size, hd], all 16-byte
-// aligned.  tile_seq / tile_row0 [n_tiles]: request and first query row of each block's 128 rows.
-// error: a device int, zero on entry; non-zero afterwards if a wait inside the kernel ran out.
-// chunk > 0: a query at position p sees only the keys from p - p % chunk on; sink != 0: one is added to the softmax's
-// denominator.
-NI_EXPORT int ni_attention_prefill_tc_masked(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,
-                                             int n_pages, const int* tile_seq, const int* tile_row0, int n_tiles,
-                                             const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
-                                             int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
-                                             float scale, int chunk, int sink, int* error, cudaStream_t stream) {
+static int run_at(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens, int n_pages, const int* tile_seq,
+                  const int* tile_row0, int n_tiles, const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
+                  int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale, int chunk, int sink,
+                  bool diff, float lambda, float eps, float factor, int* error, cudaStream_t stream) {
     if (n_tiles <= 0) return NI_OK;
     if (n_tokens <= 0 || n_pages <= 0 || error == nullptr || chunk < 0) return NI_ERR_BAD_ARGUMENT;
-    if (!ni_attention_prefill_tc_supports(n_q_heads, n_kv_heads, head_dim, page_size)) return NI_ERR_UNSUPPORTED_SIZE;
     if (((uintptr_t)q & 15) || ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || ((uintptr_t)out & 15))
         return NI_ERR_UNSUPPORTED_SIZE;
     CUtensorMap mq, mk, mv;
@@ -741,8 +803,43 @@ NI_EXPORT int ni_attention_prefill_tc_masked(const void* q, const void* k_pages,
     p.block_table = block_table; p.bt_stride = bt_stride; p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads;
     p.page_size = page_size; p.window = window; p.scale_log2e = scale * 1.4426950408889634f; p.error = error;
     p.chunk = chunk; p.sink = sink;
-    if (head_dim == 64) return launch_at<64, 4>(mq, mk, mv, p, n_tiles, stream);
-    return launch_at<128, 2>(mq, mk, mv, p, n_tiles, stream);
+    p.lambda = lambda; p.eps = eps; p.factor = factor;
+    if (diff) {
+        if (head_dim == 64) return launch_at<64, 4, true>(mq, mk, mv, p, n_tiles, stream);
+        return launch_at<128, 2, true>(mq, mk, mv, p, n_tiles, stream);
+    }
+    if (head_dim == 64) return launch_at<64, 4, false>(mq, mk, mv, p, n_tiles, stream);
+    return launch_at<128, 2, false>(mq, mk, mv, p, n_tiles, stream);
+}
+
+// q, out: bf16 [n_tokens, Hq * hd]; k_pages, v_pages: bf16 [n_pages, Hkv, page_size, hd], all 16-byte
+// aligned.  tile_seq / tile_row0 [n_tiles]: request and first query row of each block's 128 rows.
+// error: a device int, zero on entry; non-zero afterwards if a wait inside the kernel ran out.
+// chunk > 0: a query at position p sees only the keys from p - p % chunk on; sink != 0: one is added to the softmax's
+// denominator.
+NI_EXPORT int ni_attention_prefill_tc_masked(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,
+                                             int n_pages, const int* tile_seq, const int* tile_row0, int n_tiles,
+                                             const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
+                                             int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
+                                             float scale, int chunk, int sink, int* error, cudaStream_t stream) {
+    if (n_tiles <= 0) return NI_OK;
+    if (!ni_attention_prefill_tc_supports(n_q_heads, n_kv_heads, head_dim, page_size)) return NI_ERR_UNSUPPORTED_SIZE;
+    return run_at(q, k_pages, v_pages, out, n_tokens, n_pages, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table, bt_stride,
+                  n_q_heads, n_kv_heads, head_dim, page_size, window, scale, chunk, sink, false, 0.f, 0.f, 0.f, error, stream);
+}
+
+// Differential attention: a head's row of q and of the key pages holds its two maps side by side (head_dim / 2 numbers each),
+// value rows have head_dim numbers; out[t, h] = (a_0 - lambda a_1) / sqrt(mean(.^2) + eps) * factor.
+NI_EXPORT int ni_attention_prefill_tc_difference(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,
+                                                 int n_pages, const int* tile_seq, const int* tile_row0, int n_tiles,
+                                                 const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
+                                                 int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
+                                                 float lambda, float eps, float factor, int* error, cudaStream_t stream) {
+    if (n_tiles <= 0) return NI_OK;
+    if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads) return NI_ERR_BAD_ARGUMENT;
+    if ((head_dim != 64 && head_dim != 128) || page_size < 8 || page_size > 128 || 128 % page_size) return NI_ERR_UNSUPPORTED_SIZE;
+    return run_at(q, k_pages, v_pages, out, n_tokens, n_pages, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table, bt_stride,
+                  n_heads, n_kv_heads, head_dim, page_size, 0, scale, 0, 0, true, lambda, eps, factor, error, stream);
 }
 
 NI_EXPORT int ni_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,

@@ -117,6 +117,7 @@ _SIGNATURES = {
         "ni_attention_decode": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_capped": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_masked": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _P, _P, _LL, _P, _LL, _P],
+        "ni_attention_decode_difference": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_balanced": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_fresh_keys": [],
         "ni_attention_decode_set_cluster_merge": [_I],
@@ -129,6 +130,7 @@ _SIGNATURES = {
     "attention_prefill_tc": {
         "ni_attention_prefill_tc": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P],
         "ni_attention_prefill_tc_masked": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P],
+        "ni_attention_prefill_tc_difference": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P],
         "ni_attention_prefill_tc_supports": [_I, _I, _I, _I],
         "ni_attention_prefill_tc_set_wait": [_LL, _I],
     },
@@ -1601,7 +1603,7 @@ def attention_decode(q, k_pages, v_pages, out, token_list, n_items, positions, s
             _dev(positions, "positions", torch.int32), _dev(seq_of_token, "seq_of_token", torch.int32),
             _dev(block_table, "block_table", torch.int32), block_table.shape[1], n_q_heads, n_kv_heads,
             head_dim, page_size, int(window) if window else 0, float(scale), float(score_cap or 0.0), int(chunk or 0),
-            (1 if sink else 0) | (2 if shared_pages else 0), n_splits, _dev(scratch, "scratch", torch.float32),
+            (1 if sink else 0) | ((n_kv_heads if shared_pages else 0) << 1), n_splits, _dev(scratch, "scratch", torch.float32),
             _dev(tickets, "tickets", torch.int32),
             *regions, _stream()), "attention_decode")
         return
@@ -1614,6 +1616,57 @@ def attention_decode(q, k_pages, v_pages, out, token_list, n_items, positions, s
         head_dim, page_size, int(window) if window else 0, float(scale), *((float(score_cap),) if capped else ()), n_splits,
         _dev(scratch, "scratch", torch.float32), _dev(tickets, "tickets", torch.int32),
         *regions, _stream()), "attention_decode")
+
+
+def attention_decode_difference(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, n_heads,
+                                n_kv_heads, head_dim, page_size, scale, lam, eps, factor, n_splits, scratch, tickets, share: int = 1,
+                                warm=()) -> None:
+    """Split-K differential attention of single query tokens (bfloat16): every head has two maps.  q [T, H head_dim] (a
+    head's two half rows one after the other); key pages [P, Hkv / share, page_size, head_dim] with the two maps side by
+    side, value pages of the same shape; out [T, H head_dim] = (a_1 - lam a_2) / sqrt(mean(.^2) + eps) * factor per head.
+    At most 8 heads per kv head; ``share`` > 1: that many neighbouring kv heads of the call read one head of the pages.
+    The rest as attention_decode, with 2 H rows."""
+    regions = [v for w_ in (list(warm) + [None, None])[:2] for v in warm_region(w_)]
+    rows = 2 * n_heads // n_kv_heads
+    if head_dim not in DECODE_HEAD_DIMS or rows > 16 or n_heads % n_kv_heads or n_kv_heads % share:
+        raise KernelError(f"attention_decode_difference: head_dim {head_dim} / {rows} map rows per kv head not supported")
+    if q.shape[1] != n_heads * head_dim or out.shape[1] != n_heads * head_dim or k_pages.shape[1] != n_kv_heads // share \
+            or k_pages.shape[-1] != head_dim or v_pages.shape != k_pages.shape:
+        raise KernelError("attention_decode_difference: shapes do not agree")
+    if scratch.numel() < n_items * 2 * n_heads * n_splits * (head_dim + 2) or tickets.numel() < n_items * n_kv_heads:
+        raise KernelError("attention_decode_difference: scratch or tickets too small")
+    bf = torch.bfloat16
+    _check(load("attention_decode").ni_attention_decode_difference(
+        _dev(q, "q", bf), _dev(k_pages, "k_pages", bf), _dev(v_pages, "v_pages", bf), _dev(out, "out", bf),
+        _dev(token_list, "token_list", torch.int32) if token_list is not None else None, n_items,
+        _dev(positions, "positions", torch.int32), _dev(seq_of_token, "seq_of_token", torch.int32),
+        _dev(block_table, "block_table", torch.int32), block_table.shape[1], 2 * n_heads, n_kv_heads, head_dim, page_size,
+        float(scale), float(lam), float(eps), float(factor), int(share), n_splits, _dev(scratch, "scratch", torch.float32),
+        _dev(tickets, "tickets", torch.int32), *regions, _stream()), "attention_decode_difference")
+
+
+def attention_difference_tc_supports(head_dim: int, page_size: int) -> bool:
+    """True if the tcgen05 differential attention takes the case: cached heads of 64 or 128, a page size from 8 to 128
+    that divides 128."""
+    return head_dim in (64, 128) and 8 <= page_size <= 128 and 128 % page_size == 0
+
+
+def attention_prefill_difference(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table, n_heads,
+                                 n_kv_heads, head_dim, page_size, scale, lam, eps, factor) -> None:
+    """Differential attention of prompt portions (bfloat16, tcgen05): operands as attention_decode_difference, tiles as
+    attention_prefill; one block per tile and head runs the head's two maps as its two streams."""
+    if not attention_difference_tc_supports(head_dim, page_size) or n_heads % n_kv_heads:
+        raise KernelError(f"attention_prefill_difference: head_dim {head_dim} / page size {page_size} not supported")
+    if q.shape[1] != n_heads * head_dim or out.shape != q.shape or tuple(k_pages.shape[1:]) != (n_kv_heads, page_size, head_dim) \
+            or v_pages.shape != k_pages.shape:
+        raise KernelError("attention_prefill_difference: shapes do not agree")
+    bf, i32 = torch.bfloat16, torch.int32
+    _check(load("attention_prefill_tc").ni_attention_prefill_tc_difference(
+        _dev(q, "q", bf), _dev(k_pages, "k_pages", bf), _dev(v_pages, "v_pages", bf), _dev(out, "out", bf), q.shape[0],
+        k_pages.shape[0], _dev(tile_seq, "tile_seq", i32), _dev(tile_row0, "tile_row0", i32), n_tiles, _dev(cu_q, "cu_q", i32),
+        _dev(kv_len, "kv_len", i32), _dev(block_table, "block_table", i32), block_table.shape[1], n_heads, n_kv_heads, head_dim,
+        page_size, float(scale), float(lam), float(eps), float(factor), _error_word(q.device).data_ptr(), _stream()),
+        "attention_prefill_difference")
 
 
 def attention_prefill_tc_supports(n_q_heads: int, n_kv_heads: int, head_dim: int, page_size: int) -> bool:

@@ -732,8 +732,40 @@ class DifferentialAttention(PagedAttendMixin, Part):
         table = ctx.block_tables[cache.group]
         q = self._project(x, ctx, cache, table)
         att = rt.empty(x.shape[0], self.n_heads * self.value_dim)
-        self._plain(q, cache, att, ctx, table)
+        if rt.dtype != torch.bfloat16 or not self.uniform:
+            self._plain(q, cache, att, ctx, table)
+        else:
+            self._attend_maps(q, cache, att, ctx, table)
         return rt.linear(att, self.w_o, out_dtype=torch.float32, residual=residual)
+
+    def _attend_maps(self, q, cache, att, ctx, table) -> None:
+        """As PagedAttendMixin._attend: single query tokens (and the shortest portions) to the split-K kernel, longer
+        portions to the tcgen05 kernel, sizes those do not take to the plain kernel."""
+        rt, h, hd = self.rt, self.n_heads, self.head_dim
+        finish = (self.scale, self.lam, self.eps, 1.0 - self.diff)
+        # at most 8 heads (16 rows) per kv head of the split-K kernel: more are dealt over groups that read one page head
+        per_kv = h // self.n_kv
+        share = next(g for g in range(1, per_kv + 1) if per_kv % g == 0 and per_kv // g <= 8)
+        plan = None if ctx.decode_only else ctx.plan_of(self)    # a step of single tokens needs no lists
+        n_dec = q.shape[0] if plan is None else plan.scalars["n_dec"]
+        dec_list = None if plan is None else plan.arrays["dec_tokens"]
+        if n_dec > 0 and hd in ops.DECODE_HEAD_DIMS:
+            groups = self.n_kv * share
+            splits = ops.decode_splits(n_dec, groups, hd, ctx.max_kv_len)
+            scratch = rt.workspace("attention_decode_partials", n_dec * 2 * h * splits * (hd + 2), torch.float32)
+            tickets = rt.workspace("attention_decode_tickets", n_dec * groups, torch.int32, zero=True)
+            ops.attention_decode_difference(q, cache.k_pages, cache.v_pages, att, dec_list, n_dec, ctx.positions, ctx.seq_of_token,
+                                            table, h, groups, hd, rt.page_size, *finish, splits, scratch, tickets, share=share,
+                                            warm=rt.warm_attention(self.w_o, ctx))
+        elif n_dec > 0:
+            self._plain(q, cache, att, ctx, table, token_list=dec_list)
+        if plan is not None and plan.scalars["n_tiles"] > 0:
+            if ops.attention_difference_tc_supports(hd, rt.page_size):
+                ops.attention_prefill_difference(q, cache.k_pages, cache.v_pages, att, plan.arrays["tile_seq"],
+                                                 plan.arrays["tile_row0"], plan.scalars["n_tiles"], ctx.cu_q, ctx.kv_len, table,
+                                                 h, self.n_kv, hd, rt.page_size, *finish)
+            else:
+                self._plain(q, cache, att, ctx, table, token_list=plan.arrays["long_tokens"])
 
 
 class ParallelMixers(Part):
