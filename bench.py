@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the Llama 3.2 1B shape with random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers 16] [--impl ours|reference]
-    python bench.py --design runevik|vuvalorn|tazulix|mobatar [--sizes w1024,w2048]     (another design beside the Llama model of equal size)
+    python bench.py --design runevik|vuvalorn|tazulix|mobatar|kepusun [--sizes w1024,w2048]     (another design beside the Llama model of equal size)
 
 A "step" is one decode step of the whole batch.  Every request starts at a context of 2,048
 tokens and decodes W + K tokens (by default to 4,096).  Prints ONE JSON line:
@@ -122,6 +122,8 @@ def device_weights(config, seed, device):
     for p in tensor_plan(config):
         if p.init == "ones":
             out[p.name] = torch.ones(p.shape, dtype=torch.bfloat16, device=device)
+        elif p.init == "eye":
+            out[p.name] = torch.eye(*p.shape, dtype=torch.bfloat16, device=device)
         else:
             out[p.name] = (torch.randn(p.shape, generator=g, device=device, dtype=torch.float32) * 0.02).to(torch.bfloat16)
     return out
@@ -473,7 +475,27 @@ def mobatar_config(z):
             "embedding": {"bigram": {"buckets": 8191, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
 
 
-DESIGN_CONFIGS = {"runevik": runevik_config, "vuvalorn": vuvalorn_config, "tazulix": tazulix_config, "mobatar": mobatar_config}
+def kepusun_config(z):
+    """As many layers as the Llama model has, in the order matrix memory, differential attention, matrix memory,
+    differential attention over the keys and values of the attention layer before; four residual streams.  Matrix
+    memories of 128 x 128, as many heads as the Llama model; as many attention heads, two maps of 64 each over values of
+    128.  16 squared-relu experts in four groups (two stay), 4 chosen, each three eighths of the dense width (two
+    matrices instead of three), so a token multiplies with as many feed-forward weights as in the Llama model."""
+    heads = z["width"] // 128
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"] * 3 // 8},
+           "router": {"experts": 16, "top": 4, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+
+    def layer(i):
+        if i % 2 == 0:
+            return {"type": "mlstm", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+        m = {"heads": heads, "kv_heads": z["kv_heads"], "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.4}
+        return {"type": "attention", "mlp": mlp, "mixer": dict(m, kv_from=i - 2) if i % 4 == 3 else m}
+    return {"architecture": "Kepusun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "streams": 4,
+            "layers": [layer(i) for i in range(z["layers"])]}
+
+
+DESIGN_CONFIGS = {"runevik": runevik_config, "vuvalorn": vuvalorn_config, "tazulix": tazulix_config, "mobatar": mobatar_config,
+                  "kepusun": kepusun_config}
 
 
 def llama_config(z):
