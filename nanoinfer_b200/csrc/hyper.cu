@@ -127,14 +127,23 @@ __global__ void __launch_bounds__(HY_THREADS) hyper_step_kernel(const HyArgs a) 
             } else {
 #pragma unroll
                 for (int k = 0; k < V; ++k) y[k] = 0.f;
-                for (int j = 0; j < a.top; ++j) {
-                    const size_t p = t * a.top + j;
-                    const size_t row = a.all_experts > 0 ? t * a.all_experts + a.ids[p] : (a.row_of_pair ? (size_t)a.row_of_pair[p] : p);
-                    float zv[V];
-                    hy_load_act<T, V>(reinterpret_cast<const T*>(a.z) + row * d + c, zv);
-                    const float wgt = a.weights[p];
+                // four rows at a time: their numbers, then the rows, are on their way together
+                for (int j0 = 0; j0 < a.top; j0 += 4) {
+                    size_t row[4];
+                    float wgt[4], zv[4][V];
 #pragma unroll
-                    for (int k = 0; k < V; ++k) y[k] = fmaf(wgt, zv[k], y[k]);
+                    for (int j = 0; j < 4; ++j) {
+                        const size_t p = t * a.top + min(j0 + j, a.top - 1);
+                        row[j] = a.all_experts > 0 ? t * a.all_experts + a.ids[p] : (a.row_of_pair ? (size_t)a.row_of_pair[p] : p);
+                        wgt[j] = a.weights[p];
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) hy_load_act<T, V>(reinterpret_cast<const T*>(a.z) + row[j] * d + c, zv[j]);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        if (j0 + j < a.top)
+#pragma unroll
+                            for (int k = 0; k < V; ++k) y[k] = fmaf(wgt[j], zv[j][k], y[k]);
                 }
             }
 #pragma unroll

@@ -292,45 +292,57 @@ __global__ void mlstm_scan_kernel(float* __restrict__ state, long long state_str
     if (len <= 0) return;
     const int base = lt_chunk_base(cu_q, seq, &base_s);
     const int e = blockIdx.x * blockDim.x + threadIdx.x, DV = D * V;
-    if (e >= DV + D) return;
     const size_t rec = ml_record(D, V), stride = (size_t)H * rec, first = ((size_t)base * H + head) * rec;
     float* slot = state + (size_t)slots[seq] * state_stride;
     float* S = slot + (size_t)head * rec + e;
-    float s = *S, m = m_before[(size_t)base * H + head];
+    // What happens at a chunk's end is the same for the whole head: the block's first warp works it out for 32 chunks at a
+    // time - the chain of maxima in every lane alike, the two factors of chunk i in lane i.
+    __shared__ float keep_s[32], take_s[32];
+    const bool mine = e < DV + D;
+    float s = mine ? *S : 0.f, m = m_before[(size_t)base * H + head];
     const float* own_p = sums + first + e;
     float* o32 = before + first + e;
     __nv_bfloat16* o16 = reinterpret_cast<__nv_bfloat16*>(before + first) + e;
     const bool planes = split && e < DV;
     const int chunks = (len + LT_C - 1) / LT_C;
-    for (int c = 0; c < chunks; c += 8) {
-        float own[8], A[8];                       // loaded together: the chain below waits for memory once per group
-        double F[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const bool there = c + i < chunks;
-            own[i] = there ? own_p[(size_t)(c + i) * stride] : 0.f;
-            const MlMeta mt = there ? meta[(size_t)(base + c + i) * H + head] : MlMeta{0.f, 0.0};
-            A[i] = mt.A;
-            F[i] = mt.F;
-        }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            if (c + i >= chunks) break;
-            if (planes) {
-                const __nv_bfloat16 hi = __float2bfloat16_rn(s);
-                o16[(size_t)(c + i) * stride * 2] = hi;
-                o16[(size_t)(c + i) * stride * 2 + DV] = __float2bfloat16_rn(s - __bfloat162float(hi));
-            } else {
-                o32[(size_t)(c + i) * stride] = s;
+    for (int g0 = 0; g0 < chunks; g0 += 32) {
+        const int there = min(32, chunks - g0);
+        if (threadIdx.x < 32) {
+            const int lane = threadIdx.x;
+            const MlMeta mt = lane < there ? meta[(size_t)(base + g0 + lane) * H + head] : MlMeta{0.f, 0.0};
+            float m_old = 0.f, M_own = 0.f;
+            for (int i = 0; i < there; ++i) {
+                const float M = fmaxf(m, __shfl_sync(0xffffffffu, mt.A, i));
+                if (lane == i) { m_old = m; M_own = M; }
+                m = (float)(__shfl_sync(0xffffffffu, mt.F, i) + (double)M);
             }
-            if (e == 0 && c + i > 0) m_before[(size_t)(base + c + i) * H + head] = m;
-            const float M = fmaxf(m, A[i]);
-            s = fmaf(expf(m - M), s, expf(A[i] - M) * own[i]);
-            m = (float)(F[i] + (double)M);
+            keep_s[lane] = expf(m_old - M_own);
+            take_s[lane] = expf(mt.A - M_own);
+            if (blockIdx.x == 0 && lane < there && g0 + lane > 0) m_before[(size_t)(base + g0 + lane) * H + head] = m_old;
         }
+        __syncthreads();
+        for (int c = 0; c < there && mine; c += 8) {
+            float own[8];                         // loaded together: the chain below waits for memory once per group
+#pragma unroll
+            for (int i = 0; i < 8; ++i) own[i] = c + i < there ? own_p[(size_t)(g0 + c + i) * stride] : 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                if (c + i >= there) break;
+                const size_t at = (size_t)(g0 + c + i) * stride;
+                if (planes) {
+                    const __nv_bfloat16 hi = __float2bfloat16_rn(s);
+                    o16[at * 2] = hi;
+                    o16[at * 2 + DV] = __float2bfloat16_rn(s - __bfloat162float(hi));
+                } else {
+                    o32[at] = s;
+                }
+                s = fmaf(keep_s[c + i], s, take_s[c + i] * own[i]);
+            }
+        }
+        __syncthreads();
     }
-    *S = s;
-    if (e == 0) slot[(size_t)H * rec + head] = m;
+    if (mine) *S = s;
+    if (blockIdx.x == 0 && threadIdx.x == 0) slot[(size_t)H * rec + head] = m;
 }
 
 // ---- every chunk's read-out -------------------------------------------------------------------------------------------------

@@ -26,46 +26,73 @@
 #include "common.cuh"
 
 #define RT_MAX_EXPERTS 256
-#define RT_ROUTE_WARPS 8
 
-// One block per token: the token's row is widened to FP32 in shared memory once, the warps share the experts'
-// dot products (each one warp's sum in a fixed order), and the first warp does the softmax and the choice.
-template <typename T>
-__global__ void __launch_bounds__(RT_ROUTE_WARPS * 32)
+// One block per NT tokens: their rows are widened to FP32 in shared memory once, the warps share the experts' dot products,
+// EP experts at a time against all NT rows (each dot product one warp's sum in an order that depends on neither), and
+// then one warp per token does the softmax and the choice.  NT = 1 for few tokens (WARPS warps, so that all weights are
+// on their way at once), 4 or 8 for many (a block reads the router's weights once for its tokens).
+template <typename T, int NT, int EP, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
 route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
              const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights,
              int* __restrict__ counts, int n_tokens, int d, int n_all, int n_real, int top,
              int renormalize, int sigmoid_scores, float* __restrict__ all_scores, int groups, int keep, float weight_scale) {
-    extern __shared__ __align__(16) float xs[];          // [d]
-    __shared__ float choice[RT_MAX_EXPERTS];
-    __shared__ float score[RT_MAX_EXPERTS];
-    __shared__ float group_best[RT_MAX_EXPERTS];
+    static_assert(NT <= WARPS, "a warp per token");
+    extern __shared__ __align__(16) float xs[];          // [NT][d]
+    __shared__ float s_choice[NT][RT_MAX_EXPERTS];
+    __shared__ float s_score[NT][RT_MAX_EXPERTS];
+    __shared__ float s_group[NT][RT_MAX_EXPERTS];
     const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x;
-    const T* xr = x + (size_t)t * d;
-    for (int k = threadIdx.x; k < d; k += blockDim.x) xs[k] = ni_to_float(xr[k]);
+    const int t0 = blockIdx.x * NT, rows = min(NT, n_tokens - t0);
+    const T* xr = x + (size_t)t0 * d;
+    for (int k = threadIdx.x; k < NT * d; k += blockDim.x) xs[k] = k < rows * d ? ni_to_float(xr[k]) : 0.f;
     __syncthreads();
-    for (int e = w; e < n_all; e += RT_ROUTE_WARPS) {
-        const float* wr = w_router + (size_t)e * d;
-        float acc = 0.f;
+    for (int e0 = w * EP; e0 < n_all; e0 += WARPS * EP) {
+        const float* wr[EP];
+        float acc[EP][NT];
+#pragma unroll
+        for (int i = 0; i < EP; ++i) {
+            wr[i] = w_router + (size_t)min(e0 + i, n_all - 1) * d;
+#pragma unroll
+            for (int j = 0; j < NT; ++j) acc[i][j] = 0.f;
+        }
         if ((d & 3) == 0) {
-            const float4* w4 = reinterpret_cast<const float4*>(wr);
-            const float4* x4 = reinterpret_cast<const float4*>(xs);
+#pragma unroll (NT == 1 ? 8 : 2)
             for (int k = lane; k < (d >> 2); k += 32) {
-                const float4 a = x4[k], b = w4[k];
-                acc = fmaf(a.x, b.x, acc);
-                acc = fmaf(a.y, b.y, acc);
-                acc = fmaf(a.z, b.z, acc);
-                acc = fmaf(a.w, b.w, acc);
+                float4 b[EP];
+#pragma unroll
+                for (int i = 0; i < EP; ++i) b[i] = reinterpret_cast<const float4*>(wr[i])[k];
+#pragma unroll
+                for (int j = 0; j < NT; ++j) {
+                    const float4 a = reinterpret_cast<const float4*>(xs + (size_t)j * d)[k];
+#pragma unroll
+                    for (int i = 0; i < EP; ++i) {
+                        acc[i][j] = fmaf(a.x, b[i].x, acc[i][j]);
+                        acc[i][j] = fmaf(a.y, b[i].y, acc[i][j]);
+                        acc[i][j] = fmaf(a.z, b[i].z, acc[i][j]);
+                        acc[i][j] = fmaf(a.w, b[i].w, acc[i][j]);
+                    }
+                }
             }
         } else {
-            for (int k = lane; k < d; k += 32) acc = fmaf(xs[k], wr[k], acc);
+            for (int k = lane; k < d; k += 32)
+#pragma unroll
+                for (int i = 0; i < EP; ++i)
+#pragma unroll
+                    for (int j = 0; j < NT; ++j) acc[i][j] = fmaf(xs[(size_t)j * d + k], wr[i][k], acc[i][j]);
         }
-        acc = ni_warp_sum(acc);
-        if (lane == 0) score[e] = acc;
+#pragma unroll
+        for (int i = 0; i < EP; ++i)
+#pragma unroll
+            for (int j = 0; j < NT; ++j) {
+                const float v = ni_warp_sum(acc[i][j]);
+                if (lane == 0 && e0 + i < n_all) s_score[j][e0 + i] = v;
+            }
     }
     __syncthreads();
-    if (w != 0) return;
+    if (w >= rows) return;
+    const int t = t0 + w;
+    float *choice = s_choice[w], *score = s_score[w], *group_best = s_group[w];
     float inv = 1.0f;
     if (!sigmoid_scores) {
         float m = -INFINITY;
@@ -440,18 +467,31 @@ NI_EXPORT int ni_route(const void* x, int dtype, const float* w_router, const fl
     if (groups > 1 && (n_all % groups || keep <= 0 || (long long)keep * (n_all / groups) < top)) return NI_ERR_BAD_ARGUMENT;
     if (n_all > RT_MAX_EXPERTS) return NI_ERR_UNSUPPORTED_SIZE;
     if (d > 12000) return NI_ERR_UNSUPPORTED_SIZE;                    // the row lies in shared memory as FP32
-    const size_t smem = (size_t)d * sizeof(float);
-    if (dtype == NI_DTYPE_F32)
-        route_kernel<float><<<n_tokens, RT_ROUTE_WARPS * 32, smem, stream>>>((const float*)x, w_router, bias, ids, weights,
-                                                                           counts, n_tokens, d, n_all, n_real, top, renormalize,
-                                                                           sigmoid_scores, all_scores, groups, keep, weight_scale);
-    else if (dtype == NI_DTYPE_BF16)
-        route_kernel<__nv_bfloat16><<<n_tokens, RT_ROUTE_WARPS * 32, smem, stream>>>((const __nv_bfloat16*)x, w_router, bias,
-                                                                                   ids, weights, counts, n_tokens, d, n_all,
-                                                                                   n_real, top, renormalize, sigmoid_scores,
-                                                                                   all_scores, groups, keep, weight_scale);
-    else
-        return NI_ERR_BAD_ARGUMENT;
+    // many tokens: as many to a block as fit twice into an SM's shared memory
+    const int nt = n_tokens < 512 ? 1 : (d <= 3072 ? 8 : (d <= 6144 ? 4 : 1));
+    const size_t smem = (size_t)nt * d * sizeof(float);
+    const int blocks = (n_tokens + nt - 1) / nt;
+#define LAUNCH(T, NT, EP, WARPS)                                                                                                      \
+    do {                                                                                                                              \
+        if (smem > 40 * 1024) {                                                                                                       \
+            cudaError_t e = cudaFuncSetAttribute(route_kernel<T, NT, EP, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                                      \
+        }                                                                                                                             \
+        route_kernel<T, NT, EP, WARPS><<<blocks, WARPS * 32, smem, stream>>>((const T*)x, w_router, bias, ids, weights, counts, n_tokens, d, \
+                                                                            n_all, n_real, top, renormalize, sigmoid_scores, all_scores, \
+                                                                            groups, keep, weight_scale);                              \
+    } while (0)
+#define LAUNCH_T(T)                                \
+    do {                                           \
+        if (nt == 8) LAUNCH(T, 8, 2, 8);           \
+        else if (nt == 4) LAUNCH(T, 4, 2, 8);      \
+        else LAUNCH(T, 1, 1, 16);                  \
+    } while (0)
+    if (dtype == NI_DTYPE_F32) LAUNCH_T(float);
+    else if (dtype == NI_DTYPE_BF16) LAUNCH_T(__nv_bfloat16);
+    else return NI_ERR_BAD_ARGUMENT;
+#undef LAUNCH_T
+#undef LAUNCH
     NI_RETURN_LAUNCH_STATUS();
 }
 

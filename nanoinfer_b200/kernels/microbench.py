@@ -18,6 +18,10 @@
     python -m nanoinfer_b200.kernels.microbench lightning --batch 1 --tokens 2048 --heads 8 --dim 128 --vdim 128 --retention
     python -m nanoinfer_b200.kernels.microbench qk_norm_rope --batch 1 --tokens 2048 --heads 16 --kv-heads 8 --dim 128 --head-unit
     python -m nanoinfer_b200.kernels.microbench capped_unit --rows 2048 --ff 8192 --width 2048
+    python -m nanoinfer_b200.kernels.microbench mlstm --batch 1 --tokens 2048 --heads 16 --dim 128 --vdim 128
+    python -m nanoinfer_b200.kernels.microbench hyper --rows 2048 --width 2048 --streams 4 --top 4
+    python -m nanoinfer_b200.kernels.microbench attention_prefill --tokens 2048 --q-heads 16 --head-dim 128 --difference
+    python -m nanoinfer_b200.kernels.microbench attention_decode --batch 8 --context 2048 --q-heads 16 --head-dim 128 --difference
 
 Each case runs its kernel over several distinct copies of its inputs in turn (together
 larger than the L2 cache, so every run reads from HBM), times it with CUDA events after
@@ -207,7 +211,13 @@ def attention_decode(args) -> None:
         positions = (torch.linspace(ctx // 4, ctx, b, device=DEV).int() - 1).contiguous()
         kv_bytes = int(2 * (positions.long() + 1).sum().item() * hkv * hd * 2)
         splits = args.splits or ops.decode_splits(b, hkv, hd, ctx)
-    if args.balanced:
+    if args.difference:      # --q-heads heads of two maps each
+        splits = args.splits or ops.decode_splits(b, hkv, hd, ctx)
+        scratch = torch.empty(b * 2 * hq * splits * (hd + 2), dtype=torch.float32, device=DEV)
+        fns = [lambda kc=kc, vc=vc: ops.attention_decode_difference(q, kc, vc, out, None, b, positions, seq_of, table, hq, hkv, hd,
+                                                                    page, 1.0 / math.sqrt(hd // 2), 0.4, 1e-6, 0.6, splits, scratch, tickets)
+               for kc, vc in caches]
+    elif args.balanced:
         scratch = torch.empty(ops.attention_decode_balanced_scratch(hq, hkv, hd), dtype=torch.float32, device=DEV)
         fns = [lambda kc=kc, vc=vc: ops.attention_decode_balanced(q, kc, vc, out, None, b, positions, seq_of, table, hq, hkv,
                                                                   hd, page, None, 1.0 / math.sqrt(hd), scratch, tickets)
@@ -221,7 +231,7 @@ def attention_decode(args) -> None:
     us = _time(fns, args.iters)
     if args.chunk:           # only the keys of the last token's own chunk are read
         kv_bytes = kv_bytes * ((ctx - 1) % args.chunk + 1) // ctx
-    print(f"attention_decode{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''}{' (merge through scratch)' if args.scratch_merge else ''}{' (balanced)' if args.balanced else ''}{' ragged' if args.ragged else ''} batch={b} context={ctx} heads={hq}/{hkv} hd={hd} page={page} splits={splits}: "
+    print(f"attention_decode{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''}{' (merge through scratch)' if args.scratch_merge else ''}{' (balanced)' if args.balanced else ''}{' ragged' if args.ragged else ''} batch={b} context={ctx} heads={hq}/{hkv} hd={hd} page={page} splits={splits}: "
           f"{us:.2f} us, {kv_bytes / us / 1e3:.0f} GB/s of cache")
 
 
@@ -242,11 +252,14 @@ def attention_prefill(args) -> None:
     fn = lambda: ops.attention_prefill(q, kc, vc, out, tile_seq, tile_row0, len(tiles), cu_q, kv_len, table, hq, hkv,
                                        hd, page, None, 1.0 / math.sqrt(hd), kernel=args.kernel, score_cap=args.score_cap,
                                        chunk=args.chunk, sink=args.sink)
+    if args.difference:      # --q-heads heads of two maps each
+        fn = lambda: ops.attention_prefill_difference(q, kc, vc, out, tile_seq, tile_row0, len(tiles), cu_q, kv_len, table, hq, hkv, hd,
+                                                      page, 1.0 / math.sqrt(hd // 2), 0.4, 1e-6, 0.6)
     us = _time([fn], args.iters)
     ops.check_device_errors()
     seen = sum(p % args.chunk + 1 for p in range(t)) if args.chunk else t * (t + 1) / 2       # (query, key) pairs inside the mask
-    flops = 4.0 * hq * hd * seen
-    print(f"attention_prefill{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''} tokens={t} "
+    flops = (6.0 if args.difference else 4.0) * hq * hd * seen      # two maps: half-wide keys twice, the values twice
+    print(f"attention_prefill{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''} tokens={t} "
           f"heads={hq}/{hkv} hd={hd} kernel={args.kernel or 'default'}: {us:.1f} us, {flops / us / 1e6:.0f} TFLOP/s (of the pairs inside the mask)")
 
 
@@ -540,6 +553,61 @@ def capped_unit(args) -> None:
           f"normed addition with bias and bfloat16 copy {us_add:.2f} us ({n * d * 14 / us_add / 1e3:.0f} GB/s)")
 
 
+def mlstm(args) -> None:
+    """A matrix memory's kernels at --batch requests of --tokens tokens each, norm per head and gate included; states of
+    several request sets are used in turn, so that single-token steps read theirs from HBM."""
+    b, t, H, D, V = args.batch, args.tokens, args.heads, args.dim, args.vdim
+    n, bf = b * t, torch.bfloat16
+    floats = ops.mlstm_state_floats(H, D, V)
+    g = torch.Generator(device=DEV).manual_seed(0)
+    states = [torch.randn(b, floats, device=DEV, generator=g) * 0.1
+              for _ in range(max(2, min(32, -(-2 * L2_BYTES // (b * floats * 4)))) if t == 1 else 2)]
+    wide = 2 * H * (D + V)
+    z = torch.randn(n, 2 * H, device=DEV, generator=g)
+    z[:, H:] += 4.0
+    zero, w = torch.zeros(H, device=DEV), torch.ones(H * V, device=DEV)
+    cu = torch.arange(0, n + 1, t, dtype=torch.int32, device=DEV)
+    slots = torch.arange(b, dtype=torch.int32, device=DEV)
+    y = torch.empty(n, H * V, dtype=bf, device=DEV)
+    proj = torch.randn(n, wide, device=DEV, generator=g) * 0.5
+    if t == 1:
+        us = _time([lambda st=st: ops.mlstm_token_step(proj, z, 0, H, zero, zero, 15.0, st, cu, slots, b, D ** -0.5, w, 1e-6, y, H, D, V)
+                    for st in states], args.iters)
+    else:
+        proj, out = proj.to(bf), torch.empty(n, H * V, device=DEV)
+        buf = torch.empty(ops.mlstm_buffer_floats(n, b, H, D, V), device=DEV)
+        us = _time([lambda st=st: ops.mlstm_chunk_step(proj, z, 0, H, zero, zero, 15.0, st, cu, slots, b, t, D ** -0.5, w, 1e-6, buf,
+                                                       out, y, H, D, V) for st in states], args.iters)
+    print(f"mlstm batch={b} tokens={t} heads={H} dim={D} vdim={V}: {us:.2f} us ({2 * b * floats * 4 / us / 1e3:.0f} GB/s of state, "
+          f"{4.0 * n * H * D * V / us / 1e6:.2f} TFLOP/s of the recurrence's own work)")
+
+
+def hyper(args) -> None:
+    """One pass over --streams residual streams: the pending update (a plain output, or --top rows of routed experts
+    per token), the streams written back, the weighted sum through the norm without statistics."""
+    n, d, s, top = args.rows, args.width, args.streams, args.top
+    bf = torch.bfloat16
+    g = torch.Generator(device=DEV).manual_seed(0)
+    copies = max(2, min(32, -(-2 * L2_BYTES // (n * s * d * 4))))
+    xs = [torch.randn(n, s, d, device=DEV, generator=g) for _ in range(copies)]
+    mix, out, coef = torch.eye(s, device=DEV), torch.ones(s, device=DEV), torch.ones(s, device=DEV)
+    norm = (torch.ones(1, device=DEV), torch.ones(d, device=DEV), torch.zeros(d, device=DEV))
+    h = torch.empty(n, d, dtype=bf, device=DEV)
+    ys = [torch.randn(n, d, device=DEV, generator=g) for _ in range(copies)]
+    us = _time([lambda x=x, y=y: ops.hyper_step(x, None, s, (y, mix, out), coef, norm, h, None, True) for x, y in zip(xs, ys)], args.iters)
+    nbytes = n * d * (8 * s + 4 + 2)
+    print(f"hyper rows={n} width={d} streams={s}: {us:.2f} us, {nbytes / us / 1e3:.0f} GB/s")
+    if top:
+        zs = [torch.randn(n * top, d, device=DEV, generator=g).to(bf) for _ in range(copies)]
+        ids = torch.zeros(n, top, dtype=torch.int32, device=DEV)
+        wts = torch.full((n, top), 0.25, device=DEV)
+        rows = torch.randperm(n * top, device=DEV, generator=g).int()
+        us = _time([lambda x=x, z=z: ops.hyper_step(x, None, s, (ops.RoutedRows(z, ids, wts, rows), mix, out), coef, norm, h, None, True)
+                    for x, z in zip(xs, zs)], args.iters)
+        nbytes = n * d * (8 * s + 2 * top + 2)
+        print(f"hyper with {top} routed rows per token: {us:.2f} us, {nbytes / us / 1e3:.0f} GB/s")
+
+
 def routed(args) -> None:
     """The routed feed-forward at --tokens rows: the router, then the whole part (all its launches, its output normed
     and added into an FP32 stream as a sandwich layer asks for it), in bfloat16."""
@@ -681,6 +749,7 @@ def main() -> None:
         p.add_argument("--score-cap", type=float, default=0.0, help="bound the scaled scores by cap * tanh(s / cap)")
         p.add_argument("--chunk", type=int, default=0, help="a token sees only the keys of its own chunk of this many positions")
         p.add_argument("--sink", action="store_true", help="one is added to the softmax's denominator")
+        p.add_argument("--difference", action="store_true", help="differential attention: two maps of half the head size per query head")
         p.add_argument("--copies", type=int, default=0, help="decode: cache copies used in turn (default: enough to exceed L2; 1: the cache stays in L2)")
         p.add_argument("--balanced", action="store_true", help="decode: the kernel that deals the keys evenly over a fixed grid")
         p.add_argument("--ragged", action="store_true", help="decode: contexts from a quarter of --context up to it")
@@ -733,6 +802,19 @@ def main() -> None:
     p.add_argument("--plain-add", action="store_true", help="the output is added into the stream without a norm")
     p.add_argument("--flat-router", action="store_true", help="router weights so small that the choice bias decides (all tokens choose alike)")
     p.set_defaults(fn=routed)
+    p = sub.add_parser("mlstm")
+    p.add_argument("--batch", type=int, default=1)
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--dim", type=int, default=128)
+    p.add_argument("--vdim", type=int, default=128)
+    p.set_defaults(fn=mlstm)
+    p = sub.add_parser("hyper")
+    p.add_argument("--rows", type=int, default=2048)
+    p.add_argument("--width", type=int, default=2048)
+    p.add_argument("--streams", type=int, default=4)
+    p.add_argument("--top", type=int, default=4)
+    p.set_defaults(fn=hyper)
     for sp in sub.choices.values():
         sp.add_argument("--iters", type=int, default=200)
     args = ap.parse_args()

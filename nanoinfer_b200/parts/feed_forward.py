@@ -342,13 +342,12 @@ class RoutedExperts(Part):
                 raise ConfigError("routed experts: the shared unit's limit must be positive")
             self.w_shared_gate_up = rt.weight(torch.cat([weights["shared.gate"], weights["shared.up"]], dim=0))
             self.w_shared_down = rt.weight(weights["shared.down"])
+        # forward accepts leave_rows=True and hands the chosen experts' rows over (a hook for arrangements that sum them)
+        self.leaves_rows = n_real == self.n_all and self.shared_inter <= 0 and not self.weight_on_input
 
     def weights_in_order(self) -> tuple:
         routed = (self.w_gate_up, self.w_down) if self.n_real > 0 else ()
         return routed + ((self.w_shared_gate_up, self.w_shared_down) if self.shared_inter > 0 else ())
-
-        # forward accepts leave_rows=True and hands the chosen experts' rows over (a hook for arrangements that sum them)
-        self.leaves_rows = n_real == self.n_all and self.shared_inter <= 0 and not self.weight_on_input
 
     adds_normed = True          # forward accepts normed_into=(h, gain, eps): h += RMSNorm(output) * gain, returns None
 
