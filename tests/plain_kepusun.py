@@ -36,9 +36,14 @@ def capped(z, cap):
     return cap * torch.tanh(z / cap)
 
 
+def value_size(m):
+    """The size of a value: that of a key unless the mixer says otherwise."""
+    return m["dim"] if m.get("vdim") is None else m["vdim"]
+
+
 def fresh_memory(m):
     """[matrix [dim, vdim], normaliser [dim], running maximum] per head, all zero."""
-    return [[torch.zeros(m["dim"], m["vdim"], dtype=F64), torch.zeros(m["dim"], dtype=F64), torch.zeros((), dtype=F64)]
+    return [[torch.zeros(m["dim"], value_size(m), dtype=F64), torch.zeros(m["dim"], dtype=F64), torch.zeros((), dtype=F64)]
             for _ in range(m["heads"])]
 
 
@@ -57,7 +62,7 @@ def memory_step(mem, q, k, v, i_log, f_log):
 def memory_mixer(w, pre, m, h, mem, eps):
     """The matrix-memory mixer: exponential input gate, sigmoid forget gate, both logs capped; a norm per head, a
     weight over all heads, a sigmoid gate."""
-    H, D, V, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
+    H, D, V, cap = m["heads"], m["dim"], value_size(m), m["gate_cap"]
     q, k, v = (w[pre + "q"] @ h).view(H, D) * D ** -0.5, (w[pre + "k"] @ h).view(H, D), (w[pre + "v"] @ h).view(H, V)
     i_log = capped(w[pre + "i"] @ h + w[pre + "i.b"], cap)
     f_log = torch.nn.functional.logsigmoid(capped(w[pre + "f"] @ h + w[pre + "f.b"], cap))
@@ -79,7 +84,8 @@ def difference_attention(w, pre, m, h, cache, eps, own):
     """Two attention maps per head over the same values, the second taken off the first; the rest to unit root mean
     square, times 1 - diff.  ``cache`` is the list of (keys [G, 2, dim], values [G, vdim]) of the tokens so far; a
     layer with projections of its own (``own``) appends this token's."""
-    H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    H, D, V = m["heads"], m["dim"], value_size(m)
+    G = H if m.get("kv_heads") is None else m["kv_heads"]
     q = (w[pre + "q"] @ h).view(H, 2, D)
     if own:
         cache.append(((w[pre + "k"] @ h).view(G, 2, D), (w[pre + "v"] @ h).view(G, V)))
