@@ -234,11 +234,7 @@ mlstm_chunk_kv_tc_kernel(const __nv_bfloat16* __restrict__ proj, int ld, const M
     const int gq = lane >> 2, tq = lane & 3, blk = lane >> 3, rr = lane & 7;
     const int k_steps = (n + 15) / 16;
     float* out = sums + ((size_t)c.index * H + head) * ml_record(D, V);
-    for (int d = tid; d < D; d += LT_THREADS) {
-        float s = 0.f;
-        for (int j = 0; j < n; ++j) s += __bfloat162float(Khi[j * KS + d]) + __bfloat162float(Klo[j * KS + d]);
-        out[(size_t)D * V + d] = s;
-    }
+    const uint32_t ones = 0x3f803f80u;                     // two bfloat16 ones: the normaliser is a product with a column of them
     for (int mt = warp; mt < D / 16; mt += LT_THREADS / 32) {
         const int d0 = mt * 16;
         for (int vb = 0; vb < V; vb += 64) {
@@ -248,12 +244,17 @@ mlstm_chunk_kv_tc_kernel(const __nv_bfloat16* __restrict__ proj, int ld, const M
             for (int a = 0; a < 8; ++a)
 #pragma unroll
                 for (int b = 0; b < 4; ++b) acc[a][b] = 0.f;
+            float accn[4] = {0.f, 0.f, 0.f, 0.f};
             for (int kt = 0; kt < k_steps; ++kt) {
                 const int j0 = kt * 16;
                 uint32_t ahi[4], alo[4];
                 const int a_off = (j0 + (blk >> 1) * 8 + rr) * KS + d0 + (blk & 1) * 8;
                 lt_ldsm_x4_trans(ahi, Khi + a_off);
                 lt_ldsm_x4_trans(alo, Klo + a_off);
+                if (vb == 0) {
+                    lt_mma(accn, ahi, ones, ones);
+                    lt_mma(accn, alo, ones, ones);
+                }
                 const __nv_bfloat16* vp = Vs + (j0 + (blk & 1) * 8 + rr) * VS + vb + (blk >> 1) * 8;
 #pragma unroll
                 for (int np = 0; np < 4; ++np) {
@@ -266,6 +267,10 @@ mlstm_chunk_kv_tc_kernel(const __nv_bfloat16* __restrict__ proj, int ld, const M
                         lt_mma(acc[2 * np + 1], alo, b[2], b[3]);
                     }
                 }
+            }
+            if (vb == 0 && tq == 0) {
+                out[(size_t)D * V + d0 + gq] = accn[0];
+                out[(size_t)D * V + d0 + gq + 8] = accn[2];
             }
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {

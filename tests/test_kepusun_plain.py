@@ -35,7 +35,7 @@ def test_parser_reads_every_size_and_constant():
     assert a.feed_forward.extra_dict()["groups"] == 1
     assert b.feed_forward is None and b.ffn_norm is None and not b.mixer.extra_dict()["own_kv"]
     assert [r.cache_of for r in cfg.schedule] == [None, None, 1, None]
-    assert [r.cache_of for r in config_from_dict(tk.U4).schedule] == [None, None, 0, None, 0]
+    assert [r.cache_of for r in config_from_dict(tk.U4).schedule] == [None, None, 0, None, 0, None]
     third = config_from_dict(tk.U3).layers
     assert third[2].mixer.extra_dict()["value_dim"] == 8 and third[3].mixer.num_kv_heads == 3
 

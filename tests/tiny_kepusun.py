@@ -8,7 +8,7 @@ U2 has sizes the tensor-core kernels take (maps of 64 over values of 128, maps o
 64 x 128 and 32 x 32), four streams.
 U3 has values that are 1 or absent elsewhere: one stream, one head, one key head per query head, one expert, one chosen
 expert, a weight factor of 1, as many groups as experts, all groups kept, keys and values whose size is not said.
-U4 has sizes that are no multiple of 8 anywhere, five streams, memories larger than a warp's rows, and two layers that
+U4 has sizes that are no multiple of 8 anywhere, five streams, a memory with more rows than columns, and two layers that
 read the same layer's keys and values.
 """
 import json
@@ -60,7 +60,8 @@ U4 = model(173, 76, 5, [attention(3, 1, 18, 11, 0.33, 0.25, moe(9, 4, 12, 1.1, (
                         memory(5, 9, 37, 7.0, moe(3, 3, 20, 0.9)),
                         attention(5, 1, 18, 11, 0.27, 0.5, moe(6, 2, 28, 1.3, (2, 1)), kv_from=0),
                         memory(1, 70, 5, 12.0, None),
-                        attention(1, 1, 18, 11, 0.4, 0.1, moe(4, 2, 12, 1.0), kv_from=0)])
+                        attention(1, 1, 18, 11, 0.4, 0.1, moe(4, 2, 12, 1.0), kv_from=0),
+                        attention(2, 1, 9, 18, 0.3, 0.3, None)])
 
 # Standard deviations (by the last part of a tensor's slot) that make every mechanism matter in a random model without
 # making it chaotic: matrices (relative to one over the root of what they sum over) whose results are of order one, gates
