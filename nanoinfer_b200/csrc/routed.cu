@@ -468,12 +468,12 @@ NI_EXPORT int ni_route(const void* x, int dtype, const float* w_router, const fl
     if (n_all > RT_MAX_EXPERTS) return NI_ERR_UNSUPPORTED_SIZE;
     if (d > 12000) return NI_ERR_UNSUPPORTED_SIZE;                    // the row lies in shared memory as FP32
     // many tokens: as many to a block as fit twice into an SM's shared memory
-    const int nt = n_tokens < 512 ? 1 : (d <= 3072 ? 8 : (d <= 6144 ? 4 : 1));
+    const int nt = n_tokens < 512 ? 1 : (d <= 2560 ? 8 : (d <= 5632 ? 4 : 1));
     const size_t smem = (size_t)nt * d * sizeof(float);
     const int blocks = (n_tokens + nt - 1) / nt;
 #define LAUNCH(T, NT, EP, WARPS)                                                                                                      \
     do {                                                                                                                              \
-        if (smem > 40 * 1024) {                                                                                                       \
+        if (smem + (NT) * 3 * RT_MAX_EXPERTS * sizeof(float) > 48 * 1024) {  /* beside the kernel's own arrays */                                                                                                      \
             cudaError_t e = cudaFuncSetAttribute(route_kernel<T, NT, EP, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                                      \
         }                                                                                                                             \

@@ -395,6 +395,29 @@ def test_router_with_groups(dtype, E, top, groups, keep, scale, n):
     assert same >= n - max(1 if top > 8 else 0, n // 50)
 
 
+@pytest.mark.parametrize("d", [1024, 1026, 2560, 2568, 5640, 12000])
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_router_at_other_widths(dtype, d):
+    """Many tokens at widths that put eight, four and one of them into a block: the same choices and, bit for bit, the same
+    weights as a few tokens at a time."""
+    from nanoinfer_b200.kernels import ops
+    g = torch.Generator().manual_seed(d)
+    n, E, top = 530, 17, 3
+    x, w = _rand(g, n, d).to(dtype).to(DEV), _rand(g, E, d, scale=2.0 * d ** -0.5).to(DEV)
+
+    def run(rows):
+        ids, wts = torch.empty(rows.shape[0], top, **I32), torch.empty(rows.shape[0], top, device=DEV)
+        ops.route(rows, w, None, ids, wts, None, E, top, renormalize=True)
+        return ids, wts
+
+    many = run(x)
+    few = [run(x[a:a + 53].contiguous()) for a in range(0, n, 53)]
+    assert torch.equal(many[0], torch.cat([f[0] for f in few])) and torch.equal(many[1], torch.cat([f[1] for f in few]))
+    z = x.double() @ w.double().T
+    want = torch.topk(torch.softmax(z, 1), top).values
+    torch.testing.assert_close(many[1].double(), want / want.sum(1, keepdim=True), rtol=2e-4, atol=1e-6)
+
+
 @pytest.mark.parametrize("E, top, F, d", [(12, 3, 96, 128), (8, 2, 40, 96), (6, 4, 20, 76), (1, 1, 16, 64)])
 @pytest.mark.parametrize("n", [1, 4, 8, 20, 90])
 @pytest.mark.parametrize("dtype", DTYPES)
