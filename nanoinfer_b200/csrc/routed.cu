@@ -45,7 +45,20 @@ route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
     const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * NT, rows = min(NT, n_tokens - t0);
     const T* xr = x + (size_t)t0 * d;
-    for (int k = threadIdx.x; k < NT * d; k += blockDim.x) xs[k] = k < rows * d ? ni_to_float(xr[k]) : 0.f;
+    if (d % 8 == 0 && (reinterpret_cast<size_t>(x) & 15) == 0) {        // 16 bytes per load, four of them under way
+        constexpr int V = NiVec16<T>::N;
+#pragma unroll 4
+        for (int k = threadIdx.x * V; k < NT * d; k += WARPS * 32 * V) {
+            float v[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = 0.f;
+            if (k < rows * d) NiVec16<T>::load(xr + k, v);
+#pragma unroll
+            for (int i = 0; i < V; i += 4) NiVec16<float>::store(xs + k + i, v + i);
+        }
+    } else {
+        for (int k = threadIdx.x; k < NT * d; k += blockDim.x) xs[k] = k < rows * d ? ni_to_float(xr[k]) : 0.f;
+    }
     __syncthreads();
     for (int e0 = w * EP; e0 < n_all; e0 += WARPS * EP) {
         const float* wr[EP];
@@ -57,7 +70,7 @@ route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
             for (int j = 0; j < NT; ++j) acc[i][j] = 0.f;
         }
         if ((d & 3) == 0) {
-#pragma unroll (NT == 1 ? 8 : 2)
+#pragma unroll (NT == 1 ? 8 : 4)
             for (int k = lane; k < (d >> 2); k += 32) {
                 float4 b[EP];
 #pragma unroll
