@@ -3,8 +3,8 @@
 //   route     z = W_router x, s = softmax(z) over all experts - or s = sigmoid(z), each expert on its own -, all FP32;
 //             the `top` experts with the largest s + bias are chosen (ties: the lower index), their weights are s
 //             (optionally divided by their sum + 1e-20), times a factor.  Experts numbered n_real and above are identity
-//             experts: their output is x itself.  With groups > 1 the experts form that many equal groups of neighbours, a
-//             group counts as much as its best expert, and only experts of the best `keep` groups can be chosen.
+//             experts: their output is x itself.  With groups > 1 the experts, in their order, are split into that many
+//             groups of one size; groups are ranked by their best expert, and all but the first `keep` drop out.
 //   unit      an expert is W_down act(W_gate x, W_up x) with act(g, u) = g' * sigmoid(slope * g') * (u' + shift),
 //             g' = min(r g, limit), u' = clamp(r u, -limit, limit): limit = infinity, slope = 1, shift = 0, r = 1 is
 //             silu(g) * u; r is a number per row - the token's weight where a design multiplies the expert's INPUT by

@@ -994,9 +994,9 @@ def route(x, w_router, bias, ids, weights, counts, n_real, top, renormalize=Fals
     (float32; w_router float32 [E, d]); ``all_scores`` float32 [T, n_real] (or None) receives every real expert's score;
     the ``top`` experts with the
     largest score + bias (``bias`` float32 [E] or None) -> ids int32 [T, top], their scores -> weights float32
-    [T, top] (divided by their sum if ``renormalize``, then times ``weight_scale``).  ``groups`` > 1: the experts form that
-    many equal groups of neighbours, and only experts of the ``keep_groups`` groups with the best single experts can be
-    chosen.  ``counts`` int32 [n_real] (or None) receives how many
+    [T, top] (divided by their sum if ``renormalize``, then times ``weight_scale``).  ``groups`` > 1: the experts, in
+    their order, are split into that many groups of one size, ranked by their best expert, and all but the first
+    ``keep_groups`` drop out.  ``counts`` int32 [n_real] (or None) receives how many
     tokens chose each of the first ``n_real`` experts (added to what it holds)."""
     n, d = x.shape
     e = w_router.shape[0]

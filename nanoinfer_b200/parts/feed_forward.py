@@ -252,9 +252,8 @@ class RoutedExperts(Part):
     shift) that every token runs on its plain input; its output is added.
 
     ``unit`` "relu2" instead of the default "gated": an expert is W_down relu(W_up x)^2, with no gate.  ``weight_scale``
-    multiplies the weights (after the division by their sum, if any).  ``groups`` = n > 1: the experts form n equal groups
-    of neighbours, a group counts as much as its best expert, and only experts of the ``keep_groups`` best groups can be
-    chosen.  With ``leave_rows`` forward hands the chosen experts' rows over unsummed (ops.RoutedRows), for an
+    multiplies the weights (after the division by their sum, if any).  ``groups`` = n > 1: the experts, in their order, are
+    split into n groups of one size, ranked by their best expert, and all but the first ``keep_groups`` drop out.  With ``leave_rows`` forward hands the chosen experts' rows over unsummed (ops.RoutedRows), for an
     arrangement whose next kernel sums them on its way (no identity experts, no shared unit).
 
     The experts' matrices are stacked ([E, 2F, d] gate rows then up rows, and [E, d, F]).  In bfloat16, steps of a

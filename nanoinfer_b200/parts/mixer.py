@@ -624,7 +624,7 @@ class DifferentialAttention(PagedAttendMixin, Part):
 
         q = W_q x  [H, 2, D],  k = W_k x  [G, 2, D],  v = W_v x  [G, V]        (head by head: map 1, map 2; no positions)
         a_m = softmax over the earlier keys of (q_m . k_m softmax_scale), times v          for each map m
-        lambda = exp(sum lq1 lk1) - exp(sum lq2 lk2) + ``diff``                            one number for the layer
+        lambda = exp(sum lq1 lk1) - exp(sum lq2 lk2) + ``diff``                            the same for every head
         o = a_1 - lambda a_2;   o / sqrt(mean(o^2) + ``norm_eps``) * (1 - diff) per head;  then W_o on the heads side by side
 
     ``own_kv`` false in the extra: no W_k and W_v; the layer reads the pages of the run whose cache it shares
