@@ -108,8 +108,9 @@ __device__ __forceinline__ void dec_warm(const unsigned char* p, unsigned long l
 // every split writes its partial result into the shared memory of the cluster's first block, one
 // cluster barrier, and that block merges them in split order - no scratch in global memory, no
 // fence, no ticket.
-// chunk > 0: the token at position p sees only the keys from p - p % chunk on; flags bit 0 (sink): one is added to the
-// softmax's denominator; flags >> 1 = n > 1: n neighbouring kv heads of the launch read one head of the pages.
+// chunk > 0: the token at position p sees only the keys from p - p % chunk on; sinks (a number per query head; null:
+// none): exp(sinks[head]) is added to the softmax's denominator; share = n > 1: n neighbouring kv heads of the launch read
+// one head of the pages (0 or 1: each has its own).
 // DIFF (differential attention): a query head has two maps, which are two rows of the tile; a query row has HD / 2 numbers
 // and stands in the half of the tile's row that its map's keys stand in (a key row holds both maps side by side), zeros in
 // the other half.  The result of a head is u = a_0 - lambda a_1 of its two rows, u / sqrt(mean(u^2) + eps) * factor.
@@ -127,12 +128,10 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                         int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                         float scale_log2e, float cap_l2, int n_splits, float* __restrict__ scratch,
                         int* __restrict__ tickets, const unsigned char* __restrict__ warm_a, unsigned long long warm_a_bytes,
-                        const unsigned char* __restrict__ warm_b, unsigned long long warm_b_bytes, int chunk, int flags,
-                        const DecDiff diff) {
-    // flags: bit 0 - the sink; the rest - how many of the launch's kv heads share one head of the pages (0: each has its
-    // own): more than 16 query rows over one page head are dealt over several "kv heads" of at most 16 rows each
-    const int sink = flags & 1;
-    const int share = flags >> 1 > 1 ? flags >> 1 : 1;
+                        const unsigned char* __restrict__ warm_b, unsigned long long warm_b_bytes, int chunk,
+                        const float* __restrict__ sinks, int share_heads, const DecDiff diff) {
+    // more than 16 query rows over one page head are dealt over several "kv heads" of at most 16 rows each
+    const int share = share_heads > 1 ? share_heads : 1;
     // Weights that the kernels after this one will read (the caller's hint, up to two regions): asked
     // into L2 now, in pieces dealt over the blocks, while this kernel - which waits on latencies
     // more than on bandwidth - leaves the memory system room.  Nothing here depends on the kernel before.
@@ -173,10 +172,11 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
 #pragma unroll
     for (int j = 0; j < NT_O; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;   // rows g and g + 8
-    if (sink && split == 0 && warp == 0) {
-        // one more term in every row's denominator: a key of score 0 without a value, counted once - by the first
-        // warp of the first split (which always has the token's own key), in one lane of each row's four
-        m0 = m1 = 0.f;
+    if (sinks && split == 0 && warp == 0) {
+        // one more term in every row's denominator: a key without a value, counted once - by the first warp of the first
+        // split (which always has a key), in one lane of each row's four
+        m0 = g < G ? sinks[kvh * G + g] * 1.4426950408889634f : 0.f;
+        m1 = g + 8 < G ? sinks[kvh * G + g + 8] * 1.4426950408889634f : 0.f;
         if (t == 0) l0 = l1 = 1.f;
     }
     uint32_t qa[KS][4];
@@ -874,7 +874,7 @@ static int launch_decode_cl(const void* q, const void* k_pages, const void* v_pa
                          int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                          float scale_log2e, float cap_l2, int n_splits, float* scratch, int* tickets, const void* warm_a,
                          unsigned long long warm_a_bytes, const void* warm_b, unsigned long long warm_b_bytes,
-                         int chunk, int flags, const DecDiff& diff, cudaStream_t stream) {
+                         int chunk, const float* sinks, int share, const DecDiff& diff, cudaStream_t stream) {
     const size_t kv_smem = (size_t)(16 + 4 * SEG) * HD * sizeof(__nv_bfloat16);
     const size_t smem = kv_smem + (CL ? (size_t)n_splits * (n_q_heads / n_kv_heads) * (HD + 2) * sizeof(float) : 0);
     static size_t configured = 0;
@@ -911,7 +911,7 @@ static int launch_decode_cl(const void* q, const void* k_pages, const void* v_pa
                                        (__nv_bfloat16*)out, token_list, positions, seq_of_token, block_table,
                                        bt_stride, n_q_heads, n_kv_heads, page_size, window, scale_log2e, cap_l2, n_splits,
                                        scratch, tickets, (const unsigned char*)warm_a, warm_a_bytes,
-                                       (const unsigned char*)warm_b, warm_b_bytes, chunk, flags, diff);
+                                       (const unsigned char*)warm_b, warm_b_bytes, chunk, sinks, share, diff);
     return e == cudaSuccess ? NI_OK : (int)e;
 }
 
@@ -929,7 +929,7 @@ static int launch_decode(const void* q, const void* k_pages, const void* v_pages
                          int bt_stride, int n_q_heads, int n_kv_heads, int page_size, int window,
                          float scale_log2e, float cap_l2, int n_splits, float* scratch, int* tickets, const void* warm_a,
                          unsigned long long warm_a_bytes, const void* warm_b, unsigned long long warm_b_bytes,
-                         int chunk, int flags, const DecDiff* diff, cudaStream_t stream) {
+                         int chunk, const float* sinks, int share, const DecDiff* diff, cudaStream_t stream) {
     const DecDiff none = {0.f, 0.f, 0.f};
     const size_t slot_bytes = (size_t)n_splits * (n_q_heads / n_kv_heads) * (HD + 2) * sizeof(float);
     const bool few_blocks = (long long)n_items * n_kv_heads * n_splits <= 2LL * ni_sm_count() && slot_bytes <= 65536;
@@ -938,7 +938,7 @@ static int launch_decode(const void* q, const void* k_pages, const void* v_pages
     launch_decode_cl<HD, SEG, CL, CAP, DIFF>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,    \
                                              block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,          \
                                              scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, warm_a_bytes,     \
-                                             warm_b, warm_b_bytes, chunk, flags, diff ? *diff : none, stream)
+                                             warm_b, warm_b_bytes, chunk, sinks, share, diff ? *diff : none, stream)
         return diff ? NI_DEC_GO(true, false, true) : (cap_l2 > 0.f ? NI_DEC_GO(true, true, false) : NI_DEC_GO(true, false, false));
     return diff ? NI_DEC_GO(false, false, true) : (cap_l2 > 0.f ? NI_DEC_GO(false, true, false) : NI_DEC_GO(false, false, false));
 #undef NI_DEC_GO
@@ -954,9 +954,10 @@ static int decode_dispatch(const void* q, const void* k_pages, const void* v_pag
                                   int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                   float scale, float score_cap, int n_splits, float* scratch, int* tickets,
                                   const void* warm_a, long long warm_a_bytes, const void* warm_b,
-                                  long long warm_b_bytes, int chunk, int flags, const DecDiff* diff, cudaStream_t stream) {
+                                  long long warm_b_bytes, int chunk, const float* sinks, int share, const DecDiff* diff,
+                                  cudaStream_t stream) {
     if (n_items <= 0) return NI_OK;
-    if (chunk < 0 || (flags >> 1 > 1 && n_kv_heads % (flags >> 1))) return NI_ERR_BAD_ARGUMENT;
+    if (chunk < 0 || (share > 1 && n_kv_heads % share)) return NI_ERR_BAD_ARGUMENT;
     if (warm_a_bytes < 0 || (warm_a_bytes & 15) || (warm_a_bytes && (!warm_a || ((uintptr_t)warm_a & 15)))) return NI_ERR_BAD_ARGUMENT;
     if (warm_b_bytes < 0 || (warm_b_bytes & 15) || (warm_b_bytes && (!warm_b || ((uintptr_t)warm_b & 15)))) return NI_ERR_BAD_ARGUMENT;
     if (n_q_heads <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads || page_size <= 0 || n_splits <= 0 ||
@@ -975,16 +976,16 @@ static int decode_dispatch(const void* q, const void* k_pages, const void* v_pag
                 return launch_decode<64, 128>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                               block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                               scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, sinks, share, diff, stream);
             return launch_decode<64, 64>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                           block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                           scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, sinks, share, diff, stream);
         case 128:
             return launch_decode<128, 64>(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token,
                                            block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window,
                                            scale_log2e, cap_l2, n_splits, scratch, tickets, warm_a, (unsigned long long)warm_a_bytes, warm_b,
-                                              (unsigned long long)warm_b_bytes, chunk, flags, diff, stream);
+                                              (unsigned long long)warm_b_bytes, chunk, sinks, share, diff, stream);
         default: return NI_ERR_UNSUPPORTED_SIZE;
     }
 }
@@ -998,24 +999,24 @@ NI_EXPORT int ni_attention_decode(const void* q, const void* k_pages, const void
                                   long long warm_b_bytes, cudaStream_t stream) {
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, 0.f, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, nullptr, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, nullptr, 0, nullptr, stream);
 }
 
-// The same with a chunk mask (chunk > 0: the token at position p sees only the keys from p - p % chunk on) and flags:
-// bit 0 - one is added to the softmax's denominator (a sink); flags >> 1 = n > 1 - n neighbouring kv heads of the call read
-// one head of k_pages / v_pages ([P, n_kv_heads / n, page_size, hd]), so that more than 16 query heads over one page head
+// The same with a chunk mask (chunk > 0: the token at position p sees only the keys from p - p % chunk on), sinks (FP32, one
+// per query head, or null: exp(sinks[head]) is added to the softmax's denominator) and share = n > 1: n neighbouring kv heads
+// of the call read one head of k_pages / v_pages ([P, n_kv_heads / n, page_size, hd]), so that more than 16 query heads over one page head
 // can be dealt over several groups of at most 16.  score_cap 0: scores are not bounded.
 NI_EXPORT int ni_attention_decode_masked(const void* q, const void* k_pages, const void* v_pages, void* out,
                                          const int* token_list, int n_items, const int* positions,
                                          const int* seq_of_token, const int* block_table, int bt_stride,
                                          int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
-                                         float scale, float score_cap, int chunk, int flags, int n_splits, float* scratch,
+                                         float scale, float score_cap, int chunk, const float* sinks, int share, int n_splits, float* scratch,
                                          int* tickets, const void* warm_a, long long warm_a_bytes, const void* warm_b,
                                          long long warm_b_bytes, cudaStream_t stream) {
     if (score_cap < 0.f) return NI_ERR_BAD_ARGUMENT;
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, score_cap, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, chunk, flags, nullptr, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, chunk, sinks, share, nullptr, stream);
 }
 
 // Differential attention: two maps per head.  q [n_tokens, Hm, head_dim / 2], Hm = n_map_heads counting maps (a head's two
@@ -1033,7 +1034,7 @@ NI_EXPORT int ni_attention_decode_difference(const void* q, const void* k_pages,
     const DecDiff d = {lambda, eps, factor};
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_map_heads, n_kv_heads, head_dim, page_size, 0, scale, 0.f, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, share << 1, &d, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, nullptr, share, &d, stream);
 }
 
 // The same with the scaled scores bounded by score_cap * tanh(s / score_cap) (score_cap > 0).
@@ -1047,7 +1048,7 @@ NI_EXPORT int ni_attention_decode_capped(const void* q, const void* k_pages, con
     if (!(score_cap > 0.f)) return NI_ERR_BAD_ARGUMENT;
     return decode_dispatch(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table, bt_stride,
                            n_q_heads, n_kv_heads, head_dim, page_size, window, scale, score_cap, n_splits, scratch, tickets,
-                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, 0, nullptr, stream);
+                           warm_a, warm_a_bytes, warm_b, warm_b_bytes, 0, nullptr, 0, nullptr, stream);
 }
 
 // ---- the variant that allocates nothing (see attention_decode_noalloc.h) ----------------------

@@ -10,8 +10,9 @@
 // Values may have a size of their own (v_dim): the value pages are then [P, Hkv, page, v_dim] and the output
 // [T, Hq, v_dim].
 // Two more masks and one more denominator, all parameters: `chunk` > 0 lets a token see only the keys of its own
-// chunk, [p - p % chunk, p], chunks counted from the sequence's position 0; `sink` adds one to the softmax's
-// denominator - a key of score 0 without a value - so the weights of a token sum to less than one.
+// chunk, [p - p % chunk, p], chunks counted from the sequence's position 0; `sinks` (one number per query head) adds
+// exp(sinks[head]) to the softmax's denominator - a key of that score without a value - so the weights of a token sum to
+// less than one.
 // `maps` > 1: every head has that many attention maps of its own over the same values.  q is then [T, Hq] rows of
 // head_dim, Hq counting maps (head h's map m is row h * maps + m), a key row holds the maps side by side (maps * head_dim
 // numbers), and every map has an output row of v_dim numbers.  The output may be FP32 whatever the inputs' type.
@@ -38,7 +39,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
                                          int n_tokens, int n_q_heads, int n_kv_heads, int head_dim,
                                          int page_size, int window, float scale,
                                          const float* __restrict__ head_slopes, float score_cap, int v_dim, int chunk,
-                                         int sink, int maps) {
+                                         const float* __restrict__ sinks, int maps) {
     const int warps_per_block = blockDim.x >> 5;
     const long long item = (long long)blockIdx.x * warps_per_block + (threadIdx.x >> 5);
     if (item >= (long long)n_tokens * n_q_heads) return;
@@ -62,7 +63,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
         qr[r] = dim < head_dim ? ni_to_float(qrow[dim]) : 0.f;
         acc[r] = 0.f;
     }
-    float m = sink ? 0.f : -INFINITY, l = sink ? 1.f : 0.f;      // the sink: a key of score 0 that is there from the start
+    float m = sinks ? sinks[head] : -INFINITY, l = sinks ? 1.f : 0.f;      // the sink: a key that is there from the start
     for (int j = lo; j <= pos; ++j) {
         const int page = table[j / page_size];
         const size_t slot = ((size_t)page * n_kv_heads + kvh) * page_size + (j % page_size);
@@ -103,7 +104,7 @@ NI_EXPORT int ni_attention_generic(const void* q, int dtype, const void* k_pages
                                    const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
                                    int n_tokens, int n_q_heads, int n_kv_heads, int head_dim,
                                    int page_size, int window, float scale, const float* head_slopes,
-                                   float score_cap, int v_dim, int chunk, int sink, int maps, cudaStream_t stream) {
+                                   float score_cap, int v_dim, int chunk, const float* sinks, int maps, cudaStream_t stream) {
     if (n_tokens <= 0) return NI_OK;
     if (n_q_heads <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads || head_dim <= 0 || page_size <= 0 || v_dim < 0 || chunk < 0 ||
         maps <= 0 || (n_q_heads / n_kv_heads) % maps)
@@ -118,7 +119,7 @@ NI_EXPORT int ni_attention_generic(const void* q, int dtype, const void* k_pages
     attention_generic_kernel<T, TO, R><<<(int)blocks, warps * 32, 0, stream>>>(                     \
         (const T*)q, (const T*)k_pages, (const T*)v_pages, (TO*)out, token_list, positions,        \
         seq_of_token,                                                                               \
-        block_table, bt_stride, n_tokens, n_q_heads, n_kv_heads, head_dim, page_size, window, scale, head_slopes, score_cap, v_dim, chunk, sink, maps)
+        block_table, bt_stride, n_tokens, n_q_heads, n_kv_heads, head_dim, page_size, window, scale, head_slopes, score_cap, v_dim, chunk, sinks, maps)
 #define LAUNCH(T, TO)                      \
     do {                                   \
         if (head_dim <= 256 && v_dim <= 256) LAUNCH_R(T, TO, 8); \

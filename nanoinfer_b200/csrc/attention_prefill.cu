@@ -59,7 +59,8 @@ template <int HD> __device__ __forceinline__ int sw(int row, int chunk) {
 }
 
 // chunk > 0: a query at position p sees only the keys of its own chunk, p - p % chunk .. p (chunks counted from the
-// sequence's position 0).  sink: one is added to every row's softmax denominator (a key of score 0 without a value).
+// sequence's position 0).  sinks (a number per query head): exp(sinks[head]) is added to every
+// row's softmax denominator (a key of that score without a value).
 // CAP: the scaled scores are bounded smoothly, s <- cap * tanh(s / cap), before mask and softmax.  The kernel is
 // then handed scale_log2e = 2 log2(e) scale / cap and cap_l2 = cap log2(e): with x = exp2(raw * scale_log2e),
 // cap_l2 * tanh(.) = cap_l2 - 2 cap_l2 / (x + 1) is the capped score in the exponent's base; its error is a few
@@ -72,7 +73,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ cu_q, const int* __restrict__ kv_len,
                          const int* __restrict__ block_table, int bt_stride, int n_q_heads,
                          int n_kv_heads, int page_size, int window, float scale_log2e, float cap_l2, int chunk,
-                         int sink) {
+                         const float* __restrict__ sinks) {
     constexpr int CH = HD / 8;        // 16-byte chunks per row
     constexpr int KS = HD / 16;       // k-steps over the head size
     constexpr int NT_O = HD / 8;      // output column tiles
@@ -258,9 +259,10 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     cp_async_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    if (sink) {        // a key of score 0: its weight relative to the row's maximum (0 is the reference of a row without keys)
-        l0 += pf_exp2(-(m0 == -INFINITY ? 0.f : m0));
-        l1 += pf_exp2(-(m1 == -INFINITY ? 0.f : m1));
+    if (sinks) {       // its weight relative to the row's maximum (0 is the reference of a row without keys)
+        const float sk = sinks[head] * 1.4426950408889634f;
+        l0 += pf_exp2(sk - (m0 == -INFINITY ? 0.f : m0));
+        l1 += pf_exp2(sk - (m1 == -INFINITY ? 0.f : m1));
     }
     const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
     const int ra = row0 + warp * 16 + g, rb = ra + 8;
@@ -282,7 +284,7 @@ template <int HD, bool CAP> static int launch_prefill(const void* q, const void*
                                             const int* tile_seq, const int* tile_row0, int n_tiles,
                                             const int* cu_q, const int* kv_len, const int* block_table,
                                             int bt_stride, int n_q_heads, int n_kv_heads, int page_size,
-                                            int window, float scale_log2e, float cap_l2, int chunk, int sink,
+                                            int window, float scale_log2e, float cap_l2, int chunk, const float* sinks,
                                             cudaStream_t stream) {
     const size_t smem = (size_t)(PF_BM + 4 * PF_BN) * HD * sizeof(__nv_bfloat16);
     static bool configured = false;
@@ -298,7 +300,7 @@ template <int HD, bool CAP> static int launch_prefill(const void* q, const void*
     attention_prefill_kernel<HD, CAP><<<grid, PF_WARPS * 32, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
         (__nv_bfloat16*)out, tile_seq, tile_row0, cu_q, kv_len, block_table, bt_stride, n_q_heads,
-        n_kv_heads, page_size, window, scale_log2e, cap_l2, chunk, sink);
+        n_kv_heads, page_size, window, scale_log2e, cap_l2, chunk, sinks);
     NI_RETURN_LAUNCH_STATUS();
 }
 
@@ -308,7 +310,7 @@ NI_EXPORT int ni_attention_prefill(const void* q, const void* k_pages, const voi
                                    const int* tile_seq, const int* tile_row0, int n_tiles, const int* cu_q,
                                    const int* kv_len, const int* block_table, int bt_stride, int n_q_heads,
                                    int n_kv_heads, int head_dim, int page_size, int window, float scale,
-                                   float score_cap, int chunk, int sink, cudaStream_t stream) {
+                                   float score_cap, int chunk, const float* sinks, cudaStream_t stream) {
     if (n_tiles <= 0) return NI_OK;
     if (n_q_heads <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads || page_size <= 0 || chunk < 0)
         return NI_ERR_BAD_ARGUMENT;
@@ -317,9 +319,9 @@ NI_EXPORT int ni_attention_prefill(const void* q, const void* k_pages, const voi
     const float cl = cap ? score_cap * 1.4426950408889634f : 0.f;
 #define GO(HD)                                                                                                         \
     return cap ? launch_prefill<HD, true>(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu_q, kv_len,       \
-                                          block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window, sl, cl, chunk, sink, stream) \
+                                          block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window, sl, cl, chunk, sinks, stream) \
                : launch_prefill<HD, false>(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu_q, kv_len,      \
-                                           block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window, sl, cl, chunk, sink, stream)
+                                           block_table, bt_stride, n_q_heads, n_kv_heads, page_size, window, sl, cl, chunk, sinks, stream)
     switch (head_dim) {
         case 16: GO(16);
         case 32: GO(32);

@@ -236,7 +236,8 @@ struct AtParams {
     float scale_log2e;
     int* error;
     int chunk;                     // > 0: a query at position p sees only the keys from p - p % chunk on
-    int sink;                      // != 0: one is added to every row's softmax denominator (a key of score 0 without a value)
+    const float* sinks;            // a number per query head (null: none): exp(sinks[head]) is added to every row's softmax
+                                   // denominator (a key of that score without a value)
     float lambda, eps, factor;     // DIFF
 };
 
@@ -626,7 +627,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             at_mbar_arrive(&p_full[s]);
         }
         // ---- the finished rows: O / l -> bfloat16; the row's sum is the two halves' together ----
-        if (p.sink && half == 0) l += at_exp2(-(m_used == -INFINITY ? 0.f : m_used));      // the sink's weight, counted once per row
+        if (p.sinks && half == 0)      // the sink's weight, counted once per row
+            l += at_exp2(p.sinks[s ? head1 : head0] * 1.4426950408889634f - (m_used == -INFINITY ? 0.f : m_used));
         const bool finished = ok && n_tiles > 0 &&
                               __all_sync(0xffffffffu, at_wait(&o_done[s], (uint32_t)(n_tiles - 1) & 1u, abort_flag, p.error, AT_ERR_SOFTMAX));
         if (DIFF) {
@@ -784,7 +786,7 @@ NI_EXPORT int ni_attention_prefill_tc_supports(int n_q_heads, int n_kv_heads, in
 
 static int run_at(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens, int n_pages, const int* tile_seq,
                   const int* tile_row0, int n_tiles, const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
-                  int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale, int chunk, int sink,
+                  int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale, int chunk, const float* sinks,
                   bool diff, float lambda, float eps, float factor, int* error, cudaStream_t stream) {
     if (n_tiles <= 0) return NI_OK;
     if (n_tokens <= 0 || n_pages <= 0 || error == nullptr || chunk < 0) return NI_ERR_BAD_ARGUMENT;
@@ -802,7 +804,7 @@ static int run_at(const void* q, const void* k_pages, const void* v_pages, void*
     p.out = (__nv_bfloat16*)out; p.tile_seq = tile_seq; p.tile_row0 = tile_row0; p.cu_q = cu_q; p.kv_len = kv_len;
     p.block_table = block_table; p.bt_stride = bt_stride; p.n_q_heads = n_q_heads; p.n_kv_heads = n_kv_heads;
     p.page_size = page_size; p.window = window; p.scale_log2e = scale * 1.4426950408889634f; p.error = error;
-    p.chunk = chunk; p.sink = sink;
+    p.chunk = chunk; p.sinks = sinks;
     p.lambda = lambda; p.eps = eps; p.factor = factor;
     if (diff) {
         if (head_dim == 64) return launch_at<64, 4, true>(mq, mk, mv, p, n_tiles, stream);
@@ -815,17 +817,17 @@ static int run_at(const void* q, const void* k_pages, const void* v_pages, void*
 // q, out: bf16 [n_tokens, Hq * hd]; k_pages, v_pages: bf16 [n_pages, Hkv, page_size, hd], all 16-byte
 // aligned.  tile_seq / tile_row0 [n_tiles]: request and first query row of each block's 128 rows.
 // error: a device int, zero on entry; non-zero afterwards if a wait inside the kernel ran out.
-// chunk > 0: a query at position p sees only the keys from p - p % chunk on; sink != 0: one is added to the softmax's
-// denominator.
+// chunk > 0: a query at position p sees only the keys from p - p % chunk on; sinks (FP32, one per query head; null:
+// none): exp(sinks[head]) is added to the softmax's denominator.
 NI_EXPORT int ni_attention_prefill_tc_masked(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,
                                              int n_pages, const int* tile_seq, const int* tile_row0, int n_tiles,
                                              const int* cu_q, const int* kv_len, const int* block_table, int bt_stride,
                                              int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
-                                             float scale, int chunk, int sink, int* error, cudaStream_t stream) {
+                                             float scale, int chunk, const float* sinks, int* error, cudaStream_t stream) {
     if (n_tiles <= 0) return NI_OK;
     if (!ni_attention_prefill_tc_supports(n_q_heads, n_kv_heads, head_dim, page_size)) return NI_ERR_UNSUPPORTED_SIZE;
     return run_at(q, k_pages, v_pages, out, n_tokens, n_pages, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table, bt_stride,
-                  n_q_heads, n_kv_heads, head_dim, page_size, window, scale, chunk, sink, false, 0.f, 0.f, 0.f, error, stream);
+                  n_q_heads, n_kv_heads, head_dim, page_size, window, scale, chunk, sinks, false, 0.f, 0.f, 0.f, error, stream);
 }
 
 // Differential attention: a head's row of q and of the key pages holds its two maps side by side (head_dim / 2 numbers each),
@@ -839,7 +841,7 @@ NI_EXPORT int ni_attention_prefill_tc_difference(const void* q, const void* k_pa
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads) return NI_ERR_BAD_ARGUMENT;
     if ((head_dim != 64 && head_dim != 128) || page_size < 8 || page_size > 128 || 128 % page_size) return NI_ERR_UNSUPPORTED_SIZE;
     return run_at(q, k_pages, v_pages, out, n_tokens, n_pages, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table, bt_stride,
-                  n_heads, n_kv_heads, head_dim, page_size, 0, scale, 0, 0, true, lambda, eps, factor, error, stream);
+                  n_heads, n_kv_heads, head_dim, page_size, 0, scale, 0, nullptr, true, lambda, eps, factor, error, stream);
 }
 
 NI_EXPORT int ni_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, void* out, int n_tokens,
@@ -848,6 +850,6 @@ NI_EXPORT int ni_attention_prefill_tc(const void* q, const void* k_pages, const 
                                       int n_q_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                       float scale, int* error, cudaStream_t stream) {
     return ni_attention_prefill_tc_masked(q, k_pages, v_pages, out, n_tokens, n_pages, tile_seq, tile_row0, n_tiles, cu_q, kv_len,
-                                          block_table, bt_stride, n_q_heads, n_kv_heads, head_dim, page_size, window, scale, 0, 0,
-                                          error, stream);
+                                          block_table, bt_stride, n_q_heads, n_kv_heads, head_dim, page_size, window, scale, 0,
+                                          nullptr, error, stream);
 }

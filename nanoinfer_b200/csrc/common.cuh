@@ -84,6 +84,16 @@ __device__ __forceinline__ float ni_block_max(float v, float* scratch) {
     return t;
 }
 
+// Activation of a gated unit's gate: g * sigmoid(g (c1 + c2 g^2)).  (1, 0) is silu; (2 sqrt(2 / pi), 0.044715 of that) is the
+// tanh form of gelu, since (1 + tanh y) / 2 = sigmoid(2 y).
+#define NI_GELU_C1 1.5957691216057308f
+#define NI_GELU_C2 0.07135481627159896f
+__device__ __forceinline__ float ni_gate_act(float g, float c1, float c2) {
+    return g / (1.0f + expf(-(g * fmaf(c2 * g, g, c1))));
+}
+// The mode of a product with a gated epilogue may carry this flag: gelu instead of silu.
+#define NI_MODE_GELU 16
+
 // 16 bytes of a row at once: 8 bfloat16 or 4 float values, widened to FP32 (the address must be 16-byte aligned).
 template <typename T> struct NiVec16;
 template <> struct NiVec16<float> {

@@ -2,12 +2,13 @@
 //
 // Per head (state S [D, V] in FP32, carried from token to token of a request):
 //     S *= decay;   e = beta * (v - k S);   S += outer(k, e);   y = q S        (k, q: rows of D; v, e, y: rows of V)
-// with q and k unit vectors per head (q also times D^-1/2), decay = exp(-exp(A_log) softplus(a + dt_bias))
-// and beta = sigmoid(b).  q, k and v first pass a short causal convolution over time per channel
-// and silu; the last taps-1 inputs of every channel are part of a request's state.
+// with q and k unit vectors per head (q also times D^-1/2) and beta = sigmoid(b).  The decay is one number per head,
+// exp(-exp(A_log) softplus(a + dt_bias)), or one per head and key channel (then it multiplies the rows of S), whose
+// logits come from elsewhere (a product with two thin matrices).  q, k and v first pass a short causal convolution over
+// time per channel and silu; the last taps-1 inputs of every channel are part of a request's state.
 //
-// The step's tokens arrive as ONE fused projection `proj` (FP32 [T, ld]) with the columns
-//     [ q: G D | k: G D | v: H V | gate: H V | b: H | a: H ]
+// The step's tokens arrive as ONE fused projection `proj` ([T, ld], FP32 or bfloat16) whose first columns are
+//     [ q: G D | k: G D | v: H V ],   with b (H) and, one decay per head, a (H) at offsets the caller names
 // (G heads of q/k, H heads of v; head h reads q/k head h / (H / G)).  A request's state is a flat
 // FP32 vector [ S: H D V | history: (taps-1) C ] with C = 2 G D + H V, found through slots[].
 //
@@ -16,27 +17,30 @@
 //   (delta_history     per request: the new last taps-1 inputs; extra blocks of the gated norm's launch, which
 //                      comes after delta_prepare has read the old ones)
 //   delta_recurrence   per (request, head, a few value columns): its tokens one after the other
-//   delta_gated_norm   per token and head: o / rms(o) * weight * silu(gate)
+//   delta_gated_norm   per token and head: o / rms(o) * weight * silu or sigmoid(gate)
 // Prompt portions and single tokens are the same case; a token's result depends only on its own
 // request's state and tokens, in a fixed order of operations, however the step is cut.
+//
+// A step of single tokens with decays per channel has a fourth kernel, delta_token_step, that does all of it - the thin
+// second products of decay and gate included - in one launch.
 #include "common.cuh"
 
 struct DeltaDims {
     int G, H, D, V, taps, ld;  // ld: row stride of proj
+    int b_off, a_off;          // columns of b and a in proj (a_off < 0: decays per channel)
     __host__ __device__ int C() const { return 2 * G * D + H * V; }
-    __host__ __device__ int gate_off() const { return 2 * G * D + H * V; }
-    __host__ __device__ int b_off() const { return 2 * G * D + 2 * H * V; }
-    __host__ __device__ int a_off() const { return 2 * G * D + 2 * H * V + H; }
     __host__ __device__ size_t hist_off() const { return (size_t)H * D * V; }
 };
 
 __device__ __forceinline__ float dr_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float dr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float dr_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float dr_decay(float a_log, float logit) { return expf(-expf(a_log) * dr_softplus(logit)); }
 
 // Convolution of channel c at token t: taps inputs ending at this token.  Inputs before the
 // portion's first token come from the request's history, zeros before the sequence's start.
-__device__ __forceinline__ float dr_conv(const float* __restrict__ proj, const float* __restrict__ conv_w,
+template <typename T>
+__device__ __forceinline__ float dr_conv(const T* __restrict__ proj, const float* __restrict__ conv_w,
                                          const float* __restrict__ hist, const DeltaDims& dm, int t, int in_portion,
                                          int c) {
     float acc = 0.f;
@@ -44,7 +48,7 @@ __device__ __forceinline__ float dr_conv(const float* __restrict__ proj, const f
     for (int j = 0; j < dm.taps; ++j) {
         const int back = dm.taps - 1 - j;
         float x;
-        if (back <= in_portion) x = proj[(size_t)(t - back) * dm.ld + c];
+        if (back <= in_portion) x = ni_to_float(proj[(size_t)(t - back) * dm.ld + c]);
         else x = hist[(size_t)(dm.taps - 1 - (back - in_portion)) * C + c];
         acc = fmaf(conv_w[(size_t)c * dm.taps + j], x, acc);
     }
@@ -52,23 +56,32 @@ __device__ __forceinline__ float dr_conv(const float* __restrict__ proj, const f
 }
 
 // qkv [T, C]: q (unit, times D^-1/2), k (unit), v after convolution and silu; gates [T, H, 2]: decay, beta.
-// One warp per unit of work of a token: a q or k head (unit norm over its D channels), or 128 channels of v;
-// the first warp of a token also computes beta and decay.  grid = (tokens, units / warps per block).
+// One warp per unit of work of a token: a q or k head (unit norm over its D channels), 128 channels of v, or - decays
+// per channel - 128 logits of z [T, ld_z], which become decays in place; the first warp of a token also computes beta and
+// the decays per head.  grid = (tokens, units / warps per block).
 #define DP_WARPS 4
 #define DP_VCHUNK 128
+template <typename T>
 __global__ void __launch_bounds__(DP_WARPS * 32)
-delta_prepare_kernel(const float* __restrict__ proj, const float* __restrict__ conv_w,
+delta_prepare_kernel(const T* __restrict__ proj, const float* __restrict__ conv_w,
                      const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                      const float* __restrict__ state, long long state_stride,
                      const int* __restrict__ seq_of_token, const int* __restrict__ cu_q,
                      const int* __restrict__ slots, DeltaDims dm, float* __restrict__ qkv,
-                     float* __restrict__ gates) {
+                     float* __restrict__ gates, float* __restrict__ z, int ld_z) {
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31;
-    const int unit = blockIdx.y * DP_WARPS + (threadIdx.x >> 5);
-    const int C = dm.C(), HV = dm.H * dm.V;
+    int unit = blockIdx.y * DP_WARPS + (threadIdx.x >> 5);
+    const int C = dm.C(), HV = dm.H * dm.V, HD = dm.H * dm.D;
     const int n_units = 2 * dm.G + (HV + DP_VCHUNK - 1) / DP_VCHUNK;
-    if (unit >= n_units) return;
+    if (unit >= n_units) {
+        unit -= n_units;
+        if (z == nullptr || unit * DP_VCHUNK >= HD) return;
+        float* row = z + (size_t)t * ld_z;
+        for (int c = unit * DP_VCHUNK + lane; c < (unit + 1) * DP_VCHUNK && c < HD; c += 32)
+            row[c] = dr_decay(a_log[c / dm.D], row[c] + dt_bias[c]);
+        return;
+    }
     const int seq = seq_of_token[t];
     const int in_portion = t - cu_q[seq];
     const float* hist = state + (size_t)slots[seq] * state_stride + dm.hist_off();
@@ -91,17 +104,19 @@ delta_prepare_kernel(const float* __restrict__ proj, const float* __restrict__ c
             out[c] = dr_conv(proj, conv_w, hist, dm, t, in_portion, c);
     }
     if (unit == 0) {
-        const float* row = proj + (size_t)t * dm.ld;
+        const T* row = proj + (size_t)t * dm.ld;
         for (int h = lane; h < dm.H; h += 32) {
-            gates[((size_t)t * dm.H + h) * 2] = expf(-expf(a_log[h]) * dr_softplus(row[dm.a_off() + h] + dt_bias[h]));
-            gates[((size_t)t * dm.H + h) * 2 + 1] = dr_sigmoid(row[dm.b_off() + h]);
+            gates[((size_t)t * dm.H + h) * 2] =
+                dm.a_off >= 0 ? dr_decay(a_log[h], ni_to_float(row[dm.a_off + h]) + dt_bias[h]) : 1.0f;
+            gates[((size_t)t * dm.H + h) * 2 + 1] = dr_sigmoid(ni_to_float(row[dm.b_off + h]));
         }
     }
 }
 
 // The request's new history: its last taps-1 inputs.  One thread per channel walks j upwards, so a
 // portion shorter than the history shifts the old entries in place (it reads index j + q_len > j).
-__device__ __forceinline__ void delta_history(const float* __restrict__ proj, float* __restrict__ state,
+template <typename T>
+__device__ __forceinline__ void delta_history(const T* __restrict__ proj, float* __restrict__ state,
                                               long long state_stride, const int* __restrict__ cu_q,
                                               const int* __restrict__ slots, const DeltaDims& dm, int seq, int c) {
     const int C = dm.C();
@@ -110,7 +125,7 @@ __device__ __forceinline__ void delta_history(const float* __restrict__ proj, fl
     float* hist = state + (size_t)slots[seq] * state_stride + dm.hist_off();
     for (int j = 0; j < dm.taps - 1; ++j) {
         const int idx = q_len - (dm.taps - 1 - j);      // index into the portion; negative: before it
-        hist[(size_t)j * C + c] = idx >= 0 ? proj[(size_t)(first + idx) * dm.ld + c] : hist[(size_t)(j + q_len) * C + c];
+        hist[(size_t)j * C + c] = idx >= 0 ? ni_to_float(proj[(size_t)(first + idx) * dm.ld + c]) : hist[(size_t)(j + q_len) * C + c];
     }
 }
 
@@ -139,14 +154,17 @@ __device__ __forceinline__ void dr_copy16(float* dst_smem, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 
-template <int CHUNKS, int RG>
+// CHANNEL: the decays are one per row of S, decay [T, ld_z] with head h's D numbers from column h D on; they travel with k
+// and q.  Otherwise they are the first number of a head's pair in gates.
+template <int CHUNKS, int RG, bool CHANNEL>
 __global__ void __launch_bounds__(32)
 delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__ gates,
+                        const float* __restrict__ decay, int ld_z,
                         float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                         const int* __restrict__ slots, DeltaDims dm, float* __restrict__ out) {
     constexpr int ROWS = 8 * CHUNKS, COLS = 32 / RG, DP = ROWS * RG;   // rows per lane; columns per warp; D rounded up
-    constexpr int STAGE = 2 * DP + 12;                     // k | q | v of the warp's columns (up to 8) | decay, beta, -, -
-    constexpr int STAGES = DP >= 1024 ? 4 : DR_MAX_STAGES;
+    constexpr int STAGE = 2 * DP + 12 + (CHANNEL ? DP : 0);   // k | q | v of the warp's columns (up to 8) | decay, beta, -, - | decays per row
+    constexpr int STAGES = CHANNEL ? (DP >= 1024 ? 3 : (DP >= 512 ? 4 : DR_MAX_STAGES)) : (DP >= 1024 ? 4 : DR_MAX_STAGES);
     __shared__ __align__(16) float ring[STAGES][STAGE];
     const int lane = threadIdx.x, rg = lane / COLS, cl = lane % COLS;
     const int h = blockIdx.y, seq = blockIdx.z;
@@ -156,13 +174,16 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
     const int g = h / (dm.H / dm.G);
     const int first = cu_q[seq], last = cu_q[seq + 1];
     if (first >= last) return;
-    const bool wide = (D % 4 == 0) && (C % 4 == 0);        // rows of k and q start on 16-byte boundaries
+    const bool wide = (D % 4 == 0) && (C % 4 == 0) && (!CHANNEL || ld_z % 4 == 0);        // rows of k, q and the decays start on 16-byte boundaries
     const bool padded = D != DP;                           // same for the whole launch
     const bool ragged = blockIdx.x * COLS + COLS > dm.V;   // same for the whole warp: some of its columns do not exist
     if (padded || ragged) {                                // entries that no copy ever writes
         for (int st = 0; st < STAGES; ++st) {
             for (int i = lane; i < DP; i += 32)
-                if (i >= D) ring[st][i] = ring[st][DP + i] = 0.f;
+                if (i >= D) {
+                    ring[st][i] = ring[st][DP + i] = 0.f;
+                    if (CHANNEL) ring[st][2 * DP + 12 + i] = 0.f;
+                }
             if (lane < COLS && !live) ring[st][2 * DP + lane] = 0.f;
         }
     }
@@ -172,6 +193,7 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
     const float* q_src = row + g * D + (wide ? 4 * lane : lane);
     const float* v_src = row + 2 * dm.G * D + h * dm.V + col;
     const float* g_src = gates + ((size_t)first * dm.H + h) * 2;
+    const float* d_src = CHANNEL ? decay + (size_t)first * ld_z + h * D + (wide ? 4 * lane : lane) : nullptr;
     int fetch_t = first, fetch_stage = 0;
     auto fetch = [&]() {                                   // the next token into its stage (nothing past the portion)
         if (fetch_t < last) {
@@ -182,6 +204,7 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
                     if (4 * lane + 128 * m < D) {
                         dr_copy16(sg + 4 * lane + 128 * m, k_src + 128 * m);
                         dr_copy16(sg + DP + 4 * lane + 128 * m, q_src + 128 * m);
+                        if (CHANNEL) dr_copy16(sg + 2 * DP + 12 + 4 * lane + 128 * m, d_src + 128 * m);
                     }
             } else {
 #pragma unroll
@@ -189,11 +212,13 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
                     if (lane + 32 * m < D) {
                         dr_copy4(sg + lane + 32 * m, k_src + 32 * m);
                         dr_copy4(sg + DP + lane + 32 * m, q_src + 32 * m);
+                        if (CHANNEL) dr_copy4(sg + 2 * DP + 12 + lane + 32 * m, d_src + 32 * m);
                     }
             }
             if (lane < COLS && live) dr_copy4(sg + 2 * DP + lane, v_src);        // rg == 0 here
             if (lane == 31) dr_copy8(sg + 2 * DP + 8, g_src);                   // decay, beta
             k_src += C; q_src += C; v_src += C; g_src += 2 * dm.H;
+            if (CHANNEL) d_src += ld_z;
         }
         ++fetch_t;
         fetch_stage = fetch_stage + 1 == STAGES ? 0 : fetch_stage + 1;
@@ -229,8 +254,15 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
             const float4 ka = *reinterpret_cast<const float4*>(kc + 8 * c);
             const float4 kb = *reinterpret_cast<const float4*>(kc + 8 * c + 4);
             float* sc = s + 8 * c;
+            if (CHANNEL) {
+                const float4 ga = *reinterpret_cast<const float4*>(sg + 2 * DP + 12 + row0 + 8 * c);
+                const float4 gb = *reinterpret_cast<const float4*>(sg + 2 * DP + 12 + row0 + 8 * c + 4);
+                sc[0] *= ga.x; sc[1] *= ga.y; sc[2] *= ga.z; sc[3] *= ga.w;
+                sc[4] *= gb.x; sc[5] *= gb.y; sc[6] *= gb.z; sc[7] *= gb.w;
+            } else {
 #pragma unroll
-            for (int j = 0; j < 8; ++j) sc[j] *= gd;
+                for (int j = 0; j < 8; ++j) sc[j] *= gd;
+            }
             const float d0 = fmaf(sc[4], kb.x, sc[0] * ka.x), d1 = fmaf(sc[5], kb.y, sc[1] * ka.y);
             const float d2 = fmaf(sc[6], kb.z, sc[2] * ka.z), d3 = fmaf(sc[7], kb.w, sc[3] * ka.w);
             part[c] = (d0 + d1) + (d2 + d3);
@@ -285,15 +317,17 @@ delta_recurrence_kernel(const float* __restrict__ qkv, const float* __restrict__
     }
 }
 
-// y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * silu(gate[t, h, :]); one warp per (t, h).
-// The blocks behind those (from norm_blocks on) write the requests' new convolution history: by now the
-// preparation, which read the old one, has ended, and one launch less stands between two steps' products.
-template <typename T>
-__global__ void delta_gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj,
-                                        const float* __restrict__ weight, float eps, DeltaDims dm, int n_tokens,
-                                        T* __restrict__ y, int norm_blocks, int hist_blocks_per_seq,
-                                        float* __restrict__ state, long long state_stride,
-                                        const int* __restrict__ cu_q, const int* __restrict__ slots) {
+// y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * act(gate[t, h, :]) * scale, act silu or sigmoid; one
+// warp per (t, h); gate and y have row strides of their own.  The blocks behind those (from norm_blocks on) write the
+// requests' new convolution history: by now the preparation, which read the old one, has ended, and one launch less stands
+// between two steps' products.
+template <typename T, typename TP>
+__global__ void delta_gated_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int ld_gate,
+                                        int sigmoid_gate, const float* __restrict__ weight, float eps, float scale,
+                                        DeltaDims dm, int n_tokens, T* __restrict__ y, int ld_y, int norm_blocks,
+                                        int hist_blocks_per_seq, const TP* __restrict__ proj, float* __restrict__ state,
+                                        long long state_stride, const int* __restrict__ cu_q,
+                                        const int* __restrict__ slots) {
     if ((int)blockIdx.x >= norm_blocks) {
         const int hb = blockIdx.x - norm_blocks;
         delta_history(proj, state, state_stride, cu_q, slots, dm, hb / hist_blocks_per_seq,
@@ -305,52 +339,71 @@ __global__ void delta_gated_norm_kernel(const float* __restrict__ o, const float
     const int lane = threadIdx.x & 31;
     const int t = (int)(item / dm.H), h = (int)(item - (long long)t * dm.H);
     const float* orow = o + ((size_t)t * dm.H + h) * dm.V;
-    const float* grow = proj + (size_t)t * dm.ld + dm.gate_off() + h * dm.V;
-    T* yrow = y + ((size_t)t * dm.H + h) * dm.V;
+    const float* grow = gate + (size_t)t * ld_gate + h * dm.V;
+    T* yrow = y + (size_t)t * ld_y + (size_t)h * dm.V;
     float ss = 0.f;
     for (int i = lane; i < dm.V; i += 32) ss += orow[i] * orow[i];
     ss = ni_warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)dm.V + eps);
-    for (int i = lane; i < dm.V; i += 32) yrow[i] = ni_from_float<T>(orow[i] * inv * weight[i] * dr_silu(grow[i]));
+    for (int i = lane; i < dm.V; i += 32) {
+        const float g = sigmoid_gate ? dr_sigmoid(grow[i]) * scale : dr_silu(grow[i]) * scale;
+        yrow[i] = ni_from_float<T>(orow[i] * inv * weight[i] * g);
+    }
 }
 
 static int dr_check(const DeltaDims& dm) {
     if (dm.G <= 0 || dm.H <= 0 || dm.D <= 0 || dm.V <= 0 || dm.taps <= 0 || dm.H % dm.G) return NI_ERR_BAD_ARGUMENT;
-    if (dm.ld < dm.a_off() + dm.H) return NI_ERR_BAD_ARGUMENT;
+    if (dm.ld < dm.C() || (dm.b_off >= 0 && dm.ld < dm.b_off + dm.H) || (dm.a_off >= 0 && dm.ld < dm.a_off + dm.H))
+        return NI_ERR_BAD_ARGUMENT;
     if (dm.D > 1024) return NI_ERR_UNSUPPORTED_SIZE;      // a warp holds whole columns of a head's state: 32 lanes x 32 rows
     return NI_OK;
 }
 
 // Convolution, activations, unit norms, beta and decay of the step's tokens (the new history is written by
-// ni_delta_gated_norm, which every step runs after this).
-NI_EXPORT int ni_delta_prepare(const float* proj, const float* conv_w, const float* a_log, const float* dt_bias,
+// ni_delta_gated_norm, which every step runs after this).  a_off < 0: the decays are one per head and key channel; their
+// logits, z [T, ld_z] (H D columns), become decays in place, dt_bias has H D entries.
+NI_EXPORT int ni_delta_prepare(const void* proj, int proj_dtype, const float* conv_w, const float* a_log, const float* dt_bias,
                                float* state, long long state_stride, const int* seq_of_token, const int* cu_q,
                                const int* slots, int n_tokens, int n_seqs, int G, int H, int D, int V, int taps, int ld,
-                               float* qkv, float* gates, cudaStream_t stream) {
+                               int b_off, int a_off, float* z, int ld_z, float* qkv, float* gates, cudaStream_t stream) {
     if (n_tokens <= 0) return NI_OK;
-    DeltaDims dm{G, H, D, V, taps, ld};
+    DeltaDims dm{G, H, D, V, taps, ld, b_off, a_off};
     if (int rc = dr_check(dm)) return rc;
-    const int C = dm.C();
-    const int n_units = 2 * G + (H * V + DP_VCHUNK - 1) / DP_VCHUNK;
+    if (b_off < 0 || (a_off < 0) != (z != nullptr) || (z && ld_z < H * D)) return NI_ERR_BAD_ARGUMENT;
+    const int n_units = 2 * G + (H * V + DP_VCHUNK - 1) / DP_VCHUNK + (z ? (H * D + DP_VCHUNK - 1) / DP_VCHUNK : 0);
     dim3 pgrid(n_tokens, (n_units + DP_WARPS - 1) / DP_WARPS);
     if (pgrid.y > 65535) return NI_ERR_UNSUPPORTED_SIZE;
-    delta_prepare_kernel<<<pgrid, DP_WARPS * 32, 0, stream>>>(proj, conv_w, a_log, dt_bias, state, state_stride,
-                                                              seq_of_token, cu_q, slots, dm, qkv, gates);
+    if (proj_dtype == NI_DTYPE_F32)
+        delta_prepare_kernel<float><<<pgrid, DP_WARPS * 32, 0, stream>>>((const float*)proj, conv_w, a_log, dt_bias, state,
+                                                                         state_stride, seq_of_token, cu_q, slots, dm, qkv,
+                                                                         gates, z, ld_z);
+    else if (proj_dtype == NI_DTYPE_BF16)
+        delta_prepare_kernel<__nv_bfloat16><<<pgrid, DP_WARPS * 32, 0, stream>>>((const __nv_bfloat16*)proj, conv_w, a_log,
+                                                                                 dt_bias, state, state_stride, seq_of_token,
+                                                                                 cu_q, slots, dm, qkv, gates, z, ld_z);
+    else
+        return NI_ERR_BAD_ARGUMENT;
     NI_RETURN_LAUNCH_STATUS();
 }
 
-NI_EXPORT int ni_delta_recurrence(const float* qkv, const float* gates, float* state,
+// decay / ld_z: decays per channel as ni_delta_prepare leaves them in z, or null (then gates holds one per head).
+NI_EXPORT int ni_delta_recurrence(const float* qkv, const float* gates, const float* decay, int ld_z, float* state,
                                   long long state_stride, const int* cu_q, const int* slots, int n_tokens, int n_seqs,
                                   int G, int H, int D, int V, float* out, cudaStream_t stream) {
     if (n_seqs <= 0) return NI_OK;
-    DeltaDims dm{G, H, D, V, 1, 2 * G * D + 2 * H * V + 2 * H};
+    DeltaDims dm{G, H, D, V, 1, 2 * G * D + H * V, -1, -1};
     if (int rc = dr_check(dm)) return rc;
+    if (decay && ld_z < H * D) return NI_ERR_BAD_ARGUMENT;
     if (H > 65535 || n_seqs > 65535) return NI_ERR_UNSUPPORTED_SIZE;
 #define LAUNCH(CHUNKS, RG)                                                                                       \
     do {                                                                                                         \
         dim3 grid((V + 32 / (RG) - 1) / (32 / (RG)), H, n_seqs);                                                 \
-        delta_recurrence_kernel<CHUNKS, RG><<<grid, 32, 0, stream>>>(qkv, gates, state, state_stride, cu_q,       \
-                                                                     slots, dm, out);                            \
+        if (decay)                                                                                               \
+            delta_recurrence_kernel<CHUNKS, RG, true><<<grid, 32, 0, stream>>>(qkv, gates, decay, ld_z, state,    \
+                                                                               state_stride, cu_q, slots, dm, out); \
+        else                                                                                                     \
+            delta_recurrence_kernel<CHUNKS, RG, false><<<grid, 32, 0, stream>>>(qkv, gates, nullptr, 0, state,    \
+                                                                                state_stride, cu_q, slots, dm, out); \
     } while (0)
     // Lanes per column (RG): single tokens take the fewest (whole sectors of S); long portions take the fewest that
     // still give every scheduler a warp or so (3 warps per SM and more: measured at key size 128, one request of
@@ -382,26 +435,29 @@ NI_EXPORT int ni_delta_recurrence(const float* qkv, const float* gates, float* s
     NI_RETURN_LAUNCH_STATUS();
 }
 
-// The gated norm of the step's read-outs, and the requests' new convolution history (taps > 1).
-NI_EXPORT int ni_delta_gated_norm(const float* o, const float* proj, const float* weight, float eps, int n_tokens,
-                                  int n_seqs, int G, int H, int D, int V, int taps, int ld, void* y, int y_dtype,
-                                  float* state, long long state_stride, const int* cu_q, const int* slots,
-                                  cudaStream_t stream) {
+// The gated norm of the step's read-outs, and the requests' new convolution history (taps > 1) from proj.  gate: FP32 rows
+// ld_gate apart; sigmoid_gate 0: silu; scale: one more factor; y rows ld_y apart.
+NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate, int sigmoid_gate, const float* weight,
+                                  float eps, float scale, int n_tokens, int n_seqs, int G, int H, int D, int V, int taps,
+                                  void* y, int y_dtype, int ld_y, const void* proj, int proj_dtype, int ld, float* state,
+                                  long long state_stride, const int* cu_q, const int* slots, cudaStream_t stream) {
     if (n_tokens <= 0) return NI_OK;
-    DeltaDims dm{G, H, D, V, taps, ld};
+    DeltaDims dm{G, H, D, V, taps, ld, -1, -1};
     if (int rc = dr_check(dm)) return rc;
+    if (ld_gate < H * V || ld_y < H * V) return NI_ERR_BAD_ARGUMENT;
     const int warps = 4;
     const long long norm_blocks = ((long long)n_tokens * H + warps - 1) / warps;
     const int per_seq = taps > 1 ? (dm.C() + warps * 32 - 1) / (warps * 32) : 0;
     const long long blocks = norm_blocks + (long long)per_seq * n_seqs;
     if (blocks > 2147483647LL) return NI_ERR_UNSUPPORTED_SIZE;
-    if (y_dtype == NI_DTYPE_F32)
-        delta_gated_norm_kernel<float><<<(int)blocks, warps * 32, 0, stream>>>(
-            o, proj, weight, eps, dm, n_tokens, (float*)y, (int)norm_blocks, per_seq, state, state_stride, cu_q, slots);
-    else if (y_dtype == NI_DTYPE_BF16)
-        delta_gated_norm_kernel<__nv_bfloat16><<<(int)blocks, warps * 32, 0, stream>>>(
-            o, proj, weight, eps, dm, n_tokens, (__nv_bfloat16*)y, (int)norm_blocks, per_seq, state, state_stride, cu_q, slots);
-    else
-        return NI_ERR_BAD_ARGUMENT;
+#define GO(T, TP)                                                                                                        \
+    delta_gated_norm_kernel<T, TP><<<(int)blocks, warps * 32, 0, stream>>>(                                              \
+        o, gate, ld_gate, sigmoid_gate, weight, eps, scale, dm, n_tokens, (T*)y, ld_y, (int)norm_blocks, per_seq,        \
+        (const TP*)proj, state, state_stride, cu_q, slots)
+    if (y_dtype == NI_DTYPE_F32 && proj_dtype == NI_DTYPE_F32) GO(float, float);
+    else if (y_dtype == NI_DTYPE_BF16 && proj_dtype == NI_DTYPE_F32) GO(__nv_bfloat16, float);
+    else if (y_dtype == NI_DTYPE_BF16 && proj_dtype == NI_DTYPE_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else return NI_ERR_BAD_ARGUMENT;
+#undef GO
     NI_RETURN_LAUNCH_STATUS();
 }

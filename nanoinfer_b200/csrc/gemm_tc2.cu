@@ -149,6 +149,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t r[32]) {
 struct TcParams {
     void* out;
     int M, N, K, mode;
+    float act1, act2; // the gate's activation (ni_gate_act)
     int* error;       // device word: 0, or where a wait gave up
 };
 
@@ -202,7 +203,7 @@ __device__ __forceinline__ void tc_epilogue_row(const TcParams& p, int row, int 
             for (int j = 0; j < 4; ++j) {
                 const float g0 = __uint_as_float(v[16 * b + 2 * j]), g1 = __uint_as_float(v[16 * b + 2 * j + 1]);
                 const float u0 = __uint_as_float(v[16 * b + 8 + 2 * j]), u1 = __uint_as_float(v[16 * b + 8 + 2 * j + 1]);
-                __nv_bfloat162 r = __floats2bfloat162_rn((g0 / (1.0f + expf(-g0))) * u0, (g1 / (1.0f + expf(-g1))) * u1);
+                __nv_bfloat162 r = __floats2bfloat162_rn(ni_gate_act(g0, p.act1, p.act2) * u0, ni_gate_act(g1, p.act1, p.act2) * u1);
                 wp[j] = *reinterpret_cast<uint32_t*>(&r);
             }
             *reinterpret_cast<uint4*>(o + 8 * b) = w;
@@ -427,13 +428,16 @@ NI_EXPORT int ni_gemm_tc2_set_wait(long long ticks, int extra_wait) {
 }
 
 // a: bf16 [M, K]; b: bf16 [N, K]; K a multiple of 8; both 16-byte aligned.  mode 0 store bf16 [M, N],
-// 1 store FP32, 2 add into FP32 [M, N], 3 SwiGLU over blocked columns -> bf16 [M, N / 2].
+// 1 store FP32, 2 add into FP32 [M, N], 3 SwiGLU over blocked columns -> bf16 [M, N / 2] (with NI_MODE_GELU
+// added: the gate's activation is gelu).
 // error: a device int, zero on entry; non-zero afterwards if a wait inside the kernel ran out.
 // accumulators: 1 or 2 per block.  tile_n: 128, 192 or 256 columns per tile, or 0: as many as give every
 // pair of SMs about two tiles.
 NI_EXPORT int ni_gemm_tc2(const void* a, const void* b, void* out, int M, int N, int K, int mode, int accumulators,
                           int tile_n, int* error, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return NI_OK;
+    const bool gelu = mode == (TC_SWIGLU | NI_MODE_GELU);
+    if (gelu) mode = TC_SWIGLU;
     if (K <= 0 || mode < 0 || mode > TC_SWIGLU || error == nullptr) return NI_ERR_BAD_ARGUMENT;
     if (K % 8 || ((uintptr_t)a & 15) || ((uintptr_t)b & 15)) return NI_ERR_UNSUPPORTED_SIZE;
     if (mode == TC_SWIGLU && N % 16) return NI_ERR_UNSUPPORTED_SIZE;
@@ -451,6 +455,7 @@ NI_EXPORT int ni_gemm_tc2(const void* a, const void* b, void* out, int M, int N,
     if (rc != NI_OK) return rc;
     TcParams p;
     p.out = out; p.M = M; p.N = N; p.K = K; p.mode = mode; p.error = error;
+    p.act1 = gelu ? NI_GELU_C1 : 1.f; p.act2 = gelu ? NI_GELU_C2 : 0.f;
     const bool one = accumulators == 1;
     if (tile_n == 128) return one ? launch_tc2<128, 1>(ma, mb, p, stream) : launch_tc2<128, 2>(ma, mb, p, stream);
     if (tile_n == 192) return one ? launch_tc2<192, 1>(ma, mb, p, stream) : launch_tc2<192, 2>(ma, mb, p, stream);

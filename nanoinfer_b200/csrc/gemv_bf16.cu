@@ -62,6 +62,10 @@ struct GemvParams {
     __nv_bfloat16* next_x;
     float* next_ssq;          // [8 rows][next_parts]: a row's partial sums lie together (parts: a multiple of 4; what no tile writes stays 0)
     int next_parts;
+    // GV_ADD_F32: out += product * add_scale[n] + add_shift[n] (null: 1 and 0)
+    const float* add_scale;
+    const float* add_shift;
+    float act1, act2;         // GV_SWIGLU: the gate's activation (ni_gate_act)
     const float* pre_ssq;     // [8 rows][pre_parts]
     int pre_parts;
     float pre_eps;
@@ -101,6 +105,13 @@ __device__ __forceinline__ void gv_warm(const GemvParams& p) {
         const unsigned int sz = p.warm_bytes - off < PIECE ? (unsigned int)(p.warm_bytes - off) : PIECE;
         asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;\n" ::"l"(p.warm + off), "r"(sz) : "memory");
     }
+}
+
+// What a finished product adds to its column of the stream.
+__device__ __forceinline__ float gv_scaled(const GemvParams& p, float s, int n) {
+    if (p.add_scale) s *= p.add_scale[n];
+    if (p.add_shift) s += p.add_shift[n];
+    return s;
 }
 
 // One lane's share of the sum of a row of n floats (n a multiple of 4, the row 16-byte aligned).
@@ -333,7 +344,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32, (NT == 1 && U <= 4) ? 2 : 1) ge
                 float v = 0.f;
                 if (ok) {
                     const size_t o = (size_t)m * N + n;
-                    v = reinterpret_cast<float*>(p.out)[o] + tile[m][row];
+                    v = reinterpret_cast<float*>(p.out)[o] + gv_scaled(p, tile[m][row], n);
                     reinterpret_cast<float*>(p.out)[o] = v;
                     p.next_x[o] = __float2bfloat16_rn(v * p.next_gain[n]);
                 }
@@ -350,7 +361,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32, (NT == 1 && U <= 4) ? 2 : 1) ge
                 const size_t o = (size_t)m * N + n;
                 if (mode == GV_STORE_BF16) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(s);
                 else if (mode == GV_STORE_F32) reinterpret_cast<float*>(p.out)[o] = s;
-                else reinterpret_cast<float*>(p.out)[o] += s;
+                else reinterpret_cast<float*>(p.out)[o] += gv_scaled(p, s, n);
             }
         } else if (mode == GV_SWIGLU) {
             // rows 0..7 of the tile: gate; rows 8..15: the matching up rows (RN == 16)
@@ -359,7 +370,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32, (NT == 1 && U <= 4) ? 2 : 1) ge
                 if (m >= M || n0 + r + 8 >= N) continue;
                 const float gt = tile[m][r], up = tile[m][r + 8];
                 reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * (N / 2) + (n0 >> 1) + r] =
-                    __float2bfloat16_rn((gt / (1.0f + expf(-gt))) * up);
+                    __float2bfloat16_rn(ni_gate_act(gt, p.act1, p.act2) * up);
             }
         } else {  // GV_ROPE_KV: rows come in adjacent rotary pairs; a tile never straddles a head
             const int hd = p.head_dim, nq = p.n_q_heads, nkv = p.n_kv_heads;
@@ -446,12 +457,16 @@ static int launch_gemv(const GemvParams& p, int tiles_per_block, cudaStream_t st
     return launch_gemv_w<RN, NT, NORM, KEEP, U, false, 0>(p, tiles_per_block, stream);
 }
 
-static int dispatch_gemv(const GemvParams& p, bool norm, cudaStream_t stream) {
+static int dispatch_gemv(GemvParams& p, bool norm, cudaStream_t stream) {
+    const bool gelu = p.mode == (GV_SWIGLU | NI_MODE_GELU);
+    if (gelu) p.mode = GV_SWIGLU;
+    p.act1 = gelu ? NI_GELU_C1 : 1.f; p.act2 = gelu ? NI_GELU_C2 : 0.f;
     if (p.M <= 0 || p.N <= 0) return NI_OK;
     if (p.K <= 0 || p.mode < 0 || p.mode > GV_ROPE_KV) return NI_ERR_BAD_ARGUMENT;
     if (p.M > 16 || p.K % 8) return NI_ERR_UNSUPPORTED_SIZE;
     // 16 rows per tile unless that leaves SMs idle; the fused epilogues need whole 16-row tiles
-    const bool rn16 = p.mode >= GV_SWIGLU || (p.N + 15) / 16 >= 2 * ni_sm_count();
+    // ... and so does the reader of a handed-over norm
+    const bool rn16 = p.mode >= GV_SWIGLU || p.pre_ssq || (p.N + 15) / 16 >= 2 * ni_sm_count();
     if (p.mode == GV_SWIGLU && p.N % 16) return NI_ERR_UNSUPPORTED_SIZE;
     if (p.mode == GV_ROPE_KV && (p.head_dim % 16 || p.rotary_dim % 2 ||
                                  p.N != (p.n_q_heads + 2 * p.n_kv_heads) * p.head_dim))
@@ -511,21 +526,24 @@ NI_EXPORT int ni_gemv_bf16_writes_handoff(int M, int N, int K) { return M >= 1 &
 NI_EXPORT int ni_gemv_bf16_reads_handoff(int M, int K) { return M >= 1 && M <= 8 && K >= 8 && K % 8 == 0 && K <= 64 * GV_WARPS * 8; }
 
 // next_gain / next_x / next_ssq: with mode 2, also prepare the norm that follows (see GemvParams);
+// add_scale / add_shift [N], with mode 2: out += product * add_scale[n] + add_shift[n] (null: 1 and 0).  Mode 3 with
+// NI_MODE_GELU added: the gate's activation is gelu.
 // pre_ssq / pre_parts / pre_eps: x is such a prepared input.  Null pointers switch either off; sizes for
 // which the variant does not exist are refused (-2).
 NI_EXPORT int ni_gemv_bf16(const void* x, const void* w, void* out, int M, int N, int K, int mode,
                            const void* warm, long long warm_bytes, const float* next_gain, void* next_x,
                            float* next_ssq, int next_parts, const float* pre_ssq, int pre_parts, float pre_eps,
-                           cudaStream_t stream) {
+                           const float* add_scale, const float* add_shift, cudaStream_t stream) {
     if (mode == GV_ROPE_KV || !gv_warm_ok(warm, warm_bytes)) return NI_ERR_BAD_ARGUMENT;
+    if ((add_scale || add_shift) && mode != GV_ADD_F32) return NI_ERR_BAD_ARGUMENT;
     if (next_gain && (mode != GV_ADD_F32 || !next_x || !next_ssq || pre_ssq || next_parts % 4 ||
                       next_parts < ni_gemv_bf16_out_tiles(N, mode)))
         return NI_ERR_BAD_ARGUMENT;
     if (pre_ssq && (pre_parts <= 0 || pre_parts % 4 || ((uintptr_t)pre_ssq & 15))) return NI_ERR_BAD_ARGUMENT;
-    if (pre_ssq && mode != GV_SWIGLU && (N + 15) / 16 < 2 * ni_sm_count()) return NI_ERR_UNSUPPORTED_SIZE;   // (the reader has 16-row tiles)
     GemvParams p = {};
     p.next_gain = next_gain; p.next_x = (__nv_bfloat16*)next_x; p.next_ssq = next_ssq; p.next_parts = next_parts;
     p.pre_ssq = pre_ssq; p.pre_parts = pre_parts; p.pre_eps = pre_eps;
+    p.add_scale = add_scale; p.add_shift = add_shift;
     p.warm = (const unsigned char*)warm; p.warm_bytes = (unsigned long long)warm_bytes;
     p.x = x; p.w = (const __nv_bfloat16*)w; p.out = out; p.M = M; p.N = N; p.K = K; p.mode = mode;
     return dispatch_gemv(p, false, stream);

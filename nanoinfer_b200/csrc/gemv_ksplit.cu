@@ -49,7 +49,15 @@ struct KsParams {
     __nv_bfloat16* next_x;
     float* next_ssq;          // [8 rows][next_parts]
     int next_parts;
+    const float* add_scale;   // KS_ADD_F32: out += product * add_scale[n] + add_shift[n] (null: 1 and 0)
+    const float* add_shift;
 };
+
+__device__ __forceinline__ float ks_scaled(const KsParams& p, float s, int n) {
+    if (p.add_scale) s *= p.add_scale[n];
+    if (p.add_shift) s += p.add_shift[n];
+    return s;
+}
 
 __device__ __forceinline__ void ks_mma(float c[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
                                        uint32_t b0, uint32_t b1) {
@@ -198,7 +206,7 @@ __global__ void __launch_bounds__(KS_WARPS * 32, 2) gemv_ksplit_kernel(const KsP
             float v = 0.f;
             if (m < M && n < N) {
                 const size_t o = (size_t)m * N + n;
-                v = reinterpret_cast<float*>(p.out)[o] + s;
+                v = reinterpret_cast<float*>(p.out)[o] + ks_scaled(p, s, n);
                 reinterpret_cast<float*>(p.out)[o] = v;
                 p.next_x[o] = __float2bfloat16_rn(v * p.next_gain[n]);
             }
@@ -218,7 +226,7 @@ __global__ void __launch_bounds__(KS_WARPS * 32, 2) gemv_ksplit_kernel(const KsP
         const size_t o = (size_t)m * N + n;
         if (mode == KS_STORE_BF16) reinterpret_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(s);
         else if (mode == KS_STORE_F32) reinterpret_cast<float*>(p.out)[o] = s;
-        else reinterpret_cast<float*>(p.out)[o] += s;
+        else reinterpret_cast<float*>(p.out)[o] += ks_scaled(p, s, n);
     }
 }
 
@@ -288,10 +296,12 @@ NI_EXPORT int ni_gemv_ksplit_out_tiles(int N, int K) {
 // next_gain / next_x / next_ssq: with mode 2, also prepare the norm that follows (null: off).
 NI_EXPORT int ni_gemv_ksplit(const void* x, const void* w, void* out, int M, int N, int K, int mode,
                              const void* warm, long long warm_bytes, const float* next_gain, void* next_x,
-                             float* next_ssq, int next_parts, cudaStream_t stream) {
+                             float* next_ssq, int next_parts, const float* add_scale, const float* add_shift,
+                             cudaStream_t stream) {
     if (M <= 0 || N <= 0) return NI_OK;
     if (mode < KS_STORE_BF16 || mode > KS_ADD_F32) return NI_ERR_BAD_ARGUMENT;
     if (next_gain && (mode != KS_ADD_F32 || !next_x || !next_ssq)) return NI_ERR_BAD_ARGUMENT;
+    if ((add_scale || add_shift) && mode != KS_ADD_F32) return NI_ERR_BAD_ARGUMENT;
     if (warm_bytes < 0 || (warm_bytes & 15) || (warm_bytes && (!warm || ((uintptr_t)warm & 15)))) return NI_ERR_BAD_ARGUMENT;
     KsPlan plan;
     if (M > 8 || K <= 0 || K % 8 || !ks_plan(N, K, &plan)) return NI_ERR_UNSUPPORTED_SIZE;
@@ -300,6 +310,7 @@ NI_EXPORT int ni_gemv_ksplit(const void* x, const void* w, void* out, int M, int
     p.M = M; p.N = N; p.K = K; p.mode = mode;
     p.splits = plan.splits; p.slice_blocks = plan.slice_blocks; p.tiles_per_cluster = plan.tiles_per_cluster;
     p.warm = (const unsigned char*)warm; p.warm_bytes = (unsigned long long)warm_bytes;
+    p.add_scale = add_scale; p.add_shift = add_shift;
     p.next_gain = next_gain; p.next_x = (__nv_bfloat16*)next_x; p.next_ssq = next_ssq; p.next_parts = next_parts;
     if (next_gain && (next_parts % 4 || next_parts < (N + plan.rn - 1) / plan.rn)) return NI_ERR_BAD_ARGUMENT;
 #define KS_GO(RN)                                                                       \

@@ -103,6 +103,53 @@ NI_EXPORT int ni_head_gate(void* x, int dtype, const void* proj, int ld, int col
 }
 
 
+// One gate per ELEMENT: out[t, out_col + i] = x[t, i] * sigmoid(gate[t, i]) * scale, i < n; x [T, n], gate rows ld_g apart,
+// out rows ld_o apart (out may be x itself).  VEC numbers per thread.
+template <typename T, typename TG, int VEC>
+__global__ void element_gate_kernel(const T* __restrict__ x, const TG* __restrict__ gate, int ld_g, T* out, int ld_o, int n,
+                                    long long total, float scale) {
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (i >= total) return;
+    const long long t = i / n;
+    const int c = (int)(i - t * n);
+    if (VEC == 1) {
+        const float g = scale / (1.0f + expf(-ni_to_float(gate[t * ld_g + c])));
+        out[t * ld_o + c] = ni_from_float<T>(ni_to_float(x[i]) * g);
+        return;
+    }
+    float v[VEC], g[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; k += NiVec16<T>::N) NiVec16<T>::load(x + i + k, v + k);
+#pragma unroll
+    for (int k = 0; k < VEC; k += NiVec16<TG>::N) NiVec16<TG>::load(gate + t * ld_g + c + k, g + k);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] *= scale / (1.0f + expf(-g[k]));
+#pragma unroll
+    for (int k = 0; k < VEC; k += NiVec16<T>::N) NiVec16<T>::store(out + t * ld_o + c + k, v + k);
+}
+
+NI_EXPORT int ni_element_gate(const void* x, int dtype, const void* gate, int gate_dtype, int ld_g, void* out, int ld_o,
+                              int n_tokens, int n, float scale, cudaStream_t stream) {
+    if (n_tokens <= 0) return NI_OK;
+    if (n <= 0 || ld_g < n || ld_o < n) return NI_ERR_BAD_ARGUMENT;
+    const long long total = (long long)n_tokens * n;
+    const auto aligned = [](const void* p) { return (reinterpret_cast<size_t>(p) & 15) == 0; };
+    const bool wide = n % 8 == 0 && ld_g % 8 == 0 && ld_o % 8 == 0 && aligned(x) && aligned(gate) && aligned(out);
+    const long long blocks = ((wide ? total / 8 : total) + 255) / 256;
+    if (blocks > 2147483647LL) return NI_ERR_UNSUPPORTED_SIZE;
+#define GO(T, TG)                                                                                                          \
+    do {                                                                                                                   \
+        if (wide) element_gate_kernel<T, TG, 8><<<(int)blocks, 256, 0, stream>>>((const T*)x, (const TG*)gate, ld_g, (T*)out, ld_o, n, total, scale); \
+        else element_gate_kernel<T, TG, 1><<<(int)blocks, 256, 0, stream>>>((const T*)x, (const TG*)gate, ld_g, (T*)out, ld_o, n, total, scale);      \
+    } while (0)
+    if (dtype == NI_DTYPE_F32 && gate_dtype == NI_DTYPE_F32) GO(float, float);
+    else if (dtype == NI_DTYPE_BF16 && gate_dtype == NI_DTYPE_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else if (dtype == NI_DTYPE_BF16 && gate_dtype == NI_DTYPE_F32) GO(__nv_bfloat16, float);
+    else return NI_ERR_BAD_ARGUMENT;
+#undef GO
+    NI_RETURN_LAUNCH_STATUS();
+}
+
 // A latent cache row with a rotated key part: beside c = RMSNorm(first R columns) * weight a token keeps rot_dim more
 // numbers - one key part that all heads share and that is rotated by position - so a page row is [c | rot(k_r)], R +
 // rot_dim wide.  The same launch rotates the last rot_dim dimensions of every head of q [T, H (R + rot_dim)] in place

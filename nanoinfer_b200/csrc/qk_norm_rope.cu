@@ -9,17 +9,38 @@
 //            a = float(position) * inv_freq[i]  (m = `magnitude`: an encoding that also scales what it rotates)
 //   (optional, `head_unit`) every head of q and of k divided by its own root mean square over D, eps inside the
 //            root, no weight - after the rotation
+//   (optional, temp_coef) q <- q * (1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)): a factor on the finished
+//            query that grows with the position
+//   (optional, first_v) v <- (1 - lambda) v + lambda (first + first_bias): another layer's values of the same token, as
+//            that layer's projection holds them, mixed in
 //   q -> q_out [T, H D];  k -> key pages [P, G, page, D];  v -> value pages [P, G, page, V]
 //
 // One block per token.  The row's queries and keys are widened once into shared memory, where the two sums of
 // squares and the partner of every rotated dimension are found; the angles' cosines and sines are computed
-// once per token and shared by all heads.
+// once per token and shared by all heads.  The projection may be FP32 where queries and pages are bfloat16.
 #include "common.cuh"
+
+// What the options need beyond sizes and tables.
+template <typename TI> struct QkExtra {
+    float temp_coef, temp_every;      // temp_coef 0: no factor
+    const TI* first_v;                // the other layer's value columns [T, first_ld], or null
+    int first_ld;
+    const float* first_bias;          // [G V] or null
+    float lambda;
+};
+__device__ __forceinline__ float qk_temperature(float coef, float every, int pos) {
+    return coef == 0.f ? 1.f : 1.f + coef * logf(floorf((float)(pos + 1) / every) + 1.f);
+}
+// VEC neighbouring numbers of a row (16-byte aligned), widened.
+template <typename T, int VEC> __device__ __forceinline__ void qk_load(const T* p, float* v) {
+#pragma unroll
+    for (int k = 0; k < VEC; k += NiVec16<T>::N) NiVec16<T>::load(p + k, v + k);
+}
 
 // The heads' own norms: vals [(H + G) D] in shared memory holds the token's finished queries and keys; a warp takes
 // a head at a time, divides it by its root mean square and writes it out (a key only where there are pages).
 template <typename T>
-__device__ __forceinline__ void qk_head_unit_write(const float* __restrict__ vals, float eps, T* __restrict__ q_row,
+__device__ __forceinline__ void qk_head_unit_write(const float* __restrict__ vals, float eps, float temp, T* __restrict__ q_row,
                                                    T* __restrict__ kdst, int H, int G, int D, int page_size) {
     __syncthreads();
     const int lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -28,29 +49,30 @@ __device__ __forceinline__ void qk_head_unit_write(const float* __restrict__ val
         float ss = 0.f;
         for (int d = lane; d < D; d += 32) ss = fmaf(x[d], x[d], ss);
         ss = ni_warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss / (float)D + eps);
+        const float inv = (head < H ? temp : 1.0f) / sqrtf(ss / (float)D + eps);
         T* dst = head < H ? q_row + (size_t)head * D : (kdst ? kdst + (size_t)(head - H) * page_size * D : nullptr);
         if (dst)
             for (int d = lane; d < D; d += 32) dst[d] = ni_from_float<T>(x[d] * inv);
     }
 }
 
-template <typename T>
+template <typename TI, typename T>
 __global__ void __launch_bounds__(256)
-qk_norm_rope_kernel(const T* __restrict__ qkv, int ld, const float* __restrict__ bias,
+qk_norm_rope_kernel(const TI* __restrict__ qkv, int ld, const float* __restrict__ bias,
                     const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                     const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                     const int* __restrict__ block_table, int bt_stride, const float* __restrict__ inv_freq,
                     float magnitude, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                    int H, int G, int D, int V, int rotary_dim, int page_size, int head_unit) {
+                    int H, int G, int D, int V, int rotary_dim, int page_size, int head_unit, const QkExtra<TI> ex) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float scratch[32];
     const int nq = H * D, nk = G * D, nv = G * V, half = rotary_dim >> 1;
     float* row = sm;                 // [nq + nk]: queries, then keys, bias added
     float* cs = sm + nq + nk;        // [2 half]: m cos, then m sin
     const int t = blockIdx.x;
-    const T* x = qkv + (size_t)t * ld;
+    const TI* x = qkv + (size_t)t * ld;
     const int pos = positions[t];
+    const float temp = qk_temperature(ex.temp_coef, ex.temp_every, pos);
     float sq = 0.f, sk = 0.f;
     for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
         const float v = ni_to_float(x[i]) + (bias ? bias[i] : 0.f);
@@ -90,14 +112,18 @@ qk_norm_rope_kernel(const T* __restrict__ qkv, int ld, const float* __restrict__
             a = first ? a * cs[f] - b * cs[half + f] : a * cs[f] + b * cs[half + f];
         }
         if (head_unit) cs[rotary_dim + i] = a;            // kept for the heads' own norms below
-        else if (is_q) q_out[(size_t)t * nq + e] = ni_from_float<T>(a);
+        else if (is_q) q_out[(size_t)t * nq + e] = ni_from_float<T>(a * temp);
         else if (kdst) kdst[(size_t)head * page_size * D + dim] = ni_from_float<T>(a);
     }
-    if (head_unit) qk_head_unit_write<T>(cs + rotary_dim, eps, q_out + (size_t)t * nq, kdst, H, G, D, page_size);
+    if (head_unit) qk_head_unit_write<T>(cs + rotary_dim, eps, temp, q_out + (size_t)t * nq, kdst, H, G, D, page_size);
     if (vdst) {
         for (int i = threadIdx.x; i < nv; i += blockDim.x) {
             const int head = i / V, dim = i - head * V;
-            const float v = ni_to_float(x[nq + nk + i]) + (bias ? bias[nq + nk + i] : 0.f);
+            float v = ni_to_float(x[nq + nk + i]) + (bias ? bias[nq + nk + i] : 0.f);
+            if (ex.first_v) {
+                const float f = ni_to_float(ex.first_v[(size_t)t * ex.first_ld + i]) + (ex.first_bias ? ex.first_bias[i] : 0.f);
+                v = (1.0f - ex.lambda) * v + ex.lambda * f;
+            }
             vdst[(size_t)head * page_size * V + dim] = ni_from_float<T>(v);
         }
     }
@@ -105,14 +131,14 @@ qk_norm_rope_kernel(const T* __restrict__ qkv, int ld, const float* __restrict__
 
 // The same with 16 bytes per load and store: a thread owns VEC neighbouring dimensions (8 bfloat16 or 4 floats).
 // For sizes whose heads, rotated halves and rows all start on 16 bytes (the launcher checks).
-template <typename T>
+template <typename TI, typename T>
 __global__ void __launch_bounds__(256)
-qk_norm_rope_vec_kernel(const T* __restrict__ qkv, int ld, const float* __restrict__ bias,
+qk_norm_rope_vec_kernel(const TI* __restrict__ qkv, int ld, const float* __restrict__ bias,
                         const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                         const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                         const int* __restrict__ block_table, int bt_stride, const float* __restrict__ inv_freq,
                         float magnitude, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                        int H, int G, int D, int V, int rotary_dim, int page_size, int head_unit) {
+                        int H, int G, int D, int V, int rotary_dim, int page_size, int head_unit, const QkExtra<TI> ex) {
     constexpr int VEC = 16 / sizeof(T);
     extern __shared__ __align__(16) float sm[];
     __shared__ float scratch[32];
@@ -120,15 +146,13 @@ qk_norm_rope_vec_kernel(const T* __restrict__ qkv, int ld, const float* __restri
     float* row = sm;                 // [nq + nk]: queries, then keys, bias added
     float* cs = sm + nq + nk;        // [2 half]: m cos, then m sin
     const int t = blockIdx.x;
-    const T* x = qkv + (size_t)t * ld;
+    const TI* x = qkv + (size_t)t * ld;
     const int pos = positions[t];
+    const float temp = qk_temperature(ex.temp_coef, ex.temp_every, pos);
     float sq = 0.f, sk = 0.f;
     for (int i = threadIdx.x * VEC; i < nq + nk; i += blockDim.x * VEC) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(x + i);
-        const T* e = reinterpret_cast<const T*>(&raw);
         float v[VEC];
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) v[k] = ni_to_float(e[k]);
+        qk_load<TI, VEC>(x + i, v);
         if (bias) {
 #pragma unroll
             for (int k = 0; k < VEC; k += 4) {
@@ -160,13 +184,20 @@ qk_norm_rope_vec_kernel(const T* __restrict__ qkv, int ld, const float* __restri
     if (vdst) {                               // the values do not wait for the sums
         for (int i = threadIdx.x * VEC; i < nv; i += blockDim.x * VEC) {
             const int head = i / V, dim = i - head * V;
-            uint4 raw = *reinterpret_cast<const uint4*>(x + nq + nk + i);
+            float v[VEC];
+            qk_load<TI, VEC>(x + nq + nk + i, v);
             if (bias) {
-                T* e = reinterpret_cast<T*>(&raw);
 #pragma unroll
-                for (int k = 0; k < VEC; ++k) e[k] = ni_from_float<T>(ni_to_float(e[k]) + bias[nq + nk + i + k]);
+                for (int k = 0; k < VEC; ++k) v[k] += bias[nq + nk + i + k];
             }
-            *reinterpret_cast<uint4*>(vdst + (size_t)head * page_size * V + dim) = raw;
+            if (ex.first_v) {
+                float f[VEC];
+                qk_load<TI, VEC>(ex.first_v + (size_t)t * ex.first_ld + i, f);
+#pragma unroll
+                for (int k = 0; k < VEC; ++k)
+                    v[k] = (1.0f - ex.lambda) * v[k] + ex.lambda * (f[k] + (ex.first_bias ? ex.first_bias[i + k] : 0.f));
+            }
+            NiVec16<T>::store(vdst + (size_t)head * page_size * V + dim, v);
         }
     }
     sq = ni_block_sum(sq, scratch);
@@ -200,59 +231,57 @@ qk_norm_rope_vec_kernel(const T* __restrict__ qkv, int ld, const float* __restri
         uint4 packed;
         T* o = reinterpret_cast<T*>(&packed);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) o[k] = ni_from_float<T>(a[k]);
+        for (int k = 0; k < VEC; ++k) o[k] = ni_from_float<T>(is_q ? a[k] * temp : a[k]);
         if (is_q) *reinterpret_cast<uint4*>(q_out + (size_t)t * nq + e) = packed;
         else if (kdst) *reinterpret_cast<uint4*>(kdst + (size_t)head * page_size * D + dim) = packed;
     }
-    if (head_unit) qk_head_unit_write<T>(cs + rotary_dim, eps, q_out + (size_t)t * nq, kdst, H, G, D, page_size);
+    if (head_unit) qk_head_unit_write<T>(cs + rotary_dim, eps, temp, q_out + (size_t)t * nq, kdst, H, G, D, page_size);
 }
 
 // qkv [T, ld] with columns q (H D) | k (G D) | v (G V); bias FP32 [H D + G D + G V] or null; q_gain FP32 [H D] and
 // k_gain FP32 [G D], or null for no norm; head_unit: the heads' own norms after the rotation; k_pages / v_pages null: nothing is written (a run that reads another's cache).
-NI_EXPORT int ni_qk_norm_rope(const void* qkv, int dtype, int ld, const float* bias, const float* q_gain,
+// dtype: queries and pages; in_dtype: qkv and first_v (FP32 beside bfloat16 is allowed).  temp_coef 0: no factor on the
+// query.  first_v null: no mixing of values; else the other layer's value columns, row stride first_ld (see QkExtra).
+NI_EXPORT int ni_qk_norm_rope(const void* qkv, int in_dtype, int dtype, int ld, const float* bias, const float* q_gain,
                               const float* k_gain, float eps, const int* positions, const int* seq_of_token,
                               const int* block_table, int bt_stride, const float* inv_freq, float magnitude, void* q_out,
                               void* k_pages, void* v_pages, int n_tokens, int H, int G, int D, int V, int rotary_dim,
-                              int page_size, int head_unit, cudaStream_t stream) {
+                              int page_size, int head_unit, float temp_coef, float temp_every, const void* first_v,
+                              int first_ld, const float* first_bias, float lambda, cudaStream_t stream) {
     if (n_tokens <= 0) return NI_OK;
     if (H <= 0 || G <= 0 || D <= 0 || V <= 0 || page_size <= 0 || rotary_dim < 0 || rotary_dim > D || (rotary_dim & 1) ||
-        ld < (H + G) * D + G * V || (q_gain == nullptr) != (k_gain == nullptr))
+        ld < (H + G) * D + G * V || (q_gain == nullptr) != (k_gain == nullptr) || (first_v && first_ld < G * V) ||
+        (temp_coef != 0.f && !(temp_every > 0.f)))
         return NI_ERR_BAD_ARGUMENT;
     const size_t smem = ((size_t)(H + G) * D * (head_unit ? 2 : 1) + rotary_dim) * sizeof(float);
     if (smem > 200 * 1024) return NI_ERR_UNSUPPORTED_SIZE;
-    const int vec = dtype == NI_DTYPE_F32 ? 4 : 8;       // elements in 16 bytes
+    const int vec = dtype == NI_DTYPE_F32 ? 4 : 8;       // elements in 16 bytes of the output
     const auto aligned = [](const void* p) { return (reinterpret_cast<size_t>(p) & 15) == 0; };
     const bool wide = D % vec == 0 && V % vec == 0 && (rotary_dim / 2) % vec == 0 && ld % vec == 0 && aligned(qkv) &&
-                      aligned(q_out) && aligned(k_pages) && aligned(v_pages) && aligned(bias);
-#define LAUNCH_VEC(T)                                                                                                \
+                      aligned(q_out) && aligned(k_pages) && aligned(v_pages) && aligned(bias) && first_ld % vec == 0 &&
+                      aligned(first_v);
+    const int work = ((H + G) * D + vec - 1) / vec;
+    const int threads = !wide ? 256 : (work >= 256 ? 256 : (work >= 128 ? 128 : 64));
+#define LAUNCH_K(KERNEL, TI, T)                                                                                      \
     do {                                                                                                             \
+        const QkExtra<TI> ex = {temp_coef, temp_every, (const TI*)first_v, first_ld, first_bias, lambda};            \
         if (smem > 48 * 1024)                                                                                        \
-            cudaFuncSetAttribute(qk_norm_rope_vec_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        qk_norm_rope_vec_kernel<T><<<n_tokens, threads, smem, stream>>>((const T*)qkv, ld, bias, q_gain, k_gain, eps, \
-                                                                    positions, seq_of_token, block_table, bt_stride, \
-                                                                    inv_freq, magnitude, (T*)q_out, (T*)k_pages,     \
-                                                                    (T*)v_pages, H, G, D, V, rotary_dim, page_size, head_unit); \
+            cudaFuncSetAttribute(KERNEL<TI, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);             \
+        KERNEL<TI, T><<<n_tokens, threads, smem, stream>>>((const TI*)qkv, ld, bias, q_gain, k_gain, eps, positions, \
+                                                           seq_of_token, block_table, bt_stride, inv_freq, magnitude, \
+                                                           (T*)q_out, (T*)k_pages, (T*)v_pages, H, G, D, V,          \
+                                                           rotary_dim, page_size, head_unit, ex);                    \
     } while (0)
-    if (wide && (dtype == NI_DTYPE_F32 || dtype == NI_DTYPE_BF16)) {
-        const int work = ((H + G) * D + vec - 1) / vec;
-        const int threads = work >= 256 ? 256 : (work >= 128 ? 128 : 64);
-        if (dtype == NI_DTYPE_F32) LAUNCH_VEC(float);
-        else LAUNCH_VEC(__nv_bfloat16);
-        NI_RETURN_LAUNCH_STATUS();
-    }
-#undef LAUNCH_VEC
-#define LAUNCH(T)                                                                                                    \
-    do {                                                                                                             \
-        if (smem > 48 * 1024)                                                                                        \
-            cudaFuncSetAttribute(qk_norm_rope_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-        qk_norm_rope_kernel<T><<<n_tokens, 256, smem, stream>>>((const T*)qkv, ld, bias, q_gain, k_gain, eps,       \
-                                                                positions, seq_of_token, block_table, bt_stride,     \
-                                                                inv_freq, magnitude, (T*)q_out, (T*)k_pages,         \
-                                                                (T*)v_pages, H, G, D, V, rotary_dim, page_size, head_unit);     \
+#define LAUNCH(TI, T)                                                \
+    do {                                                             \
+        if (wide) LAUNCH_K(qk_norm_rope_vec_kernel, TI, T);          \
+        else LAUNCH_K(qk_norm_rope_kernel, TI, T);                   \
     } while (0)
-    if (dtype == NI_DTYPE_F32) LAUNCH(float);
-    else if (dtype == NI_DTYPE_BF16) LAUNCH(__nv_bfloat16);
+    if (dtype == NI_DTYPE_F32 && in_dtype == NI_DTYPE_F32) LAUNCH(float, float);
+    else if (dtype == NI_DTYPE_BF16 && in_dtype == NI_DTYPE_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
+    else if (dtype == NI_DTYPE_BF16 && in_dtype == NI_DTYPE_F32) LAUNCH(float, __nv_bfloat16);
     else return NI_ERR_BAD_ARGUMENT;
 #undef LAUNCH
+#undef LAUNCH_K
     NI_RETURN_LAUNCH_STATUS();
 }

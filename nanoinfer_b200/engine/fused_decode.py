@@ -44,6 +44,8 @@ class FusedDecode:
         for b in blocks:
             if type(b) is not PreNormBlock or type(b.mixer) is not PagedAttention or type(b.feed_forward) is not SwiGLU:
                 return None
+            if b.feed_forward.gelu or b.feed_forward.affine is not None or b.scales != [None, None]:
+                return None
             if type(b.mixer_norm) is not RMSNorm or type(b.ffn_norm) is not RMSNorm or not b.feed_forward.blocked:
                 return None
         first = blocks[0].mixer

@@ -140,22 +140,24 @@ class Runtime:
         return ops.NormHandoff(norm, norm.gain, norm.eps, n_rows, n_out, tiles, self.device) if tiles > 0 else None
 
     def linear(self, x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-               residual: Optional[torch.Tensor] = None, warm=None, handoff=None) -> Optional[torch.Tensor]:
+               residual: Optional[torch.Tensor] = None, warm=None, handoff=None, affine=None):
         """y[M, N] = x[M, K] . w[N, K]^T.  ``out_dtype`` float32 asks for FP32 results
         (logits); the default is the compute dtype.  With ``residual`` (the FP32 residual
         stream) the kernel MAY add the product into it and return None; otherwise the product
-        is returned and the caller adds it.  ``warm``: a hint that the skinny kernel takes (see warm())."""
+        is returned and the caller adds it.  ``affine`` (scale, shift), float32 per column, either may be None: what is
+        added is the product * scale + shift (returned as an ops.ScaledAddition where it stays pending).  ``warm``: a hint
+        that the skinny kernel takes (see warm())."""
         m, n = x.shape[0], w.shape[0]
         out_dtype = out_dtype or self.dtype
         if self.dtype == torch.float32:
             out = self.empty(m, n, dtype=torch.float32)
             ops.gemm_f32(x, w, out)
-            return out
+            return out if affine is None else ops.ScaledAddition(out, *affine)
         if residual is None and self.swapped_gemm(m, n, x.shape[1]):
             out = self.empty(m, n, dtype=out_dtype)
             ops.gemm_swap_tc(x, w, out, ops.STORE_BF16 if out_dtype == torch.bfloat16 else ops.STORE_F32)
             return out
-        return ops.linear_bf16(x, w, out_dtype, residual, warm, handoff)
+        return ops.linear_bf16(x, w, out_dtype, residual, warm, handoff, affine)
 
     def heads_linear(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         """One product per head: y[t, h, :] = x[t, h, :] . w[h]^T for x [T, H K] (some columns of a wider

@@ -82,6 +82,8 @@ class StepContext:
     room may ask the head of them into L2 (``Runtime.warm``).
     norm_after: the norm part that reads the residual stream after the running block, if it can come
     prepared by the kernel that last adds into the stream (``ops.NormHandoff``); else None.
+    shared: what a layer leaves for later layers of the same step, by name (a projection whose columns others mix in);
+    written anew in every forward pass.
     """
     n_tokens: int
     n_seqs: int
@@ -103,6 +105,7 @@ class StepContext:
     plans: Dict[type, DevicePlan] = field(default_factory=dict)
     read_after: tuple = ()
     norm_after: object = None
+    shared: Dict[str, object] = field(default_factory=dict)
 
     def plan_of(self, part) -> DevicePlan:
         owner = plan_owner(type(part))

@@ -25,16 +25,17 @@ _ERRORS = {-1: "bad argument", -2: "size not supported by this kernel",
 _SIGNATURES = {
     "elementwise": {
         "ni_embedding": [_P, _P, _I, _P, _I, _I, _I, _P],
-        "ni_add_rmsnorm": [_P, _P, _I, _P, _F, _P, _I, _P, _I, _I, _P],
+        "ni_add_rmsnorm": [_P, _P, _I, _P, _F, _P, _I, _P, _I, _I, _P, _P, _P],
         "ni_residual_add": [_P, _P, _I, _LL, _P],
-        "ni_swiglu": [_P, _P, _I, _I, _I, _P],
-        "ni_swiglu_blocked": [_P, _P, _I, _I, _I, _P],
+        "ni_residual_add_scaled": [_P, _P, _I, _LL, _I, _P, _P, _P],
+        "ni_swiglu": [_P, _P, _I, _I, _I, _I, _P],
+        "ni_swiglu_blocked": [_P, _P, _I, _I, _I, _I, _P],
     },
     "rope_kv": {
         "ni_rope_kv_write": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     },
     "attention_generic": {
-        "ni_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _F, _I, _I, _I, _I, _P],
+        "ni_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _F, _I, _I, _P, _I, _P],
     },
     "gemm_f32": {
         "ni_gemm_f32": [_P, _P, _P, _I, _I, _I, _P],
@@ -56,7 +57,7 @@ _SIGNATURES = {
         "ni_embedding_pairs": [_P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P],
     },
     "qk_norm_rope": {
-        "ni_qk_norm_rope": [_P, _I, _I, _P, _P, _P, _F, _P, _P, _P, _I, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+        "ni_qk_norm_rope": [_P, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _I, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P, _F, _P],
     },
     "lightning": {
         "ni_lightning_recurrence": [_P, _I, _I, _P, _LL, _P, _P, _P, _P, _I, _I, _I, _P, _LL, _I, _I, _I, _I, _P],
@@ -91,17 +92,18 @@ _SIGNATURES = {
         "ni_route_combine_add_normed": [_P, _P, _I, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P],
     },
     "delta_rule": {
-        "ni_delta_prepare": [_P, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P],
-        "ni_delta_recurrence": [_P, _P, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
-        "ni_delta_gated_norm": [_P, _P, _P, _F, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _LL, _P, _P, _P],
+        "ni_delta_prepare": [_P, _I, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P],
+        "ni_delta_recurrence": [_P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
+        "ni_delta_gated_norm": [_P, _P, _I, _I, _P, _F, _F, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _LL, _P, _P, _P],
     },
     "latent": {
         "ni_latent_norm_write": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
         "ni_head_gate": [_P, _I, _P, _I, _I, _I, _I, _I, _F, _P],
+        "ni_element_gate": [_P, _I, _P, _I, _I, _P, _I, _I, _I, _F, _P],
         "ni_latent_rope_write": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _I, _P],
     },
     "gemv_bf16": {
-        "ni_gemv_bf16": [_P, _P, _P, _I, _I, _I, _I, _P, _LL, _P, _P, _P, _I, _P, _I, _F, _P],
+        "ni_gemv_bf16": [_P, _P, _P, _I, _I, _I, _I, _P, _LL, _P, _P, _P, _I, _P, _I, _F, _P, _P, _P],
         "ni_gemv_bf16_out_tiles": [_I, _I],
         "ni_gemv_bf16_writes_handoff": [_I, _I, _I],
         "ni_gemv_bf16_reads_handoff": [_I, _I],
@@ -109,14 +111,14 @@ _SIGNATURES = {
         "ni_gemv_qkv_rope": [_P, _P, _F, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _I, _F, _P],
     },
     "gemv_ksplit": {
-        "ni_gemv_ksplit": [_P, _P, _P, _I, _I, _I, _I, _P, _LL, _P, _P, _P, _I, _P],
+        "ni_gemv_ksplit": [_P, _P, _P, _I, _I, _I, _I, _P, _LL, _P, _P, _P, _I, _P, _P, _P],
         "ni_gemv_ksplit_out_tiles": [_I, _I],
         "ni_gemv_ksplit_supports": [_I, _I, _I],
     },
     "attention_decode": {
         "ni_attention_decode": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_capped": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P, _P, _LL, _P, _LL, _P],
-        "ni_attention_decode_masked": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _P, _P, _LL, _P, _LL, _P],
+        "ni_attention_decode_masked": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _I, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_difference": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _I, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_balanced": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _LL, _P, _LL, _P],
         "ni_attention_decode_fresh_keys": [],
@@ -125,11 +127,11 @@ _SIGNATURES = {
         "ni_attention_decode_noalloc": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     },
     "attention_prefill": {
-        "ni_attention_prefill": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I, _P],
+        "ni_attention_prefill": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P, _P],
     },
     "attention_prefill_tc": {
         "ni_attention_prefill_tc": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P],
-        "ni_attention_prefill_tc_masked": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P],
+        "ni_attention_prefill_tc_masked": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
         "ni_attention_prefill_tc_difference": [_P, _P, _P, _P, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P],
         "ni_attention_prefill_tc_supports": [_I, _I, _I, _I],
         "ni_attention_prefill_tc_set_wait": [_LL, _I],
@@ -287,16 +289,41 @@ def embedding(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor) -> N
                                             n, d, table.shape[0], _stream()), "embedding")
 
 
-def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
+class ScaledAddition:
+    """An addition still pending on the residual stream whose columns have a factor and a shift of their own: the stream
+    becomes h + y * scale + shift, with ``scale`` and ``shift`` float32 [d] or None.  Where a pending addition may be a
+    tensor it may be one of these."""
+
+    def __init__(self, y: torch.Tensor, scale: Optional[torch.Tensor], shift: Optional[torch.Tensor]) -> None:
+        self.y, self.scale, self.shift = y, scale, shift
+
+
+def _pending(delta) -> tuple:
+    """(tensor, scale, shift) of a pending addition: a tensor, a ScaledAddition or None."""
+    if isinstance(delta, ScaledAddition):
+        d = delta.y.shape[1]
+        for v in (delta.scale, delta.shift):
+            if v is not None and v.numel() != d:
+                raise KernelError("a pending addition's scale and shift must have its width")
+        return delta.y, delta.scale, delta.shift
+    return delta, None, None
+
+
+def _f32_or_none(t: Optional[torch.Tensor], name: str):
+    return _dev(t, name, torch.float32) if t is not None else None
+
+
+def add_rmsnorm(h: torch.Tensor, delta, gain: torch.Tensor, eps: float,
                 out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
     """Residual add fused with RMSNorm.
 
-    h float32 [T, d]; delta [T, d] or None; gain float32 [d]; out [R, d].
+    h float32 [T, d]; delta [T, d], a ScaledAddition or None; gain float32 [d]; out [R, d].
     rows None: R = T, h += delta in place, out = norm(h) * gain.
     rows int32 [R]: out[r] = norm(h[rows[r]] + delta[rows[r]]) * gain, h untouched.
     """
     d = h.shape[1]
     n_out = out.shape[0]
+    delta, scale, shift = _pending(delta)
     if out.shape[1] != d or gain.numel() != d:
         raise KernelError("add_rmsnorm: widths do not agree")
     if rows is None and n_out != h.shape[0]:
@@ -309,11 +336,20 @@ def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tens
         _dev(h, "h", torch.float32), _dev(delta, "delta") if delta is not None else None,
         _code(delta, "delta") if delta is not None else F32, _dev(gain, "gain", torch.float32),
         float(eps), _dev(out, "out"), _code(out, "out"),
-        _dev(rows, "rows", torch.int32) if rows is not None else None, n_out, d, _stream()),
-        "add_rmsnorm")
+        _dev(rows, "rows", torch.int32) if rows is not None else None, n_out, d, _f32_or_none(scale, "scale"),
+        _f32_or_none(shift, "shift"), _stream()), "add_rmsnorm")
 
 
-def residual_add(h: torch.Tensor, delta: torch.Tensor) -> None:
+def residual_add(h: torch.Tensor, delta) -> None:
+    """h += delta; delta [T, d] or a ScaledAddition."""
+    delta, scale, shift = _pending(delta)
+    if scale is not None or shift is not None:
+        if delta.shape != h.shape:
+            raise KernelError("residual_add: shapes do not agree")
+        _check(load("elementwise").ni_residual_add_scaled(
+            _dev(h, "h", torch.float32), _dev(delta, "delta"), _code(delta, "delta"), h.numel(), h.shape[1],
+            _f32_or_none(scale, "scale"), _f32_or_none(shift, "shift"), _stream()), "residual_add")
+        return
     if delta.shape != h.shape:
         raise KernelError("residual_add: shapes do not agree")
     _check(load("elementwise").ni_residual_add(_dev(h, "h", torch.float32), _dev(delta, "delta"),
@@ -321,8 +357,8 @@ def residual_add(h: torch.Tensor, delta: torch.Tensor) -> None:
            "residual_add")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, blocked: bool = False) -> None:
-    """out[t, i] = silu(gate[t, i]) * up[t, i].  Plain layout: gate_up = [gate | up] along the
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, blocked: bool = False, gelu: bool = False) -> None:
+    """out[t, i] = silu(gate[t, i]) * up[t, i] (``gelu``: the tanh form of gelu instead of silu).  Plain layout: gate_up = [gate | up] along the
     columns.  Blocked layout (I a multiple of 8): columns in blocks of 8 gate values followed by
     their 8 up values."""
     n, inter = out.shape
@@ -331,7 +367,7 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, blocked: bool = False) -> N
     if blocked and inter % 8:
         raise KernelError("swiglu: the blocked layout needs I to be a multiple of 8")
     fn = load("elementwise").ni_swiglu_blocked if blocked else load("elementwise").ni_swiglu
-    _check(fn(_dev(gate_up, "gate_up"), _dev(out, "out"), _code(out, "out"), n, inter, _stream()), "swiglu")
+    _check(fn(_dev(gate_up, "gate_up"), _dev(out, "out"), _code(out, "out"), n, inter, 1 if gelu else 0, _stream()), "swiglu")
 
 
 def rope_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, k_pages: Optional[torch.Tensor],
@@ -360,20 +396,32 @@ def rope_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, k_pages: Optional[torc
         1 if interleaved else 0, page_size, 1 if write else 0, _stream()), "rope_kv_write")
 
 
+def _sinks(sink, n_q_heads: int, device):
+    """The sinks of an attention call as float32 [Hq] on the device, or None: ``sink`` is None or False (none), True (a
+    key of score 0 for every head, so that one is added to the denominators) or that tensor."""
+    if sink is None or sink is False:
+        return None
+    if sink is True:
+        return torch.zeros(n_q_heads, dtype=torch.float32, device=device)
+    if sink.numel() != n_q_heads:
+        raise KernelError("attention: one sink per query head")
+    return sink
+
+
 def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       out: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
                       block_table: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int,
                       page_size: int, window: Optional[int], scale: float,
                       token_list: Optional[torch.Tensor] = None, head_slopes: Optional[torch.Tensor] = None,
                       score_cap: float = 0.0, value_dim: Optional[int] = None, chunk: int = 0,
-                      sink: bool = False, maps: int = 1) -> None:
+                      sink=None, maps: int = 1) -> None:
     """The plain attention kernel (any dtype, any head size up to 1,024).  ``token_list``
     int32 [n] restricts it to those tokens of the step.  ``head_slopes`` float32 [Hq] adds
     slope[h] * (key position - query position) to the scaled scores of head h.  ``score_cap`` c > 0
     bounds the scaled scores: s <- c * tanh(s / c).  ``value_dim``: the size of a value where it differs
     from the keys' (value pages [P, Hkv, page_size, value_dim], out [T, Hq * value_dim]).  ``chunk`` c > 0: a token at
-    position p sees only the keys from p - p % c on.  ``sink``: one is added to the softmax's denominator.  ``maps`` = m >
-    1: every head has m attention maps over the same values; ``n_q_heads`` counts maps (head h's map i is row h m + i of
+    position p sees only the keys from p - p % c on.  ``sink`` float32 [Hq] (or True for zeros): exp(sink[h]) is added to
+    the softmax's denominator of head h.  ``maps`` = m > 1: every head has m attention maps over the same values; ``n_q_heads`` counts maps (head h's map i is row h m + i of
     q), and a key row holds m parts of ``head_dim`` side by side.  ``out`` may be float32 where the rest is bfloat16."""
     if head_slopes is not None and head_slopes.numel() != n_q_heads:
         raise KernelError("attention: one slope per query head")
@@ -387,6 +435,7 @@ def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         raise KernelError(f"attention: head_dim {head_dim} or value_dim {v_dim} beyond 1,024 is not supported")
     if k_pages.shape[-1] != maps * head_dim or v_pages.shape[-1] != v_dim:
         raise KernelError("attention: the pages' rows must have the keys' and the values' sizes")
+    sink = _sinks(sink, n_q_heads, q.device)
     _check(load("attention_generic").ni_attention_generic(
         _dev(q, "q"), _code(q, "q"), _dev(k_pages, "k_pages"), _dev(v_pages, "v_pages"),
         _dev(out, "out"), _code(out, "out"), _dev(token_list, "token_list", torch.int32) if token_list is not None else None,
@@ -395,7 +444,7 @@ def attention_generic(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         block_table.shape[1], n if token_list is None else token_list.numel(), n_q_heads, n_kv_heads, head_dim, page_size,
         int(window) if window else 0, float(scale),
         _dev(head_slopes, "head_slopes", torch.float32) if head_slopes is not None else None, float(score_cap),
-        v_dim, int(chunk or 0), 1 if sink else 0, int(maps), _stream()), "attention_generic")
+        v_dim, int(chunk or 0), _f32_or_none(sink, "sink"), int(maps), _stream()), "attention_generic")
 
 
 def gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -479,49 +528,70 @@ def gelu_table_gate(gate: torch.Tensor, tokens: torch.Tensor, table: torch.Tenso
 
 
 def delta_prepare(proj, conv_w, a_log, dt_bias, state, seq_of_token, cu_q, slots, n_seqs, n_q_heads_kv, n_heads, dim,
-                  vdim, taps, qkv, gates) -> None:
-    """The gated delta rule's per-token inputs from the fused projection ``proj`` (float32 [T, ld], columns
-    q | k | v | gate | b | a): convolution + silu, unit q and k -> qkv [T, C]; decay and beta -> gates [T, H, 2].
+                  vdim, taps, qkv, gates, col0: int = 0, b_col: Optional[int] = None, z=None) -> None:
+    """The gated delta rule's per-token inputs from the fused projection ``proj`` ([T, ld], float32 or bfloat16; from column
+    ``col0`` on q | k | v; b at ``b_col``): convolution + silu, unit q and k -> qkv [T, C]; decay and beta -> gates
+    [T, H, 2].  Without ``z`` the decays are one per head, their logits at the columns after b, and ``b_col`` defaults to
+    the column after q | k | v and a gate of H V.  ``z`` (float32 [T, *], the first H D columns): the decays are one per
+    head and key channel; z holds their logits and, afterwards, the decays; ``dt_bias`` then has H D entries.
     It reads each request's convolution history in ``state`` (float32 [slots, H D V + (taps - 1) C]); the new
     history is written by delta_gated_norm, which must follow in the same step."""
     n = proj.shape[0]
     c = 2 * n_q_heads_kv * dim + n_heads * vdim
+    if b_col is None:
+        b_col = col0 + c + n_heads * vdim
+    a_rel = b_col - col0 + n_heads if z is None else -1
     if qkv.shape != (n, c) or gates.shape != (n, n_heads, 2) or conv_w.shape != (c, taps):
         raise KernelError("delta_prepare: shapes do not agree")
+    if proj.shape[1] < max(col0 + c, b_col + n_heads * (2 if z is None else 1)):
+        raise KernelError("delta_prepare: the projection has too few columns")
+    if dt_bias.numel() != n_heads * (dim if z is not None else 1) or a_log.numel() != n_heads or \
+            (z is not None and (z.shape[0] != n or z.shape[1] < n_heads * dim)):
+        raise KernelError("delta_prepare: the decay's constants or logits have another size")
     if state.shape[1] != n_heads * dim * vdim + (taps - 1) * c:
         raise KernelError("delta_prepare: the state has another size")
     f32 = torch.float32
     _check(load("delta_rule").ni_delta_prepare(
-        _dev(proj, "proj", f32), _dev(conv_w, "conv_w", f32), _dev(a_log, "a_log", f32), _dev(dt_bias, "dt_bias", f32),
+        _dev(proj, "proj") + col0 * proj.element_size(), _code(proj, "proj"), _dev(conv_w, "conv_w", f32),
+        _dev(a_log, "a_log", f32), _dev(dt_bias, "dt_bias", f32),
         _dev(state, "state", f32), state.shape[1], _dev(seq_of_token, "seq_of_token", torch.int32),
         _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), n, n_seqs, n_q_heads_kv, n_heads, dim, vdim,
-        taps, proj.shape[1], _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _stream()),
-        "delta_prepare")
+        taps, proj.shape[1], b_col - col0, a_rel, _f32_or_none(z, "z"), z.shape[1] if z is not None else 0,
+        _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _stream()), "delta_prepare")
 
 
-def delta_recurrence(qkv, gates, state, cu_q, slots, n_seqs, n_q_heads_kv, n_heads, dim, vdim, out) -> None:
+def delta_recurrence(qkv, gates, state, cu_q, slots, n_seqs, n_q_heads_kv, n_heads, dim, vdim, out, z=None) -> None:
     """Per head and token, in order: the state M [D, V] decays (M *= decay), the error e = beta * (v - k M) is
     written back (M += outer(k, e)) and the token reads y = q M - for every token of every request;
-    S float32 [H, D, V] at the start of each row of ``state``; out float32 [T, H V]."""
+    S float32 [H, D, V] at the start of each row of ``state``; out float32 [T, H V].  ``z``: decays per head and key channel,
+    as delta_prepare leaves them (they multiply the rows of M)."""
     f32 = torch.float32
-    if out.shape != (qkv.shape[0], n_heads * vdim):
-        raise KernelError("delta_recurrence: out must be [T, H V]")
+    if out.shape != (qkv.shape[0], n_heads * vdim) or (z is not None and (z.shape[0] != out.shape[0] or z.shape[1] < n_heads * dim)):
+        raise KernelError("delta_recurrence: out must be [T, H V] (and z [T, H D] or wider)")
     _check(load("delta_rule").ni_delta_recurrence(
-        _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _dev(state, "state", f32),
-        state.shape[1], _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), qkv.shape[0], n_seqs,
-        n_q_heads_kv, n_heads, dim, vdim, _dev(out, "out", f32), _stream()), "delta_recurrence")
+        _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _f32_or_none(z, "z"), z.shape[1] if z is not None else 0,
+        _dev(state, "state", f32), state.shape[1], _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32),
+        qkv.shape[0], n_seqs, n_q_heads_kv, n_heads, dim, vdim, _dev(out, "out", f32), _stream()), "delta_recurrence")
 
 
-def delta_gated_norm(o, proj, weight, eps, n_q_heads_kv, n_heads, dim, vdim, y, state, cu_q, slots, n_seqs, taps) -> None:
-    """y[t, h, :] = o[t, h, :] / rms * weight * silu(gate[t, h, :]), gate = its columns of ``proj``; and each
-    request's new convolution history (its last taps - 1 rows of ``proj``) into ``state``."""
+def delta_gated_norm(o, proj, weight, eps, n_q_heads_kv, n_heads, dim, vdim, y, state, cu_q, slots, n_seqs, taps, col0: int = 0,
+                     gate=None, gate_col: Optional[int] = None, sigmoid: bool = False, scale: float = 1.0, y_col: int = 0) -> None:
+    """y[t, y_col + h vdim ..] = o[t, h, :] / rms * weight * silu(gate[t, h, :]) * scale (``sigmoid``: instead of silu); gate
+    = columns ``gate_col`` on of the float32 tensor ``gate`` (default: of proj, behind q | k | v); and each request's new
+    convolution history (its last taps - 1 rows of ``proj``, columns ``col0`` on) into ``state``."""
     n = o.shape[0]
-    if y.shape != o.shape or weight.numel() != vdim:
+    f32 = torch.float32
+    hv, c = n_heads * vdim, 2 * n_q_heads_kv * dim + n_heads * vdim
+    gate = proj if gate is None else gate
+    gate_col = col0 + c if gate_col is None else gate_col
+    if o.shape != (n, hv) or y.shape[0] != n or y.shape[1] < y_col + hv or weight.numel() != vdim or gate.shape[0] != n or \
+            gate.shape[1] < gate_col + hv or proj.shape[0] != n or proj.shape[1] < col0 + c:
         raise KernelError("delta_gated_norm: shapes do not agree")
     _check(load("delta_rule").ni_delta_gated_norm(
-        _dev(o, "o", torch.float32), _dev(proj, "proj", torch.float32), _dev(weight, "weight", torch.float32), float(eps),
-        n, n_seqs, n_q_heads_kv, n_heads, dim, vdim, taps, proj.shape[1], _dev(y, "y"), _code(y, "y"),
-        _dev(state, "state", torch.float32), state.shape[1], _dev(cu_q, "cu_q", torch.int32),
+        _dev(o, "o", f32), _dev(gate, "gate", f32) + gate_col * 4, gate.shape[1], 1 if sigmoid else 0,
+        _dev(weight, "weight", f32), float(eps), float(scale), n, n_seqs, n_q_heads_kv, n_heads, dim, vdim, taps,
+        _dev(y, "y") + y_col * y.element_size(), _code(y, "y"), y.shape[1], _dev(proj, "proj") + col0 * proj.element_size(),
+        _code(proj, "proj"), proj.shape[1], _dev(state, "state", f32), state.shape[1], _dev(cu_q, "cu_q", torch.int32),
         _dev(slots, "slots", torch.int32), _stream()), "delta_gated_norm")
 
 
@@ -564,6 +634,19 @@ def head_gate(x, proj, col0, n_heads, vdim, scale: float = 1.0) -> None:
         raise KernelError("head_gate: shapes or dtypes do not agree")
     _check(load("latent").ni_head_gate(_dev(x, "x"), _code(x, "x"), _dev(proj, "proj"), proj.shape[1], int(col0), n,
                                        n_heads, vdim, float(scale), _stream()), "head_gate")
+
+
+def element_gate(x, gate, col0, out=None, out_col: int = 0, scale: float = 1.0) -> None:
+    """out[t, out_col + i] = x[t, i] * sigmoid(gate[t, col0 + i]) * scale for every column i of x [T, n]; ``gate`` [T, *] of
+    x's dtype or float32; ``out`` (default x itself) [T, *] of x's dtype."""
+    n_rows, n = x.shape
+    out = x if out is None else out
+    if gate.shape[0] != n_rows or gate.shape[1] < col0 + n or out.shape[0] != n_rows or out.shape[1] < out_col + n or \
+            out.dtype != x.dtype or gate.dtype not in (x.dtype, torch.float32):
+        raise KernelError("element_gate: shapes or dtypes do not agree")
+    _check(load("latent").ni_element_gate(
+        _dev(x, "x"), _code(x, "x"), _dev(gate, "gate") + col0 * gate.element_size(), _code(gate, "gate"), gate.shape[1],
+        _dev(out, "out") + out_col * out.element_size(), out.shape[1], n_rows, n, float(scale), _stream()), "element_gate")
 
 
 def embedding_scaled(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: torch.Tensor) -> None:
@@ -648,34 +731,49 @@ def relu_squared(z: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def qk_norm_rope(qkv, bias, q_gain, k_gain, eps, positions, seq_of_token, block_table, inv_freq, magnitude, q_out,
-                 k_pages, v_pages, n_heads, n_kv_heads, head_dim, value_dim, rotary_dim, page_size, head_unit=False) -> None:
+                 k_pages, v_pages, n_heads, n_kv_heads, head_dim, value_dim, rotary_dim, page_size, head_unit=False,
+                 col0=0, temperature=None, first_values=None) -> None:
     """From the fused projection ``qkv`` [T, ld] (columns q | k | v): + ``bias`` (float32 over those columns, or
     None); RMS norm of all the row's query values together and of all its key values together (``q_gain`` float32
     [H hd], ``k_gain`` float32 [Hkv hd]; both None: no norm); rotation of the first ``rotary_dim`` dimensions of every
     head, dimension i paired with i + rotary_dim / 2, cosine and sine times ``magnitude``; with ``head_unit`` every
     head of q and k is then divided by its own root mean square (``eps`` inside the root, no weight); queries -> q_out [T, H hd],
-    keys -> k_pages [P, Hkv, page_size, hd], values -> v_pages [P, Hkv, page_size, value_dim] (None: nothing written)."""
+    keys -> k_pages [P, Hkv, page_size, hd], values -> v_pages [P, Hkv, page_size, value_dim] (None: nothing written).
+    The columns start at ``col0`` of qkv, which may be float32 where q_out and the pages are bfloat16.  ``temperature``
+    (coef, every): the finished query times 1 + coef ln(floor((position + 1) / every) + 1).  ``first_values`` (rows, column,
+    bias, lambda): v <- (1 - lambda) v + lambda (rows[t, column : column + Hkv value_dim] + bias), rows [T, *] of qkv's
+    dtype, bias float32 [Hkv value_dim] or None."""
     n = qkv.shape[0]
     f32, i32 = torch.float32, torch.int32
     cols = (n_heads + n_kv_heads) * head_dim + n_kv_heads * value_dim
     write = k_pages is not None
-    if qkv.shape[1] < cols or q_out.shape != (n, n_heads * head_dim) or q_out.dtype != qkv.dtype:
+    if qkv.shape[1] < col0 + cols or q_out.shape != (n, n_heads * head_dim) or (q_out.dtype != qkv.dtype and qkv.dtype != f32):
         raise KernelError("qk_norm_rope: shapes or dtypes do not agree")
-    if write and (tuple(k_pages.shape[1:]) != (n_kv_heads, page_size, head_dim) or k_pages.dtype != qkv.dtype
-                  or tuple(v_pages.shape[1:]) != (n_kv_heads, page_size, value_dim) or v_pages.dtype != qkv.dtype):
+    if write and (tuple(k_pages.shape[1:]) != (n_kv_heads, page_size, head_dim) or k_pages.dtype != q_out.dtype
+                  or tuple(v_pages.shape[1:]) != (n_kv_heads, page_size, value_dim) or v_pages.dtype != q_out.dtype):
         raise KernelError("qk_norm_rope: pages must be [P, Hkv, page_size, head_dim] and [P, Hkv, page_size, value_dim]")
     if (bias is not None and bias.numel() != cols) or (q_gain is None) != (k_gain is None) or \
             (q_gain is not None and (q_gain.numel() != n_heads * head_dim or k_gain.numel() != n_kv_heads * head_dim)):
         raise KernelError("qk_norm_rope: the bias or a gain has another size")
     if rotary_dim > 0 and inv_freq.numel() != rotary_dim // 2:
         raise KernelError("qk_norm_rope: inv_freq must have rotary_dim / 2 entries")
+    coef, every = temperature if temperature is not None else (0.0, 1.0)
+    first, first_ld, first_bias, lam = None, 0, None, 0.0
+    if first_values is not None:
+        rows, column, bias_v, lam = first_values
+        nv = n_kv_heads * value_dim
+        if rows.shape[0] != n or rows.shape[1] < column + nv or rows.dtype != qkv.dtype or (bias_v is not None and bias_v.numel() != nv):
+            raise KernelError("qk_norm_rope: the values to mix in must be rows of qkv's dtype with the values' columns")
+        first, first_ld = _dev(rows, "first values") + column * rows.element_size(), rows.shape[1]
+        first_bias = _dev(bias_v, "first values' bias", f32) if bias_v is not None else None
     _check(load("qk_norm_rope").ni_qk_norm_rope(
-        _dev(qkv, "qkv"), _code(qkv, "qkv"), qkv.shape[1], _dev(bias, "bias", f32) if bias is not None else None,
+        _dev(qkv, "qkv") + col0 * qkv.element_size(), _code(qkv, "qkv"), _code(q_out, "q_out"), qkv.shape[1], _dev(bias, "bias", f32) if bias is not None else None,
         _dev(q_gain, "q_gain", f32) if q_gain is not None else None, _dev(k_gain, "k_gain", f32) if k_gain is not None else None,
         float(eps), _dev(positions, "positions", i32), _dev(seq_of_token, "seq_of_token", i32),
         _dev(block_table, "block_table", i32), block_table.shape[1], _dev(inv_freq, "inv_freq", f32), float(magnitude),
         _dev(q_out, "q_out"), _dev(k_pages, "k_pages") if write else None, _dev(v_pages, "v_pages") if write else None,
-        n, n_heads, n_kv_heads, head_dim, value_dim, rotary_dim, page_size, 1 if head_unit else 0, _stream()), "qk_norm_rope")
+        n, n_heads, n_kv_heads, head_dim, value_dim, rotary_dim, page_size, 1 if head_unit else 0, float(coef),
+        float(every), first, first_ld, first_bias, float(lam), _stream()), "qk_norm_rope")
 
 
 LIGHTNING_MAX_DIM = 256      # the largest key size whose chunk buffers fit a block's shared memory
@@ -1115,6 +1213,7 @@ GEMV_MAX_ROWS = 16      # what the skinny kernels take
 # 1.40 ms against 1.21 ms for the library product with separate element-wise kernels.
 SKINNY_ROWS = 8
 STORE_BF16, STORE_F32, ADD_F32, SWIGLU_BF16 = 0, 1, 2, 3
+GEGLU_BF16 = SWIGLU_BF16 | 16      # as SWIGLU_BF16 with the tanh form of gelu for the gate (NI_MODE_GELU)
 
 
 def _gemv_check(m: int, n: int, k: int, w: torch.Tensor, out: torch.Tensor, mode: int, what: str) -> None:
@@ -1123,7 +1222,7 @@ def _gemv_check(m: int, n: int, k: int, w: torch.Tensor, out: torch.Tensor, mode
     if m > GEMV_MAX_ROWS or k % 8:
         raise KernelError(f"{what}: takes at most {GEMV_MAX_ROWS} rows and K a multiple of 8 "
                           f"(got M={m}, K={k})")
-    if mode == SWIGLU_BF16:
+    if mode in (SWIGLU_BF16, GEGLU_BF16):
         if n % 16 or out.shape != (m, n // 2) or out.dtype != torch.bfloat16:
             raise KernelError(f"{what}: the SwiGLU epilogue needs N a multiple of 16 and out bf16 [M, N/2]")
     else:
@@ -1201,10 +1300,11 @@ def gemv_reads_handoff(m: int, k: int) -> bool:
 
 
 def gemv_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, warm=None,
-              handoff: Optional["NormHandoff"] = None, pre: Optional["NormHandoff"] = None) -> None:
+              handoff: Optional["NormHandoff"] = None, pre: Optional["NormHandoff"] = None, affine=None) -> None:
     """x[M, K] . w[N, K]^T for M <= 16, K % 8 == 0.  mode STORE_BF16 / STORE_F32: out[M, N] =;
     ADD_F32: out[M, N] +=; SWIGLU_BF16: w's rows in blocks of 8 gate + 8 up rows,
-    out[M, N/2] = silu(gate) * up.  ``warm`` (tensor, first byte, bytes): weights of the kernels
+    out[M, N/2] = silu(gate) * up (GEGLU_BF16: gelu).  ``affine`` (scale, shift), each float32 [N] or None, with ADD_F32:
+    out[M, N] += product * scale + shift.  ``warm`` (tensor, first byte, bytes): weights of the kernels
     after this one, asked into L2 when this kernel's own loads have been issued.  ``handoff`` (with
     ADD_F32, up to 8 rows): also prepare the norm that follows; ``pre``: x is such a prepared input."""
     if (handoff is not None or pre is not None) and x.shape[0] > HANDOFF_ROWS:
@@ -1217,7 +1317,18 @@ def gemv_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, wa
     _check(load("gemv_bf16").ni_gemv_bf16(_dev(x, "x", torch.bfloat16), _dev(w, "w", torch.bfloat16),
                                           _dev(out, "out"), m, n, k, mode, *warm_region(warm),
                                           *(handoff.producer_args() if handoff is not None else _NO_HANDOFF),
-                                          *(pre.reader_args() if pre is not None else _NO_PRE), _stream()), "gemv_bf16")
+                                          *(pre.reader_args() if pre is not None else _NO_PRE),
+                                          *_affine_args(affine, n), _stream()), "gemv_bf16")
+
+
+def _affine_args(affine, n: int) -> tuple:
+    """(scale, shift) of an adding product as pointers (null where absent)."""
+    if affine is None:
+        return None, None
+    scale, shift = affine
+    if any(v is not None and v.numel() != n for v in (scale, shift)):
+        raise KernelError("an adding product's scale and shift must have one number per column")
+    return _f32_or_none(scale, "scale"), _f32_or_none(shift, "shift")
 
 
 KSPLIT_ROWS = 8          # rows the cluster split-K skinny product takes
@@ -1233,10 +1344,10 @@ def gemv_ksplit_supports(m: int, n: int, k: int) -> bool:
 
 
 def gemv_ksplit(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, warm=None,
-                handoff: Optional["NormHandoff"] = None, pre=None) -> None:
+                handoff: Optional["NormHandoff"] = None, pre=None, affine=None) -> None:
     """x[M, K] . w[N, K]^T for M <= 8 and a long K, split over the blocks of a cluster (each keeps
     its slice of the activations in registers; the slices' sums are added in slice order).
-    mode STORE_BF16 / STORE_F32 / ADD_F32 as gemv_bf16."""
+    mode STORE_BF16 / STORE_F32 / ADD_F32 (with ``affine``) as gemv_bf16."""
     m, k = x.shape
     n = w.shape[0]
     if mode not in (STORE_BF16, STORE_F32, ADD_F32):
@@ -1252,7 +1363,7 @@ def gemv_ksplit(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int, 
     _check(load("gemv_ksplit").ni_gemv_ksplit(_dev(x, "x", torch.bfloat16), _dev(w, "w", torch.bfloat16),
                                               _dev(out, "out"), m, n, k, mode, *warm_region(warm),
                                               *(handoff.producer_args() if handoff is not None else _NO_HANDOFF),
-                                              _stream()), "gemv_ksplit")
+                                              *_affine_args(affine, n), _stream()), "gemv_ksplit")
 
 
 def gemv_norm_bf16(h: torch.Tensor, gain: torch.Tensor, eps: float, rows: Optional[torch.Tensor],
@@ -1303,13 +1414,16 @@ def gemv_qkv_rope(x: torch.Tensor, gain: Optional[torch.Tensor], eps: float, w: 
 
 
 def linear_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype,
-                residual: Optional[torch.Tensor] = None, warm=None, handoff: Optional["NormHandoff"] = None) -> Optional[torch.Tensor]:
+                residual: Optional[torch.Tensor] = None, warm=None, handoff: Optional["NormHandoff"] = None,
+                affine=None):
     """y = x . w^T for bfloat16 operands with FP32 accumulation.
 
     Up to SKINNY_ROWS rows (decode): the package's own bandwidth kernel; with ``residual`` (float32
     [M, N]) the product is added into it and None is returned.  More rows: a library matrix
     product (cuBLASLt through torch), as the reference's projections are cuBLAS calls
     (src/op/kernels/cuda/matmul_kernel.cu:76-86); the caller adds the result to the residual.
+    ``affine`` (scale, shift), with ``residual``: what is added is y * scale + shift (float32 per column, either may be
+    None); where the kernel cannot add it, a ScaledAddition is returned.
     """
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("linear_bf16: operands must be bfloat16")
@@ -1321,16 +1435,15 @@ def linear_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype,
         product = gemv_ksplit if (m <= KSPLIT_ROWS and KSPLIT_MIN_K <= k <= KSPLIT_MAX_K
                                   and gemv_ksplit_supports(m, w.shape[0], k)) else gemv_bf16
         if residual is not None:
-            product(x, w, residual, ADD_F32, warm, handoff=handoff)
+            product(x, w, residual, ADD_F32, warm, handoff=handoff, affine=affine)
             return None
         out = torch.empty(m, w.shape[0], dtype=out_dtype, device=x.device)
         product(x, w, out, STORE_BF16 if out_dtype == torch.bfloat16 else STORE_F32, warm)
         return out
     if handoff is not None:
         raise KernelError("linear_bf16: a norm can only be handed over by the skinny product (up to 8 rows)")
-    if out_dtype == torch.bfloat16:
-        return torch.matmul(x, w.t())
-    return torch.mm(x, w.t(), out_dtype=torch.float32)
+    y = torch.matmul(x, w.t()) if out_dtype == torch.bfloat16 else torch.mm(x, w.t(), out_dtype=torch.float32)
+    return y if affine is None else ScaledAddition(y, *affine)
 
 
 _error_words: Dict[torch.device, torch.Tensor] = {}
@@ -1412,7 +1525,7 @@ def gemm_tc(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, mode: int, kern
         raise KernelError("gemm_tc: inner sizes do not agree")
     if k % 8:
         raise KernelError(f"gemm_tc: K must be a multiple of 8 (got {k})")
-    if mode == SWIGLU_BF16:
+    if mode in (SWIGLU_BF16, GEGLU_BF16):
         if n % 16 or out.shape != (m, n // 2) or out.dtype != torch.bfloat16:
             raise KernelError("gemm_tc: the SwiGLU epilogue needs N a multiple of 16 and out bf16 [M, N/2]")
     else:
@@ -1576,11 +1689,11 @@ def attention_decode_cluster_merge(on: bool) -> None:
 
 def attention_decode(q, k_pages, v_pages, out, token_list, n_items, positions, seq_of_token, block_table,
                      n_q_heads, n_kv_heads, head_dim, page_size, window, scale, n_splits, scratch,
-                     tickets, warm=(), score_cap: float = 0.0, chunk: int = 0, sink: bool = False,
+                     tickets, warm=(), score_cap: float = 0.0, chunk: int = 0, sink=None,
                      shared_pages: bool = False) -> None:
     """Split-K attention of single query tokens (bfloat16).  ``score_cap`` c > 0 bounds the scaled scores:
-    s <- c * tanh(s / c).  ``chunk`` c > 0: the token at position p sees only the keys from p - p % c on; ``sink``: one
-    is added to the softmax's denominator.  ``shared_pages``: the pages hold ONE head that all ``n_kv_heads`` of the
+    s <- c * tanh(s / c).  ``chunk`` c > 0: the token at position p sees only the keys from p - p % c on; ``sink``
+    float32 [Hq] (or True for zeros): exp(sink[h]) is added to head h's softmax denominator.  ``shared_pages``: the pages hold ONE head that all ``n_kv_heads`` of the
     call read (more than 16 query heads over one shared head, dealt over groups of at most 16).  ``token_list`` int32 [n_items] or
     None for tokens 0..n_items-1.  scratch: float32, at least n_items * Hq * n_splits *
     (head_dim + 2); tickets: int32 zeros, at least n_items * Hkv (left zero by the kernel).
@@ -1595,7 +1708,8 @@ def attention_decode(q, k_pages, v_pages, out, token_list, n_items, positions, s
     capped = score_cap and score_cap > 0.0
     if shared_pages and k_pages.shape[1] != 1:
         raise KernelError("attention_decode: shared pages hold one head")
-    if chunk or sink or shared_pages:
+    sink = _sinks(sink, n_q_heads, q.device)
+    if chunk or sink is not None or shared_pages:
         _check(lib.ni_attention_decode_masked(
             _dev(q, "q", torch.bfloat16), _dev(k_pages, "k_pages", torch.bfloat16),
             _dev(v_pages, "v_pages", torch.bfloat16), _dev(out, "out", torch.bfloat16),
@@ -1603,7 +1717,7 @@ def attention_decode(q, k_pages, v_pages, out, token_list, n_items, positions, s
             _dev(positions, "positions", torch.int32), _dev(seq_of_token, "seq_of_token", torch.int32),
             _dev(block_table, "block_table", torch.int32), block_table.shape[1], n_q_heads, n_kv_heads,
             head_dim, page_size, int(window) if window else 0, float(scale), float(score_cap or 0.0), int(chunk or 0),
-            (1 if sink else 0) | ((n_kv_heads if shared_pages else 0) << 1), n_splits, _dev(scratch, "scratch", torch.float32),
+            _f32_or_none(sink, "sink"), n_kv_heads if shared_pages else 0, n_splits, _dev(scratch, "scratch", torch.float32),
             _dev(tickets, "tickets", torch.int32),
             *regions, _stream()), "attention_decode")
         return
@@ -1679,10 +1793,10 @@ def attention_prefill_tc_supports(n_q_heads: int, n_kv_heads: int, head_dim: int
 
 def attention_prefill(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu_q, kv_len, block_table,
                       n_q_heads, n_kv_heads, head_dim, page_size, window, scale, kernel: Optional[str] = None,
-                      score_cap: float = 0.0, chunk: int = 0, sink: bool = False) -> None:
+                      score_cap: float = 0.0, chunk: int = 0, sink=None) -> None:
     """``score_cap`` c > 0 bounds the scaled scores, s <- c * tanh(s / c) (the mma.sync kernel only).  ``chunk`` c > 0:
-    a query at position p sees only the keys from p - p % c on; ``sink``: one is added to the softmax's denominator
-    (both kernels).
+    a query at position p sees only the keys from p - p % c on; ``sink`` float32 [Hq] (or True for zeros): exp(sink[h]) is
+    added to head h's softmax denominator (both kernels).
     Flash-style causal attention of prompt portions (bfloat16): one block per tile of
     PREFILL_TILE_ROWS query rows and query head (mma.sync kernel) or pair of query heads
     (tcgen05 kernel, where it takes the case); tile_seq / tile_row0 int32 [n_tiles] name each
@@ -1690,6 +1804,7 @@ def attention_prefill(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu
     if head_dim % 16 or head_dim > PREFILL_MAX_HEAD_DIM:
         raise KernelError(f"attention_prefill: head_dim {head_dim} not supported (multiples of 16 up to 128)")
     tc_ok = attention_prefill_tc_supports(n_q_heads, n_kv_heads, head_dim, page_size) and not score_cap
+    sink = _sinks(sink, n_q_heads, q.device)
     if kernel == "tc" and not tc_ok:
         raise KernelError("attention_prefill: the tcgen05 kernel does not take this case")
     if tc_ok and kernel != "mma":
@@ -1699,7 +1814,7 @@ def attention_prefill(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu
             _dev(tile_seq, "tile_seq", torch.int32), _dev(tile_row0, "tile_row0", torch.int32), n_tiles,
             _dev(cu_q, "cu_q", torch.int32), _dev(kv_len, "kv_len", torch.int32),
             _dev(block_table, "block_table", torch.int32), block_table.shape[1], n_q_heads, n_kv_heads,
-            head_dim, page_size, int(window) if window else 0, float(scale), int(chunk or 0), 1 if sink else 0,
+            head_dim, page_size, int(window) if window else 0, float(scale), int(chunk or 0), _f32_or_none(sink, "sink"),
             _error_word(q.device).data_ptr(), _stream()), "attention_prefill_tc")
         return
     _check(load("attention_prefill").ni_attention_prefill(
@@ -1709,7 +1824,7 @@ def attention_prefill(q, k_pages, v_pages, out, tile_seq, tile_row0, n_tiles, cu
         _dev(cu_q, "cu_q", torch.int32), _dev(kv_len, "kv_len", torch.int32),
         _dev(block_table, "block_table", torch.int32), block_table.shape[1], n_q_heads, n_kv_heads,
         head_dim, page_size, int(window) if window else 0, float(scale), float(score_cap or 0.0), int(chunk or 0),
-        1 if sink else 0, _stream()), "attention_prefill")
+        _f32_or_none(sink, "sink"), _stream()), "attention_prefill")
 
 
 _argmax_keys: Dict[torch.device, torch.Tensor] = {}   # per device: merge keys, zero between calls

@@ -1,2 +1,2 @@
 """Architectures: each module registers its config parser and tensor naming."""
-from . import kepusun, llama, mobatar, runevik, tazulix, vuvalorn  # noqa: F401
+from . import kepusun, llama, lomopel, mobatar, runevik, tazulix, vuvalorn  # noqa: F401

@@ -59,9 +59,22 @@ from dataclasses import dataclass, field
 from typing import Dict, Optional, Tuple
 
 
+class FreeDim(int):
+    """A size that no configuration key gives: the stored tensor decides it (the inner size of two thin matrices that
+    stand in for one, say).  Its value is the size that random weights are made with.  Free sizes with one label must
+    agree within a part; the part reads them off the tensors it is handed."""
+
+    label: str
+
+    def __new__(cls, default: int, label: str) -> "FreeDim":
+        self = super().__new__(cls, default)
+        self.label = label
+        return self
+
+
 @dataclass(frozen=True)
 class WeightSlot:
-    """Shape and initialisation rule of one weight of a part.
+    """Shape and initialisation rule of one weight of a part; a size may be a FreeDim.
 
     init "normal": N(0, std) in random-weights mode; "ones": 1.0 (norm gains); "zeros"; "eye": the identity matrix.
     """

@@ -7,7 +7,7 @@ import torch
 
 from ..config.registry import part, register_part
 from ..kernels import ops
-from ..kernels.ops import NormHandoff, StreamCopy
+from ..kernels.ops import NormHandoff, ScaledAddition, StreamCopy
 from .base import WeightSlot
 
 
@@ -18,7 +18,18 @@ class PreNormBlock:
     The residual stream h is FP32 and updated in place.  Each addition is fused into the
     norm that follows it, so a block takes the addition still pending from the block before
     and returns its own.
+
+    With ``layer_scale`` in the layer's extra every sublayer's output is multiplied column by column by a learned vector
+    ("ls1", "ls2") before it joins the stream.  A sublayer that adds into the stream itself may take the vector along
+    (``bind_output_scale``: its last product adds scaled columns); for the others it rides in the pending addition.
     """
+
+    @staticmethod
+    def weight_slots(layer_spec, hidden_size: int):
+        if not layer_spec.extra_dict().get("layer_scale", False):
+            return {}
+        n = 1 if layer_spec.feed_forward is None else 2
+        return {f"ls{i}": WeightSlot((hidden_size,), init="ones") for i in range(1, n + 1)}
 
     def __init__(self, layer_spec, hidden_size: int, weights_of, rt) -> None:
         """``weights_of(what)`` returns {slot: tensor} for what in
@@ -35,6 +46,18 @@ class PreNormBlock:
                 layer_spec.ffn_norm, hidden_size, weights_of("ffn_norm"), rt)
             self.feed_forward = part("feed_forward", layer_spec.feed_forward.kind)(
                 layer_spec.feed_forward, hidden_size, weights_of("feed_forward"), rt)
+        # scales that the sublayer itself does not take: (mixer's, feed-forward's)
+        self.scales = [None, None]
+        if layer_spec.extra_dict().get("layer_scale", False):
+            own = weights_of("block")
+            for i, sub in enumerate((self.mixer, self.feed_forward)):
+                if sub is None:
+                    continue
+                scale = rt.gain(own[f"ls{i + 1}"])
+                if hasattr(sub, "bind_output_scale"):
+                    sub.bind_output_scale(scale)
+                else:
+                    self.scales[i] = scale
 
     def weights_in_order(self) -> tuple:
         return tuple(getattr(self.mixer, "weights_in_order", tuple)()) + tuple(getattr(self.feed_forward, "weights_in_order", tuple)())
@@ -42,7 +65,7 @@ class PreNormBlock:
     def first_norm(self):
         """The norm that reads the residual stream first, if its reader (the mixer) can take it
         prepared by the kernel that last added into the stream (a NormHandoff); else None."""
-        return self.mixer_norm if hasattr(self.mixer, "forward_prenormed") else None
+        return self.mixer_norm if hasattr(self.mixer, "forward_prenormed") and self.scales[0] is None else None
 
     def forward(self, h: torch.Tensor, delta, ctx, cache):
         """``delta``: what the block before left - None, an addition still pending on the stream, or a
@@ -53,18 +76,20 @@ class PreNormBlock:
         pre = None
         if isinstance(delta, NormHandoff):
             pre, delta = delta, None
-            if pre.norm is not self.mixer_norm or not hasattr(mixer, "forward_prenormed"):
+            if pre.norm is not self.mixer_norm or self.first_norm() is None:
                 pre = None                              # not for this block's norm: it is computed as usual
         after = ctx.read_after                       # what runs after this block
         ctx.read_after = tuple(getattr(ffn, "weights_in_order", tuple)()) + tuple(after)   # ... after the mixer
         # the norms that may be handed from kernel to kernel: this block's second one, the next block's first
-        to_ffn = self.ffn_norm if hasattr(ffn, "forward_prenormed") and _fuses(ffn, self.ffn_norm, n) else None
+        to_ffn = self.ffn_norm if self.scales[1] is None and hasattr(ffn, "forward_prenormed") and _fuses(ffn, self.ffn_norm, n) else None
         try:
             a = self._mix(h, delta, pre, ctx, cache, n, to_ffn)
         finally:
             ctx.read_after = after
         if ffn is None:
             return a                                 # the mixer's addition, pending or made
+        if self.scales[1] is not None:
+            return ScaledAddition(ffn.forward(self.ffn_norm.forward(h, a), ctx), self.scales[1], None)
         then = ctx.norm_after if getattr(ffn, "hands_off_norm", False) else None
         if isinstance(a, NormHandoff):
             return ffn.forward_prenormed(a, ctx, residual=h, then_norm=then)
@@ -79,6 +104,8 @@ class PreNormBlock:
 
     def _mix(self, h, delta, pre, ctx, cache, n, to_ffn):
         mixer = self.mixer
+        if self.scales[0] is not None:
+            return ScaledAddition(mixer.forward(self.mixer_norm.forward(h, delta), ctx, cache), self.scales[0], None)
         then = {"then_norm": to_ffn} if to_ffn is not None and getattr(mixer, "hands_off_norm", False) else {}
         if pre is not None:
             return mixer.forward_prenormed(pre, ctx, cache, residual=h, **then)

@@ -13,7 +13,9 @@ from .base import Part, WeightSlot
 
 class SwiGLU(Part):
     """y = down(silu(gate(x)) * up(x)); gate and up are one fused projection
-    (src/model/llama.cpp:364-379, src/op/kernels/cuda/swiglu_kernel.cu:25-40)."""
+    (src/model/llama.cpp:364-379, src/op/kernels/cuda/swiglu_kernel.cu:25-40).  ``activation`` "gelu_tanh" in the spec's
+    extra: the tanh form of gelu instead of silu; ``f32_out``: the output leaves in FP32 where it is not added in place.
+    A layer may hand it a scale per output column (``bind_output_scale``)."""
 
     kernel_modules_bf16 = ("gemm_tc", "gemm_tc2", "gemm_swap_tc")      # libraries of csrc: the tcgen05 products with the activation inside
 
@@ -37,9 +39,21 @@ class SwiGLU(Part):
             w13 = torch.cat([gate, up], dim=0)
         self.w_gate_up = rt.weight(w13)
         self.w_down = rt.weight(weights["down"])
+        e = spec.extra_dict()
+        activation = e.get("activation", "silu")
+        if activation not in ("silu", "gelu_tanh"):
+            raise ConfigError(f"gated unit: activation '{activation}' is not known (silu, gelu_tanh)")
+        self.gelu = activation == "gelu_tanh"
+        self.act_mode = ops.GEGLU_BF16 if self.gelu else ops.SWIGLU_BF16
+        self.out_dtype = torch.float32 if e.get("f32_out", False) else None
+        self.affine = None
 
     adds_into_residual = True   # forward() accepts residual= and may add its output there
     graph_safe = "all"
+
+    def bind_output_scale(self, scale) -> None:
+        """The output's columns are multiplied by ``scale`` as they join the stream."""
+        self.affine = (scale, None)
 
     def weights_in_order(self) -> tuple:
         return (self.w_gate_up, self.w_down)
@@ -54,19 +68,20 @@ class SwiGLU(Part):
         n = x.shape[0]
         act = rt.empty(n, self.inter)
         if self.blocked and rt.skinny(n, self.hidden_size):
-            ops.gemv_bf16(x, self.w_gate_up, act, ops.SWIGLU_BF16,     # activation in the epilogue
+            ops.gemv_bf16(x, self.w_gate_up, act, self.act_mode,       # activation in the epilogue
                           warm=rt.warm(self.w_down, 0, which=2))
         elif self.blocked and rt.tensor_core_gemm(n, self.hidden_size):
-            ops.gemm_tc(x, self.w_gate_up, act, ops.SWIGLU_BF16)       # tcgen05 product, activation fused
-        elif self.blocked and rt.mid_batch(n, self.hidden_size, rt.MID_GATE_UP):
+            ops.gemm_tc(x, self.w_gate_up, act, self.act_mode)         # tcgen05 product, activation fused
+        elif self.blocked and not self.gelu and rt.mid_batch(n, self.hidden_size, rt.MID_GATE_UP):
             ops.gemm_swap_tc(x, self.w_gate_up, act, ops.SWIGLU_BF16)  # weights on the tile's lanes, activation fused
         else:
             gate_up = rt.linear(x, self.w_gate_up)
-            ops.swiglu(gate_up, act, blocked=self.blocked)
-        if residual is not None and rt.mid_batch(n, self.inter, rt.MID_DOWN):
+            ops.swiglu(gate_up, act, blocked=self.blocked, gelu=self.gelu)
+        if residual is not None and self.affine is None and rt.mid_batch(n, self.inter, rt.MID_DOWN):
             ops.gemm_swap_tc(act, self.w_down, residual, ops.ADD_F32)
             return None
-        return rt.linear(act, self.w_down, residual=residual, warm=rt.warm_after(ctx, which=4))
+        return rt.linear(act, self.w_down, out_dtype=self.out_dtype, residual=residual, warm=rt.warm_after(ctx, which=4),
+                         affine=self.affine)
 
     def forward_fused_norm(self, h: torch.Tensor, norm, ctx, residual=None, then_norm=None):
         """As forward, with x = norm(h): norm, projection and activation in one launch.  ``then_norm``:
@@ -74,7 +89,7 @@ class SwiGLU(Part):
         NormHandoff is returned instead of None."""
         rt = self.rt
         act = rt.empty(h.shape[0], self.inter)
-        ops.gemv_norm_bf16(h, norm.gain, norm.eps, None, self.w_gate_up, act, ops.SWIGLU_BF16,
+        ops.gemv_norm_bf16(h, norm.gain, norm.eps, None, self.w_gate_up, act, self.act_mode,
                            warm=rt.warm(self.w_down, 0, which=2))
         return self._down(act, ctx, residual, then_norm)
 
@@ -82,13 +97,14 @@ class SwiGLU(Part):
         """As forward_fused_norm, with the norm prepared by the kernel that last added into the stream."""
         rt = self.rt
         act = rt.empty(pre.x.shape[0], self.inter)
-        ops.gemv_bf16(pre.x, self.w_gate_up, act, ops.SWIGLU_BF16, warm=rt.warm(self.w_down, 0, which=2), pre=pre)
+        ops.gemv_bf16(pre.x, self.w_gate_up, act, self.act_mode, warm=rt.warm(self.w_down, 0, which=2), pre=pre)
         return self._down(act, ctx, residual, then_norm)
 
     def _down(self, act, ctx, residual, then_norm):
         rt = self.rt
         handoff = rt.handoff(then_norm, act.shape[0], self.hidden_size, self.inter) if residual is not None else None
-        out = rt.linear(act, self.w_down, residual=residual, warm=rt.warm_after(ctx, which=4), handoff=handoff)
+        out = rt.linear(act, self.w_down, out_dtype=self.out_dtype, residual=residual, warm=rt.warm_after(ctx, which=4),
+                        handoff=handoff, affine=self.affine)
         return handoff if handoff is not None else out
 
 

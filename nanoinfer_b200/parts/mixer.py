@@ -1,6 +1,7 @@
 """Token mixers.  The one built in is grouped-query attention over the paged cache."""
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List, Optional
 
 import numpy as np
@@ -9,14 +10,15 @@ import torch
 from ..config.model_config import ConfigError
 from ..config.registry import part, register_part
 from ..kernels import ops
-from .base import PagedKVNeed, PagedNeed, Part, StateNeed, StepPlan, WeightSlot
+from .base import FreeDim, PagedKVNeed, PagedNeed, Part, StateNeed, StepPlan, WeightSlot
 
 
 class PagedAttendMixin:
     """What every mixer that attends over pages of keys and values shares: the step's plan (which tokens
     go to which kernel) and the choice among the attention kernels.  A class that uses it sets n_heads,
     n_kv, head_dim, window, scale, position and w_o; optionally ``chunk`` (c > 0: a token at position p sees only the
-    keys from p - p % c on) and ``sink`` (one is added to the softmax's denominator)."""
+    keys from p - p % c on) and ``sink`` (float32 [n_heads] on the device: exp(sink[h]) is added to the softmax's
+    denominator of head h)."""
 
     # How the attention kernels split a step.  Requests that bring at most SHORT_PORTION tokens are
     # handled token by token by the split-K kernel (which fetches a token's last
@@ -65,7 +67,7 @@ class PagedAttendMixin:
         n = q.shape[0]
         slopes = getattr(self.position, "head_slopes", None)
         cap = float(getattr(self, "score_cap", 0.0))       # > 0: scores are bounded by cap * tanh(s / cap)
-        chunk, sink = int(getattr(self, "chunk", 0) or 0), bool(getattr(self, "sink", False))
+        chunk, sink = int(getattr(self, "chunk", 0) or 0), getattr(self, "sink", None)
         if rt.dtype != torch.bfloat16 or slopes is not None:
             # float32, or a position encoding that acts on the scores (a bias slope[h] * (k_pos - q_pos)): the plain
             # kernel takes both.  (A chunk mask and a sink are known to the split-K kernel for single tokens and to both
@@ -86,7 +88,7 @@ class PagedAttendMixin:
         n_dec = n if plan is None else plan.scalars["n_dec"]
         dec_list = None if plan is None else plan.arrays["dec_tokens"]
         if n_dec > 0:
-            if (decode_ok and cap == 0.0 and chunk == 0 and not sink and not shared and rt.balanced_attention(n_dec, self.n_kv, self.head_dim)
+            if (decode_ok and cap == 0.0 and chunk == 0 and sink is None and not shared and rt.balanced_attention(n_dec, self.n_kv, self.head_dim)
                     and n_dec <= ops.DECODE_BALANCED_MAX_ITEMS):
                 # many tokens: their keys dealt evenly over a fixed set of blocks, whatever their lengths
                 scratch = rt.workspace("attention_decode_balanced_partials",
@@ -492,18 +494,29 @@ class NormedQKAttention(PagedAttendMixin, Part):
         s = (q . k) softmax_scale;  causal softmax;  sum p v;   then W_o on the heads side by side
 
     More options in the spec's extra: ``chunk`` = c > 0 - a token at position p sees only the keys of its own chunk,
-    positions p - p % c .. p, chunks counted from the sequence's start; ``sink`` - one is added to the softmax's
-    denominator (a key of score 0 that has no value); ``head_gate`` - head h's output is multiplied by
-    sigmoid(W_g x)_h, one more row per head in the fused projection ("g").
+    positions p - p % c .. p, chunks counted from the sequence's start; ``spec.window`` = w - a token sees itself and the
+    w - 1 tokens before it; ``sink`` - True: one is added to the softmax's denominator (a key of score 0 that has no
+    value), "learned": exp(sink_h) with a number per head ("sink"), not scaled; ``head_gate`` - head h's output is
+    multiplied by sigmoid(W_g x)_h, one more row per head in the fused projection ("g"); ``element_gate`` - every
+    coordinate of the output by its own sigmoid(W_g x)_i ("g" has a row per coordinate); ``temperature`` = (coef, every) -
+    the finished query at position p times 1 + coef ln(floor((p + 1) / every) + 1); ``value_mix`` - "first": this layer's
+    values v_0 go along to later layers of the step, "later": v <- (1 - lambda) v + lambda v_0 with the learned number
+    "vmix", and the mixed values are cached; ``output_bias`` - the output projection has one ("o.b").
 
     Keys have ``head_dim`` entries, values ``value_dim`` (the same unless the extra says otherwise).  The three
     projections are one product; bias, both norms, the rotation and the cache write are one kernel
     (csrc/qk_norm_rope.cu), FP32 inside whatever the tensors' type.  With values of the keys' size the attention
     runs on the package's paged kernels (tcgen05 flash attention for prompt portions, split-K for single tokens);
-    other value sizes take the plain kernel, which knows them."""
+    other value sizes take the plain kernel, which knows them.
+
+    ``joined`` in the extra: the part is one side of mixers that share their input and their output projection
+    (ParallelMixers): it hands over its matrices (``in_rows``, ``out_matrix``) and runs what lies between (``between``)."""
 
     kernel_modules = ("qk_norm_rope",)       # libraries of csrc that this part's kernels live in
     kernel_modules_bf16 = ("attention_prefill_tc",)
+
+    JOINS = True                # can be a side of mixers with joined projections
+    wants_f32_tokens = False    # a joined projection of single tokens need not be FP32 for this side's sake
 
     adds_into_residual = True
     graph_safe = "all"
@@ -517,15 +530,24 @@ class NormedQKAttention(PagedAttendMixin, Part):
     @staticmethod
     def weight_slots(spec, hidden_size: int) -> Dict[str, WeightSlot]:
         h, g, d, v, bias, qk_norm = NormedQKAttention._dims(spec)
+        e = spec.extra_dict()
         slots = {"q": WeightSlot((h * d, hidden_size)), "k": WeightSlot((g * d, hidden_size)),
                  "v": WeightSlot((g * v, hidden_size))}
         if bias:
             slots.update({"q.b": WeightSlot((h * d,)), "k.b": WeightSlot((g * d,)), "v.b": WeightSlot((g * v,))})
         if qk_norm:
             slots.update({"q.norm": WeightSlot((h * d,), init="ones"), "k.norm": WeightSlot((g * d,), init="ones")})
-        if spec.extra_dict().get("head_gate", False):
+        if e.get("head_gate", False):
             slots["g"] = WeightSlot((h, hidden_size))
+        if e.get("element_gate", False):
+            slots["g"] = WeightSlot((h * v, hidden_size))
+        if e.get("sink", False) == "learned":
+            slots["sink"] = WeightSlot((h,))
+        if e.get("value_mix"):
+            slots["vmix"] = WeightSlot(())
         slots["o"] = WeightSlot((hidden_size, h * v))
+        if e.get("output_bias", False):
+            slots["o.b"] = WeightSlot((hidden_size,))
         return slots
 
     def __init__(self, spec, hidden_size, weights, rt) -> None:
@@ -535,20 +557,33 @@ class NormedQKAttention(PagedAttendMixin, Part):
             raise ConfigError("normed-qk attention: heads must be a positive multiple of kv_heads")
         if not 0 < d <= 512 or not 0 < v <= 512:
             raise ConfigError(f"normed-qk attention: key size {d} and value size {v} must lie in 1 .. 512")
-        if spec.window is not None:
-            raise ConfigError("normed-qk attention sees every earlier key, or those of its chunk (no window)")
         e = spec.extra_dict()
         self.n_heads, self.n_kv, self.head_dim, self.value_dim = h, g, d, v
-        self.window = None
-        self.chunk, self.sink = int(e.get("chunk", 0) or 0), bool(e.get("sink", False))
-        self.head_unit_norm, self.head_gate = bool(e.get("head_unit_norm", False)), bool(e.get("head_gate", False))
-        if self.chunk < 0:
-            raise ConfigError("normed-qk attention: a chunk must be a positive number of tokens")
+        self.window = spec.window
+        self.chunk = int(e.get("chunk", 0) or 0)
+        if self.chunk < 0 or (self.window is not None and (self.window <= 0 or self.chunk > 0)):
+            raise ConfigError("normed-qk attention: a chunk or a window must be a positive number of tokens, and not both given")
+        sink = e.get("sink", False)
+        if sink not in (False, True, "learned"):
+            raise ConfigError(f"normed-qk attention: sink '{sink}' is not known")
+        self.sink = None if not sink else (rt.gain(weights["sink"]) if sink == "learned" else
+                                           torch.zeros(h, dtype=torch.float32, device=rt.device))
+        self.head_unit_norm = bool(e.get("head_unit_norm", False))
+        self.head_gate, self.element_gate = bool(e.get("head_gate", False)), bool(e.get("element_gate", False))
+        if self.head_gate and self.element_gate:
+            raise ConfigError("normed-qk attention: one gate per head or one per coordinate, not both")
+        self.temperature = tuple(float(x) for x in e["temperature"]) if e.get("temperature") is not None else None
+        if self.temperature is not None and not self.temperature[1] > 0:
+            raise ConfigError("normed-qk attention: the temperature's stretch must be positive")
+        self.value_mix = e.get("value_mix")
+        if self.value_mix not in (None, "first", "later"):
+            raise ConfigError(f"normed-qk attention: value_mix '{self.value_mix}' is not known (first, later)")
+        self.mix_weight = float(weights["vmix"].float()) if self.value_mix == "later" else 0.0
         # A factor on the mixer's output that whoever owns it may set (mixers side by side weight their outputs): with a
-        # gate per head it rides in the gate, before the output projection, which is linear.
-        self.takes_output_scale, self.output_scale = self.head_gate, 1.0
-        if self.head_gate:
-            self.kernel_modules = ("latent",)         # the library of csrc that holds the per-head gate
+        # gate it rides in the gate, before the output projection, which is linear.
+        self.takes_output_scale, self.output_scale = self.head_gate or self.element_gate, 1.0
+        if self.takes_output_scale:
+            self.kernel_modules = ("latent",)         # the library of csrc that holds the gates
         self.scale = float(spec.softmax_scale)
         self.eps = float(e.get("norm_eps", 1e-6))
         self.position = part("position", spec.position.kind)(spec.position, hidden_size, {}, rt)
@@ -559,23 +594,37 @@ class NormedQKAttention(PagedAttendMixin, Part):
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         self.inv_freq = self.position.inv_freq if self.position.rotary_dim > 0 else \
             torch.zeros(0, dtype=torch.float32, device=rt.device)
-        self.cols = (h + g) * d + g * v               # the gates' columns follow these
-        rows = [weights["q"], weights["k"], weights["v"]] + ([weights["g"]] if self.head_gate else [])
-        pad = -(self.cols + (h if self.head_gate else 0)) % 8     # zero rows, so that every row of the result starts on 16 bytes
-        if pad:
-            rows.append(torch.zeros(pad, hidden_size, dtype=weights["q"].dtype, device=weights["q"].device))
-        self.w_qkv = rt.weight(torch.cat(rows, dim=0))
-        self.w_o = rt.weight(weights["o"])
+        self.cols = (h + g) * d + g * v               # the gates' columns follow these (from a multiple of 8 on: 16-byte rows)
+        rows = [weights["q"], weights["k"], weights["v"]]
+        if self.element_gate:
+            rows += _zero_rows(-self.cols % 8, weights["q"])
+        self.gate_col = sum(x.shape[0] for x in rows)
+        if self.takes_output_scale:
+            rows.append(weights["g"])
+        rows += _zero_rows(-sum(x.shape[0] for x in rows) % 8, weights["q"])       # every row of the result starts on 16 bytes
         self.bias = rt.gain(torch.cat([weights["q.b"], weights["k.b"], weights["v.b"]])) if bias else None
         self.q_gain = rt.gain(weights["q.norm"]) if qk_norm else None
         self.k_gain = rt.gain(weights["k.norm"]) if qk_norm else None
+        self.output_bias = rt.gain(weights["o.b"]) if e.get("output_bias", False) else None
+        self.affine = (None, self.output_bias) if self.output_bias is not None else None
+        if e.get("joined", False):
+            if self.output_bias is not None:
+                raise ConfigError("normed-qk attention: a side of joined mixers has no bias on its output projection")
+            self.in_rows, self.out_matrix = torch.cat(rows, dim=0), weights["o"]
+        else:
+            self.w_qkv = rt.weight(torch.cat(rows, dim=0))
+            self.w_o = rt.weight(weights["o"])
+
+    def bind_output_scale(self, scale) -> None:
+        """The output's columns are multiplied by ``scale`` as they join the stream (the output bias too)."""
+        self.affine = (scale, scale * self.output_bias if self.output_bias is not None else None)
 
     def cache_need(self):
-        # with a chunk mask the keys before the running chunk are never read again: the cache gives their pages back
+        # with a chunk mask or a window the keys before it are never read again: the cache gives their pages back
         chunk = self.chunk or None
         if self.value_dim == self.head_dim:
-            return PagedKVNeed(self.n_kv, self.head_dim, None, chunk)
-        return PagedNeed((("k", (self.n_kv, self.head_dim)), ("v", (self.n_kv, self.value_dim))), None, chunk)
+            return PagedKVNeed(self.n_kv, self.head_dim, self.window, chunk)
+        return PagedNeed((("k", (self.n_kv, self.head_dim)), ("v", (self.n_kv, self.value_dim))), self.window, chunk)
 
     def weights_in_order(self) -> tuple:
         return (self.w_qkv, self.w_o)
@@ -583,39 +632,77 @@ class NormedQKAttention(PagedAttendMixin, Part):
     def can_fuse_norm(self, norm, n_rows: int) -> bool:
         return self.rt.skinny(n_rows, self.hidden_size) and self.rt.fuses_norm(norm)
 
+    hands_off_norm = True       # forward_fused_norm / forward_prenormed accept then_norm= and may return its NormHandoff
+
     def forward(self, x: torch.Tensor, ctx, cache, residual=None):
         return self.finish(self.rt.linear(x, self.w_qkv), ctx, cache, residual=residual)
 
-    def forward_fused_norm(self, h: torch.Tensor, norm, ctx, cache, residual=None):
+    def forward_fused_norm(self, h: torch.Tensor, norm, ctx, cache, residual=None, then_norm=None):
         """As forward, with x = norm(h): the norm runs inside the projection (steps of a few rows)."""
-        return self.finish(self.project(h, norm), ctx, cache, residual=residual)
+        return self.finish(self.project(h, norm), ctx, cache, residual=residual, then_norm=then_norm)
+
+    def forward_prenormed(self, pre, ctx, cache, residual=None, then_norm=None):
+        """As forward_fused_norm, with the norm prepared by the kernel that last added into the stream."""
+        qkv = self.rt.empty(pre.x.shape[0], self.w_qkv.shape[0])
+        ops.gemv_bf16(pre.x, self.w_qkv, qkv, ops.STORE_BF16, pre=pre)
+        return self.finish(qkv, ctx, cache, residual=residual, then_norm=then_norm)
 
     def project(self, h: torch.Tensor, norm) -> torch.Tensor:
         qkv = self.rt.empty(h.shape[0], self.w_qkv.shape[0])
         ops.gemv_norm_bf16(h, norm.gain, norm.eps, None, self.w_qkv, qkv, ops.STORE_BF16)
         return qkv
 
-    def finish(self, qkv: torch.Tensor, ctx, cache, residual=None):
+    def finish(self, qkv: torch.Tensor, ctx, cache, residual=None, then_norm=None):
+        rt = self.rt
+        att = self.between(qkv, 0, ctx, cache)
+        # the product leaves in FP32 (or is added into the FP32 stream by the kernel itself): the residual sum
+        # sees it unrounded
+        handoff = rt.handoff(then_norm, qkv.shape[0], self.hidden_size, att.shape[1]) if residual is not None else None
+        if residual is None and self.affine is not None:
+            raise ConfigError("normed-qk attention: a bias or scale on the output needs an arrangement that hands over the stream")
+        out = rt.linear(att, self.w_o, out_dtype=torch.float32, residual=residual, handoff=handoff, affine=self.affine)
+        return handoff if handoff is not None else out
+
+    def between(self, qkv: torch.Tensor, col0: int, ctx, cache, out=None, out_col: int = 0) -> torch.Tensor:
+        """Everything between the projections: from columns ``col0`` on of qkv to the gated heads [T, H V] - or into those
+        columns of ``out``.  Single tokens may come projected in FP32."""
         rt = self.rt
         n = qkv.shape[0]
         h, g, d, v = self.n_heads, self.n_kv, self.head_dim, self.value_dim
         table = ctx.block_tables[cache.group]
         q = rt.empty(n, h * d)
+        v_col = col0 + (h + g) * d
+        first = None
+        if self.value_mix == "first":
+            # later layers read this layer's values from its projection
+            ctx.shared["first_values"] = (qkv, v_col, self.bias[(h + g) * d:self.cols] if self.bias is not None else None)
+        elif self.value_mix == "later":
+            first = ctx.shared["first_values"] + (self.mix_weight,)
         ops.qk_norm_rope(qkv, self.bias, self.q_gain, self.k_gain, self.eps, ctx.positions, ctx.seq_of_token, table,
                          self.inv_freq, self.magnitude, q, cache.k_pages if cache.writable else None,
                          cache.v_pages if cache.writable else None, h, g, d, v, self.position.rotary_dim, rt.page_size,
-                         head_unit=self.head_unit_norm)
-        att = rt.empty(n, h * v)
+                         head_unit=self.head_unit_norm, col0=col0, temperature=self.temperature, first_values=first)
+        plain = out is not None and not self.element_gate and not self.head_gate
+        att = out if plain and out_col == 0 and out.shape[1] == h * v else rt.empty(n, h * v)
         if v == d:
             self._attend(q, cache, att, ctx, table)
         else:
             ops.attention_generic(q, cache.k_pages, cache.v_pages, att, ctx.positions, ctx.seq_of_token, table,
-                                  h, g, d, rt.page_size, None, self.scale, value_dim=v, chunk=self.chunk, sink=self.sink)
-        if self.head_gate:
-            ops.head_gate(att, qkv, self.cols, h, v, scale=self.output_scale)
-        # the product leaves in FP32 (or is added into the FP32 stream by the kernel itself): the residual sum
-        # sees it unrounded
-        return rt.linear(att, self.w_o, out_dtype=torch.float32, residual=residual)
+                                  h, g, d, rt.page_size, self.window, self.scale, value_dim=v, chunk=self.chunk, sink=self.sink)
+        if self.element_gate:
+            ops.element_gate(att, qkv, col0 + self.gate_col, out=out, out_col=out_col, scale=self.output_scale)
+        elif self.head_gate:
+            gates, col = (qkv, col0 + self.gate_col) if qkv.dtype == att.dtype else (qkv[:, col0:].to(att.dtype).contiguous(), self.gate_col)
+            ops.head_gate(att, gates, col, h, v, scale=self.output_scale)
+        if out is None:
+            return att
+        if not self.element_gate and att is not out:
+            out[:, out_col:out_col + h * v].copy_(att)
+        return out
+
+
+def _zero_rows(n: int, like: torch.Tensor) -> list:
+    return [torch.zeros(n, like.shape[1], dtype=like.dtype, device=like.device)] if n > 0 else []
 
 
 class DifferentialAttention(PagedAttendMixin, Part):
@@ -773,14 +860,16 @@ class ParallelMixers(Part):
     specs (``left``, ``right``: MixerSpec of any registered kinds) and the two scales come in the spec's extra; the
     weights of each lie under its side's name ("left.q", "right.o", ...).  Each side keeps what it needs between steps
     in the layer run's one cache view - so at most one of them may need pages, and at most one a state (attention beside
-    a recurrence, say).  The sum is FP32.  Where both sides can carry a factor on their output themselves
-    (``takes_output_scale``) and the second can add its output projection into a given FP32 tensor, the scales ride in
-    the sides' own kernels and the second side's last product adds into the first side's result; otherwise one more
-    kernel forms the weighted sum."""
+    a recurrence, say).  The sum is FP32.  Three ways of running them:
+
+    joined      (``join`` in the extra, sides whose class says ``JOINS``) one product for everything both sides project,
+                both sides write what their output projections read side by side into one matrix - each with its scale
+                inside its own last kernel -, and one product with [W_o left | W_o right] gives the weighted sum;
+    folded      both sides can carry a factor on their output themselves (``takes_output_scale``) and the second can add
+                its output projection into a given FP32 tensor: the second side's last product adds into the first's result;
+    plain       one more kernel forms the weighted sum."""
 
     kernel_modules = ("pointwise",)       # the library of csrc that holds the weighted sum
-
-    adds_into_residual = False
 
     @staticmethod
     def _sides(spec):
@@ -792,21 +881,46 @@ class ParallelMixers(Part):
         slots = {}
         for name, sub, _ in ParallelMixers._sides(spec):
             for slot, ws in part("mixer", sub.kind).weight_slots(sub, hidden_size).items():
+                if any(isinstance(n, FreeDim) for n in ws.shape):            # free sizes are a side's own
+                    ws = replace(ws, shape=tuple(FreeDim(n, f"{name}.{n.label}") if isinstance(n, FreeDim) else n for n in ws.shape))
                 slots[f"{name}.{slot}"] = ws
         return slots
 
     def __init__(self, spec, hidden_size, weights, rt) -> None:
         Part.__init__(self, spec, hidden_size, weights, rt)
         self.sub_parts, self.scales = [], []
+        self.joined = bool(spec.extra_dict().get("join", False)) and \
+            all(getattr(part("mixer", sub.kind), "JOINS", False) for _, sub, _ in self._sides(spec))
         for name, sub, scale in self._sides(spec):
             own = {slot[len(name) + 1:]: w for slot, w in weights.items() if slot.startswith(name + ".")}
+            if self.joined:
+                sub = replace(sub, extra=sub.extra + (("joined", True),))
             self.sub_parts.append(part("mixer", sub.kind)(sub, hidden_size, own, rt))
             self.scales.append(scale)
         first, second = self.sub_parts
-        self.folded = (all(getattr(p, "takes_output_scale", False) for p in self.sub_parts)
-                       and getattr(second, "adds_into_residual", False))
-        if self.folded:
+        if self.joined and not all(getattr(p, "takes_output_scale", False) for p in self.sub_parts):
+            raise ConfigError("mixers side by side: joined sides must be able to carry a factor on their output")
+        self.folded = not self.joined and (all(getattr(p, "takes_output_scale", False) for p in self.sub_parts)
+                                           and getattr(second, "adds_into_residual", False))
+        if self.folded or self.joined:
             first.output_scale, second.output_scale = self.scales
+        self.affine = None
+        self.adds_into_residual = self.joined
+        if self.joined:
+            self.in_cols = (0, first.in_rows.shape[0])
+            self.out_cols = (0, first.out_matrix.shape[1])
+            self.w_in = rt.weight(torch.cat([p.in_rows for p in self.sub_parts], dim=0))
+            outs = [p.out_matrix for p in self.sub_parts]
+            self.out_width = sum(w.shape[1] for w in outs)
+            self.pad = -self.out_width % 8                        # zero columns: rows of 16 bytes for the products
+            if self.pad:
+                outs.append(torch.zeros(hidden_size, self.pad, dtype=outs[0].dtype, device=outs[0].device))
+            self.w_out = rt.weight(torch.cat(outs, dim=1))
+            for p in self.sub_parts:
+                p.w_o = self.w_out                                # what a side may ask into L2 ahead of its product
+                del p.in_rows, p.out_matrix
+            self.forward_fused_norm, self.forward_prenormed = self._forward_fused_norm, self._forward_prenormed
+            self.bind_output_scale = self._bind_output_scale
         safety = [getattr(p, "graph_safe", "none") for p in self.sub_parts]
         self.graph_safe = "all" if all(x == "all" for x in safety) else \
             ("decode" if all(x in ("decode", "all") for x in safety) else "none")
@@ -823,9 +937,55 @@ class ParallelMixers(Part):
         return tuple(needs) if len(needs) > 1 else (needs[0] if needs else None)
 
     def weights_in_order(self) -> tuple:
+        if self.joined:
+            return (self.w_in, self.w_out)
         return tuple(w for p in self.sub_parts for w in getattr(p, "weights_in_order", tuple)())
 
-    def forward(self, x: torch.Tensor, ctx, cache):
+    # ---- joined -----------------------------------------------------------------------------------------
+    hands_off_norm = True       # _forward_fused_norm / _forward_prenormed accept then_norm=
+
+    def _bind_output_scale(self, scale) -> None:
+        self.affine = (scale, None)
+
+    def can_fuse_norm(self, norm, n_rows: int) -> bool:
+        return self.joined and self.rt.skinny(n_rows, self.hidden_size) and self.rt.fuses_norm(norm)
+
+    def _token_dtype(self, ctx):
+        """What the joined projection of a few rows leaves in: FP32 where a side asks for it in steps of single tokens."""
+        f32 = ctx.max_q_len == 1 and any(p.wants_f32_tokens for p in self.sub_parts)
+        return (torch.float32, ops.STORE_F32) if f32 else (self.rt.dtype, ops.STORE_BF16)
+
+    def _forward_fused_norm(self, h, norm, ctx, cache, residual=None, then_norm=None):
+        dtype, mode = self._token_dtype(ctx)
+        proj = self.rt.empty(h.shape[0], self.w_in.shape[0], dtype=dtype)
+        ops.gemv_norm_bf16(h, norm.gain, norm.eps, None, self.w_in, proj, mode)
+        return self._between(proj, ctx, cache, residual, then_norm)
+
+    def _forward_prenormed(self, pre, ctx, cache, residual=None, then_norm=None):
+        dtype, mode = self._token_dtype(ctx)
+        proj = self.rt.empty(pre.x.shape[0], self.w_in.shape[0], dtype=dtype)
+        ops.gemv_bf16(pre.x, self.w_in, proj, mode, pre=pre)
+        return self._between(proj, ctx, cache, residual, then_norm)
+
+    def _between(self, proj, ctx, cache, residual, then_norm=None):
+        rt = self.rt
+        n = proj.shape[0]
+        mixed = rt.empty(n, self.out_width + self.pad)
+        if self.pad:
+            mixed[:, self.out_width:].zero_()
+        for p, col, out_col in zip(self.sub_parts, self.in_cols, self.out_cols):
+            p.between(proj, col, ctx, cache, out=mixed, out_col=out_col)
+        if residual is None and self.affine is not None:
+            raise ConfigError("mixers side by side: a scale on the output needs an arrangement that hands over the stream")
+        handoff = rt.handoff(then_norm, n, self.hidden_size, mixed.shape[1]) if residual is not None else None
+        out = rt.linear(mixed, self.w_out, out_dtype=torch.float32, residual=residual, handoff=handoff, affine=self.affine)
+        return handoff if handoff is not None else out
+
+    # ---- folded and plain ---------------------------------------------------------------------------------
+    def forward(self, x: torch.Tensor, ctx, cache, residual=None):
+        if self.joined:
+            dtype, _ = self._token_dtype(ctx) if self.rt.skinny(x.shape[0], self.hidden_size) else (None, None)
+            return self._between(self.rt.linear(x, self.w_in, out_dtype=dtype), ctx, cache, residual)
         first, second = self.sub_parts
         left = first.forward(x, ctx, cache)
         if left.dtype != torch.float32:

@@ -8,7 +8,7 @@ import torch
 from ..config.model_config import ConfigError
 from ..config.registry import part, register_part
 from ..kernels import ops
-from .base import Part, StateNeed, WeightSlot
+from .base import FreeDim, Part, StateNeed, WeightSlot
 
 
 class GatedDeltaRule(Part):
@@ -21,16 +21,27 @@ class GatedDeltaRule(Part):
     v (``num_heads`` heads of ``value_dim``) pass a short causal convolution over time per channel
     (``conv_taps`` taps, the last one the current token's, no bias) and silu; q and k are then unit
     vectors per head (1e-6 under the root), q also times head_dim^-1/2.  beta = sigmoid(W_b x), one per
-    head; decay = exp(-exp(A_log) softplus(W_a x + dt_bias)), one per head.  Each head's y is divided by its
-    root mean square (``norm_eps``), multiplied by a weight [value_dim] shared by the heads and by
-    silu(W_g x), and leaves through W_o.
+    head.  Each head's y is divided by its root mean square (``norm_eps``), multiplied by a weight [value_dim] shared by
+    the heads and by a gate, and leaves through W_o.  Two options in the spec's extra:
 
-    All projections of x are ONE product (rows q | k | v | gate | b | a) whose results stay FP32;
-    everything from there to the gated norm is FP32 on the device.  A request's state is one FP32 vector:
-    M of every head, then the last conv_taps - 1 inputs of every convolved channel.  A step's kernels
-    run exactly once, so the state advances by exactly the step's tokens."""
+    ``decay``  "head" (the default): one decay per head, exp(-exp(A_log) softplus(W_a x + dt_bias));
+               "key_channel": one per head and key channel, exp(-exp(A_log_h) softplus(W_a2 (W_a1 x) + dt_bias)), which
+               multiplies the rows of M - W_a1 and W_a2 are thin, their inner size follows from the stored tensors;
+    ``gate``   "silu" (the default): silu(W_g x); "low_rank_sigmoid": sigmoid(W_g2 (W_g1 x)), thin in the same way.
+
+    All projections of x are ONE product (rows q | k | v | gate | b | a, or q | k | v | b | a1 | g1); with thin matrices a
+    second, block-diagonal product turns (W_a1 x, W_g1 x) into the logits of decay and gate in FP32.  Everything from there
+    to the gated norm is FP32 on the device.  A request's state is one FP32 vector: M of every head, then the last
+    conv_taps - 1 inputs of every convolved channel.  A step's kernels run exactly once, so the state advances by exactly
+    the step's tokens.
+
+    ``joined`` in the extra: one side of mixers that share their input and output projections (ParallelMixers)."""
 
     kernel_modules = ("delta_rule",)       # libraries of csrc that this part's kernels live in
+
+    JOINS = True                # can be a side of mixers with joined projections
+    takes_output_scale = True   # a factor on the output rides in the gated norm, before the output projection
+    output_scale = 1.0
 
     adds_into_residual = True
     graph_safe = "all"
@@ -41,14 +52,34 @@ class GatedDeltaRule(Part):
         return spec.num_kv_heads, spec.num_heads, spec.head_dim, int(e["value_dim"]), int(e["conv_taps"])
 
     @staticmethod
+    def _options(spec):
+        e = spec.extra_dict()
+        decay, gate = e.get("decay", "head"), e.get("gate", "silu")
+        if decay not in ("head", "key_channel") or gate not in ("silu", "low_rank_sigmoid"):
+            raise ConfigError(f"gated delta rule: decay '{decay}' (head, key_channel) or gate '{gate}' (silu, low_rank_sigmoid) "
+                              f"is not known")
+        return decay == "key_channel", gate == "low_rank_sigmoid"
+
+    @staticmethod
     def weight_slots(spec, hidden_size: int) -> Dict[str, WeightSlot]:
         g, h, d, v, taps = GatedDeltaRule._dims(spec)
-        return {"q": WeightSlot((g * d, hidden_size)), "q.conv": WeightSlot((g * d, taps)),
-                "k": WeightSlot((g * d, hidden_size)), "k.conv": WeightSlot((g * d, taps)),
-                "v": WeightSlot((h * v, hidden_size)), "v.conv": WeightSlot((h * v, taps)),
-                "b": WeightSlot((h, hidden_size)), "A_log": WeightSlot((h,)), "norm": WeightSlot((v,), init="ones"),
-                "a": WeightSlot((h, hidden_size)), "dt_bias": WeightSlot((h,)),
-                "g": WeightSlot((h * v, hidden_size)), "o": WeightSlot((hidden_size, h * v))}
+        channel, thin_gate = GatedDeltaRule._options(spec)
+        slots = {"q": WeightSlot((g * d, hidden_size)), "q.conv": WeightSlot((g * d, taps)),
+                 "k": WeightSlot((g * d, hidden_size)), "k.conv": WeightSlot((g * d, taps)),
+                 "v": WeightSlot((h * v, hidden_size)), "v.conv": WeightSlot((h * v, taps)),
+                 "b": WeightSlot((h, hidden_size)), "A_log": WeightSlot((h,)), "norm": WeightSlot((v,), init="ones")}
+        if channel:
+            rank = FreeDim(d, "decay_rank")
+            slots.update({"a1": WeightSlot((rank, hidden_size)), "a2": WeightSlot((h * d, rank)), "dt_bias": WeightSlot((h * d,))})
+        else:
+            slots.update({"a": WeightSlot((h, hidden_size)), "dt_bias": WeightSlot((h,))})
+        if thin_gate:
+            rank = FreeDim(v, "gate_rank")
+            slots.update({"g1": WeightSlot((rank, hidden_size)), "g2": WeightSlot((h * v, rank))})
+        else:
+            slots["g"] = WeightSlot((h * v, hidden_size))
+        slots["o"] = WeightSlot((hidden_size, h * v))
+        return slots
 
     def __init__(self, spec, hidden_size, weights, rt) -> None:
         super().__init__(spec, hidden_size, weights, rt)
@@ -60,13 +91,58 @@ class GatedDeltaRule(Part):
         if v <= 0 or taps <= 0:
             raise ConfigError("gated delta rule: value size and convolution taps must be positive")
         self.G, self.H, self.D, self.V, self.taps = g, h, d, v, taps
+        self.channel, self.thin_gate = self._options(spec)
         self.eps = float(spec.extra_dict().get("norm_eps", 1e-6))
         self.channels = 2 * g * d + h * v
-        self.w_in = rt.weight(torch.cat([weights[s] for s in ("q", "k", "v", "g", "b", "a")], dim=0))
-        self.w_o = rt.weight(weights["o"])
+        rows = [weights[s] for s in ("q", "k", "v")]
+        at = self.channels
+        self.gate_col = at                                     # (a full gate's)
+        if not self.thin_gate:
+            rows.append(weights["g"])
+            at += h * v
+        self.b_col = at
+        rows.append(weights["b"])
+        at += h
+        if not self.channel:
+            rows.append(weights["a"])
+            at += h
+        joined = bool(spec.extra_dict().get("joined", False))
+        like = weights["q"]
+
+        def zeros(n, k):
+            return torch.zeros(n, k, dtype=like.dtype, device=like.device)
+
+        # the thin matrices: their inner sizes padded with zeros to multiples of 8, from a multiple of 8 columns on
+        self.thin_col = self.thin_k = 0
+        self.w_thin = None
+        if self.channel or self.thin_gate:
+            if at % 8:
+                rows.append(zeros(-at % 8, hidden_size))
+            self.thin_col = at + -at % 8
+            pairs = ([("a1", "a2")] if self.channel else []) + ([("g1", "g2")] if self.thin_gate else [])
+            second, self.ranks = [], {}
+            for one, two in pairs:
+                rank = weights[one].shape[0]
+                if weights[two].shape[1] != rank:
+                    raise ConfigError(f"gated delta rule: {one} and {two} differ in their inner size")
+                rows += [weights[one]] + ([zeros(-rank % 8, hidden_size)] if rank % 8 else [])
+                padded = torch.cat([weights[two], zeros(weights[two].shape[0], -rank % 8)], dim=1)
+                second.append(padded)
+                self.ranks[one] = padded.shape[1]
+                self.thin_k += padded.shape[1]
+            self.w_thin = rt.weight(torch.block_diag(*[x.float() for x in second]).to(like.dtype))        # [H D (+ H V), ranks]
+            at = self.thin_col + self.thin_k
+        if joined and at % 8:
+            rows.append(zeros(-at % 8, hidden_size))
+        if joined:
+            self.in_rows, self.out_matrix = torch.cat(rows, dim=0), weights["o"]
+        else:
+            self.w_in = rt.weight(torch.cat(rows, dim=0))
+            self.w_o = rt.weight(weights["o"])
         self.conv_w = rt.gain(torch.cat([weights[s] for s in ("q.conv", "k.conv", "v.conv")], dim=0))
         self.a_log, self.dt_bias = rt.gain(weights["A_log"]), rt.gain(weights["dt_bias"])
         self.norm_w = rt.gain(weights["norm"])
+        self.wants_f32_tokens = False
 
     def cache_need(self):
         return StateNeed((self.H * self.D * self.V + (self.taps - 1) * self.channels,), "float32")
@@ -85,19 +161,45 @@ class GatedDeltaRule(Part):
         return proj
 
     def finish(self, proj: torch.Tensor, ctx, cache, residual=None):
+        y = self.rt.empty(proj.shape[0], self.H * self.V)
+        self.between(proj, 0, ctx, cache, out=y)
+        return self.rt.linear(y, self.w_o, residual=residual)
+
+    def _thin_logits(self, proj: torch.Tensor, col0: int):
+        """FP32 [T, H D (+ H V)]: the logits of decay and gate from their thin first products in ``proj``."""
+        rt = self.rt
+        n = proj.shape[0]
+        x = proj[:, col0 + self.thin_col:col0 + self.thin_col + self.thin_k]
+        if rt.dtype == torch.float32:
+            z = rt.empty(n, self.w_thin.shape[0])
+            ops.gemm_f32_heads(x, self.w_thin.view(1, *self.w_thin.shape), z)
+            return z
+        if x.dtype != torch.bfloat16 or rt.skinny(n, self.thin_k):
+            x = x.to(torch.bfloat16).contiguous()
+        return rt.linear(x, self.w_thin, out_dtype=torch.float32)
+
+    def between(self, proj: torch.Tensor, col0: int, ctx, cache, out: torch.Tensor, out_col: int = 0) -> torch.Tensor:
+        """Everything between the projections: from columns ``col0`` on of proj to the gated, normed read-outs in columns
+        ``out_col`` on of ``out``."""
         rt = self.rt
         n = proj.shape[0]
         f32 = torch.float32
         g, h, d, v = self.G, self.H, self.D, self.V
+        z = self._thin_logits(proj, col0) if self.w_thin is not None else None
+        decay = z if self.channel else None
         qkv = rt.empty(n, self.channels, dtype=f32)
         gates = rt.empty(n, h, 2, dtype=f32)
         ops.delta_prepare(proj, self.conv_w, self.a_log, self.dt_bias, cache.state, ctx.seq_of_token, ctx.cu_q,
-                          ctx.slots, ctx.n_seqs, g, h, d, v, self.taps, qkv, gates)
+                          ctx.slots, ctx.n_seqs, g, h, d, v, self.taps, qkv, gates, col0=col0, b_col=col0 + self.b_col, z=decay)
         o = rt.empty(n, h * v, dtype=f32)
-        ops.delta_recurrence(qkv, gates, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, g, h, d, v, o)
-        y = rt.empty(n, h * v)
-        ops.delta_gated_norm(o, proj, self.norm_w, self.eps, g, h, d, v, y, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, self.taps)
-        return rt.linear(y, self.w_o, residual=residual)
+        ops.delta_recurrence(qkv, gates, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, g, h, d, v, o, z=decay)
+        gate, gate_col = (z, h * d if self.channel else 0) if self.thin_gate else (proj, col0 + self.gate_col)
+        if gate.dtype != f32:
+            gate, gate_col = gate[:, gate_col:gate_col + h * v].to(f32).contiguous(), 0
+        ops.delta_gated_norm(o, proj, self.norm_w, self.eps, g, h, d, v, out, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs,
+                             self.taps, col0=col0, gate=gate, gate_col=gate_col, sigmoid=self.thin_gate,
+                             scale=self.output_scale, y_col=out_col)
+        return out
 
 
 class LightningAttention(Part):

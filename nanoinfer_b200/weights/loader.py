@@ -16,6 +16,7 @@ from typing import Dict, List
 import torch
 
 from ..config.model_config import ConfigError, ModelConfig
+from ..parts.base import FreeDim
 from . import safetensors_io as sio
 from .plan import tensor_plan
 
@@ -46,6 +47,26 @@ def _stored_dtype(t: torch.Tensor) -> torch.Tensor:
     return t
 
 
+def _wrong_shapes(plan, found) -> list:
+    """(name, planned shape, found shape) where the two differ.  A free size takes any positive number, but the same one
+    for every tensor of its scope that has it under that label."""
+    wrong, seen = [], {}
+    for name, p in plan.items():
+        if name not in found:
+            continue
+        shape = tuple(found[name])
+        ok = len(shape) == len(p.shape)
+        if ok:
+            for want, have in zip(p.shape, shape):
+                if isinstance(want, FreeDim):
+                    ok = ok and have > 0 and seen.setdefault((p.scope, want.label), have) == have
+                else:
+                    ok = ok and want == have
+        if not ok:
+            wrong.append((name, p.shape, shape))
+    return wrong
+
+
 def check_tensors(model_dir: str, config: ModelConfig, found: Dict[str, tuple]) -> None:
     """Compare {name: shape} of a folder with the configuration's plan; raise WeightError."""
     plan = {p.name: p for p in tensor_plan(config)}
@@ -61,7 +82,7 @@ def check_tensors(model_dir: str, config: ModelConfig, found: Dict[str, tuple]) 
             pass                      # an architecture whose output is always the embedding's table names none
     unexpected = [n for n in found if n not in plan and n not in allowed_extra
                   and not any(fnmatchcase(n, pat) for pat in arch.ignored_tensors)]
-    wrong = [(n, plan[n].shape, found[n]) for n in plan if n in found and tuple(found[n]) != plan[n].shape]
+    wrong = _wrong_shapes(plan, found)
     if missing or unexpected or wrong:
         raise WeightError(model_dir, sorted(missing), sorted(unexpected), sorted(wrong))
 
