@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the Llama 3.2 1B shape with random weights.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers 16] [--impl ours|reference]
-    python bench.py --design runevik|vuvalorn|tazulix|mobatar|kepusun [--sizes w1024,w2048]     (another design beside the Llama model of equal size)
+    python bench.py --design runevik|vuvalorn|tazulix|mobatar|kepusun|lomopel [--sizes w1024,w2048]     (another design beside the Llama model of equal size)
 
 A "step" is one decode step of the whole batch.  Every request starts at a context of 2,048
 tokens and decodes W + K tokens (by default to 4,096).  Prints ONE JSON line:
@@ -494,8 +494,28 @@ def kepusun_config(z):
             "layers": [layer(i) for i in range(z["layers"])]}
 
 
+def lomopel_config(z):
+    """As many layers as the Llama model has, every third (from the first on) attention over all keys, the others side-by-side
+    layers.  Heads of 128 throughout, the Llama model's head counts in both kinds of attention (the side-by-side layers' under a
+    window of 1,024), half as many delta heads of 128 x 128, each with query and key heads of its own; thin matrices of 128.  The
+    feed-forward is the Llama model's with gelu."""
+    heads = z["width"] // 128
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    att = {"heads": heads, "kv_heads": z["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    n_right = max(heads // 2, 1)
+    left = dict(att, mask={"size": 1024}, rot={"dims": 128, "base": 500000.0})
+    right = {"heads": n_right, "kv_heads": n_right, "dim": 128, "vdim": 128, "conv": 4}
+
+    def layer(i):
+        if i % 3 == 0:
+            return {"type": "attention", "mlp": mlp, "mixer": dict(att, v_mix=True, q_temp={"coef": 0.1, "every": 2000})}
+        return {"type": "parallel", "mlp": mlp, "mixer": {"left": left, "right": right, "left_scale": 0.9, "right_scale": 1.2}}
+    return {"architecture": "Lomopel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "layers": [layer(i) for i in range(z["layers"])]}
+
+
 DESIGN_CONFIGS = {"runevik": runevik_config, "vuvalorn": vuvalorn_config, "tazulix": tazulix_config, "mobatar": mobatar_config,
-                  "kepusun": kepusun_config}
+                  "kepusun": kepusun_config, "lomopel": lomopel_config}
 
 
 def llama_config(z):

@@ -461,3 +461,208 @@ NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate
 #undef GO
     NI_RETURN_LAUNCH_STATUS();
 }
+// ---- a step of single tokens with decays per channel: everything between the projections in one launch -------------------
+//
+// One block of 8 warps per (head, request).  A warp owns every 8th row of S, a lane every 32nd column; S is read into
+// registers first, before anything else is needed.  Meanwhile: the convolution of the head's q, k and v channels (a thread
+// per channel), the thin second products of its D decay logits and V gate logits (a thread per row of the weights, which
+// are bfloat16 rows of 16-byte pieces; the thin first products stand in shared memory), unit norms.  Then k S, the error,
+// the update, q S and the gated norm; S is written back once.
+// The convolution history of the value channels is moved on by their own block.  A query/key channel belongs to the H / G
+// heads that share it: the last of their blocks to have read the old inputs (an atomic ticket per request and q/k head, left
+// zero) moves them on.  No block waits for another.
+#define DT_WARPS 8
+struct DeltaTokenParams {
+    const float* proj;                 // [T, ld] FP32: q | k | v | ... b at b_off, the thin first products at thin_off
+    const __nv_bfloat16* w_decay;      // [H D, ra]
+    const __nv_bfloat16* w_gate;       // [H V, rg]
+    const float *conv_w, *a_log, *dt_bias, *norm_w;
+    float* state;
+    long long state_stride;
+    const int *cu_q, *slots;
+    int* tickets;                      // [requests, G], zero
+    __nv_bfloat16* y;
+    int ld_y, thin_off, ra, rg;
+    float eps, scale;
+};
+
+// Row . x for a row of n bfloat16 (n a multiple of 8, 16-byte aligned) and x in shared memory.
+__device__ __forceinline__ float dt_thin_dot(const __nv_bfloat16* __restrict__ row, const float* x, int n) {
+    float a0 = 0.f, a1 = 0.f;
+    for (int i = 0; i < n; i += 8) {
+        float w[8];
+        NiVec16<__nv_bfloat16>::load(row + i, w);
+        const float4 x0 = *reinterpret_cast<const float4*>(x + i), x1 = *reinterpret_cast<const float4*>(x + i + 4);
+        a0 = fmaf(w[0], x0.x, a0); a1 = fmaf(w[1], x0.y, a1);
+        a0 = fmaf(w[2], x0.z, a0); a1 = fmaf(w[3], x0.w, a1);
+        a0 = fmaf(w[4], x1.x, a0); a1 = fmaf(w[5], x1.y, a1);
+        a0 = fmaf(w[6], x1.z, a0); a1 = fmaf(w[7], x1.w, a1);
+    }
+    return a0 + a1;
+}
+
+// DR: rows of S per warp (D <= 8 DR); VC: columns per lane (V <= 32 VC).
+template <int DR, int VC>
+__global__ void __launch_bounds__(DT_WARPS * 32)
+delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
+    constexpr int DP = DT_WARPS * DR, VP = 32 * VC;
+    __shared__ float sq[DP], sk[DP], sg[DP], sv[VP], sgate[VP], su[VP], red[DT_WARPS][VP], scratch[32];
+    __shared__ float unit[2];          // what q and k are multiplied by
+    __shared__ int s_last;
+    extern __shared__ __align__(16) float thin[];       // [ra + rg]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.x, seq = blockIdx.y;
+    const int D = dm.D, V = dm.V, G = dm.G, C = dm.C(), per = dm.H / G, g = h / per, taps = dm.taps;
+    const int t = p.cu_q[seq];
+    float* st = p.state + (size_t)p.slots[seq] * p.state_stride;
+    float* S = st + (size_t)h * D * V;
+    float* hist = st + dm.hist_off();
+    float s[DR][VC];
+#pragma unroll
+    for (int i = 0; i < DR; ++i)
+#pragma unroll
+        for (int j = 0; j < VC; ++j) {
+            const int row = warp + DT_WARPS * i, col = lane + 32 * j;
+            s[i][j] = (row < D && col < V) ? S[(size_t)row * V + col] : 0.f;
+        }
+    const float* row = p.proj + (size_t)t * dm.ld;
+    for (int i = tid; i < p.ra + p.rg; i += blockDim.x) thin[i] = row[p.thin_off + i];
+    for (int i = tid; i < 2 * D + V; i += blockDim.x) {
+        const int c = i < D ? g * D + i : (i < 2 * D ? G * D + g * D + i - D : 2 * G * D + h * V + i - 2 * D);
+        const float x = row[c];
+        float acc = 0.f;
+        for (int j = 0; j + 1 < taps; ++j) acc = fmaf(p.conv_w[(size_t)c * taps + j], hist[(size_t)j * C + c], acc);
+        const float y = dr_silu(fmaf(p.conv_w[(size_t)c * taps + taps - 1], x, acc));
+        if (i < D) sq[i] = y;
+        else if (i < 2 * D) sk[i - D] = y;
+        else sv[i - 2 * D] = y;
+    }
+    __syncthreads();
+    if (tid == 0 && taps > 1) {
+        int last = 1;
+        if (per > 1) {
+            __threadfence();
+            int* ticket = p.tickets + (size_t)seq * G + g;
+            last = atomicAdd(ticket, 1) == per - 1;
+            if (last) *ticket = 0;
+        }
+        s_last = last;
+    }
+    for (int r = tid; r < D + V; r += blockDim.x) {
+        if (r < D) {
+            const int c = h * D + r;
+            sg[r] = dr_decay(p.a_log[h], dt_thin_dot(p.w_decay + (size_t)c * p.ra, thin, p.ra) + p.dt_bias[c]);
+        } else {
+            const int c = h * V + r - D;
+            sgate[r - D] = dr_sigmoid(dt_thin_dot(p.w_gate + (size_t)c * p.rg, thin + p.ra, p.rg)) * p.scale;
+        }
+    }
+    if (warp < 2) {
+        const float* v = warp == 0 ? sq : sk;
+        float ss = 0.f;
+        for (int i = lane; i < D; i += 32) ss = fmaf(v[i], v[i], ss);
+        ss = ni_warp_sum(ss);
+        if (lane == 0) unit[warp] = 1.0f / sqrtf(ss + 1e-6f) * (warp == 0 ? 1.0f / sqrtf((float)D) : 1.0f);
+    }
+    __syncthreads();
+    const float rq = unit[0], rk = unit[1];
+    float acc[VC];
+#pragma unroll
+    for (int j = 0; j < VC; ++j) acc[j] = 0.f;
+#pragma unroll
+    for (int i = 0; i < DR; ++i) {
+        const int r = warp + DT_WARPS * i;
+        const float gd = r < D ? sg[r] : 0.f, kk = r < D ? sk[r] * rk : 0.f;
+#pragma unroll
+        for (int j = 0; j < VC; ++j) {
+            s[i][j] *= gd;
+            acc[j] = fmaf(kk, s[i][j], acc[j]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < VC; ++j) red[warp][lane + 32 * j] = acc[j];
+    __syncthreads();
+    for (int c = tid; c < V; c += blockDim.x) {
+        float d = 0.f;
+#pragma unroll
+        for (int w = 0; w < DT_WARPS; ++w) d += red[w][c];
+        su[c] = dr_sigmoid(row[dm.b_off + h]) * (sv[c] - d);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < VC; ++j) acc[j] = 0.f;
+    float u[VC];
+#pragma unroll
+    for (int j = 0; j < VC; ++j) u[j] = lane + 32 * j < V ? su[lane + 32 * j] : 0.f;
+#pragma unroll
+    for (int i = 0; i < DR; ++i) {
+        const int r = warp + DT_WARPS * i;
+        const float kk = r < D ? sk[r] * rk : 0.f, qq = r < D ? sq[r] * rq : 0.f;
+#pragma unroll
+        for (int j = 0; j < VC; ++j) {
+            const int col = lane + 32 * j;
+            s[i][j] = fmaf(kk, u[j], s[i][j]);
+            acc[j] = fmaf(qq, s[i][j], acc[j]);
+            if (r < D && col < V) S[(size_t)r * V + col] = s[i][j];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < VC; ++j) red[warp][lane + 32 * j] = acc[j];
+    __syncthreads();
+    float o = 0.f;                     // V <= 128 < blockDim.x: a thread per column
+    if (tid < V) {
+#pragma unroll
+        for (int w = 0; w < DT_WARPS; ++w) o += red[w][tid];
+    }
+    const float ss = ni_block_sum(o * o, scratch);
+    if (tid < V)
+        p.y[(size_t)t * p.ld_y + (size_t)h * V + tid] =
+            __float2bfloat16_rn(o * (1.0f / sqrtf(ss / (float)V + p.eps)) * p.norm_w[tid] * sgate[tid]);
+    if (taps > 1) {
+        const int first = s_last ? 0 : 2 * D;          // the q and k channels only by the last of the heads that share them
+        for (int i = first + tid; i < 2 * D + V; i += blockDim.x) {
+            const int c = i < D ? g * D + i : (i < 2 * D ? G * D + g * D + i - D : 2 * G * D + h * V + i - 2 * D);
+            for (int j = 0; j + 2 < taps; ++j) hist[(size_t)j * C + c] = hist[(size_t)(j + 1) * C + c];
+            hist[(size_t)(taps - 2) * C + c] = row[c];
+        }
+    }
+}
+
+// The largest key and value sizes of ni_delta_token_step.
+NI_EXPORT int ni_delta_token_max_dim() { return 128; }
+
+// One token per request: proj FP32 [T, ld] (q | k | v from column 0, b at b_off, the thin first products - ra of the decay,
+// then rg of the gate, both multiples of 8 - at thin_off), w_decay bf16 [H D, ra], w_gate bf16 [H V, rg]; y bf16, rows ld_y
+// apart.  tickets: int32 zeros, at least n_seqs * G.  The state moves on, convolution history included.
+NI_EXPORT int ni_delta_token_step(const float* proj, int ld, int b_off, int thin_off, const void* w_decay, int ra,
+                                  const void* w_gate, int rg, const float* conv_w, const float* a_log, const float* dt_bias,
+                                  const float* norm_w, float eps, float scale, float* state, long long state_stride,
+                                  const int* cu_q, const int* slots, int* tickets, int n_seqs, int G, int H, int D, int V,
+                                  int taps, void* y, int ld_y, cudaStream_t stream) {
+    if (n_seqs <= 0) return NI_OK;
+    DeltaDims dm{G, H, D, V, taps, ld, b_off, -1};
+    if (int rc = dr_check(dm)) return rc;
+    if (b_off < 0 || thin_off < 0 || ra <= 0 || rg <= 0 || ra % 8 || rg % 8 || ld < thin_off + ra + rg || ld_y < H * V ||
+        (reinterpret_cast<size_t>(w_decay) & 15) || (reinterpret_cast<size_t>(w_gate) & 15))
+        return NI_ERR_BAD_ARGUMENT;
+    if (D > 128 || V > 128 || n_seqs > 65535 || ra + rg > 8192) return NI_ERR_UNSUPPORTED_SIZE;
+    DeltaTokenParams p = {};
+    p.proj = proj; p.w_decay = (const __nv_bfloat16*)w_decay; p.w_gate = (const __nv_bfloat16*)w_gate;
+    p.conv_w = conv_w; p.a_log = a_log; p.dt_bias = dt_bias; p.norm_w = norm_w;
+    p.state = state; p.state_stride = state_stride; p.cu_q = cu_q; p.slots = slots; p.tickets = tickets;
+    p.y = (__nv_bfloat16*)y; p.ld_y = ld_y; p.thin_off = thin_off; p.ra = ra; p.rg = rg; p.eps = eps; p.scale = scale;
+    const size_t smem = (size_t)(ra + rg) * sizeof(float);
+#define GO(DR, VC) delta_token_kernel<DR, VC><<<dim3(H, n_seqs), DT_WARPS * 32, smem, stream>>>(p, dm)
+#define GO_V(DR)                          \
+    do {                                  \
+        if (V <= 32) GO(DR, 1);           \
+        else if (V <= 64) GO(DR, 2);      \
+        else GO(DR, 4);                   \
+    } while (0)
+    if (D <= 32) GO_V(4);
+    else if (D <= 64) GO_V(8);
+    else GO_V(16);
+#undef GO_V
+#undef GO
+    NI_RETURN_LAUNCH_STATUS();
+}

@@ -7,6 +7,7 @@
     python -m nanoinfer_b200.kernels.microbench gemm_swap --m 64 --n 2048 --k 2048 --mode add --milestones
     python -m nanoinfer_b200.kernels.microbench decode_fused --batch 8 --context 2048
     python -m nanoinfer_b200.kernels.microbench delta_rule --batch 8 --tokens 1 --heads 16 --dim 128 --vdim 128
+    python -m nanoinfer_b200.kernels.microbench delta_rule --batch 1 --tokens 2048 --heads 16 --dim 128 --vdim 128 --channel
     python -m nanoinfer_b200.kernels.microbench attention_prefill --tokens 2048 --q-heads 16 --head-dim 128 --score-cap 30
     python -m nanoinfer_b200.kernels.microbench conv_attention --batch 1 --tokens 2048 --heads 16 --kv-heads 8 --dim 128
     python -m nanoinfer_b200.kernels.microbench routed --tokens 2048 --width 2048 --ff 2048 --experts 16 --identity 2 --top 4
@@ -385,6 +386,8 @@ def delta_rule(args) -> None:
     unit norms, gates), the recurrence, the gated norm.  States of several request sets are used in turn, so that
     single-token steps read theirs from HBM."""
     b, t, G, H, D, V, taps = args.batch, args.tokens, args.kv_heads, args.heads, args.dim, args.vdim, args.taps
+    if args.channel:
+        return delta_rule_channel(args)
     n = b * t
     C, N = 2 * G * D + H * V, 2 * G * D + 2 * H * V + 2 * H
     size = H * D * V + (taps - 1) * C
@@ -413,6 +416,53 @@ def delta_rule(args) -> None:
           f"({n * (N + C + 2 * H) * 4 / us_prep / 1e3:.0f} GB/s), recurrence {us_rec:.2f} us "
           f"({state_bytes / us_rec / 1e3:.0f} GB/s of state, {flops / us_rec / 1e6:.2f} TFLOP/s FP32), "
           f"gated norm {us_norm:.2f} us ({n * H * V * (4 + 4 + 2) / us_norm / 1e3:.0f} GB/s)")
+
+
+def delta_rule_channel(args) -> None:
+    """The delta rule with decays per key channel: a step of single tokens (one launch; thin matrices of --rank), or prompt
+    portions (the preparation, the recurrence in chunks and, beside it, token by token, the gated norm)."""
+    b, t, G, H, D, V, taps, rank = args.batch, args.tokens, args.kv_heads, args.heads, args.dim, args.vdim, args.taps, args.rank
+    n, C = b * t, 2 * G * D + H * V
+    b_col, thin = C, C + -(-H // 8) * 8
+    size = H * D * V + (taps - 1) * C
+    copies = max(2, min(32, -(-2 * L2_BYTES // (b * size * 4)))) if t == 1 else 2
+    g = torch.Generator(device=DEV).manual_seed(0)
+    states = [torch.randn(b, size, device=DEV, generator=g) * 0.1 for _ in range(copies)]
+    conv_w = torch.randn(C, taps, device=DEV, generator=g) * 0.5
+    a_log, dt_bias, norm_w = torch.zeros(H, device=DEV), torch.full((H * D,), -3.0, device=DEV), torch.ones(V, device=DEV)
+    cu = torch.arange(0, n + 1, t, dtype=torch.int32, device=DEV)
+    seq = torch.repeat_interleave(torch.arange(b, device=DEV), t).int()
+    slots = torch.arange(b, dtype=torch.int32, device=DEV)
+    y = torch.empty(n, H * V, dtype=torch.bfloat16, device=DEV)
+    what = f"delta_rule, decays per channel, batch={b} tokens={t} heads={H}/{G} dim={D} vdim={V} taps={taps}"
+    state_bytes = 2 * b * H * D * V * 4                      # S read and written once per step
+    if t == 1:
+        proj = torch.randn(n, thin + 2 * rank, device=DEV, generator=g)
+        w_decay, w_gate = ((torch.randn(H * m, rank, device=DEV, generator=g) * 0.1).to(torch.bfloat16) for m in (D, V))
+        tickets = torch.zeros(b * G, dtype=torch.int32, device=DEV)
+        us = _time([lambda st=st: ops.delta_token_step(proj, 0, b_col, thin, w_decay, w_gate, conv_w, a_log, dt_bias, norm_w, 1e-6, 1.0,
+                                                       st, cu, slots, tickets, b, G, H, D, V, taps, y) for st in states], args.iters)
+        total = state_bytes + 2 * H * (D + V) * rank + n * proj.shape[1] * 4
+        print(f"{what}: token step {us:.2f} us ({state_bytes / us / 1e3:.0f} GB/s of state, {total / us / 1e3:.0f} GB/s of all)")
+        return
+    proj = torch.randn(n, thin + 2 * rank, device=DEV, generator=g).to(torch.bfloat16)
+    z0 = torch.randn(n, H * (D + V), device=DEV, generator=g)
+    z = z0.clone()
+    qkv, gates, o = torch.empty(n, C, device=DEV), torch.empty(n, H, 2, device=DEV), torch.empty(n, H * V, device=DEV)
+    us_prep = _time([lambda st=st: ops.delta_prepare(proj, conv_w, a_log, dt_bias, st, seq, cu, slots, b, G, H, D, V, taps, qkv, gates,
+                                                     b_col=b_col, z=z) for st in states], args.iters)
+    z.copy_(z0)
+    ops.delta_prepare(proj, conv_w, a_log, dt_bias, states[0], seq, cu, slots, b, G, H, D, V, taps, qkv, gates, b_col=b_col, z=z)
+    buf = torch.empty(ops.delta_chunk_buffer_bytes(n, b, H, D, V) // 4, device=DEV)
+    us_chunk = _time([lambda st=st: ops.delta_chunk_recurrence(qkv, gates, z, st, cu, slots, b, t, G, H, D, V, buf, o) for st in states],
+                     args.iters)
+    us_rec = _time([lambda st=st: ops.delta_recurrence(qkv, gates, st, cu, slots, b, G, H, D, V, o, z=z) for st in states], args.iters)
+    us_norm = _time([lambda: ops.delta_gated_norm(o, proj, norm_w, 1e-6, G, H, D, V, y, states[0], cu, slots, b, taps, gate=z,
+                                                  gate_col=H * D, sigmoid=True)], args.iters)
+    flops = 8.0 * n * H * D * V
+    print(f"{what}: prepare {us_prep:.2f} us ({n * (C * 6 + H * D * 8) / us_prep / 1e3:.0f} GB/s), in chunks {us_chunk:.2f} us "
+          f"({flops / us_chunk / 1e6:.2f} TFLOP/s of the recurrence), token by token {us_rec:.2f} us ({flops / us_rec / 1e6:.2f}), "
+          f"gated norm {us_norm:.2f} us ({n * H * V * 10 / us_norm / 1e3:.0f} GB/s)")
 
 
 def conv_attention(args) -> None:
@@ -734,6 +784,8 @@ def main() -> None:
     p.add_argument("--dim", type=int, default=128)
     p.add_argument("--vdim", type=int, default=128)
     p.add_argument("--taps", type=int, default=4)
+    p.add_argument("--channel", action="store_true", help="decays per key channel and a gate from thin matrices")
+    p.add_argument("--rank", type=int, default=128, help="--channel: inner size of the thin matrices")
     p.set_defaults(fn=delta_rule)
     for name, fn in (("attention_decode", attention_decode), ("attention_prefill", attention_prefill)):
         p = sub.add_parser(name)

@@ -93,8 +93,14 @@ _SIGNATURES = {
     },
     "delta_rule": {
         "ni_delta_prepare": [_P, _I, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P, _P],
+        "ni_delta_token_step": [_P, _I, _I, _I, _P, _I, _P, _I, _P, _P, _P, _P, _F, _F, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P],
+        "ni_delta_token_max_dim": [],
         "ni_delta_recurrence": [_P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
         "ni_delta_gated_norm": [_P, _P, _I, _I, _P, _F, _F, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _LL, _P, _P, _P],
+    },
+    "delta_chunk": {
+        "ni_delta_chunk_recurrence": [_P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _P],
+        "ni_delta_chunk_max_dim": [],
     },
     "latent": {
         "ni_latent_norm_write": [_P, _I, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _P],
@@ -194,6 +200,10 @@ def load(module: str) -> ctypes.CDLL:
             lib.ni_attention_decode_set_cluster_merge(0)
         if module == "attention_decode" and lib.ni_attention_decode_fresh_keys() != DECODE_FRESH_KEYS:
             raise KernelError("attention_decode: DEC_FRESH_KEYS of the built kernel differs from ops.DECODE_FRESH_KEYS")
+        if module == "delta_chunk" and lib.ni_delta_chunk_max_dim() != DELTA_CHUNK_MAX_DIM:
+            raise KernelError("delta_chunk: the built kernel's largest key size differs from ops.DELTA_CHUNK_MAX_DIM")
+        if module == "delta_rule" and lib.ni_delta_token_max_dim() != DELTA_TOKEN_MAX_DIM:
+            raise KernelError("delta_rule: the built kernel's largest sizes differ from ops.DELTA_TOKEN_MAX_DIM")
         if module == "hyper" and lib.ni_hyper_max_streams() != HYPER_MAX_STREAMS:
             raise KernelError("hyper: HY_MAX_STREAMS of the built kernel differs from ops.HYPER_MAX_STREAMS")
         _libs[module] = lib
@@ -593,6 +603,59 @@ def delta_gated_norm(o, proj, weight, eps, n_q_heads_kv, n_heads, dim, vdim, y, 
         _dev(y, "y") + y_col * y.element_size(), _code(y, "y"), y.shape[1], _dev(proj, "proj") + col0 * proj.element_size(),
         _code(proj, "proj"), proj.shape[1], _dev(state, "state", f32), state.shape[1], _dev(cu_q, "cu_q", torch.int32),
         _dev(slots, "slots", torch.int32), _stream()), "delta_gated_norm")
+
+
+DELTA_CHUNK_MAX_DIM = 128      # the largest key size that the chunked delta rule takes
+
+
+def delta_chunk_buffer_bytes(n_tokens: int, n_seqs: int, n_heads: int, dim: int, vdim: int) -> int:
+    """Bytes of the buffer that delta_chunk_recurrence needs for a step."""
+    f = load("delta_chunk").ni_delta_chunk_buffer_bytes
+    f.restype, f.argtypes = ctypes.c_longlong, [_I] * 5
+    return int(f(n_tokens, n_seqs, n_heads, dim, vdim))
+
+
+def delta_chunk_recurrence(qkv, gates, z, state, cu_q, slots, n_seqs, max_q_len, n_q_heads_kv, n_heads, dim, vdim, buf, out) -> None:
+    """As delta_recurrence with decays per key channel (``z`` as delta_prepare leaves it), for prompt portions: chunks of 32
+    tokens, their products on the tensor cores with every FP32 operand split into two bfloat16 halves.  ``max_q_len``: the
+    most tokens that one request brings; ``buf``: delta_chunk_buffer_bytes bytes on the device."""
+    f32 = torch.float32
+    n = qkv.shape[0]
+    if out.shape != (n, n_heads * vdim) or z.shape[0] != n or z.shape[1] < n_heads * dim or gates.shape != (n, n_heads, 2) or \
+            qkv.shape[1] != 2 * n_q_heads_kv * dim + n_heads * vdim:
+        raise KernelError("delta_chunk_recurrence: shapes do not agree")
+    _check(load("delta_chunk").ni_delta_chunk_recurrence(
+        _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _dev(z, "z", f32), z.shape[1], _dev(state, "state", f32), state.shape[1],
+        _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), n, n_seqs, int(max_q_len), n_q_heads_kv, n_heads, dim,
+        vdim, _dev(buf, "buf"), buf.numel() * buf.element_size(), _dev(out, "out", f32), _stream()), "delta_chunk_recurrence")
+
+
+DELTA_TOKEN_MAX_DIM = 128      # the largest key and value sizes whose state a block of the token kernel holds in registers
+
+
+def delta_token_step(proj, col0, b_col, thin_col, w_decay, w_gate, conv_w, a_log, dt_bias, norm_w, eps, scale, state, cu_q, slots,
+                     tickets, n_seqs, n_q_heads_kv, n_heads, dim, vdim, taps, y, y_col: int = 0) -> None:
+    """A step of single tokens of the delta rule with decays per key channel in one launch: from ``proj`` (float32 [T, *], from
+    column ``col0`` on q | k | v, beta's logits at ``b_col``, the thin first products of decay and gate at ``thin_col``) to
+    the gated, normed read-outs in columns ``y_col`` on of ``y`` (bfloat16); the thin second products with ``w_decay``
+    (bfloat16 [H D, ra]) and ``w_gate`` ([H V, rg]; ra and rg multiples of 8) inside.  The state moves on, convolution
+    history included.  tickets: int32 zeros, at least n_seqs * q/k heads (left zero)."""
+    n = proj.shape[0]
+    f32, bf, i32 = torch.float32, torch.bfloat16, torch.int32
+    c, hd, hv = 2 * n_q_heads_kv * dim + n_heads * vdim, n_heads * dim, n_heads * vdim
+    ra, rg = w_decay.shape[1], w_gate.shape[1]
+    if n != n_seqs or y.shape[0] != n or y.shape[1] < y_col + hv or w_decay.shape[0] != hd or w_gate.shape[0] != hv or \
+            conv_w.shape != (c, taps) or a_log.numel() != n_heads or dt_bias.numel() != hd or norm_w.numel() != vdim or \
+            proj.shape[1] < max(col0 + c, b_col + n_heads, thin_col + ra + rg) or min(b_col, thin_col) < col0:
+        raise KernelError("delta_token_step: shapes do not agree")
+    if state.shape[1] != hd * vdim + (taps - 1) * c or tickets.numel() < n_seqs * n_q_heads_kv:
+        raise KernelError("delta_token_step: the state has another size, or too few tickets")
+    _check(load("delta_rule").ni_delta_token_step(
+        _dev(proj, "proj", f32) + 4 * col0, proj.shape[1], b_col - col0, thin_col - col0, _dev(w_decay, "w_decay", bf), ra,
+        _dev(w_gate, "w_gate", bf), rg, _dev(conv_w, "conv_w", f32), _dev(a_log, "a_log", f32), _dev(dt_bias, "dt_bias", f32),
+        _dev(norm_w, "norm_w", f32), float(eps), float(scale), _dev(state, "state", f32), state.shape[1], _dev(cu_q, "cu_q", i32),
+        _dev(slots, "slots", i32), _dev(tickets, "tickets", i32), n_seqs, n_q_heads_kv, n_heads, dim, vdim, taps,
+        _dev(y, "y", bf) + 2 * y_col, y.shape[1], _stream()), "delta_token_step")
 
 
 def latent_norm_write(proj, col0, rank, weight, eps, pages, positions, seq_of_token, block_table, page_size) -> None:

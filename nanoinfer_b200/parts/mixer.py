@@ -951,7 +951,7 @@ class ParallelMixers(Part):
         return self.joined and self.rt.skinny(n_rows, self.hidden_size) and self.rt.fuses_norm(norm)
 
     def _token_dtype(self, ctx):
-        """What the joined projection of a few rows leaves in: FP32 where a side asks for it in steps of single tokens."""
+        """What the joined projection leaves in: FP32 where a side asks for it in steps of single tokens."""
         f32 = ctx.max_q_len == 1 and any(p.wants_f32_tokens for p in self.sub_parts)
         return (torch.float32, ops.STORE_F32) if f32 else (self.rt.dtype, ops.STORE_BF16)
 
@@ -984,8 +984,7 @@ class ParallelMixers(Part):
     # ---- folded and plain ---------------------------------------------------------------------------------
     def forward(self, x: torch.Tensor, ctx, cache, residual=None):
         if self.joined:
-            dtype, _ = self._token_dtype(ctx) if self.rt.skinny(x.shape[0], self.hidden_size) else (None, None)
-            return self._between(self.rt.linear(x, self.w_in, out_dtype=dtype), ctx, cache, residual)
+            return self._between(self.rt.linear(x, self.w_in, out_dtype=self._token_dtype(ctx)[0]), ctx, cache, residual)
         first, second = self.sub_parts
         left = first.forward(x, ctx, cache)
         if left.dtype != torch.float32:

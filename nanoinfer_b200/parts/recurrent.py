@@ -31,13 +31,17 @@ class GatedDeltaRule(Part):
 
     All projections of x are ONE product (rows q | k | v | gate | b | a, or q | k | v | b | a1 | g1); with thin matrices a
     second, block-diagonal product turns (W_a1 x, W_g1 x) into the logits of decay and gate in FP32.  Everything from there
-    to the gated norm is FP32 on the device.  A request's state is one FP32 vector: M of every head, then the last
+    to the gated norm is FP32 on the device; in bfloat16 a step of single tokens with both options is one launch (from an
+    FP32 projection, thin products included), and portions of CHUNK_FROM tokens and more run in chunks on the tensor cores
+    (csrc/delta_chunk.cu).  A request's state is one FP32 vector: M of every head, then the last
     conv_taps - 1 inputs of every convolved channel.  A step's kernels run exactly once, so the state advances by exactly
     the step's tokens.
 
     ``joined`` in the extra: one side of mixers that share their input and output projections (ParallelMixers)."""
 
     kernel_modules = ("delta_rule",)       # libraries of csrc that this part's kernels live in
+
+    CHUNK_FROM = 16             # a step whose longest portion has this many tokens takes the chunked recurrence
 
     JOINS = True                # can be a side of mixers with joined projections
     takes_output_scale = True   # a factor on the output rides in the gated norm, before the output projection
@@ -130,6 +134,7 @@ class GatedDeltaRule(Part):
                 second.append(padded)
                 self.ranks[one] = padded.shape[1]
                 self.thin_k += padded.shape[1]
+            self.w_second = [rt.weight(x) for x in second]
             self.w_thin = rt.weight(torch.block_diag(*[x.float() for x in second]).to(like.dtype))        # [H D (+ H V), ranks]
             at = self.thin_col + self.thin_k
         if joined and at % 8:
@@ -142,7 +147,12 @@ class GatedDeltaRule(Part):
         self.conv_w = rt.gain(torch.cat([weights[s] for s in ("q.conv", "k.conv", "v.conv")], dim=0))
         self.a_log, self.dt_bias = rt.gain(weights["A_log"]), rt.gain(weights["dt_bias"])
         self.norm_w = rt.gain(weights["norm"])
-        self.wants_f32_tokens = False
+        # single tokens go through one kernel, which reads an FP32 projection
+        self.wants_f32_tokens = (rt.dtype == torch.bfloat16 and self.channel and self.thin_gate
+                                 and max(d, v) <= ops.DELTA_TOKEN_MAX_DIM and self.thin_k <= 8192)
+        self.chunked = rt.dtype == torch.bfloat16 and self.channel and d <= ops.DELTA_CHUNK_MAX_DIM
+        if self.chunked:
+            self.kernel_modules = ("delta_chunk",)
 
     def cache_need(self):
         return StateNeed((self.H * self.D * self.V + (self.taps - 1) * self.channels,), "float32")
@@ -185,6 +195,12 @@ class GatedDeltaRule(Part):
         n = proj.shape[0]
         f32 = torch.float32
         g, h, d, v = self.G, self.H, self.D, self.V
+        if self.wants_f32_tokens and ctx.max_q_len == 1 and proj.dtype == f32:
+            tickets = rt.workspace("delta_token_tickets", ctx.n_seqs * g, torch.int32, zero=True)
+            ops.delta_token_step(proj, col0, col0 + self.b_col, col0 + self.thin_col, *self.w_second, self.conv_w, self.a_log,
+                                 self.dt_bias, self.norm_w, self.eps, self.output_scale, cache.state, ctx.cu_q, ctx.slots,
+                                 tickets, ctx.n_seqs, g, h, d, v, self.taps, out, y_col=out_col)
+            return out
         z = self._thin_logits(proj, col0) if self.w_thin is not None else None
         decay = z if self.channel else None
         qkv = rt.empty(n, self.channels, dtype=f32)
@@ -192,7 +208,13 @@ class GatedDeltaRule(Part):
         ops.delta_prepare(proj, self.conv_w, self.a_log, self.dt_bias, cache.state, ctx.seq_of_token, ctx.cu_q,
                           ctx.slots, ctx.n_seqs, g, h, d, v, self.taps, qkv, gates, col0=col0, b_col=col0 + self.b_col, z=decay)
         o = rt.empty(n, h * v, dtype=f32)
-        ops.delta_recurrence(qkv, gates, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, g, h, d, v, o, z=decay)
+        if self.chunked and ctx.max_q_len >= self.CHUNK_FROM:
+            need = ops.delta_chunk_buffer_bytes(n, ctx.n_seqs, h, d, v)
+            buf = rt.workspace("delta_chunks", -(-need // 4), f32)                 # one buffer for all layers
+            ops.delta_chunk_recurrence(qkv, gates, decay, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, ctx.max_q_len, g, h, d, v,
+                                       buf, o)
+        else:
+            ops.delta_recurrence(qkv, gates, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, g, h, d, v, o, z=decay)
         gate, gate_col = (z, h * d if self.channel else 0) if self.thin_gate else (proj, col0 + self.gate_col)
         if gate.dtype != f32:
             gate, gate_col = gate[:, gate_col:gate_col + h * v].to(f32).contiguous(), 0
