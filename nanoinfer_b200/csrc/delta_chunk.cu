@@ -12,19 +12,20 @@
 // channel decays.  The sum over s < i is resolved once per chunk: u = U0 - W S with U0 and W the forward substitutions of
 // beta v and beta P k.
 //
-// Two launches:
-//   delta_chunk_prepare   per (chunk, head), all at once: A, B (a group of 8 lanes per s walks i upwards with k_s times the
-//                         decays in registers - what is left at the end is the last line's factor), then a thread per column
-//                         of [W | U0] does the substitution
+// Two launches, from the projection (bfloat16) on; the projection's q, k and v never exist in FP32 in memory:
+//   delta_chunk_prepare   per (chunk, head), all at once: convolution and silu of the head's channels (a thread per channel
+//                         walks the tokens), unit norms, decays, beta - all into shared memory -; A, B (a group of 8 lanes
+//                         per s walks i upwards with k_s times the decays in registers - what is left at the end is the
+//                         last line's factor); then a thread per column of [W | U0] does the substitution
 //   delta_chunk_scan      per (request, head, 16 value columns): the chunks one after the other; S stands in the
-//                         accumulators of its four warps, and as two bfloat16 planes in shared memory for the products that
+//                         accumulators of its warps, and as two bfloat16 planes in shared memory for the products that
 //                         read it; the next chunk's operands are copied while this one's are used
+// The convolution's history is read here and moved on by the gated norm's launch (delta_rule.cu), which follows.
 // A chunk begins at a portion's first token, so where a prompt is cut changes results by roundings only.
 #include "linear_attention.cuh"
 
 #define DC_C 32          // tokens per chunk
-#define DC_THREADS 256   // of the preparation
-#define DC_SCAN_THREADS 128
+#define DC_THREADS 256
 #define DC_VS 16         // value columns per block of the scan
 #define DC_AS 36         // row stride of A in shared memory
 #define DC_BS (DC_C + 8) // row stride of the planes of B
@@ -58,14 +59,61 @@ __device__ __forceinline__ void dc_store_split(__nv_bfloat16* hi, __nv_bfloat16*
     *lo = __float2bfloat16_rn(v - __bfloat162float(h));
 }
 
-// qkv FP32 [T, C] (q | k | v of every head, q and k unit vectors per head, q scaled), gates [T, H, 2] (beta second), decay
-// [T, ld_z] (H D).  grid (chunks of the longest portion, H, requests).  DP: the padded key size; a lane owns DP / 32 groups
+// What the preparation reads: proj bfloat16 [T, ld] with q (G D) | k (G D) | v (H V) from column 0, beta's logits at b_off;
+// z FP32 [T, ld_z], the decays' logits in its first H D columns; a request's convolution history behind its S in state.
+struct DcInput {
+    const __nv_bfloat16* proj;
+    const float *conv_w, *a_log, *dt_bias, *z, *state;
+    long long state_stride;
+    const int *cu_q, *slots;
+    int ld, b_off, ld_z, G, H, D, V, taps;
+};
+
+__device__ __forceinline__ float dc_silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+
+// Channel c (of the projection) of the chunk's tokens `first` .. `first + n - 1` through the convolution and silu, rows n ..
+// DC_C - 1 zero: dst[r * stride].  TAPS: 4, or 0 for any number.
+template <int TAPS>
+__device__ __forceinline__ void dc_conv_column(const DcInput& in, const float* __restrict__ hist, int seq_first, int first, int n,
+                                               int c, float* dst, int stride) {
+    const int taps = TAPS ? TAPS : in.taps, C = 2 * in.G * in.D + in.H * in.V;
+    const __nv_bfloat16* x = in.proj + (size_t)first * in.ld + c;
+    const int before = first - seq_first;           // tokens of this portion before the chunk
+    // the input `back` tokens before the chunk's first: from the portion, or from the history
+    const auto earlier = [&](int back) {
+        return back <= before ? __bfloat162float(x[-(long long)back * in.ld]) : hist[(size_t)(taps - 1 - (back - before)) * C + c];
+    };
+    if (TAPS == 4) {
+        const float4 w = *reinterpret_cast<const float4*>(in.conv_w + (size_t)c * 4);
+        float x3 = earlier(3), x2 = earlier(2), x1 = earlier(1);
+        float v[DC_C];
+#pragma unroll
+        for (int r = 0; r < DC_C; ++r) v[r] = r < n ? __bfloat162float(x[(size_t)r * in.ld]) : 0.f;
+#pragma unroll
+        for (int r = 0; r < DC_C; ++r) {
+            const float y = fmaf(w.w, v[r], fmaf(w.z, x1, fmaf(w.y, x2, w.x * x3)));
+            x3 = x2; x2 = x1; x1 = v[r];
+            dst[r * stride] = r < n ? dc_silu(y) : 0.f;
+        }
+    } else {
+        for (int r = 0; r < DC_C; ++r) {
+            float y = 0.f;
+            if (r < n)
+                for (int j = 0; j < taps; ++j) {
+                    const int back = taps - 1 - j;
+                    const float v = back <= r ? __bfloat162float(x[(size_t)(r - back) * in.ld]) : earlier(back - r);
+                    y = fmaf(in.conv_w[(size_t)c * taps + j], v, y);
+                }
+            dst[r * stride] = r < n ? dc_silu(y) : 0.f;
+        }
+    }
+}
+
+// grid (chunks of the longest portion, H, requests).  DP: the padded key size; a lane of the pairs' phase owns DP / 32 groups
 // of four channels.
-template <int DP>
-__global__ void __launch_bounds__(DC_THREADS)
-delta_chunk_prepare_kernel(const float* __restrict__ qkv, const float* __restrict__ gates, const float* __restrict__ decay,
-                           int ld_z, const int* __restrict__ cu_q, int G, int H, int D, int V, unsigned char* __restrict__ buf,
-                           DcLayout lay) {
+template <int DP, int TAPS>
+__global__ void __launch_bounds__(DC_THREADS, 2)
+delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, DcLayout lay) {
     constexpr int M = DP / 32;
     extern __shared__ __align__(16) float dc_smem[];
     float* sq = dc_smem;                       // [DC_C][DP]
@@ -73,29 +121,59 @@ delta_chunk_prepare_kernel(const float* __restrict__ qkv, const float* __restric
     float* sg = sk + DC_C * DP;
     float* sA = sg + DC_C * DP;                // [DC_C][DC_AS], times beta of the row
     float* sB = sA + DC_C * DC_AS;             // [DC_C][DC_AS]
+    float* sv = sB + DC_C * DC_AS;             // [DC_C][VP]
     __shared__ float beta[DC_C];
     __shared__ int base_scratch;
     const int seq = blockIdx.z, h = blockIdx.y;
-    const int first = cu_q[seq] + blockIdx.x * DC_C, last = cu_q[seq + 1];
+    const int seq_first = in.cu_q[seq], first = seq_first + blockIdx.x * DC_C, last = in.cu_q[seq + 1];
     if (first >= last) return;
     const int n = min(DC_C, last - first);
-    const int g = h / (H / G), C = 2 * G * D + H * V;
-    unsigned char* rec = buf + ((size_t)(dc_chunk_base(cu_q, seq, &base_scratch) + blockIdx.x) * H + h) * lay.bytes();
-    const int tid = threadIdx.x;
-    for (int i = tid; i < DC_C * DP; i += DC_THREADS) {
-        const int r = i / DP, d = i - r * DP;
-        const bool ok = r < n && d < D;
-        const float* row = qkv + (size_t)(first + r) * C;
-        sq[i] = ok ? row[g * D + d] : 0.f;
-        sk[i] = ok ? row[G * D + g * D + d] : 0.f;
-        sg[i] = ok ? decay[(size_t)(first + r) * ld_z + h * D + d] : 1.f;
+    const int H = in.H, G = in.G, D = in.D, V = in.V, VP = lay.VP, g = h / (H / G);
+    unsigned char* rec = buf + ((size_t)(dc_chunk_base(in.cu_q, seq, &base_scratch) + blockIdx.x) * H + h) * lay.bytes();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const float* hist = in.state + (size_t)in.slots[seq] * in.state_stride + (size_t)H * D * V;
+    // ---- q, k, v of the chunk; decays; beta ----
+    for (int i = tid; i < 2 * DP + VP; i += DC_THREADS) {
+        const int part = i < DP ? 0 : (i < 2 * DP ? 1 : 2), e = i - part * DP;
+        float* dst = part == 0 ? sq + e : (part == 1 ? sk + e : sv + e);
+        const int stride = part == 2 ? VP : DP;
+        if (e < (part == 2 ? V : D)) {
+            dc_conv_column<TAPS>(in, hist, seq_first, first, n, part == 2 ? 2 * G * D + h * V + e : part * G * D + g * D + e, dst, stride);
+        } else {
+            for (int r = 0; r < DC_C; ++r) dst[r * stride] = 0.f;
+        }
     }
-    for (int i = tid; i < DC_C * DC_AS; i += DC_THREADS) sA[i] = sB[i] = 0.f;
-    if (tid < DC_C) beta[tid] = tid < n ? gates[((size_t)(first + tid) * H + h) * 2 + 1] : 0.f;
+    {
+        const float ea = -expf(in.a_log[h]);
+#pragma unroll 4
+        for (int i = tid; i < DC_C * DP; i += DC_THREADS) {
+            const int r = i / DP, d = i - r * DP;
+            float gd = 1.f;
+            if (r < n && d < D) {
+                const float x = in.z[(size_t)(first + r) * in.ld_z + h * D + d] + in.dt_bias[h * D + d];
+                gd = expf(ea * (x > 20.0f ? x : log1pf(expf(x))));
+            }
+            sg[i] = gd;
+        }
+    }
+    for (int i = tid; i < 2 * DC_C * DC_AS; i += DC_THREADS) sA[i] = 0.f;       // A and B
+    if (tid < DC_C)
+        beta[tid] = tid < n ? 1.0f / (1.0f + expf(-__bfloat162float(in.proj[(size_t)(first + tid) * in.ld + in.b_off + h]))) : 0.f;
+    __syncthreads();
+    // ---- unit norms: a warp per row ----
+    for (int r = warp; r < 2 * DC_C; r += DC_THREADS / 32) {
+        float4* row = reinterpret_cast<float4*>((r < DC_C ? sq : sk) + (r & (DC_C - 1)) * DP);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (lane < DP / 4) v = row[lane];
+        const float ss = ni_warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
+        const float f = 1.0f / sqrtf(ss + 1e-6f) * (r < DC_C ? 1.0f / sqrtf((float)D) : 1.0f);
+        if (lane < DP / 4) row[lane] = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+    }
     __syncthreads();
     {
-        // warp w: the tokens s = w, 15 - w, 16 + w, 31 - w (early and late ones together); 8 lanes each
-        const int warp = tid >> 5, lane = tid & 31, q4 = lane >> 3, l = lane & 7;
+        // warp w: the tokens s = w, 15 - w, 16 + w, 31 - w (early and late ones together); 8 lanes each.  Four i at a time;
+        // their eight sums over the 8 lanes end up one per lane (seven shuffles).
+        const int q4 = lane >> 3, l = lane & 7;
         const int s = q4 == 0 ? warp : (q4 == 1 ? 15 - warp : (q4 == 2 ? 16 + warp : 31 - warp));
         float kp[4 * M];
 #pragma unroll
@@ -103,33 +181,41 @@ delta_chunk_prepare_kernel(const float* __restrict__ qkv, const float* __restric
             const float4 v = *reinterpret_cast<const float4*>(sk + s * DP + 4 * (l + 8 * m));
             kp[4 * m] = v.x; kp[4 * m + 1] = v.y; kp[4 * m + 2] = v.z; kp[4 * m + 3] = v.w;
         }
-        for (int i = warp; i < DC_C; ++i) {            // (every s of the warp is at least `warp`)
-            float a = 0.f, b = 0.f;
-            if (i >= s) {
+        for (int i0 = warp & ~3; i0 < DC_C; i0 += 4) {
+            float t[8];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int i = i0 + u;
+                const bool decays = i > s;
+                float a = 0.f, b = 0.f;
 #pragma unroll
                 for (int m = 0; m < M; ++m) {
                     const int c = 4 * (l + 8 * m);
-                    if (i > s) {
-                        const float4 gg = *reinterpret_cast<const float4*>(sg + i * DP + c);
-                        kp[4 * m] *= gg.x; kp[4 * m + 1] *= gg.y; kp[4 * m + 2] *= gg.z; kp[4 * m + 3] *= gg.w;
-                    }
+                    const float4 gg = *reinterpret_cast<const float4*>(sg + i * DP + c);
                     const float4 kk = *reinterpret_cast<const float4*>(sk + i * DP + c);
                     const float4 qq = *reinterpret_cast<const float4*>(sq + i * DP + c);
+                    kp[4 * m] *= decays ? gg.x : 1.f; kp[4 * m + 1] *= decays ? gg.y : 1.f;
+                    kp[4 * m + 2] *= decays ? gg.z : 1.f; kp[4 * m + 3] *= decays ? gg.w : 1.f;
                     a = fmaf(kk.x, kp[4 * m], a); a = fmaf(kk.y, kp[4 * m + 1], a);
                     a = fmaf(kk.z, kp[4 * m + 2], a); a = fmaf(kk.w, kp[4 * m + 3], a);
                     b = fmaf(qq.x, kp[4 * m], b); b = fmaf(qq.y, kp[4 * m + 1], b);
                     b = fmaf(qq.z, kp[4 * m + 2], b); b = fmaf(qq.w, kp[4 * m + 3], b);
                 }
+                t[u] = a;
+                t[4 + u] = b;
             }
 #pragma unroll
-            for (int off = 4; off > 0; off >>= 1) {
-                a += __shfl_xor_sync(0xffffffffu, a, off);
-                b += __shfl_xor_sync(0xffffffffu, b, off);
+            for (int half = 4; half > 0; half >>= 1) {
+                const bool upper = l & half;
+#pragma unroll
+                for (int e = 0; e < half; ++e) {
+                    const float mine = upper ? t[e + half] : t[e], send = upper ? t[e] : t[e + half];
+                    t[e] = mine + __shfl_xor_sync(0xffffffffu, send, half);
+                }
             }
-            if (l == 0 && i >= s) {
-                if (i > s) sA[i * DC_AS + s] = a * beta[i];
-                sB[i * DC_AS + s] = b;
-            }
+            const int i = i0 + (l & 3);              // lane l holds the sum of t[l]: A of i0 + l, or B of i0 + l - 4
+            if (l < 4 && i > s) sA[i * DC_AS + s] = t[0] * beta[i];
+            if (l >= 4 && i >= s) sB[i * DC_AS + s] = t[0];
         }
         __nv_bfloat16* k_hi = reinterpret_cast<__nv_bfloat16*>(rec + 4 * lay.plane()) + s * DP;
         __nv_bfloat16* k_lo = k_hi + DC_C * DP;
@@ -145,19 +231,22 @@ delta_chunk_prepare_kernel(const float* __restrict__ qkv, const float* __restric
     __syncthreads();
     {
         __nv_bfloat16* b_hi = reinterpret_cast<__nv_bfloat16*>(rec + lay.b_off());
-        for (int i = tid; i < DC_C * DC_C; i += DC_THREADS)
-            dc_store_split(b_hi + i, b_hi + DC_C * DC_C + i, sB[(i / DC_C) * DC_AS + i % DC_C]);
+        for (int i = tid; i < DC_C * DC_C / 2; i += DC_THREADS) {
+            const float2 v = *reinterpret_cast<const float2*>(sB + (i / (DC_C / 2)) * DC_AS + 2 * (i % (DC_C / 2)));
+            uint32_t hi, lo;
+            lt_split2(v.x, v.y, hi, lo);
+            *reinterpret_cast<uint32_t*>(b_hi + 2 * i) = hi;
+            *reinterpret_cast<uint32_t*>(b_hi + DC_C * DC_C + 2 * i) = lo;
+        }
     }
     __nv_bfloat16* w_hi = reinterpret_cast<__nv_bfloat16*>(rec);
     __nv_bfloat16* w_lo = w_hi + DC_C * DP;
     __nv_bfloat16* q_hi = w_lo + DC_C * DP;
     __nv_bfloat16* q_lo = q_hi + DC_C * DP;
     float* u0 = reinterpret_cast<float*>(rec + lay.u_off());
-    for (int col = tid; col < DP + lay.VP; col += DC_THREADS) {
+    for (int col = tid; col < DP + VP; col += DC_THREADS) {
         const bool is_k = col < DP;
         const int vc = col - DP;
-        const bool live = is_k || vc < V;
-        const float* vrow = qkv + (size_t)first * C + 2 * G * D + h * V + vc;
         float x[DC_C], P = 1.f;
 #pragma unroll
         for (int i = 0; i < DC_C; ++i) {
@@ -167,20 +256,20 @@ delta_chunk_prepare_kernel(const float* __restrict__ qkv, const float* __restric
                 rhs = sk[i * DP + col] * P;
                 dc_store_split(q_hi + i * DP + col, q_lo + i * DP + col, sq[i * DP + col] * P);
             } else {
-                rhs = live && i < n ? vrow[(size_t)i * C] : 0.f;
+                rhs = sv[i * VP + vc];
             }
-            float acc0 = beta[i] * rhs, acc1 = 0.f;
+            float acc[4] = {beta[i] * rhs, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int s = 0; s < i; s += 4) {
                 const float4 a = *reinterpret_cast<const float4*>(sA + i * DC_AS + s);      // zero from column i on
-                acc0 = fmaf(-a.x, x[s], acc0);
-                if (s + 1 < i) acc1 = fmaf(-a.y, x[s + 1], acc1);
-                if (s + 2 < i) acc0 = fmaf(-a.z, x[s + 2], acc0);
-                if (s + 3 < i) acc1 = fmaf(-a.w, x[s + 3], acc1);
+                acc[0] = fmaf(-a.x, x[s], acc[0]);
+                if (s + 1 < i) acc[1] = fmaf(-a.y, x[s + 1], acc[1]);
+                if (s + 2 < i) acc[2] = fmaf(-a.z, x[s + 2], acc[2]);
+                if (s + 3 < i) acc[3] = fmaf(-a.w, x[s + 3], acc[3]);
             }
-            x[i] = acc0 + acc1;
+            x[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
             if (is_k) dc_store_split(w_hi + i * DP + col, w_lo + i * DP + col, x[i]);
-            else u0[i * lay.VP + vc] = x[i];
+            else u0[i * VP + vc] = x[i];
         }
         if (is_k) reinterpret_cast<float*>(rec + lay.p_off())[col] = P;
     }
@@ -198,14 +287,14 @@ template <int DP> __host__ __device__ constexpr int dc_stage_bytes() {
 #define DC_SS (DC_VS + 8)          // row stride of the planes of S and of u
 template <int DP> __host__ __device__ constexpr int dc_scan_smem() { return 2 * dc_stage_bytes<DP>() + 2 * DP * DC_SS * 2 + 2 * DC_C * DC_SS * 2; }
 
-// grid (value slices, H, requests); 4 warps.
+// grid (value slices, H, requests); 8 warps: warp w multiplies row tile w % 4 of [W; Q] with column tile w / 4 of S, and owns
+// rows 16 w .. 16 w + 15 of S itself.
 template <int DP>
-__global__ void __launch_bounds__(DC_SCAN_THREADS)
+__global__ void __launch_bounds__(DC_THREADS)
 delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, float* __restrict__ state, long long state_stride,
                         const int* __restrict__ cu_q, const int* __restrict__ slots, int H, int D, int V,
                         float* __restrict__ out) {
     constexpr int RS = DP + 8;                       // row stride of the operand planes
-    constexpr int MT = DP / 16 < 4 ? 1 : DP / 64;    // row tiles of S per warp
     extern __shared__ __align__(16) unsigned char dc_raw[];
     __shared__ int base_scratch;
     const int seq = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * DC_VS;
@@ -225,54 +314,51 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
         const unsigned char* rec = rec0 + (size_t)c * rec_step;
         unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>();
         constexpr int PIECES = DP / 8;
-        for (int i = tid; i < 6 * DC_C * PIECES; i += DC_SCAN_THREADS) {
+        for (int i = tid; i < 6 * DC_C * PIECES; i += DC_THREADS) {
             const int r = i / PIECES, p = i - r * PIECES;                    // r: row of plane r / DC_C
             lt_cp_async16(st + ((size_t)r * RS + 8 * p) * 2, rec + ((size_t)r * DP + 8 * p) * 2);
         }
         unsigned char* sb = st + 6 * DC_C * RS * 2;
-        for (int i = tid; i < 2 * DC_C * (DC_C / 8); i += DC_SCAN_THREADS) {
+        for (int i = tid; i < 2 * DC_C * (DC_C / 8); i += DC_THREADS) {
             const int r = i / (DC_C / 8), p = i % (DC_C / 8);
             lt_cp_async16(sb + (r * DC_BS + 8 * p) * 2, rec + lay.b_off() + (r * DC_C + 8 * p) * 2);
         }
         unsigned char* su = sb + 2 * DC_C * DC_BS * 2;
-        for (int i = tid; i < DC_C * (DC_VS / 4); i += DC_SCAN_THREADS) {
+        for (int i = tid; i < DC_C * (DC_VS / 4); i += DC_THREADS) {
             const int r = i / (DC_VS / 4), p = i % (DC_VS / 4);
             lt_cp_async16(su + (r * DC_VS + 4 * p) * 4, rec + lay.u_off() + ((size_t)r * lay.VP + v0 + 4 * p) * 4);
         }
         unsigned char* sp = su + DC_C * DC_VS * 4;
-        for (int i = tid; i < DP / 4; i += DC_SCAN_THREADS) lt_cp_async16(sp + 16 * i, rec + lay.p_off() + 16 * i);
+        for (int i = tid; i < DP / 4; i += DC_THREADS) lt_cp_async16(sp + 16 * i, rec + lay.p_off() + 16 * i);
     };
     fetch(0);
     lt_cp_async_commit();
-    // this warp's rows of S: tiles warp, warp + 4; two column tiles of 8
-    float s[MT][2][4];
+    // this warp's 16 rows of S; two column tiles of 8
+    const bool owns = warp < DP / 16;
+    float s[2][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int row = 16 * warp + g + 8 * (e >> 1), col = v0 + 8 * j + 2 * t + (e & 1);
+            s[j][e] = (row < D && col < V) ? S[(size_t)row * V + col] : 0.f;
+        }
+    auto publish = [&]() {                           // S as two planes, for the products of the next chunk
+        if (!owns) return;
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int row = 16 * (warp + 4 * m) + g + 8 * (e >> 1), col = v0 + 8 * j + 2 * t + (e & 1);
-                s[m][j][e] = (row < D && col < V) ? S[(size_t)row * V + col] : 0.f;
+            for (int half = 0; half < 2; ++half) {
+                uint32_t hi, lo;
+                lt_split2(s[j][2 * half], s[j][2 * half + 1], hi, lo);
+                const int at = (16 * warp + g + 8 * half) * DC_SS + 8 * j + 2 * t;
+                *reinterpret_cast<uint32_t*>(s_hi + at) = hi;
+                *reinterpret_cast<uint32_t*>(s_lo + at) = lo;
             }
-    auto publish = [&]() {                           // S as two planes, for the products of the next chunk
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-            if (warp + 4 * m >= DP / 16) continue;
-#pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    uint32_t hi, lo;
-                    lt_split2(s[m][j][2 * half], s[m][j][2 * half + 1], hi, lo);
-                    const int at = (16 * (warp + 4 * m) + g + 8 * half) * DC_SS + 8 * j + 2 * t;
-                    *reinterpret_cast<uint32_t*>(s_hi + at) = hi;
-                    *reinterpret_cast<uint32_t*>(s_lo + at) = lo;
-                }
-        }
     };
     publish();
     const int mi = lane >> 3, lr = lane & 7;
+    const int rt = warp & 3, ct = warp >> 2;         // row tile of [W; Q] (0, 1: W), column tile
     for (int c = 0; c < n_chunks; ++c) {
         lt_cp_async_wait<0>();
         __syncthreads();                             // chunk c's operands and the planes of S are there; the other stage is free
@@ -283,43 +369,41 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
         const __nv_bfloat16* b_hi = planes + 6 * DC_C * RS;
         const float* su = reinterpret_cast<const float*>(b_hi + 2 * DC_C * DC_BS);
         const float* sp = su + DC_C * DC_VS;
-        // ---- [W; Q] S: warps 0 and 1 the 32 rows of W, 2 and 3 those of Q ----
-        float acc[2][2][4];                          // [high x high | the two mixed terms][column tile]
+        // ---- [W; Q] S ----
+        float acc[3][4];                             // high x high, low x high, high x low
 #pragma unroll
-        for (int k = 0; k < 2; ++k)
-#pragma unroll
-            for (int j = 0; j < 2; ++j) acc[k][j][0] = acc[k][j][1] = acc[k][j][2] = acc[k][j][3] = 0.f;
-        const __nv_bfloat16* a_hi = planes + (warp >> 1) * 2 * DC_C * RS + 16 * (warp & 1) * RS;
+        for (int k = 0; k < 3; ++k) acc[k][0] = acc[k][1] = acc[k][2] = acc[k][3] = 0.f;
+        const __nv_bfloat16* a_hi = planes + (rt >> 1) * 2 * DC_C * RS + 16 * (rt & 1) * RS;
         const __nv_bfloat16* a_lo = a_hi + DC_C * RS;
 #pragma unroll
-        for (int kk = 0; kk < DP / 16; ++kk) {
-            uint32_t ah[4], al[4], bh[4], bl[4];
-            const int a_at = (lr + 8 * (mi & 1)) * RS + 16 * kk + 8 * (mi >> 1);
-            const int b_at = (16 * kk + lr + 8 * (mi & 1)) * DC_SS + 8 * (mi >> 1);
-            dc_ldsm_x4(ah, a_hi + a_at);
-            dc_ldsm_x4(al, a_lo + a_at);
+        for (int k2 = 0; k2 < DP / 32; ++k2) {       // 32 rows of S at a time: one transposing load per plane
+            uint32_t bh[4], bl[4];
+            const int b_at = (32 * k2 + lr + 8 * mi) * DC_SS + 8 * ct;
             lt_ldsm_x4_trans(bh, s_hi + b_at);
             lt_ldsm_x4_trans(bl, s_lo + b_at);
-            lt_mma(acc[0][0], ah, bh[0], bh[1]);
-            lt_mma(acc[0][1], ah, bh[2], bh[3]);
-            lt_mma(acc[1][0], al, bh[0], bh[1]);
-            lt_mma(acc[1][1], al, bh[2], bh[3]);
-            lt_mma(acc[1][0], ah, bl[0], bl[1]);
-            lt_mma(acc[1][1], ah, bl[2], bl[3]);
+#pragma unroll
+            for (int kk = 0; kk < 2; ++kk) {
+                uint32_t ah[4], al[4];
+                const int a_at = (lr + 8 * (mi & 1)) * RS + 32 * k2 + 16 * kk + 8 * (mi >> 1);
+                dc_ldsm_x4(ah, a_hi + a_at);
+                dc_ldsm_x4(al, a_lo + a_at);
+                lt_mma(acc[0], ah, bh[2 * kk], bh[2 * kk + 1]);
+                lt_mma(acc[1], al, bh[2 * kk], bh[2 * kk + 1]);
+                lt_mma(acc[2], ah, bl[2 * kk], bl[2 * kk + 1]);
+            }
         }
-        if (warp < 2) {                              // u = U0 - W S
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
+        for (int e = 0; e < 4; ++e) acc[0][e] += acc[1][e] + acc[2][e];
+        if (rt < 2) {                                // u = U0 - W S
 #pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    const int r = 16 * warp + g + 8 * half, cl = 8 * j + 2 * t;
-                    const float2 u0 = *reinterpret_cast<const float2*>(su + r * DC_VS + cl);
-                    uint32_t hi, lo;
-                    lt_split2(u0.x - (acc[0][j][2 * half] + acc[1][j][2 * half]),
-                              u0.y - (acc[0][j][2 * half + 1] + acc[1][j][2 * half + 1]), hi, lo);
-                    *reinterpret_cast<uint32_t*>(u_hi + r * DC_SS + cl) = hi;
-                    *reinterpret_cast<uint32_t*>(u_lo + r * DC_SS + cl) = lo;
-                }
+            for (int half = 0; half < 2; ++half) {
+                const int r = 16 * rt + g + 8 * half, cl = 8 * ct + 2 * t;
+                const float2 u0 = *reinterpret_cast<const float2*>(su + r * DC_VS + cl);
+                uint32_t hi, lo;
+                lt_split2(u0.x - acc[0][2 * half], u0.y - acc[0][2 * half + 1], hi, lo);
+                *reinterpret_cast<uint32_t*>(u_hi + r * DC_SS + cl) = hi;
+                *reinterpret_cast<uint32_t*>(u_lo + r * DC_SS + cl) = lo;
+            }
         }
         __syncthreads();                             // u is there; nobody reads the planes of S any more
         uint32_t uh[DC_C / 16][4], ul[DC_C / 16][4];
@@ -330,70 +414,66 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
             lt_ldsm_x4_trans(ul[ks], u_lo + at);
         }
         // ---- S <- P S + K^T u ----
+        if (owns) {
+            const float p0 = sp[16 * warp + g], p1 = sp[16 * warp + g + 8];
+            float add[2][2][4];                      // [column tile][high x high | mixed]
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-            const int tile = warp + 4 * m;
-            if (tile >= DP / 16) continue;
-            const float p0 = sp[16 * tile + g], p1 = sp[16 * tile + g + 8];
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                s[m][j][0] *= p0; s[m][j][1] *= p0;
-                s[m][j][2] *= p1; s[m][j][3] *= p1;
-            }
+                for (int k = 0; k < 2; ++k) add[j][k][0] = add[j][k][1] = add[j][k][2] = add[j][k][3] = 0.f;
             const __nv_bfloat16* kt = planes + 4 * DC_C * RS;
 #pragma unroll
             for (int ks = 0; ks < DC_C / 16; ++ks) {
                 uint32_t ah[4], al[4];
-                const int at = (16 * ks + lr + 8 * (mi >> 1)) * RS + 16 * tile + 8 * (mi & 1);
+                const int at = (16 * ks + lr + 8 * (mi >> 1)) * RS + 16 * warp + 8 * (mi & 1);
                 lt_ldsm_x4_trans(ah, kt + at);
                 lt_ldsm_x4_trans(al, kt + DC_C * RS + at);
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
-                    lt_mma(s[m][j], ah, uh[ks][2 * j], uh[ks][2 * j + 1]);
-                    lt_mma(s[m][j], al, uh[ks][2 * j], uh[ks][2 * j + 1]);
-                    lt_mma(s[m][j], ah, ul[ks][2 * j], ul[ks][2 * j + 1]);
+                    lt_mma(add[j][0], ah, uh[ks][2 * j], uh[ks][2 * j + 1]);
+                    lt_mma(add[j][1], al, uh[ks][2 * j], uh[ks][2 * j + 1]);
+                    lt_mma(add[j][1], ah, ul[ks][2 * j], ul[ks][2 * j + 1]);
                 }
             }
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[j][e] = fmaf(s[j][e], e < 2 ? p0 : p1, add[j][0][e] + add[j][1][e]);
+            if (c + 1 < n_chunks) publish();
         }
-        if (c + 1 < n_chunks) publish();
         // ---- o = Q S + B u ----
-        if (warp >= 2) {
+        if (rt >= 2) {
+            acc[1][0] = acc[1][1] = acc[1][2] = acc[1][3] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < DC_C / 16; ++ks) {
                 uint32_t ah[4], al[4];
-                const int at = (16 * (warp - 2) + lr + 8 * (mi & 1)) * DC_BS + 16 * ks + 8 * (mi >> 1);
+                const int at = (16 * (rt - 2) + lr + 8 * (mi & 1)) * DC_BS + 16 * ks + 8 * (mi >> 1);
                 dc_ldsm_x4(ah, b_hi + at);
                 dc_ldsm_x4(al, b_hi + DC_C * DC_BS + at);
-#pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    lt_mma(acc[0][j], ah, uh[ks][2 * j], uh[ks][2 * j + 1]);
-                    lt_mma(acc[1][j], al, uh[ks][2 * j], uh[ks][2 * j + 1]);
-                    lt_mma(acc[1][j], ah, ul[ks][2 * j], ul[ks][2 * j + 1]);
-                }
+                const uint32_t h0 = ct ? uh[ks][2] : uh[ks][0], h1 = ct ? uh[ks][3] : uh[ks][1];
+                lt_mma(acc[0], ah, h0, h1);
+                lt_mma(acc[1], al, h0, h1);
+                lt_mma(acc[1], ah, ct ? ul[ks][2] : ul[ks][0], ct ? ul[ks][3] : ul[ks][1]);
             }
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
-                const int tok = first + c * DC_C + 16 * (warp - 2) + g + 8 * half;
+                const int tok = first + c * DC_C + 16 * (rt - 2) + g + 8 * half;
                 if (tok >= last) continue;
 #pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const int col = v0 + 8 * j + 2 * t + e;
-                        if (col < V) out[((size_t)tok * H + h) * V + col] = acc[0][j][2 * half + e] + acc[1][j][2 * half + e];
-                    }
+                for (int e = 0; e < 2; ++e) {
+                    const int col = v0 + 8 * ct + 2 * t + e;
+                    if (col < V) out[((size_t)tok * H + h) * V + col] = acc[0][2 * half + e] + acc[1][2 * half + e];
+                }
             }
         }
     }
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int row = 16 * (warp + 4 * m) + g + 8 * (e >> 1), col = v0 + 8 * j + 2 * t + (e & 1);
-                if (row < D && col < V) S[(size_t)row * V + col] = s[m][j][e];
-            }
+        for (int e = 0; e < 4; ++e) {
+            const int row = 16 * warp + g + 8 * (e >> 1), col = v0 + 8 * j + 2 * t + (e & 1);
+            if (row < D && col < V) S[(size_t)row * V + col] = s[j][e];
+        }
 }
 
 // Bytes of the buffer that ni_delta_chunk_recurrence needs.
@@ -404,44 +484,47 @@ NI_EXPORT long long ni_delta_chunk_buffer_bytes(int n_tokens, int n_seqs, int H,
 }
 NI_EXPORT int ni_delta_chunk_max_dim() { return 128; }
 
-template <int DP>
-static int dc_launch(const float* qkv, const float* gates, const float* decay, int ld_z, float* state, long long state_stride,
-                     const int* cu_q, const int* slots, int n_seqs, int max_q_len, int G, int H, int D, int V, void* buf,
-                     float* out, cudaStream_t stream) {
-    const DcLayout lay{DP, (V + DC_VS - 1) / DC_VS * DC_VS};
-    const size_t smem_p = (size_t)(3 * DC_C * DP + 2 * DC_C * DC_AS) * sizeof(float), smem_s = dc_scan_smem<DP>();
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(delta_chunk_prepare_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
+template <int DP, int TAPS>
+static int dc_launch(const DcInput& in, float* state, int n_seqs, int max_q_len, void* buf, float* out, cudaStream_t stream) {
+    const DcLayout lay{DP, (in.V + DC_VS - 1) / DC_VS * DC_VS};
+    const size_t smem_p = (size_t)(3 * DC_C * DP + 2 * DC_C * DC_AS + DC_C * lay.VP) * sizeof(float), smem_s = dc_scan_smem<DP>();
+    static size_t configured = 0;
+    if (configured < smem_p) {
+        cudaError_t e = cudaFuncSetAttribute(delta_chunk_prepare_kernel<DP, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
         if (e == cudaSuccess)
             e = cudaFuncSetAttribute(delta_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s);
         if (e != cudaSuccess) return (int)e;
-        configured = true;
+        configured = smem_p;
     }
-    dim3 grid_p((max_q_len + DC_C - 1) / DC_C, H, n_seqs), grid_s(lay.VP / DC_VS, H, n_seqs);
-    delta_chunk_prepare_kernel<DP><<<grid_p, DC_THREADS, smem_p, stream>>>(qkv, gates, decay, ld_z, cu_q, G, H, D, V,
-                                                                           (unsigned char*)buf, lay);
+    dim3 grid_p((max_q_len + DC_C - 1) / DC_C, in.H, n_seqs), grid_s(lay.VP / DC_VS, in.H, n_seqs);
+    delta_chunk_prepare_kernel<DP, TAPS><<<grid_p, DC_THREADS, smem_p, stream>>>(in, (unsigned char*)buf, lay);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
-    delta_chunk_scan_kernel<DP><<<grid_s, DC_SCAN_THREADS, smem_s, stream>>>((const unsigned char*)buf, lay, state, state_stride,
-                                                                             cu_q, slots, H, D, V, out);
+    delta_chunk_scan_kernel<DP><<<grid_s, DC_THREADS, smem_s, stream>>>((const unsigned char*)buf, lay, state, in.state_stride,
+                                                                        in.cu_q, in.slots, in.H, in.D, in.V, out);
     NI_RETURN_LAUNCH_STATUS();
 }
 
-// The recurrence over a step's tokens: qkv, gates and decay as ni_delta_prepare leaves them (decays per channel); the state
-// [H, D, V] at the start of a request's row moves on; out FP32 [T, H V].  max_q_len: the most tokens a request brings.  buf:
-// 16-byte aligned, ni_delta_chunk_buffer_bytes long.
-NI_EXPORT int ni_delta_chunk_recurrence(const float* qkv, const float* gates, const float* decay, int ld_z, float* state,
-                                        long long state_stride, const int* cu_q, const int* slots, int n_tokens, int n_seqs,
-                                        int max_q_len, int G, int H, int D, int V, void* buf, long long buf_bytes, float* out,
-                                        cudaStream_t stream) {
+// The rule over a step's prompt portions, from the projection (see DcInput) to the read-outs, out FP32 [T, H V]: the state
+// [H, D, V] at the start of a request's row moves on; the convolution history behind it is read (ni_delta_gated_norm, which
+// must follow, writes the new one).  max_q_len: the most tokens a request brings.  buf: 16-byte aligned,
+// ni_delta_chunk_buffer_bytes long.
+NI_EXPORT int ni_delta_chunk_recurrence(const void* proj, int ld, int b_off, const float* conv_w, const float* a_log,
+                                        const float* dt_bias, const float* z, int ld_z, float* state, long long state_stride,
+                                        const int* cu_q, const int* slots, int n_tokens, int n_seqs, int max_q_len, int G, int H,
+                                        int D, int V, int taps, void* buf, long long buf_bytes, float* out, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return NI_OK;
-    if (G <= 0 || H <= 0 || D <= 0 || V <= 0 || H % G || ld_z < H * D || max_q_len <= 0 || buf == nullptr ||
-        (reinterpret_cast<size_t>(buf) & 15) || buf_bytes < ni_delta_chunk_buffer_bytes(n_tokens, n_seqs, H, D, V) ||
-        state_stride < (long long)H * D * V)
+    if (G <= 0 || H <= 0 || D <= 0 || V <= 0 || taps <= 0 || H % G || ld_z < H * D || max_q_len <= 0 || buf == nullptr ||
+        (reinterpret_cast<size_t>(buf) & 15) || buf_bytes < ni_delta_chunk_buffer_bytes(n_tokens, n_seqs, H, D, V) || b_off < 0 ||
+        ld < b_off + H || ld < 2 * G * D + H * V || state_stride < (long long)H * D * V + (long long)(taps - 1) * (2 * G * D + H * V))
         return NI_ERR_BAD_ARGUMENT;
-    if (D > 128 || H > 65535 || n_seqs > 65535) return NI_ERR_UNSUPPORTED_SIZE;
-#define GO(DP) return dc_launch<DP>(qkv, gates, decay, ld_z, state, state_stride, cu_q, slots, n_seqs, max_q_len, G, H, D, V, buf, out, stream)
+    if (D > 128 || V > 512 || H > 65535 || n_seqs > 65535) return NI_ERR_UNSUPPORTED_SIZE;
+    const DcInput in = {(const __nv_bfloat16*)proj, conv_w, a_log, dt_bias, z, state, state_stride, cu_q, slots,
+                        ld, b_off, ld_z, G, H, D, V, taps};
+    const bool four = taps == 4 && (reinterpret_cast<size_t>(conv_w) & 15) == 0;
+#define GO(DP)                                                                                    \
+    return four ? dc_launch<DP, 4>(in, state, n_seqs, max_q_len, buf, out, stream)                \
+                : dc_launch<DP, 0>(in, state, n_seqs, max_q_len, buf, out, stream)
     if (D <= 32) GO(32);
     if (D <= 64) GO(64);
     GO(128);

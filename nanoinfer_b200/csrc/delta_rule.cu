@@ -465,8 +465,8 @@ NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate
 //
 // One block of 8 warps per (head, request).  A warp owns every 8th row of S, a lane every 32nd column; S is read into
 // registers first, before anything else is needed.  Meanwhile: the convolution of the head's q, k and v channels (a thread
-// per channel), the thin second products of its D decay logits and V gate logits (a thread per row of the weights, which
-// are bfloat16 rows of 16-byte pieces; the thin first products stand in shared memory), unit norms.  Then k S, the error,
+// per channel), the thin second products of its D decay logits and V gate logits (a group of lanes per row of the weights, 16
+// bytes each; the thin first products stand in shared memory), unit norms.  Then k S, the error,
 // the update, q S and the gated norm; S is written back once.
 // The convolution history of the value channels is moved on by their own block.  A query/key channel belongs to the H / G
 // heads that share it: the last of their blocks to have read the old inputs (an atomic ticket per request and q/k head, left
@@ -486,19 +486,48 @@ struct DeltaTokenParams {
     float eps, scale;
 };
 
-// Row . x for a row of n bfloat16 (n a multiple of 8, 16-byte aligned) and x in shared memory.
-__device__ __forceinline__ float dt_thin_dot(const __nv_bfloat16* __restrict__ row, const float* x, int n) {
-    float a0 = 0.f, a1 = 0.f;
-    for (int i = 0; i < n; i += 8) {
-        float w[8];
-        NiVec16<__nv_bfloat16>::load(row + i, w);
-        const float4 x0 = *reinterpret_cast<const float4*>(x + i), x1 = *reinterpret_cast<const float4*>(x + i + 4);
-        a0 = fmaf(w[0], x0.x, a0); a1 = fmaf(w[1], x0.y, a1);
-        a0 = fmaf(w[2], x0.z, a0); a1 = fmaf(w[3], x0.w, a1);
-        a0 = fmaf(w[4], x1.x, a0); a1 = fmaf(w[5], x1.y, a1);
-        a0 = fmaf(w[6], x1.z, a0); a1 = fmaf(w[7], x1.w, a1);
+// The dot products of `rows` rows of n bfloat16 (n a multiple of 8, rows 16-byte aligned) with x in shared memory, dealt
+// over the block's warps: L lanes share a row (L a power of two), four rows per group of lanes on their way at a time.
+// done(row, sum) is called by one lane per row.
+template <int L, typename F>
+__device__ __forceinline__ void dt_thin_rows(const __nv_bfloat16* __restrict__ w, int rows, const float* x, int n, F done) {
+    constexpr int PER_WARP = 32 / L;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane % L, sub = lane / L;
+    for (int r0 = 4 * PER_WARP * warp; r0 < rows; r0 += 4 * PER_WARP * DT_WARPS) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int k = 8 * l; k < n; k += 8 * L) {
+            uint4 raw[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int row = r0 + u * PER_WARP + sub;
+                raw[u] = row < rows ? *reinterpret_cast<const uint4*>(w + (size_t)row * n + k) : make_uint4(0u, 0u, 0u, 0u);
+            }
+            const float4 x0 = *reinterpret_cast<const float4*>(x + k), x1 = *reinterpret_cast<const float4*>(x + k + 4);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+                const float2 w0 = __bfloat1622float2(p[0]), w1 = __bfloat1622float2(p[1]), w2 = __bfloat1622float2(p[2]),
+                             w3 = __bfloat1622float2(p[3]);
+                a[u] = fmaf(w0.x, x0.x, a[u]); a[u] = fmaf(w0.y, x0.y, a[u]);
+                a[u] = fmaf(w1.x, x0.z, a[u]); a[u] = fmaf(w1.y, x0.w, a[u]);
+                a[u] = fmaf(w2.x, x1.x, a[u]); a[u] = fmaf(w2.y, x1.y, a[u]);
+                a[u] = fmaf(w3.x, x1.z, a[u]); a[u] = fmaf(w3.y, x1.w, a[u]);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+#pragma unroll
+            for (int off = L / 2; off > 0; off >>= 1) a[u] += __shfl_xor_sync(0xffffffffu, a[u], off);
+            const int row = r0 + u * PER_WARP + sub;
+            if (l == 0 && row < rows) done(row, a[u]);
+        }
     }
-    return a0 + a1;
+}
+template <typename F>
+__device__ __forceinline__ void dt_thin(const __nv_bfloat16* __restrict__ w, int rows, const float* x, int n, F done) {
+    if (n > 64) dt_thin_rows<16>(w, rows, x, n, done);
+    else if (n > 16) dt_thin_rows<8>(w, rows, x, n, done);
+    else dt_thin_rows<2>(w, rows, x, n, done);
 }
 
 // DR: rows of S per warp (D <= 8 DR); VC: columns per lane (V <= 32 VC).
@@ -548,15 +577,8 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
         }
         s_last = last;
     }
-    for (int r = tid; r < D + V; r += blockDim.x) {
-        if (r < D) {
-            const int c = h * D + r;
-            sg[r] = dr_decay(p.a_log[h], dt_thin_dot(p.w_decay + (size_t)c * p.ra, thin, p.ra) + p.dt_bias[c]);
-        } else {
-            const int c = h * V + r - D;
-            sgate[r - D] = dr_sigmoid(dt_thin_dot(p.w_gate + (size_t)c * p.rg, thin + p.ra, p.rg)) * p.scale;
-        }
-    }
+    dt_thin(p.w_decay + (size_t)h * D * p.ra, D, thin, p.ra, [&](int r, float a) { sg[r] = a; });
+    dt_thin(p.w_gate + (size_t)h * V * p.rg, V, thin + p.ra, p.rg, [&](int r, float a) { sgate[r] = dr_sigmoid(a) * p.scale; });
     if (warp < 2) {
         const float* v = warp == 0 ? sq : sk;
         float ss = 0.f;
@@ -564,6 +586,8 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
         ss = ni_warp_sum(ss);
         if (lane == 0) unit[warp] = 1.0f / sqrtf(ss + 1e-6f) * (warp == 0 ? 1.0f / sqrtf((float)D) : 1.0f);
     }
+    __syncthreads();
+    if (tid < D) sg[tid] = dr_decay(p.a_log[h], sg[tid] + p.dt_bias[h * D + tid]);        // (D <= 128 < blockDim.x)
     __syncthreads();
     const float rq = unit[0], rk = unit[1];
     float acc[VC];

@@ -452,16 +452,16 @@ def delta_rule_channel(args) -> None:
     us_prep = _time([lambda st=st: ops.delta_prepare(proj, conv_w, a_log, dt_bias, st, seq, cu, slots, b, G, H, D, V, taps, qkv, gates,
                                                      b_col=b_col, z=z) for st in states], args.iters)
     z.copy_(z0)
-    ops.delta_prepare(proj, conv_w, a_log, dt_bias, states[0], seq, cu, slots, b, G, H, D, V, taps, qkv, gates, b_col=b_col, z=z)
     buf = torch.empty(ops.delta_chunk_buffer_bytes(n, b, H, D, V) // 4, device=DEV)
-    us_chunk = _time([lambda st=st: ops.delta_chunk_recurrence(qkv, gates, z, st, cu, slots, b, t, G, H, D, V, buf, o) for st in states],
-                     args.iters)
+    us_chunk = _time([lambda st=st: ops.delta_chunk_recurrence(proj, 0, b_col, conv_w, a_log, dt_bias, z, st, cu, slots, b, t, G, H, D, V, taps,
+                                                               buf, o) for st in states], args.iters)
+    ops.delta_prepare(proj, conv_w, a_log, dt_bias, states[0], seq, cu, slots, b, G, H, D, V, taps, qkv, gates, b_col=b_col, z=z)
     us_rec = _time([lambda st=st: ops.delta_recurrence(qkv, gates, st, cu, slots, b, G, H, D, V, o, z=z) for st in states], args.iters)
     us_norm = _time([lambda: ops.delta_gated_norm(o, proj, norm_w, 1e-6, G, H, D, V, y, states[0], cu, slots, b, taps, gate=z,
                                                   gate_col=H * D, sigmoid=True)], args.iters)
     flops = 8.0 * n * H * D * V
-    print(f"{what}: prepare {us_prep:.2f} us ({n * (C * 6 + H * D * 8) / us_prep / 1e3:.0f} GB/s), in chunks {us_chunk:.2f} us "
-          f"({flops / us_chunk / 1e6:.2f} TFLOP/s of the recurrence), token by token {us_rec:.2f} us ({flops / us_rec / 1e6:.2f}), "
+    print(f"{what}: in chunks, preparation included, {us_chunk:.2f} us ({flops / us_chunk / 1e6:.2f} TFLOP/s of the recurrence); "
+          f"preparation {us_prep:.2f} us ({n * (C * 6 + H * D * 8) / us_prep / 1e3:.0f} GB/s) and token by token {us_rec:.2f} us; "
           f"gated norm {us_norm:.2f} us ({n * H * V * 10 / us_norm / 1e3:.0f} GB/s)")
 
 

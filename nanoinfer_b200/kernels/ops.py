@@ -99,7 +99,7 @@ _SIGNATURES = {
         "ni_delta_gated_norm": [_P, _P, _I, _I, _P, _F, _F, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _LL, _P, _P, _P],
     },
     "delta_chunk": {
-        "ni_delta_chunk_recurrence": [_P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _P],
+        "ni_delta_chunk_recurrence": [_P, _I, _I, _P, _P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _P],
         "ni_delta_chunk_max_dim": [],
     },
     "latent": {
@@ -615,19 +615,26 @@ def delta_chunk_buffer_bytes(n_tokens: int, n_seqs: int, n_heads: int, dim: int,
     return int(f(n_tokens, n_seqs, n_heads, dim, vdim))
 
 
-def delta_chunk_recurrence(qkv, gates, z, state, cu_q, slots, n_seqs, max_q_len, n_q_heads_kv, n_heads, dim, vdim, buf, out) -> None:
-    """As delta_recurrence with decays per key channel (``z`` as delta_prepare leaves it), for prompt portions: chunks of 32
-    tokens, their products on the tensor cores with every FP32 operand split into two bfloat16 halves.  ``max_q_len``: the
-    most tokens that one request brings; ``buf``: delta_chunk_buffer_bytes bytes on the device."""
+def delta_chunk_recurrence(proj, col0, b_col, conv_w, a_log, dt_bias, z, state, cu_q, slots, n_seqs, max_q_len, n_q_heads_kv, n_heads,
+                           dim, vdim, taps, buf, out) -> None:
+    """What delta_prepare and delta_recurrence do with decays per key channel, for prompt portions of a bfloat16 projection
+    (``proj`` [T, *], q | k | v from column ``col0`` on, beta's logits at ``b_col``; ``z`` float32 [T, *]: the decays' logits
+    in its first H D columns, left as they are): chunks of 32 tokens, their products on the tensor cores with every FP32
+    operand split into two bfloat16 halves.  ``max_q_len``: the most tokens that one request brings; ``buf``:
+    delta_chunk_buffer_bytes bytes on the device.  delta_gated_norm must follow (it moves the convolution history on)."""
     f32 = torch.float32
-    n = qkv.shape[0]
-    if out.shape != (n, n_heads * vdim) or z.shape[0] != n or z.shape[1] < n_heads * dim or gates.shape != (n, n_heads, 2) or \
-            qkv.shape[1] != 2 * n_q_heads_kv * dim + n_heads * vdim:
+    n = proj.shape[0]
+    c = 2 * n_q_heads_kv * dim + n_heads * vdim
+    if out.shape != (n, n_heads * vdim) or z.shape[0] != n or z.shape[1] < n_heads * dim or b_col < col0 or \
+            proj.shape[1] < max(col0 + c, b_col + n_heads) or conv_w.shape != (c, taps) or a_log.numel() != n_heads or \
+            dt_bias.numel() != n_heads * dim or state.shape[1] != n_heads * dim * vdim + (taps - 1) * c:
         raise KernelError("delta_chunk_recurrence: shapes do not agree")
     _check(load("delta_chunk").ni_delta_chunk_recurrence(
-        _dev(qkv, "qkv", f32), _dev(gates, "gates", f32), _dev(z, "z", f32), z.shape[1], _dev(state, "state", f32), state.shape[1],
-        _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), n, n_seqs, int(max_q_len), n_q_heads_kv, n_heads, dim,
-        vdim, _dev(buf, "buf"), buf.numel() * buf.element_size(), _dev(out, "out", f32), _stream()), "delta_chunk_recurrence")
+        _dev(proj, "proj", torch.bfloat16) + 2 * col0, proj.shape[1], b_col - col0, _dev(conv_w, "conv_w", f32),
+        _dev(a_log, "a_log", f32), _dev(dt_bias, "dt_bias", f32), _dev(z, "z", f32), z.shape[1], _dev(state, "state", f32),
+        state.shape[1], _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), n, n_seqs, int(max_q_len), n_q_heads_kv,
+        n_heads, dim, vdim, taps, _dev(buf, "buf"), buf.numel() * buf.element_size(), _dev(out, "out", f32), _stream()),
+        "delta_chunk_recurrence")
 
 
 DELTA_TOKEN_MAX_DIM = 128      # the largest key and value sizes whose state a block of the token kernel holds in registers

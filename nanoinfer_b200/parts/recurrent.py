@@ -150,7 +150,7 @@ class GatedDeltaRule(Part):
         # single tokens go through one kernel, which reads an FP32 projection
         self.wants_f32_tokens = (rt.dtype == torch.bfloat16 and self.channel and self.thin_gate
                                  and max(d, v) <= ops.DELTA_TOKEN_MAX_DIM and self.thin_k <= 8192)
-        self.chunked = rt.dtype == torch.bfloat16 and self.channel and d <= ops.DELTA_CHUNK_MAX_DIM
+        self.chunked = rt.dtype == torch.bfloat16 and self.channel and d <= ops.DELTA_CHUNK_MAX_DIM and v <= 512
         if self.chunked:
             self.kernel_modules = ("delta_chunk",)
 
@@ -161,7 +161,11 @@ class GatedDeltaRule(Part):
         return (self.w_in, self.w_o)
 
     def forward(self, x: torch.Tensor, ctx, cache, residual=None):
-        return self.finish(self.rt.linear(x, self.w_in, out_dtype=torch.float32), ctx, cache, residual=residual)
+        dtype = self.rt.dtype if self._in_chunks(ctx) else torch.float32
+        return self.finish(self.rt.linear(x, self.w_in, out_dtype=dtype), ctx, cache, residual=residual)
+
+    def _in_chunks(self, ctx) -> bool:
+        return self.chunked and ctx.max_q_len >= self.CHUNK_FROM
 
     def project(self, h: torch.Tensor, norm) -> torch.Tensor:
         """The fused input projection of norm(h), with the norm inside the product (steps of a few rows): the first
@@ -203,17 +207,17 @@ class GatedDeltaRule(Part):
             return out
         z = self._thin_logits(proj, col0) if self.w_thin is not None else None
         decay = z if self.channel else None
-        qkv = rt.empty(n, self.channels, dtype=f32)
-        gates = rt.empty(n, h, 2, dtype=f32)
-        ops.delta_prepare(proj, self.conv_w, self.a_log, self.dt_bias, cache.state, ctx.seq_of_token, ctx.cu_q,
-                          ctx.slots, ctx.n_seqs, g, h, d, v, self.taps, qkv, gates, col0=col0, b_col=col0 + self.b_col, z=decay)
         o = rt.empty(n, h * v, dtype=f32)
-        if self.chunked and ctx.max_q_len >= self.CHUNK_FROM:
+        if self._in_chunks(ctx) and proj.dtype == torch.bfloat16:
             need = ops.delta_chunk_buffer_bytes(n, ctx.n_seqs, h, d, v)
             buf = rt.workspace("delta_chunks", -(-need // 4), f32)                 # one buffer for all layers
-            ops.delta_chunk_recurrence(qkv, gates, decay, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, ctx.max_q_len, g, h, d, v,
-                                       buf, o)
+            ops.delta_chunk_recurrence(proj, col0, col0 + self.b_col, self.conv_w, self.a_log, self.dt_bias, z, cache.state,
+                                       ctx.cu_q, ctx.slots, ctx.n_seqs, ctx.max_q_len, g, h, d, v, self.taps, buf, o)
         else:
+            qkv = rt.empty(n, self.channels, dtype=f32)
+            gates = rt.empty(n, h, 2, dtype=f32)
+            ops.delta_prepare(proj, self.conv_w, self.a_log, self.dt_bias, cache.state, ctx.seq_of_token, ctx.cu_q, ctx.slots,
+                              ctx.n_seqs, g, h, d, v, self.taps, qkv, gates, col0=col0, b_col=col0 + self.b_col, z=decay)
             ops.delta_recurrence(qkv, gates, cache.state, ctx.cu_q, ctx.slots, ctx.n_seqs, g, h, d, v, o, z=decay)
         gate, gate_col = (z, h * d if self.channel else 0) if self.thin_gate else (proj, col0 + self.gate_col)
         if gate.dtype != f32:

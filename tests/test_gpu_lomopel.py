@@ -186,7 +186,8 @@ def test_gate_per_coordinate(dtype, gate_dtype, n, w, ld_g, col, ld_o, out_col):
 
 
 def _plain_delta(proj, z, conv_w, a_log, dt_bias, norm_w, hist, S, G, H, D, V, eps, scale, b_col):
-    """Gated read-outs [T, H V] of one request's rows; moves hist (a list of rows) and S (a list of matrices) on."""
+    """Gated read-outs [T, H V] of one request's rows (norm_w None: the read-outs themselves); moves hist (a list of rows)
+    and S (a list of matrices) on."""
     C, outs = 2 * G * D + H * V, []
     for row, zr in zip(proj, z):
         c = convolved(row[:C], conv_w, hist)
@@ -199,53 +200,59 @@ def _plain_delta(proj, z, conv_w, a_log, dt_bias, norm_w, hist, S, G, H, D, V, e
             kk, qq = k[h // (H // G)], q[h // (H // G)]
             kk, qq = kk / torch.sqrt((kk * kk).sum() + 1e-6), qq / torch.sqrt((qq * qq).sum() + 1e-6) * D ** -0.5
             S[h], o = delta_step(S[h], decay[h], beta[h], qq, kk, v[h])
-            heads.append(unit_rms(o, eps) * norm_w)
-        outs.append(torch.cat(heads) * gate * scale)
+            heads.append(o if norm_w is None else unit_rms(o, eps) * norm_w)
+        outs.append(torch.cat(heads) if norm_w is None else torch.cat(heads) * gate * scale)
     return torch.stack(outs)
 
 
-@pytest.mark.parametrize("G, H, D, V", [(2, 6, 20, 12), (3, 3, 32, 64), (1, 2, 64, 40), (2, 2, 128, 128), (1, 1, 7, 33), (1, 3, 96, 16)])
-@pytest.mark.parametrize("speed", [-6.0, -2.0, 3.0])
-def test_delta_rule_in_chunks(G, H, D, V, speed):
-    """The chunked recurrence against the plain rule and the kernel that goes token by token: portions around the chunk's 32
-    tokens and of many chunks beside single tokens, slots out of order, decays from slow to so fast that a chunk's product
-    vanishes; outputs and states over three steps."""
+@pytest.mark.parametrize("G, H, D, V, taps", [(2, 6, 20, 12, 4), (3, 3, 32, 64, 4), (1, 2, 64, 40, 2), (2, 2, 128, 128, 4), (1, 1, 7, 33, 1),
+                                              (1, 3, 96, 16, 5), (1, 1, 16, 200, 3)])
+@pytest.mark.parametrize("speed", [-8.0, -2.0, 4.0])
+def test_delta_rule_in_chunks(G, H, D, V, taps, speed):
+    """The chunked rule against the plain one and the kernels that go token by token: portions around the chunk's 32 tokens,
+    shorter than the convolution's history and of many chunks beside single tokens, slots out of order, decays from slow to so
+    fast that a chunk's product vanishes; read-outs and states over three steps, histories moved on between."""
     from nanoinfer_b200.kernels import ops
     g = torch.Generator().manual_seed(D * 3 + V + int(speed))
+    C, col0 = 2 * G * D + H * V, 16
+    b_col = col0 + C + 5
+    ld = b_col + H + (-(b_col + H) % 8)
+    conv_w, a_log, dt_bias = torch.randn(C, taps, generator=g) * 0.6, torch.randn(H, generator=g) * 0.5, speed + torch.randn(H * D, generator=g)
     slots = [3, 0, 2, 4]
-    state = (torch.randn(5, H * D * V + 9, generator=g) * 0.2).to(DEV)
-    state = state[:, :H * D * V].contiguous()
-    other = state.clone()
-    S = {s: list(state[s].cpu().double().view(H, D, V)) for s in slots}
+    state = (torch.randn(5, H * D * V + (taps - 1) * C, generator=g) * 0.2).to(DEV)
+    other, before = state.clone(), state.clone()
+    S = {s: list(state[s, :H * D * V].cpu().double().view(H, D, V)) for s in slots}
+    hist = {s: list(state[s, H * D * V:].cpu().double().view(taps - 1, C)) for s in slots}
     for lens in ([33, 1, 64, 150], [1, 31, 2, 32], [100, 5, 96, 1]):
         n, cu = sum(lens), [0]
         for ln in lens:
             cu.append(cu[-1] + ln)
-        q, k = (torch.nn.functional.normalize(torch.randn(n, G, D, generator=g), dim=-1) for _ in range(2))
-        k = torch.nn.functional.normalize(k + 0.7 * k[:1], dim=-1)               # keys that resemble one another
-        v = torch.randn(n, H, V, generator=g)
-        qkv = torch.cat([q.reshape(n, -1) * D ** -0.5, k.reshape(n, -1), v.reshape(n, -1)], dim=1)
-        decay = torch.exp(-torch.exp(speed + torch.randn(n, H, D, generator=g)))
-        z = torch.cat([decay.reshape(n, -1), torch.zeros(n, 8)], dim=1).to(DEV)
-        gates = torch.rand(n, H, 2, generator=g)
+        seq = [i for i, ln in enumerate(lens) for _ in range(ln)]
+        proj = (torch.randn(n, ld, generator=g) + 0.5).to(torch.bfloat16)           # (keys that resemble one another)
+        z = torch.randn(n, H * D + 8, generator=g)
+        args, pd, zd = (_i32(cu), _i32(slots), 4), proj.to(DEV), z.to(DEV)
         out, ref = torch.full((n, H * V), 7.0, device=DEV), torch.empty(n, H * V, device=DEV)
         buf = torch.empty(-(-ops.delta_chunk_buffer_bytes(n, 4, H, D, V) // 4), device=DEV)
-        args = (_i32(cu), _i32(slots), 4)
-        ops.delta_chunk_recurrence(qkv.to(DEV), gates.to(DEV), z, state, *args, max(lens), G, H, D, V, buf, out)
-        ops.delta_recurrence(qkv.to(DEV), gates.to(DEV), other, *args, G, H, D, V, ref, z=z)
-        want = torch.zeros(n, H, V, dtype=F64)
-        for i, s in enumerate(slots):
-            for t in range(cu[i], cu[i + 1]):
-                for h in range(H):
-                    S[s][h], want[t, h] = delta_step(S[s][h], decay[t, h].double(), gates[t, h, 1].double(),
-                                                     q[t, h // (H // G)].double() * D ** -0.5, k[t, h // (H // G)].double(), v[t, h].double())
+        weights = (conv_w.to(DEV), a_log.to(DEV), dt_bias.to(DEV))
+        ops.delta_chunk_recurrence(pd, col0, b_col, *weights, zd, state, *args, max(lens), G, H, D, V, taps, buf, out)
+        assert torch.equal(zd.cpu(), z)
+        qkv, gates = torch.empty(n, C, device=DEV), torch.empty(n, H, 2, device=DEV)
+        ops.delta_prepare(pd, *weights, other, _i32(seq), *args, G, H, D, V, taps, qkv, gates, col0=col0, b_col=b_col, z=zd)
+        ops.delta_recurrence(qkv, gates, other, *args, G, H, D, V, ref, z=zd)
+        for st, o in ((state, out), (other, ref)):                                  # moves the histories on
+            ops.delta_gated_norm(o, pd, torch.ones(V, device=DEV), 1e-5, G, H, D, V, torch.empty(n, H * V, device=DEV, dtype=torch.bfloat16),
+                                 st, *args, taps, col0=col0, gate=torch.zeros(n, H * V, device=DEV), gate_col=0, sigmoid=True)
+        want = torch.cat([_plain_delta(proj[cu[i]:cu[i + 1], col0:].double(), torch.cat([z[cu[i]:cu[i + 1], :H * D], torch.zeros(lens[i], H * V)], 1).double(),
+                                       conv_w.double(), a_log.double(), dt_bias.double(), None, hist[s], S[s], G, H, D, V, 0.0, 1.0, b_col - col0)
+                          for i, s in enumerate(slots)])
         size = want.abs().max().item()
-        torch.testing.assert_close(ref.cpu().double().view(n, H, V), want, rtol=1e-4, atol=1e-5 * size)
-        torch.testing.assert_close(out.cpu().double().view(n, H, V), want, rtol=1e-3, atol=2e-4 * size)
+        torch.testing.assert_close(ref.cpu().double(), want, rtol=1e-4, atol=1e-5 * size)
+        torch.testing.assert_close(out.cpu().double(), want, rtol=1e-3, atol=2e-4 * size)
     for s in slots:
         final = torch.stack(S[s])
-        torch.testing.assert_close(state[s].cpu().double().view(H, D, V), final, rtol=1e-3, atol=2e-4 * final.abs().max().item())
-    assert torch.equal(state[1], other[1])                                       # a slot that nobody has
+        torch.testing.assert_close(state[s, :H * D * V].cpu().double().view(H, D, V), final, rtol=1e-3, atol=2e-4 * final.abs().max().item())
+        assert torch.equal(state[s, H * D * V:], other[s, H * D * V:])
+    assert torch.equal(state[1], before[1])                                         # a slot that nobody has
 
 
 @pytest.mark.parametrize("G, H, D, V, taps", [(2, 6, 20, 12, 4), (3, 3, 32, 64, 4), (1, 2, 64, 64, 2), (5, 5, 40, 9, 5), (2, 2, 128, 128, 3),
