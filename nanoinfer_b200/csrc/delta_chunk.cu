@@ -30,15 +30,19 @@
 #define DC_AS 36         // row stride of A in shared memory
 #define DC_BS (DC_C + 8) // row stride of the planes of B
 
-// One (chunk, head) of the buffer, in bytes: W, Q, K as two bfloat16 planes each [DC_C][DP], the two planes of B
-// [DC_C][DC_C], U0 FP32 [DC_C][VP], P_n FP32 [DP].
+#define DC_PAD 8         // numbers behind every row of the planes of W, Q and K (rows then start in different banks)
+
+// One (chunk, head) of the buffer, in bytes - laid out as the scan keeps it in shared memory, so that it is copied as it is: W,
+// Q, K as two bfloat16 planes each [DC_C][DP + DC_PAD], the two planes of B [DC_C][DC_BS], P_n FP32 [DP]; behind that U0 FP32
+// in slices of DC_VS columns [VP / DC_VS][DC_C][DC_VS].
 struct DcLayout {
     int DP, VP;
-    __host__ __device__ size_t plane() const { return (size_t)DC_C * DP * 2; }
+    __host__ __device__ int rs() const { return DP + DC_PAD; }
+    __host__ __device__ size_t plane() const { return (size_t)DC_C * rs() * 2; }
     __host__ __device__ size_t b_off() const { return 6 * plane(); }
-    __host__ __device__ size_t u_off() const { return b_off() + 2 * DC_C * DC_C * 2; }
-    __host__ __device__ size_t p_off() const { return u_off() + (size_t)DC_C * VP * 4; }
-    __host__ __device__ size_t bytes() const { return p_off() + (size_t)DP * 4; }
+    __host__ __device__ size_t p_off() const { return b_off() + 2 * DC_C * DC_BS * 2; }
+    __host__ __device__ size_t u_off() const { return p_off() + (size_t)DP * 4; }
+    __host__ __device__ size_t bytes() const { return u_off() + (size_t)DC_C * VP * 4; }
 };
 static int dc_pad_dim(int D) { return D <= 32 ? 32 : (D <= 64 ? 64 : 128); }
 
@@ -86,13 +90,14 @@ __device__ __forceinline__ void dc_conv_column(const DcInput& in, const float* _
     if (TAPS == 4) {
         const float4 w = *reinterpret_cast<const float4*>(in.conv_w + (size_t)c * 4);
         float x3 = earlier(3), x2 = earlier(2), x1 = earlier(1);
-        float v[DC_C];
+        __nv_bfloat16 v[DC_C];
 #pragma unroll
-        for (int r = 0; r < DC_C; ++r) v[r] = r < n ? __bfloat162float(x[(size_t)r * in.ld]) : 0.f;
+        for (int r = 0; r < DC_C; ++r) v[r] = r < n ? x[(size_t)r * in.ld] : __float2bfloat16_rn(0.f);
 #pragma unroll
         for (int r = 0; r < DC_C; ++r) {
-            const float y = fmaf(w.w, v[r], fmaf(w.z, x1, fmaf(w.y, x2, w.x * x3)));
-            x3 = x2; x2 = x1; x1 = v[r];
+            const float x0 = __bfloat162float(v[r]);
+            const float y = fmaf(w.w, x0, fmaf(w.z, x1, fmaf(w.y, x2, w.x * x3)));
+            x3 = x2; x2 = x1; x1 = x0;
             dst[r * stride] = r < n ? dc_silu(y) : 0.f;
         }
     } else {
@@ -112,9 +117,9 @@ __device__ __forceinline__ void dc_conv_column(const DcInput& in, const float* _
 // grid (chunks of the longest portion, H, requests).  DP: the padded key size; a lane of the pairs' phase owns DP / 32 groups
 // of four channels.
 template <int DP, int TAPS>
-__global__ void __launch_bounds__(DC_THREADS, 2)
+__global__ void __launch_bounds__(DC_THREADS, 3)
 delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, DcLayout lay) {
-    constexpr int M = DP / 32;
+    constexpr int M = DP / 32, RS = DP + DC_PAD;
     extern __shared__ __align__(16) float dc_smem[];
     float* sq = dc_smem;                       // [DC_C][DP]
     float* sk = sq + DC_C * DP;
@@ -132,7 +137,16 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
     unsigned char* rec = buf + ((size_t)(dc_chunk_base(in.cu_q, seq, &base_scratch) + blockIdx.x) * H + h) * lay.bytes();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const float* hist = in.state + (size_t)in.slots[seq] * in.state_stride + (size_t)H * D * V;
-    // ---- q, k, v of the chunk; decays; beta ----
+    // ---- the decays' logits on their way; q, k, v of the chunk; decays; beta ----
+    const float* zrow = in.z + (size_t)first * in.ld_z + h * D;
+    const bool wide = D % 4 == 0 && in.ld_z % 4 == 0 && (reinterpret_cast<size_t>(in.z) & 15) == 0;
+    if (wide) {
+        for (int i = tid; i < DC_C * (DP / 4); i += DC_THREADS) {
+            const int r = i / (DP / 4), d = 4 * (i % (DP / 4));
+            if (r < n && d < D) lt_cp_async16(sg + r * DP + d, zrow + (size_t)r * in.ld_z + d);
+        }
+    }
+    lt_cp_async_commit();
     for (int i = tid; i < 2 * DP + VP; i += DC_THREADS) {
         const int part = i < DP ? 0 : (i < 2 * DP ? 1 : 2), e = i - part * DP;
         float* dst = part == 0 ? sq + e : (part == 1 ? sk + e : sv + e);
@@ -143,17 +157,23 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
             for (int r = 0; r < DC_C; ++r) dst[r * stride] = 0.f;
         }
     }
+    lt_cp_async_wait<0>();
     {
+        // a thread turns the pieces it copied itself into decays (or fetches number by number where rows are not aligned)
         const float ea = -expf(in.a_log[h]);
-#pragma unroll 4
-        for (int i = tid; i < DC_C * DP; i += DC_THREADS) {
-            const int r = i / DP, d = i - r * DP;
-            float gd = 1.f;
-            if (r < n && d < D) {
-                const float x = in.z[(size_t)(first + r) * in.ld_z + h * D + d] + in.dt_bias[h * D + d];
-                gd = expf(ea * (x > 20.0f ? x : log1pf(expf(x))));
+        for (int i = tid; i < DC_C * (DP / 4); i += DC_THREADS) {
+            const int r = i / (DP / 4), d = 4 * (i % (DP / 4));
+            float4* at = reinterpret_cast<float4*>(sg + r * DP + d);
+            float4 z4 = *at;
+            float* v = reinterpret_cast<float*>(&z4);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const bool live = r < n && d + e < D;
+                const float raw = wide ? v[e] : (live ? zrow[(size_t)r * in.ld_z + d + e] : 0.f);
+                const float x = live ? raw + in.dt_bias[h * D + d + e] : 0.f;
+                v[e] = live ? expf(ea * (x > 20.0f ? x : log1pf(expf(x)))) : 1.f;
             }
-            sg[i] = gd;
+            *at = z4;
         }
     }
     for (int i = tid; i < 2 * DC_C * DC_AS; i += DC_THREADS) sA[i] = 0.f;       // A and B
@@ -217,8 +237,8 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
             if (l < 4 && i > s) sA[i * DC_AS + s] = t[0] * beta[i];
             if (l >= 4 && i >= s) sB[i * DC_AS + s] = t[0];
         }
-        __nv_bfloat16* k_hi = reinterpret_cast<__nv_bfloat16*>(rec + 4 * lay.plane()) + s * DP;
-        __nv_bfloat16* k_lo = k_hi + DC_C * DP;
+        __nv_bfloat16* k_hi = reinterpret_cast<__nv_bfloat16*>(rec + 4 * lay.plane()) + s * RS;
+        __nv_bfloat16* k_lo = k_hi + DC_C * RS;
 #pragma unroll
         for (int m = 0; m < M; ++m) {
             uint2 hi, lo;
@@ -235,18 +255,19 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
             const float2 v = *reinterpret_cast<const float2*>(sB + (i / (DC_C / 2)) * DC_AS + 2 * (i % (DC_C / 2)));
             uint32_t hi, lo;
             lt_split2(v.x, v.y, hi, lo);
-            *reinterpret_cast<uint32_t*>(b_hi + 2 * i) = hi;
-            *reinterpret_cast<uint32_t*>(b_hi + DC_C * DC_C + 2 * i) = lo;
+            __nv_bfloat16* to = b_hi + (i / (DC_C / 2)) * DC_BS + 2 * (i % (DC_C / 2));
+            *reinterpret_cast<uint32_t*>(to) = hi;
+            *reinterpret_cast<uint32_t*>(to + DC_C * DC_BS) = lo;
         }
     }
     __nv_bfloat16* w_hi = reinterpret_cast<__nv_bfloat16*>(rec);
-    __nv_bfloat16* w_lo = w_hi + DC_C * DP;
-    __nv_bfloat16* q_hi = w_lo + DC_C * DP;
-    __nv_bfloat16* q_lo = q_hi + DC_C * DP;
-    float* u0 = reinterpret_cast<float*>(rec + lay.u_off());
+    __nv_bfloat16* w_lo = w_hi + DC_C * RS;
+    __nv_bfloat16* q_hi = w_lo + DC_C * RS;
+    __nv_bfloat16* q_lo = q_hi + DC_C * RS;
     for (int col = tid; col < DP + VP; col += DC_THREADS) {
         const bool is_k = col < DP;
         const int vc = col - DP;
+        float* u0 = reinterpret_cast<float*>(rec + lay.u_off()) + (size_t)(vc / DC_VS) * DC_C * DC_VS + vc % DC_VS;
         float x[DC_C], P = 1.f;
 #pragma unroll
         for (int i = 0; i < DC_C; ++i) {
@@ -254,7 +275,7 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
             if (is_k) {
                 P *= sg[i * DP + col];
                 rhs = sk[i * DP + col] * P;
-                dc_store_split(q_hi + i * DP + col, q_lo + i * DP + col, sq[i * DP + col] * P);
+                dc_store_split(q_hi + i * RS + col, q_lo + i * RS + col, sq[i * DP + col] * P);
             } else {
                 rhs = sv[i * VP + vc];
             }
@@ -268,8 +289,8 @@ delta_chunk_prepare_kernel(const DcInput in, unsigned char* __restrict__ buf, Dc
                 if (s + 3 < i) acc[3] = fmaf(-a.w, x[s + 3], acc[3]);
             }
             x[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
-            if (is_k) dc_store_split(w_hi + i * DP + col, w_lo + i * DP + col, x[i]);
-            else u0[i * VP + vc] = x[i];
+            if (is_k) dc_store_split(w_hi + i * RS + col, w_lo + i * RS + col, x[i]);
+            else u0[i * DC_VS] = x[i];
         }
         if (is_k) reinterpret_cast<float*>(rec + lay.p_off())[col] = P;
     }
@@ -282,7 +303,7 @@ __device__ __forceinline__ void dc_ldsm_x4(uint32_t (&r)[4], const void* p) {
 }
 
 template <int DP> __host__ __device__ constexpr int dc_stage_bytes() {
-    return 6 * DC_C * (DP + 8) * 2 + 2 * DC_C * DC_BS * 2 + DC_C * DC_VS * 4 + DP * 4;
+    return 6 * DC_C * (DP + DC_PAD) * 2 + 2 * DC_C * DC_BS * 2 + DP * 4 + DC_C * DC_VS * 4;
 }
 #define DC_SS (DC_VS + 8)          // row stride of the planes of S and of u
 template <int DP> __host__ __device__ constexpr int dc_scan_smem() { return 2 * dc_stage_bytes<DP>() + 2 * DP * DC_SS * 2 + 2 * DC_C * DC_SS * 2; }
@@ -294,7 +315,8 @@ __global__ void __launch_bounds__(DC_THREADS)
 delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, float* __restrict__ state, long long state_stride,
                         const int* __restrict__ cu_q, const int* __restrict__ slots, int H, int D, int V,
                         float* __restrict__ out) {
-    constexpr int RS = DP + 8;                       // row stride of the operand planes
+    constexpr int RS = DP + DC_PAD;                  // row stride of the operand planes
+    constexpr int FIXED = dc_stage_bytes<DP>() - DC_C * DC_VS * 4;      // of a stage: everything but the slice of U0
     extern __shared__ __align__(16) unsigned char dc_raw[];
     __shared__ int base_scratch;
     const int seq = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * DC_VS;
@@ -310,26 +332,14 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
     __nv_bfloat16* u_lo = u_hi + DC_C * DC_SS;
     float* S = state + (size_t)slots[seq] * state_stride + (size_t)h * D * V;
 
-    auto fetch = [&](int c) {                        // the operands of chunk c into their stage
-        const unsigned char* rec = rec0 + (size_t)c * rec_step;
-        unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>();
-        constexpr int PIECES = DP / 8;
-        for (int i = tid; i < 6 * DC_C * PIECES; i += DC_THREADS) {
-            const int r = i / PIECES, p = i - r * PIECES;                    // r: row of plane r / DC_C
-            lt_cp_async16(st + ((size_t)r * RS + 8 * p) * 2, rec + ((size_t)r * DP + 8 * p) * 2);
-        }
-        unsigned char* sb = st + 6 * DC_C * RS * 2;
-        for (int i = tid; i < 2 * DC_C * (DC_C / 8); i += DC_THREADS) {
-            const int r = i / (DC_C / 8), p = i % (DC_C / 8);
-            lt_cp_async16(sb + (r * DC_BS + 8 * p) * 2, rec + lay.b_off() + (r * DC_C + 8 * p) * 2);
-        }
-        unsigned char* su = sb + 2 * DC_C * DC_BS * 2;
-        for (int i = tid; i < DC_C * (DC_VS / 4); i += DC_THREADS) {
-            const int r = i / (DC_VS / 4), p = i % (DC_VS / 4);
-            lt_cp_async16(su + (r * DC_VS + 4 * p) * 4, rec + lay.u_off() + ((size_t)r * lay.VP + v0 + 4 * p) * 4);
-        }
-        unsigned char* sp = su + DC_C * DC_VS * 4;
-        for (int i = tid; i < DP / 4; i += DC_THREADS) lt_cp_async16(sp + 16 * i, rec + lay.p_off() + 16 * i);
+    auto fetch = [&](int c) {                        // the operands of chunk c into their stage, as they lie in the buffer
+        const unsigned char* rec = rec0 + (size_t)c * rec_step + 16 * tid;
+        unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>() + 16 * tid;
+#pragma unroll
+        for (int i = 0; i < (FIXED + 16 * DC_THREADS - 1) / (16 * DC_THREADS); ++i)
+            if ((i + 1) * 16 * DC_THREADS <= FIXED || 16 * tid + i * 16 * DC_THREADS < FIXED)
+                lt_cp_async16(st + i * 16 * DC_THREADS, rec + i * 16 * DC_THREADS);
+        if (tid < DC_C * DC_VS / 4) lt_cp_async16(st + FIXED, rec + lay.u_off() + (size_t)blockIdx.x * DC_C * DC_VS * 4);
     };
     fetch(0);
     lt_cp_async_commit();
@@ -367,8 +377,8 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
         const unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>();
         const __nv_bfloat16* planes = reinterpret_cast<const __nv_bfloat16*>(st);
         const __nv_bfloat16* b_hi = planes + 6 * DC_C * RS;
-        const float* su = reinterpret_cast<const float*>(b_hi + 2 * DC_C * DC_BS);
-        const float* sp = su + DC_C * DC_VS;
+        const float* sp = reinterpret_cast<const float*>(b_hi + 2 * DC_C * DC_BS);
+        const float* su = sp + DP;
         // ---- [W; Q] S ----
         float acc[3][4];                             // high x high, low x high, high x low
 #pragma unroll

@@ -463,7 +463,7 @@ NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate
 }
 // ---- a step of single tokens with decays per channel: everything between the projections in one launch -------------------
 //
-// One block of 8 warps per (head, request).  A warp owns every 8th row of S, a lane every 32nd column; S is read into
+// One block of 16 warps per (head, request).  A warp owns every 16th row of S, a lane every 32nd column; S is read into
 // registers first, before anything else is needed.  Meanwhile: the convolution of the head's q, k and v channels (a thread
 // per channel), the thin second products of its D decay logits and V gate logits (a group of lanes per row of the weights, 16
 // bytes each; the thin first products stand in shared memory), unit norms.  Then k S, the error,
@@ -471,7 +471,7 @@ NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate
 // The convolution history of the value channels is moved on by their own block.  A query/key channel belongs to the H / G
 // heads that share it: the last of their blocks to have read the old inputs (an atomic ticket per request and q/k head, left
 // zero) moves them on.  No block waits for another.
-#define DT_WARPS 8
+#define DT_WARPS 16
 struct DeltaTokenParams {
     const float* proj;                 // [T, ld] FP32: q | k | v | ... b at b_off, the thin first products at thin_off
     const __nv_bfloat16* w_decay;      // [H D, ra]
@@ -486,85 +486,69 @@ struct DeltaTokenParams {
     float eps, scale;
 };
 
-// The dot products of `rows` rows of n bfloat16 (n a multiple of 8, rows 16-byte aligned) with x in shared memory, dealt
-// over the block's warps: L lanes share a row (L a power of two), four rows per group of lanes on their way at a time.
-// done(row, sum) is called by one lane per row.
-template <int L, typename F>
-__device__ __forceinline__ void dt_thin_rows(const __nv_bfloat16* __restrict__ w, int rows, const float* x, int n, F done) {
-    constexpr int PER_WARP = 32 / L;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane % L, sub = lane / L;
-    for (int r0 = 4 * PER_WARP * warp; r0 < rows; r0 += 4 * PER_WARP * DT_WARPS) {
-        float a[4] = {0.f, 0.f, 0.f, 0.f};
-        for (int k = 8 * l; k < n; k += 8 * L) {
-            uint4 raw[4];
-#pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const int row = r0 + u * PER_WARP + sub;
-                raw[u] = row < rows ? *reinterpret_cast<const uint4*>(w + (size_t)row * n + k) : make_uint4(0u, 0u, 0u, 0u);
-            }
-            const float4 x0 = *reinterpret_cast<const float4*>(x + k), x1 = *reinterpret_cast<const float4*>(x + k + 4);
-#pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
-                const float2 w0 = __bfloat1622float2(p[0]), w1 = __bfloat1622float2(p[1]), w2 = __bfloat1622float2(p[2]),
-                             w3 = __bfloat1622float2(p[3]);
-                a[u] = fmaf(w0.x, x0.x, a[u]); a[u] = fmaf(w0.y, x0.y, a[u]);
-                a[u] = fmaf(w1.x, x0.z, a[u]); a[u] = fmaf(w1.y, x0.w, a[u]);
-                a[u] = fmaf(w2.x, x1.x, a[u]); a[u] = fmaf(w2.y, x1.y, a[u]);
-                a[u] = fmaf(w3.x, x1.z, a[u]); a[u] = fmaf(w3.y, x1.w, a[u]);
-            }
-        }
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-#pragma unroll
-            for (int off = L / 2; off > 0; off >>= 1) a[u] += __shfl_xor_sync(0xffffffffu, a[u], off);
-            const int row = r0 + u * PER_WARP + sub;
-            if (l == 0 && row < rows) done(row, a[u]);
-        }
-    }
-}
-template <typename F>
-__device__ __forceinline__ void dt_thin(const __nv_bfloat16* __restrict__ w, int rows, const float* x, int n, F done) {
-    if (n > 64) dt_thin_rows<16>(w, rows, x, n, done);
-    else if (n > 16) dt_thin_rows<8>(w, rows, x, n, done);
-    else dt_thin_rows<2>(w, rows, x, n, done);
-}
-
-// DR: rows of S per warp (D <= 8 DR); VC: columns per lane (V <= 32 VC).
-template <int DR, int VC>
-__global__ void __launch_bounds__(DT_WARPS * 32)
+// DR: rows of S per warp (D <= 16 DR); VC: columns per lane (V <= 32 VC).  EXACT: D and V are those bounds, taps 4.
+// Everything that does not depend on this block's own results - S, weights, constants, the history - is asked for before the
+// first barrier, so that the chain of dependent memory round trips is short.
+template <int DR, int VC, bool EXACT>
+__global__ void __launch_bounds__(DT_WARPS * 32, 1)
 delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
-    constexpr int DP = DT_WARPS * DR, VP = 32 * VC;
+    constexpr int DP = DT_WARPS * DR, VP = 32 * VC, U = 8;
     __shared__ float sq[DP], sk[DP], sg[DP], sv[VP], sgate[VP], su[VP], red[DT_WARPS][VP], scratch[32];
     __shared__ float unit[2];          // what q and k are multiplied by
     __shared__ int s_last;
     extern __shared__ __align__(16) float thin[];       // [ra + rg]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int h = blockIdx.x, seq = blockIdx.y;
-    const int D = dm.D, V = dm.V, G = dm.G, C = dm.C(), per = dm.H / G, g = h / per, taps = dm.taps;
+    const int D = EXACT ? DP : dm.D, V = EXACT ? VP : dm.V, taps = EXACT ? 4 : dm.taps;
+    const int G = dm.G, C = dm.C(), per = dm.H / G, g = h / per;
     const int t = p.cu_q[seq];
     float* st = p.state + (size_t)p.slots[seq] * p.state_stride;
     float* S = st + (size_t)h * D * V;
-    float* hist = st + dm.hist_off();
+    float* hist = st + (size_t)dm.H * D * V;
     float s[DR][VC];
 #pragma unroll
     for (int i = 0; i < DR; ++i)
 #pragma unroll
         for (int j = 0; j < VC; ++j) {
             const int row = warp + DT_WARPS * i, col = lane + 32 * j;
-            s[i][j] = (row < D && col < V) ? S[(size_t)row * V + col] : 0.f;
+            s[i][j] = (EXACT || (row < D && col < V)) ? S[(size_t)row * V + col] : 0.f;
         }
+    // the thin second products: the first half of the warps the D rows of the decay's matrix, the others the V rows of the
+    // gate's; L lanes share a row, a lane's first 16 bytes of up to U rows are asked for here
+    const bool gates = warp >= DT_WARPS / 2;
+    const int n_thin = gates ? p.rg : p.ra, rows = gates ? V : D, w8 = warp & (DT_WARPS / 2 - 1);
+    const int L = n_thin > 64 ? 16 : (n_thin > 32 ? 8 : 4), l = lane & (L - 1), sub = lane / L, per_warp = 32 / L;
+    const __nv_bfloat16* w_thin = gates ? p.w_gate + (size_t)h * V * p.rg : p.w_decay + (size_t)h * D * p.ra;
+    uint4 raw[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int row = (u * (DT_WARPS / 2) + w8) * per_warp + sub;
+        raw[u] = row < rows && 8 * l < n_thin ? *reinterpret_cast<const uint4*>(w_thin + (size_t)row * n_thin + 8 * l)
+                                              : make_uint4(0u, 0u, 0u, 0u);
+    }
     const float* row = p.proj + (size_t)t * dm.ld;
+    const float a_log = p.a_log[h], beta = dr_sigmoid(row[dm.b_off + h]);
+    const float dt = tid < D ? p.dt_bias[h * D + tid] : 0.f, norm_w = tid < V ? p.norm_w[tid] : 0.f;
     for (int i = tid; i < p.ra + p.rg; i += blockDim.x) thin[i] = row[p.thin_off + i];
-    for (int i = tid; i < 2 * D + V; i += blockDim.x) {
-        const int c = i < D ? g * D + i : (i < 2 * D ? G * D + g * D + i - D : 2 * G * D + h * V + i - 2 * D);
-        const float x = row[c];
+    // the convolution: a thread per channel (2 D + V <= 384 < blockDim.x)
+    int c = -1;
+    float x = 0.f, h0 = 0.f, h1 = 0.f, h2 = 0.f;
+    if (tid < 2 * D + V) {
+        c = tid < D ? g * D + tid : (tid < 2 * D ? G * D + g * D + tid - D : 2 * G * D + h * V + tid - 2 * D);
+        x = row[c];
         float acc = 0.f;
-        for (int j = 0; j + 1 < taps; ++j) acc = fmaf(p.conv_w[(size_t)c * taps + j], hist[(size_t)j * C + c], acc);
-        const float y = dr_silu(fmaf(p.conv_w[(size_t)c * taps + taps - 1], x, acc));
-        if (i < D) sq[i] = y;
-        else if (i < 2 * D) sk[i - D] = y;
-        else sv[i - 2 * D] = y;
+        if (EXACT) {                       // (taps 4: the weights in one load)
+            const float4 w = *reinterpret_cast<const float4*>(p.conv_w + (size_t)c * 4);
+            h0 = hist[c]; h1 = hist[(size_t)C + c]; h2 = hist[2 * (size_t)C + c];
+            acc = fmaf(w.w, x, fmaf(w.z, h2, fmaf(w.y, h1, w.x * h0)));
+        } else {
+            for (int j = 0; j + 1 < taps; ++j) acc = fmaf(p.conv_w[(size_t)c * taps + j], hist[(size_t)j * C + c], acc);
+            acc = fmaf(p.conv_w[(size_t)c * taps + taps - 1], x, acc);
+        }
+        const float y = dr_silu(acc);
+        if (tid < D) sq[tid] = y;
+        else if (tid < 2 * D) sk[tid - D] = y;
+        else sv[tid - 2 * D] = y;
     }
     __syncthreads();
     if (tid == 0 && taps > 1) {
@@ -577,8 +561,42 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
         }
         s_last = last;
     }
-    dt_thin(p.w_decay + (size_t)h * D * p.ra, D, thin, p.ra, [&](int r, float a) { sg[r] = a; });
-    dt_thin(p.w_gate + (size_t)h * V * p.rg, V, thin + p.ra, p.rg, [&](int r, float a) { sgate[r] = dr_sigmoid(a) * p.scale; });
+    {
+        const float* xs = thin + (gates ? p.ra : 0);
+        float a[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) a[u] = 0.f;
+        for (int k = 8 * l; k < n_thin; k += 8 * L) {
+            if (k != 8 * l) {
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    const int r = (u * (DT_WARPS / 2) + w8) * per_warp + sub;
+                    raw[u] = r < rows ? *reinterpret_cast<const uint4*>(w_thin + (size_t)r * n_thin + k) : make_uint4(0u, 0u, 0u, 0u);
+                }
+            }
+            const float4 x0 = *reinterpret_cast<const float4*>(xs + k), x1 = *reinterpret_cast<const float4*>(xs + k + 4);
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const __nv_bfloat162* q = reinterpret_cast<const __nv_bfloat162*>(&raw[u]);
+                const float2 w0 = __bfloat1622float2(q[0]), w1 = __bfloat1622float2(q[1]), w2 = __bfloat1622float2(q[2]),
+                             w3 = __bfloat1622float2(q[3]);
+                a[u] = fmaf(w0.x, x0.x, a[u]); a[u] = fmaf(w0.y, x0.y, a[u]);
+                a[u] = fmaf(w1.x, x0.z, a[u]); a[u] = fmaf(w1.y, x0.w, a[u]);
+                a[u] = fmaf(w2.x, x1.x, a[u]); a[u] = fmaf(w2.y, x1.y, a[u]);
+                a[u] = fmaf(w3.x, x1.z, a[u]); a[u] = fmaf(w3.y, x1.w, a[u]);
+            }
+        }
+        for (int off = L / 2; off > 0; off >>= 1)
+#pragma unroll
+            for (int u = 0; u < U; ++u) a[u] += __shfl_xor_sync(0xffffffffu, a[u], off);
+        if (l == 0) {
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int r = (u * (DT_WARPS / 2) + w8) * per_warp + sub;
+                if (r < rows) (gates ? sgate : sg)[r] = a[u];
+            }
+        }
+    }
     if (warp < 2) {
         const float* v = warp == 0 ? sq : sk;
         float ss = 0.f;
@@ -587,7 +605,7 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
         if (lane == 0) unit[warp] = 1.0f / sqrtf(ss + 1e-6f) * (warp == 0 ? 1.0f / sqrtf((float)D) : 1.0f);
     }
     __syncthreads();
-    if (tid < D) sg[tid] = dr_decay(p.a_log[h], sg[tid] + p.dt_bias[h * D + tid]);        // (D <= 128 < blockDim.x)
+    if (tid < D) sg[tid] = dr_decay(a_log, sg[tid] + dt);
     __syncthreads();
     const float rq = unit[0], rk = unit[1];
     float acc[VC];
@@ -596,7 +614,7 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
 #pragma unroll
     for (int i = 0; i < DR; ++i) {
         const int r = warp + DT_WARPS * i;
-        const float gd = r < D ? sg[r] : 0.f, kk = r < D ? sk[r] * rk : 0.f;
+        const float gd = EXACT || r < D ? sg[r] : 0.f, kk = EXACT || r < D ? sk[r] * rk : 0.f;
 #pragma unroll
         for (int j = 0; j < VC; ++j) {
             s[i][j] *= gd;
@@ -606,34 +624,34 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
 #pragma unroll
     for (int j = 0; j < VC; ++j) red[warp][lane + 32 * j] = acc[j];
     __syncthreads();
-    for (int c = tid; c < V; c += blockDim.x) {
+    if (tid < V) {                     // (V <= 128 < blockDim.x: a thread per column)
         float d = 0.f;
 #pragma unroll
-        for (int w = 0; w < DT_WARPS; ++w) d += red[w][c];
-        su[c] = dr_sigmoid(row[dm.b_off + h]) * (sv[c] - d);
+        for (int w = 0; w < DT_WARPS; ++w) d += red[w][tid];
+        su[tid] = beta * (sv[tid] - d);
     }
     __syncthreads();
 #pragma unroll
     for (int j = 0; j < VC; ++j) acc[j] = 0.f;
     float u[VC];
 #pragma unroll
-    for (int j = 0; j < VC; ++j) u[j] = lane + 32 * j < V ? su[lane + 32 * j] : 0.f;
+    for (int j = 0; j < VC; ++j) u[j] = EXACT || lane + 32 * j < V ? su[lane + 32 * j] : 0.f;
 #pragma unroll
     for (int i = 0; i < DR; ++i) {
         const int r = warp + DT_WARPS * i;
-        const float kk = r < D ? sk[r] * rk : 0.f, qq = r < D ? sq[r] * rq : 0.f;
+        const float kk = EXACT || r < D ? sk[r] * rk : 0.f, qq = EXACT || r < D ? sq[r] * rq : 0.f;
 #pragma unroll
         for (int j = 0; j < VC; ++j) {
             const int col = lane + 32 * j;
             s[i][j] = fmaf(kk, u[j], s[i][j]);
             acc[j] = fmaf(qq, s[i][j], acc[j]);
-            if (r < D && col < V) S[(size_t)r * V + col] = s[i][j];
+            if (EXACT || (r < D && col < V)) S[(size_t)r * V + col] = s[i][j];
         }
     }
 #pragma unroll
     for (int j = 0; j < VC; ++j) red[warp][lane + 32 * j] = acc[j];
     __syncthreads();
-    float o = 0.f;                     // V <= 128 < blockDim.x: a thread per column
+    float o = 0.f;
     if (tid < V) {
 #pragma unroll
         for (int w = 0; w < DT_WARPS; ++w) o += red[w][tid];
@@ -641,13 +659,13 @@ delta_token_kernel(const DeltaTokenParams p, const DeltaDims dm) {
     const float ss = ni_block_sum(o * o, scratch);
     if (tid < V)
         p.y[(size_t)t * p.ld_y + (size_t)h * V + tid] =
-            __float2bfloat16_rn(o * (1.0f / sqrtf(ss / (float)V + p.eps)) * p.norm_w[tid] * sgate[tid]);
-    if (taps > 1) {
-        const int first = s_last ? 0 : 2 * D;          // the q and k channels only by the last of the heads that share them
-        for (int i = first + tid; i < 2 * D + V; i += blockDim.x) {
-            const int c = i < D ? g * D + i : (i < 2 * D ? G * D + g * D + i - D : 2 * G * D + h * V + i - 2 * D);
+            __float2bfloat16_rn(o * (1.0f / sqrtf(ss / (float)V + p.eps)) * norm_w * dr_sigmoid(sgate[tid]) * p.scale);
+    if (taps > 1 && c >= 0 && (s_last || tid >= 2 * D)) {      // the q and k channels only by the last of the heads that share them
+        if (EXACT) {
+            hist[c] = h1; hist[(size_t)C + c] = h2; hist[2 * (size_t)C + c] = x;
+        } else {
             for (int j = 0; j + 2 < taps; ++j) hist[(size_t)j * C + c] = hist[(size_t)(j + 1) * C + c];
-            hist[(size_t)(taps - 2) * C + c] = row[c];
+            hist[(size_t)(taps - 2) * C + c] = x;
         }
     }
 }
@@ -676,17 +694,24 @@ NI_EXPORT int ni_delta_token_step(const float* proj, int ld, int b_off, int thin
     p.state = state; p.state_stride = state_stride; p.cu_q = cu_q; p.slots = slots; p.tickets = tickets;
     p.y = (__nv_bfloat16*)y; p.ld_y = ld_y; p.thin_off = thin_off; p.ra = ra; p.rg = rg; p.eps = eps; p.scale = scale;
     const size_t smem = (size_t)(ra + rg) * sizeof(float);
-#define GO(DR, VC) delta_token_kernel<DR, VC><<<dim3(H, n_seqs), DT_WARPS * 32, smem, stream>>>(p, dm)
+    const bool conv_aligned = (reinterpret_cast<size_t>(conv_w) & 15) == 0;
+#define GO_E(DR, VC, EXACT) delta_token_kernel<DR, VC, EXACT><<<dim3(H, n_seqs), DT_WARPS * 32, smem, stream>>>(p, dm)
+#define GO(DR, VC)                                                                  \
+    do {                                                                            \
+        if (D == DT_WARPS * DR && V == 32 * VC && taps == 4 && conv_aligned) GO_E(DR, VC, true); \
+        else GO_E(DR, VC, false);                                                   \
+    } while (0)
 #define GO_V(DR)                          \
     do {                                  \
         if (V <= 32) GO(DR, 1);           \
         else if (V <= 64) GO(DR, 2);      \
         else GO(DR, 4);                   \
     } while (0)
-    if (D <= 32) GO_V(4);
-    else if (D <= 64) GO_V(8);
-    else GO_V(16);
+    if (D <= 32) GO_V(2);
+    else if (D <= 64) GO_V(4);
+    else GO_V(8);
 #undef GO_V
 #undef GO
+#undef GO_E
     NI_RETURN_LAUNCH_STATUS();
 }
