@@ -85,8 +85,12 @@ qk_norm_rope_kernel(const TI* __restrict__ qkv, int ld, const float* __restrict_
         cs[i] = c * magnitude;
         cs[half + i] = s * magnitude;
     }
-    sq = ni_block_sum(sq, scratch);
-    sk = ni_block_sum(sk, scratch);          // (its barriers also publish row and cs)
+    if (q_gain) {
+        sq = ni_block_sum(sq, scratch);
+        sk = ni_block_sum(sk, scratch);      // (its barriers also publish row and cs)
+    } else {
+        __syncthreads();                     // no norm over the whole row: row and cs are all that is needed
+    }
     const float inv_q = q_gain ? 1.0f / sqrtf(sq / (float)nq + eps) : 1.0f;
     const float inv_k = k_gain ? 1.0f / sqrtf(sk / (float)nk + eps) : 1.0f;
     T* kdst = nullptr;
@@ -200,8 +204,12 @@ qk_norm_rope_vec_kernel(const TI* __restrict__ qkv, int ld, const float* __restr
             NiVec16<T>::store(vdst + (size_t)head * page_size * V + dim, v);
         }
     }
-    sq = ni_block_sum(sq, scratch);
-    sk = ni_block_sum(sk, scratch);          // (its barriers also publish row and cs)
+    if (q_gain) {
+        sq = ni_block_sum(sq, scratch);
+        sk = ni_block_sum(sk, scratch);      // (its barriers also publish row and cs)
+    } else {
+        __syncthreads();                     // no norm over the whole row: row and cs are all that is needed
+    }
     const float inv_q = q_gain ? 1.0f / sqrtf(sq / (float)nq + eps) : 1.0f;
     const float inv_k = k_gain ? 1.0f / sqrtf(sk / (float)nk + eps) : 1.0f;
     for (int i = threadIdx.x * VEC; i < nq + nk; i += blockDim.x * VEC) {

@@ -63,12 +63,35 @@ class Runtime:
             a, b = os.environ["NANOINFER_B200_BALANCED"].split(",")
             self.balanced_attention_pairs, self.balanced_attention_narrow_heads = int(a), bool(int(b))
         self._workspaces = {}
+        self._side = None
+        if os.environ.get("NANOINFER_B200_SIDE_BRANCHES"):      # for measurements: 0 runs every branch on one stream
+            self.side_branches = bool(int(os.environ["NANOINFER_B200_SIDE_BRANCHES"]))
         self._retired = []
         ops.require_cuda()
         if self.device.type != "cuda":
             raise ops.KernelError(f"device {self.device} is not a CUDA device; there is no CPU path")
         if self.balanced_attention_pairs <= 0:
             self.balanced_attention_pairs = ops.sm_count(self.device)
+
+    # Two branches of a layer that do not depend on each other may run side by side on the device (see fork).
+    side_branches: bool = True
+
+    def fork(self, one, other) -> None:
+        """Runs ``one()`` and ``other()``, neither of which reads what the other writes, as two branches: ``other`` on a
+        stream of its own that starts where the current one stands, and both joined at the end.  Inside a captured step
+        they become two branches of the graph.  Scratch tensors (``workspace``) must not be shared between the two."""
+        if not self.side_branches:
+            one()
+            other()
+            return
+        if self._side is None:
+            self._side = torch.cuda.Stream(self.device)
+        main = torch.cuda.current_stream(self.device)
+        self._side.wait_stream(main)
+        with torch.cuda.stream(self._side):
+            other()
+        one()
+        main.wait_stream(self._side)
 
     def weight(self, t: torch.Tensor) -> torch.Tensor:
         """A matrix weight on the device in the compute dtype."""

@@ -973,8 +973,9 @@ class ParallelMixers(Part):
         mixed = rt.empty(n, self.out_width + self.pad)
         if self.pad:
             mixed[:, self.out_width:].zero_()
-        for p, col, out_col in zip(self.sub_parts, self.in_cols, self.out_cols):
-            p.between(proj, col, ctx, cache, out=mixed, out_col=out_col)
+        # the sides read the projection and write columns of their own: two branches
+        rt.fork(*(lambda p=p, col=col, out_col=out_col: p.between(proj, col, ctx, cache, out=mixed, out_col=out_col)
+                  for p, col, out_col in zip(self.sub_parts, self.in_cols, self.out_cols)))
         if residual is None and self.affine is not None:
             raise ConfigError("mixers side by side: a scale on the output needs an arrangement that hands over the stream")
         handoff = rt.handoff(then_norm, n, self.hidden_size, mixed.shape[1]) if residual is not None else None
