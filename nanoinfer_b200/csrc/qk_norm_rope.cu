@@ -246,6 +246,115 @@ qk_norm_rope_vec_kernel(const TI* __restrict__ qkv, int ld, const float* __restr
     if (head_unit) qk_head_unit_write<T>(cs + rotary_dim, eps, temp, q_out + (size_t)t * nq, kdst, H, G, D, page_size);
 }
 
+// Without norms over the whole row, for heads of 64 or 128 that are rotated whole or not at all: a warp per head, the two
+// dimensions of a rotated pair in one lane (a lane owns E neighbours of the first half and their partners), the head's own norm
+// by shuffles, nothing in shared memory.  Up to four heads per warp are on their way at a time; cosines and sines once per warp.
+template <typename TI, int E> __device__ __forceinline__ void qk_load_e(const TI* p, float* v);
+template <> __device__ __forceinline__ void qk_load_e<float, 1>(const float* p, float* v) { v[0] = *p; }
+template <> __device__ __forceinline__ void qk_load_e<__nv_bfloat16, 1>(const __nv_bfloat16* p, float* v) { v[0] = __bfloat162float(*p); }
+template <> __device__ __forceinline__ void qk_load_e<float, 2>(const float* p, float* v) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    v[0] = x.x; v[1] = x.y;
+}
+template <> __device__ __forceinline__ void qk_load_e<__nv_bfloat16, 2>(const __nv_bfloat16* p, float* v) {
+    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+    v[0] = x.x; v[1] = x.y;
+}
+__device__ __forceinline__ void qk_store_e(float* p, const float* v, int e) {
+    if (e == 1) *p = v[0];
+    else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+}
+__device__ __forceinline__ void qk_store_e(__nv_bfloat16* p, const float* v, int e) {
+    if (e == 1) *p = __float2bfloat16_rn(v[0]);
+    else *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
+}
+
+template <typename TI, typename T, int E>
+__global__ void __launch_bounds__(256)
+qk_heads_kernel(const TI* __restrict__ qkv, int ld, const float* __restrict__ bias, float eps, const int* __restrict__ positions,
+                const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
+                const float* __restrict__ inv_freq, float magnitude, T* __restrict__ q_out, T* __restrict__ k_pages,
+                T* __restrict__ v_pages, int H, int G, int V, int rotated, int page_size, int head_unit,
+                const QkExtra<TI> ex) {
+    constexpr int D = 64 * E, HALF = 32 * E, VEC = 16 / sizeof(T), AT_ONCE = 4;
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const TI* x = qkv + (size_t)t * ld;
+    const int pos = positions[t], nq = H * D, nk = G * D, nv = G * V;
+    const float temp = qk_temperature(ex.temp_coef, ex.temp_every, pos);
+    T* kdst = nullptr;
+    T* vdst = nullptr;
+    if (k_pages) {
+        const int page = block_table[(size_t)seq_of_token[t] * bt_stride + pos / page_size], in_page = pos % page_size;
+        kdst = k_pages + ((size_t)page * G * page_size + in_page) * D;
+        vdst = v_pages + ((size_t)page * G * page_size + in_page) * V;
+    }
+    float cs[E], sn[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+        cs[e] = 1.f;
+        sn[e] = 0.f;
+        if (rotated) {
+            sincosf((float)pos * inv_freq[E * lane + e], &sn[e], &cs[e]);
+            cs[e] *= magnitude;
+            sn[e] *= magnitude;
+        }
+    }
+    const int heads = kdst ? H + G : H;
+    for (int h0 = warp; h0 < heads; h0 += AT_ONCE * warps) {
+        float a[AT_ONCE][E], b[AT_ONCE][E];
+#pragma unroll
+        for (int k = 0; k < AT_ONCE; ++k) {
+            const int head = h0 + k * warps;
+            if (head < heads) {
+                qk_load_e<TI, E>(x + (size_t)head * D + E * lane, a[k]);
+                qk_load_e<TI, E>(x + (size_t)head * D + HALF + E * lane, b[k]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < AT_ONCE; ++k) {
+            const int head = h0 + k * warps;
+            if (head >= heads) break;
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < E; ++e) {
+                float u = a[k][e], v = b[k][e];
+                if (bias) {
+                    u += bias[head * D + E * lane + e];
+                    v += bias[head * D + HALF + E * lane + e];
+                }
+                a[k][e] = u * cs[e] - v * sn[e];
+                b[k][e] = v * cs[e] + u * sn[e];
+                ss = fmaf(a[k][e], a[k][e], fmaf(b[k][e], b[k][e], ss));
+            }
+            float f = head < H ? temp : 1.f;
+            if (head_unit) f /= sqrtf(ni_warp_sum(ss) / (float)D + eps);
+#pragma unroll
+            for (int e = 0; e < E; ++e) { a[k][e] *= f; b[k][e] *= f; }
+            T* dst = head < H ? q_out + (size_t)t * nq + (size_t)head * D : kdst + (size_t)(head - H) * page_size * D;
+            qk_store_e(dst + E * lane, a[k], E);
+            qk_store_e(dst + HALF + E * lane, b[k], E);
+        }
+    }
+    if (!vdst) return;
+    for (int i = threadIdx.x * VEC; i < nv; i += blockDim.x * VEC) {
+        const int head = i / V, dim = i - head * V;
+        float v[VEC];
+        qk_load<TI, VEC>(x + nq + nk + i, v);
+        if (bias) {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) v[k] += bias[nq + nk + i + k];
+        }
+        if (ex.first_v) {
+            float f[VEC];
+            qk_load<TI, VEC>(ex.first_v + (size_t)t * ex.first_ld + i, f);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k)
+                v[k] = (1.0f - ex.lambda) * v[k] + ex.lambda * (f[k] + (ex.first_bias ? ex.first_bias[i + k] : 0.f));
+        }
+        NiVec16<T>::store(vdst + (size_t)head * page_size * V + dim, v);
+    }
+}
+
 // qkv [T, ld] with columns q (H D) | k (G D) | v (G V); bias FP32 [H D + G D + G V] or null; q_gain FP32 [H D] and
 // k_gain FP32 [G D], or null for no norm; head_unit: the heads' own norms after the rotation; k_pages / v_pages null: nothing is written (a run that reads another's cache).
 // dtype: queries and pages; in_dtype: qkv and first_v (FP32 beside bfloat16 is allowed).  temp_coef 0: no factor on the
@@ -280,9 +389,20 @@ NI_EXPORT int ni_qk_norm_rope(const void* qkv, int in_dtype, int dtype, int ld, 
                                                            (T*)q_out, (T*)k_pages, (T*)v_pages, H, G, D, V,          \
                                                            rotary_dim, page_size, head_unit, ex);                    \
     } while (0)
+#define LAUNCH_H(TI, T, E)                                                                                           \
+    do {                                                                                                             \
+        const QkExtra<TI> ex = {temp_coef, temp_every, (const TI*)first_v, first_ld, first_bias, lambda};            \
+        qk_heads_kernel<TI, T, E><<<n_tokens, 256, 0, stream>>>((const TI*)qkv, ld, bias, eps, positions, seq_of_token, \
+                                                                block_table, bt_stride, inv_freq, magnitude, (T*)q_out, \
+                                                                (T*)k_pages, (T*)v_pages, H, G, V, rotary_dim > 0,   \
+                                                                page_size, head_unit, ex);                           \
+    } while (0)
+    const bool by_heads = wide && !q_gain && (D == 64 || D == 128) && (rotary_dim == 0 || rotary_dim == D);
 #define LAUNCH(TI, T)                                                \
     do {                                                             \
-        if (wide) LAUNCH_K(qk_norm_rope_vec_kernel, TI, T);          \
+        if (by_heads && D == 64) LAUNCH_H(TI, T, 1);                 \
+        else if (by_heads) LAUNCH_H(TI, T, 2);                       \
+        else if (wide) LAUNCH_K(qk_norm_rope_vec_kernel, TI, T);          \
         else LAUNCH_K(qk_norm_rope_kernel, TI, T);                   \
     } while (0)
     if (dtype == NI_DTYPE_F32 && in_dtype == NI_DTYPE_F32) LAUNCH(float, float);
@@ -290,6 +410,7 @@ NI_EXPORT int ni_qk_norm_rope(const void* qkv, int in_dtype, int dtype, int ld, 
     else if (dtype == NI_DTYPE_BF16 && in_dtype == NI_DTYPE_F32) LAUNCH(float, __nv_bfloat16);
     else return NI_ERR_BAD_ARGUMENT;
 #undef LAUNCH
+#undef LAUNCH_H
 #undef LAUNCH_K
     NI_RETURN_LAUNCH_STATUS();
 }

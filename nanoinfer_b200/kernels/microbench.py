@@ -225,14 +225,17 @@ def attention_decode(args) -> None:
                for kc, vc in caches]
     else:
         scratch = torch.empty(b * hq * splits * (hd + 2), dtype=torch.float32, device=DEV)
+        sink = torch.zeros(hq, device=DEV) if args.sink else None
         fns = [lambda kc=kc, vc=vc: ops.attention_decode(q, kc, vc, out, None, b, positions, seq_of, table, hq, hkv, hd,
-                                                         page, None, 1.0 / math.sqrt(hd), splits, scratch, tickets,
-                                                         score_cap=args.score_cap, chunk=args.chunk, sink=args.sink)
+                                                         page, args.window or None, 1.0 / math.sqrt(hd), splits, scratch, tickets,
+                                                         score_cap=args.score_cap, chunk=args.chunk, sink=sink)
                for kc, vc in caches]
     us = _time(fns, args.iters)
     if args.chunk:           # only the keys of the last token's own chunk are read
         kv_bytes = kv_bytes * ((ctx - 1) % args.chunk + 1) // ctx
-    print(f"attention_decode{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''}{' (merge through scratch)' if args.scratch_merge else ''}{' (balanced)' if args.balanced else ''}{' ragged' if args.ragged else ''} batch={b} context={ctx} heads={hq}/{hkv} hd={hd} page={page} splits={splits}: "
+    if args.window:
+        kv_bytes = kv_bytes * min(ctx, args.window) // ctx
+    print(f"attention_decode{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''}{f' window of {args.window}' if args.window else ''}{' (merge through scratch)' if args.scratch_merge else ''}{' (balanced)' if args.balanced else ''}{' ragged' if args.ragged else ''} batch={b} context={ctx} heads={hq}/{hkv} hd={hd} page={page} splits={splits}: "
           f"{us:.2f} us, {kv_bytes / us / 1e3:.0f} GB/s of cache")
 
 
@@ -250,17 +253,18 @@ def attention_prefill(args) -> None:
     tile_row0 = torch.tensor(tiles, dtype=torch.int32, device=DEV)
     cu_q = torch.tensor([0, t], dtype=torch.int32, device=DEV)
     kv_len = torch.tensor([t], dtype=torch.int32, device=DEV)
+    sink = torch.zeros(hq, device=DEV) if args.sink else None
     fn = lambda: ops.attention_prefill(q, kc, vc, out, tile_seq, tile_row0, len(tiles), cu_q, kv_len, table, hq, hkv,
-                                       hd, page, None, 1.0 / math.sqrt(hd), kernel=args.kernel, score_cap=args.score_cap,
-                                       chunk=args.chunk, sink=args.sink)
+                                       hd, page, args.window or None, 1.0 / math.sqrt(hd), kernel=args.kernel, score_cap=args.score_cap,
+                                       chunk=args.chunk, sink=sink)
     if args.difference:      # --q-heads heads of two maps each
         fn = lambda: ops.attention_prefill_difference(q, kc, vc, out, tile_seq, tile_row0, len(tiles), cu_q, kv_len, table, hq, hkv, hd,
                                                       page, 1.0 / math.sqrt(hd // 2), 0.4, 1e-6, 0.6)
     us = _time([fn], args.iters)
     ops.check_device_errors()
-    seen = sum(p % args.chunk + 1 for p in range(t)) if args.chunk else t * (t + 1) / 2       # (query, key) pairs inside the mask
+    seen = sum(p % args.chunk + 1 for p in range(t)) if args.chunk else sum(min(p + 1, args.window or t) for p in range(t))       # (query, key) pairs inside the mask
     flops = (6.0 if args.difference else 4.0) * hq * hd * seen      # two maps: half-wide keys twice, the values twice
-    print(f"attention_prefill{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''} tokens={t} "
+    print(f"attention_prefill{' difference' if args.difference else ''}{' with a sink' if args.sink else ''}{f' chunks of {args.chunk}' if args.chunk else ''}{f' window of {args.window}' if args.window else ''} tokens={t} "
           f"heads={hq}/{hkv} hd={hd} kernel={args.kernel or 'default'}: {us:.1f} us, {flops / us / 1e6:.0f} TFLOP/s (of the pairs inside the mask)")
 
 
@@ -569,7 +573,11 @@ def qk_norm_rope(args) -> None:
     seq = torch.repeat_interleave(torch.arange(b, device=DEV), t).int()
     inv_freq = torch.pow(500000.0, -2.0 * torch.arange(D // 4, device=DEV) / (D // 2)).float()
     q = torch.empty(n, H * D, dtype=bf, device=DEV)
-    if args.head_unit:       # no bias, no whole-projection norms; the whole head rotated, then every head normed on its own
+    if args.mix:             # biases, the query's factor, another layer's values mixed in; no rotation
+        first = (projs[0], (H + G) * D, bias[(H + G) * D:].contiguous(), 0.3)
+        us = _time([lambda p=p: ops.qk_norm_rope(p, bias, None, None, 1e-6, pos, seq, table, inv_freq[:0], 1.0, q, k_pages, v_pages, H, G, D, D,
+                                                 0, page, temperature=(0.1, 100.0), first_values=first) for p in projs], args.iters)
+    elif args.head_unit:     # no bias, no whole-projection norms; the whole head rotated, then every head normed on its own
         inv_full = torch.pow(500000.0, -2.0 * torch.arange(D // 2, device=DEV) / D).float()
         us = _time([lambda p=p: ops.qk_norm_rope(p, None, None, None, 1e-6, pos, seq, table, inv_full, 1.0, q, k_pages, v_pages, H, G, D, D,
                                                  D, page, head_unit=True) for p in projs], args.iters)
@@ -577,7 +585,10 @@ def qk_norm_rope(args) -> None:
         us = _time([lambda p=p: ops.qk_norm_rope(p, bias, qg, kg, 1e-6, pos, seq, table, inv_freq, 1.2, q, k_pages, v_pages, H, G, D, D,
                                                  D // 2, page) for p in projs], args.iters)
     moved = n * cols * 2 * 2                              # every column read once and written once
-    print(f"qk_norm_rope{' (rotation, then a norm per head)' if args.head_unit else ''} batch={b} tokens={t} heads={H}/{G} dim={D}: "
+    att = [torch.randn(n, H * D, device=DEV, generator=g).to(bf) for _ in range(copies)]
+    us_gate = _time([lambda a=a, p=p: ops.element_gate(a, p, 0) for a, p in zip(att, projs)], args.iters)
+    print(f"element_gate tokens={n} width={H * D}: {us_gate:.2f} us ({3 * n * H * D * 2 / us_gate / 1e3:.0f} GB/s)")
+    print(f"qk_norm_rope{' (biases, temperature, value mixing)' if args.mix else ' (rotation, then a norm per head)' if args.head_unit else ''} batch={b} tokens={t} heads={H}/{G} dim={D}: "
           f"{us:.2f} us ({moved / us / 1e3:.0f} GB/s)")
 
 
@@ -800,7 +811,8 @@ def main() -> None:
         p.add_argument("--kernel", default=None, choices=["tc", "mma"], help="prefill: insist on one kernel")
         p.add_argument("--score-cap", type=float, default=0.0, help="bound the scaled scores by cap * tanh(s / cap)")
         p.add_argument("--chunk", type=int, default=0, help="a token sees only the keys of its own chunk of this many positions")
-        p.add_argument("--sink", action="store_true", help="one is added to the softmax's denominator")
+        p.add_argument("--window", type=int, default=0, help="a token sees itself and this many - 1 tokens before it")
+        p.add_argument("--sink", action="store_true", help="a sink per head in the softmax's denominator")
         p.add_argument("--difference", action="store_true", help="differential attention: two maps of half the head size per query head")
         p.add_argument("--copies", type=int, default=0, help="decode: cache copies used in turn (default: enough to exceed L2; 1: the cache stays in L2)")
         p.add_argument("--balanced", action="store_true", help="decode: the kernel that deals the keys evenly over a fixed grid")
@@ -835,6 +847,7 @@ def main() -> None:
     p.add_argument("--kv-heads", type=int, default=8)
     p.add_argument("--dim", type=int, default=128)
     p.add_argument("--head-unit", action="store_true", help="no bias and no whole-projection norm; every head normed on its own after the rotation")
+    p.add_argument("--mix", action="store_true", help="biases, a factor on the query by position and another layer's values mixed in; no norms")
     p.set_defaults(fn=qk_norm_rope)
     p = sub.add_parser("capped_unit")
     p.add_argument("--rows", type=int, default=2048)

@@ -142,7 +142,7 @@ def test_a_sink_per_head_in_every_attention_kernel(kernel, Hq, Hkv, D, V, window
         at += ln
 
 
-@pytest.mark.parametrize("H, G, D, V, col0", [(4, 2, 24, 40, 0), (5, 5, 18, 11, 0), (8, 2, 64, 64, 24), (1, 1, 16, 16, 8)])
+@pytest.mark.parametrize("H, G, D, V, col0", [(4, 2, 24, 40, 0), (5, 5, 18, 11, 0), (8, 2, 64, 64, 24), (1, 1, 16, 16, 8), (20, 5, 128, 64, 8)])
 @pytest.mark.parametrize("dtype, in_dtype", [(torch.float32, torch.float32), (torch.bfloat16, torch.bfloat16), (torch.bfloat16, torch.float32)])
 def test_bias_temperature_and_value_mixing(dtype, in_dtype, H, G, D, V, col0):
     """The kernel between projection and attention: biases, the query's factor at positions around its steps, another
@@ -170,6 +170,35 @@ def test_bias_temperature_and_value_mixing(dtype, in_dtype, H, G, D, V, col0):
         torch.testing.assert_close(k_pages[place].cpu().double().reshape(-1), x[H * D:(H + G) * D], **_tol(dtype))
         first = other[i, 16:16 + G * V].double() + first_bias.double()
         torch.testing.assert_close(v_pages[place].cpu().double().reshape(-1), mixed_value(x[(H + G) * D:], first, lam), **_tol(dtype))
+
+
+@pytest.mark.parametrize("H, G, D, rot", [(4, 2, 64, 64), (19, 1, 128, 128), (6, 3, 128, 64), (5, 5, 22, 22), (3, 3, 16, 0)])
+@pytest.mark.parametrize("dtype, in_dtype", [(torch.float32, torch.float32), (torch.bfloat16, torch.bfloat16), (torch.bfloat16, torch.float32)])
+def test_rotation_and_unit_norms_of_heads(dtype, in_dtype, H, G, D, rot):
+    """Heads rotated whole, in part and not at all, then divided by their root mean square, at positions on both sides of
+    page borders; with no pages given only the queries are written."""
+    from nanoinfer_b200.kernels import ops
+    page, n, eps, table = 16, 6, 1e-5, [2, 0, 3, 1]
+    g = torch.Generator().manual_seed(H * 100 + D)
+    cols = (H + 2 * G) * D
+    qkv = (2 * torch.randn(n, cols + (-cols % 8), generator=g)).to(in_dtype)
+    positions, r = [0, 15, 16, 17, 47, 48], {"dims": rot, "base": 300.0} if rot else None
+    freq = torch.tensor([300.0 ** (-2.0 * i / rot) for i in range(rot // 2)]) if rot else torch.zeros(0)
+    pages = [torch.zeros(4, G, page, D, dtype=dtype, device=DEV) for _ in range(2)]
+    outs = []
+    for kv in (pages, (None, None)):
+        q_out = torch.empty(n, H * D, dtype=dtype, device=DEV)
+        ops.qk_norm_rope(qkv.to(DEV), None, None, None, eps, _i32(positions), torch.zeros(n, dtype=torch.int32, device=DEV), _i32([table]),
+                         freq.to(DEV), 1.0, q_out, *kv, H, G, D, D, rot, page, head_unit=True)
+        outs.append(q_out)
+    assert torch.equal(*outs)
+    for t, p in enumerate(positions):
+        x = qkv[t].double()
+        for a in range(H + G):
+            want = unit_rms(rotate(x[a * D:(a + 1) * D], p, r), eps)
+            got = outs[0][t].view(H, D)[a] if a < H else pages[0][table[p // page], a - H, p % page]
+            torch.testing.assert_close(got.cpu().double(), want, **_tol(dtype))
+        torch.testing.assert_close(pages[1][table[p // page], :, p % page].cpu().double().reshape(-1), x[(H + G) * D:cols], **_tol(dtype))
 
 
 @pytest.mark.parametrize("n, w, ld_g, col, ld_o, out_col", [(3, 96, 200, 32, 120, 24), (5, 35, 61, 7, 40, 5), (70, 512, 1024, 512, 512, 0)])
