@@ -19,7 +19,7 @@
 //                         last line's factor); then a thread per column of [W | U0] does the substitution
 //   delta_chunk_scan      per (request, head, 16 value columns): the chunks one after the other; S stands in the
 //                         accumulators of its warps, and as two bfloat16 planes in shared memory for the products that
-//                         read it; the next chunk's operands are copied while this one's are used
+//                         read it; the operands of the next two chunks are on their way while this one's are used
 // The convolution's history is read here and moved on by the gated norm's launch (delta_rule.cu), which follows.
 // A chunk begins at a portion's first token, so where a prompt is cut changes results by roundings only.
 #include "linear_attention.cuh"
@@ -30,6 +30,7 @@
 #define DC_AS 36         // row stride of A in shared memory
 #define DC_BS (DC_C + 8) // row stride of the planes of B
 
+#define DC_STAGES 3      // chunks whose operands the scan has in shared memory or on their way
 #define DC_PAD 8         // numbers behind every row of the planes of W, Q and K (rows then start in different banks)
 
 // One (chunk, head) of the buffer, in bytes - laid out as the scan keeps it in shared memory, so that it is copied as it is: W,
@@ -306,7 +307,7 @@ template <int DP> __host__ __device__ constexpr int dc_stage_bytes() {
     return 6 * DC_C * (DP + DC_PAD) * 2 + 2 * DC_C * DC_BS * 2 + DP * 4 + DC_C * DC_VS * 4;
 }
 #define DC_SS (DC_VS + 8)          // row stride of the planes of S and of u
-template <int DP> __host__ __device__ constexpr int dc_scan_smem() { return 2 * dc_stage_bytes<DP>() + 2 * DP * DC_SS * 2 + 2 * DC_C * DC_SS * 2; }
+template <int DP> __host__ __device__ constexpr int dc_scan_smem() { return DC_STAGES * dc_stage_bytes<DP>() + 2 * DP * DC_SS * 2 + 2 * DC_C * DC_SS * 2; }
 
 // grid (value slices, H, requests); 8 warps: warp w multiplies row tile w % 4 of [W; Q] with column tile w / 4 of S, and owns
 // rows 16 w .. 16 w + 15 of S itself.
@@ -326,7 +327,7 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
     const unsigned char* rec0 = buf + ((size_t)dc_chunk_base(cu_q, seq, &base_scratch) * H + h) * lay.bytes();
     const size_t rec_step = (size_t)H * lay.bytes();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    __nv_bfloat16* s_hi = reinterpret_cast<__nv_bfloat16*>(dc_raw + 2 * dc_stage_bytes<DP>());     // [DP][DC_SS]
+    __nv_bfloat16* s_hi = reinterpret_cast<__nv_bfloat16*>(dc_raw + DC_STAGES * dc_stage_bytes<DP>());     // [DP][DC_SS]
     __nv_bfloat16* s_lo = s_hi + DP * DC_SS;
     __nv_bfloat16* u_hi = s_lo + DP * DC_SS;                                                         // [DC_C][DC_SS]
     __nv_bfloat16* u_lo = u_hi + DC_C * DC_SS;
@@ -334,15 +335,17 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
 
     auto fetch = [&](int c) {                        // the operands of chunk c into their stage, as they lie in the buffer
         const unsigned char* rec = rec0 + (size_t)c * rec_step + 16 * tid;
-        unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>() + 16 * tid;
+        unsigned char* st = dc_raw + (c % DC_STAGES) * dc_stage_bytes<DP>() + 16 * tid;
 #pragma unroll
         for (int i = 0; i < (FIXED + 16 * DC_THREADS - 1) / (16 * DC_THREADS); ++i)
             if ((i + 1) * 16 * DC_THREADS <= FIXED || 16 * tid + i * 16 * DC_THREADS < FIXED)
                 lt_cp_async16(st + i * 16 * DC_THREADS, rec + i * 16 * DC_THREADS);
         if (tid < DC_C * DC_VS / 4) lt_cp_async16(st + FIXED, rec + lay.u_off() + (size_t)blockIdx.x * DC_C * DC_VS * 4);
     };
-    fetch(0);
-    lt_cp_async_commit();
+    for (int c = 0; c < DC_STAGES - 1; ++c) {
+        if (c < n_chunks) fetch(c);
+        lt_cp_async_commit();                        // one group per chunk, empty or not
+    }
     // this warp's 16 rows of S; two column tiles of 8
     const bool owns = warp < DP / 16;
     float s[2][4];
@@ -370,11 +373,11 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
     const int mi = lane >> 3, lr = lane & 7;
     const int rt = warp & 3, ct = warp >> 2;         // row tile of [W; Q] (0, 1: W), column tile
     for (int c = 0; c < n_chunks; ++c) {
-        lt_cp_async_wait<0>();
-        __syncthreads();                             // chunk c's operands and the planes of S are there; the other stage is free
-        if (c + 1 < n_chunks) fetch(c + 1);
+        lt_cp_async_wait<DC_STAGES - 2>();
+        __syncthreads();                             // chunk c's operands and the planes of S are there; the stage of c - 1 is free
+        if (c + DC_STAGES - 1 < n_chunks) fetch(c + DC_STAGES - 1);
         lt_cp_async_commit();
-        const unsigned char* st = dc_raw + (c & 1) * dc_stage_bytes<DP>();
+        const unsigned char* st = dc_raw + (c % DC_STAGES) * dc_stage_bytes<DP>();
         const __nv_bfloat16* planes = reinterpret_cast<const __nv_bfloat16*>(st);
         const __nv_bfloat16* b_hi = planes + 6 * DC_C * RS;
         const float* sp = reinterpret_cast<const float*>(b_hi + 2 * DC_C * DC_BS);

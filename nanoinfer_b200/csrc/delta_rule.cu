@@ -327,7 +327,7 @@ __global__ void delta_gated_norm_kernel(const float* __restrict__ o, const float
                                         DeltaDims dm, int n_tokens, T* __restrict__ y, int ld_y, int norm_blocks,
                                         int hist_blocks_per_seq, const TP* __restrict__ proj, float* __restrict__ state,
                                         long long state_stride, const int* __restrict__ cu_q,
-                                        const int* __restrict__ slots) {
+                                        const int* __restrict__ slots, int wide) {
     if ((int)blockIdx.x >= norm_blocks) {
         const int hb = blockIdx.x - norm_blocks;
         delta_history(proj, state, state_stride, cu_q, slots, dm, hb / hist_blocks_per_seq,
@@ -342,6 +342,18 @@ __global__ void delta_gated_norm_kernel(const float* __restrict__ o, const float
     const float* grow = gate + (size_t)t * ld_gate + h * dm.V;
     T* yrow = y + (size_t)t * ld_y + (size_t)h * dm.V;
     float ss = 0.f;
+    if (wide) {                            // V = 128, all rows on 16 bytes: four neighbours per lane, both rows asked for at once
+        const float4 v = *reinterpret_cast<const float4*>(orow + 4 * lane), g = *reinterpret_cast<const float4*>(grow + 4 * lane);
+        const float4 w = *reinterpret_cast<const float4*>(weight + 4 * lane);
+        ss = ni_warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
+        const float f = scale / sqrtf(ss / (float)dm.V + eps);
+        const auto act = [&](float z) { return sigmoid_gate ? dr_sigmoid(z) : dr_silu(z); };
+        __align__(16) T out[4] = {ni_from_float<T>(v.x * f * w.x * act(g.x)), ni_from_float<T>(v.y * f * w.y * act(g.y)),
+                    ni_from_float<T>(v.z * f * w.z * act(g.z)), ni_from_float<T>(v.w * f * w.w * act(g.w))};
+        if (sizeof(T) == 4) *reinterpret_cast<float4*>(yrow + 4 * lane) = *reinterpret_cast<float4*>(out);
+        else *reinterpret_cast<uint2*>(yrow + 4 * lane) = *reinterpret_cast<uint2*>(out);
+        return;
+    }
     for (int i = lane; i < dm.V; i += 32) ss += orow[i] * orow[i];
     ss = ni_warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)dm.V + eps);
@@ -450,10 +462,13 @@ NI_EXPORT int ni_delta_gated_norm(const float* o, const float* gate, int ld_gate
     const int per_seq = taps > 1 ? (dm.C() + warps * 32 - 1) / (warps * 32) : 0;
     const long long blocks = norm_blocks + (long long)per_seq * n_seqs;
     if (blocks > 2147483647LL) return NI_ERR_UNSUPPORTED_SIZE;
+    const auto aligned = [](const void* q) { return (reinterpret_cast<size_t>(q) & 15) == 0; };
+    const int wide = V == 128 && y_dtype == NI_DTYPE_BF16 && ld_gate % 4 == 0 && ld_y % 8 == 0 && aligned(o) && aligned(gate) &&
+                     aligned(weight) && aligned(y);
 #define GO(T, TP)                                                                                                        \
     delta_gated_norm_kernel<T, TP><<<(int)blocks, warps * 32, 0, stream>>>(                                              \
         o, gate, ld_gate, sigmoid_gate, weight, eps, scale, dm, n_tokens, (T*)y, ld_y, (int)norm_blocks, per_seq,        \
-        (const TP*)proj, state, state_stride, cu_q, slots)
+        (const TP*)proj, state, state_stride, cu_q, slots, wide)
     if (y_dtype == NI_DTYPE_F32 && proj_dtype == NI_DTYPE_F32) GO(float, float);
     else if (y_dtype == NI_DTYPE_BF16 && proj_dtype == NI_DTYPE_F32) GO(__nv_bfloat16, float);
     else if (y_dtype == NI_DTYPE_BF16 && proj_dtype == NI_DTYPE_BF16) GO(__nv_bfloat16, __nv_bfloat16);

@@ -9,7 +9,7 @@
 //            a = float(position) * inv_freq[i]  (m = `magnitude`: an encoding that also scales what it rotates)
 //   (optional, `head_unit`) every head of q and of k divided by its own root mean square over D, eps inside the
 //            root, no weight - after the rotation
-//   (optional, temp_coef) q <- q * (1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)): a factor on the finished
+//   (optional, temp_coef) q <- q * (1 + temp_coef * ln(1 + floor((position + 1) / temp_every))): a factor on the finished
 //            query that grows with the position
 //   (optional, first_v) v <- (1 - lambda) v + lambda (first + first_bias): another layer's values of the same token, as
 //            that layer's projection holds them, mixed in

@@ -810,7 +810,7 @@ def qk_norm_rope(qkv, bias, q_gain, k_gain, eps, positions, seq_of_token, block_
     head of q and k is then divided by its own root mean square (``eps`` inside the root, no weight); queries -> q_out [T, H hd],
     keys -> k_pages [P, Hkv, page_size, hd], values -> v_pages [P, Hkv, page_size, value_dim] (None: nothing written).
     The columns start at ``col0`` of qkv, which may be float32 where q_out and the pages are bfloat16.  ``temperature``
-    (coef, every): the finished query times 1 + coef ln(floor((position + 1) / every) + 1).  ``first_values`` (rows, column,
+    (coef, every): the finished query times 1 + coef ln(1 + floor((position + 1) / every)).  ``first_values`` (rows, column,
     bias, lambda): v <- (1 - lambda) v + lambda (rows[t, column : column + Hkv value_dim] + bias), rows [T, *] of qkv's
     dtype, bias float32 [Hkv value_dim] or None."""
     n = qkv.shape[0]

@@ -499,7 +499,7 @@ class NormedQKAttention(PagedAttendMixin, Part):
     value), "learned": exp(sink_h) with a number per head ("sink"), not scaled; ``head_gate`` - head h's output is
     multiplied by sigmoid(W_g x)_h, one more row per head in the fused projection ("g"); ``element_gate`` - every
     coordinate of the output by its own sigmoid(W_g x)_i ("g" has a row per coordinate); ``temperature`` = (coef, every) -
-    the finished query at position p times 1 + coef ln(floor((p + 1) / every) + 1); ``value_mix`` - "first": this layer's
+    the finished query at position p times 1 + coef ln(1 + floor((p + 1) / every)); ``value_mix`` - "first": this layer's
     values v_0 go along to later layers of the step, "later": v <- (1 - lambda) v + lambda v_0 with the learned number
     "vmix", and the mixed values are cached; ``output_bias`` - the output projection has one ("o.b").
 

@@ -623,6 +623,26 @@ def test_replay_matches_plain(models, key, dtype, cut):
     assert runner.cache.num_free_slots == 4
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_sides_that_are_not_joined(models, dtype):
+    """The same model with side-by-side layers whose sides keep projections of their own (the weighted sum is formed in the
+    second side's last product) and with layer scales that the block carries out itself."""
+    from dataclasses import replace
+
+    from nanoinfer_b200.config import load_config
+    from nanoinfer_b200.engine import ModelRunner
+    from nanoinfer_b200.weights import load_weights
+    d, raw, reqs, want = models["l1"]
+    cfg = load_config(d)
+    layers = tuple(replace(la, mixer=replace(la.mixer, extra=tuple((k, False if k == "join" else v) for k, v in la.mixer.extra)))
+                   for la in cfg.layers)
+    cfg = replace(cfg, layers=layers)
+    steps = ru.mixed({k: reqs[k] for k in ("q2", "q4", "q5", "q6")})
+    runner = ModelRunner(cfg, load_weights(d, cfg), dtype=dtype, page_size=16, num_pages=ru.max_live_tokens(steps, 64) // 16, max_requests=4)
+    assert not runner.model.blocks[0].mixer.joined and runner.model.blocks[0].scales[0] is not None
+    _compare(ru.run_trace(runner, steps), want, dtype, "sides of their own")
+
+
 @pytest.mark.parametrize("key", list(RAW))
 def test_float32_barely_depends_on_the_cut(models, key):
     """In 32-bit, cuts may differ by roundings of the matrix products and no more."""
