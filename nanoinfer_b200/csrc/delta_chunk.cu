@@ -19,7 +19,8 @@
 //                         last line's factor); then a thread per column of [W | U0] does the substitution
 //   delta_chunk_scan      per (request, head, 16 value columns): the chunks one after the other; S stands in the
 //                         accumulators of its warps, and as two bfloat16 planes in shared memory for the products that
-//                         read it; the operands of the next two chunks are on their way while this one's are used
+//                         read it; the operands of the next two chunks are on their way (bulk copies) while this one's
+//                         are used
 // The convolution's history is read here and moved on by the gated norm's launch (delta_rule.cu), which follows.
 // A chunk begins at a portion's first token, so where a prompt is cut changes results by roundings only.
 #include "linear_attention.cuh"
@@ -303,6 +304,40 @@ __device__ __forceinline__ void dc_ldsm_x4(uint32_t (&r)[4], const void* p) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
+// Bulk copies of whole records into shared memory, counted in by an mbarrier per stage.  A wait lasts at most dc_wait_limit
+// clock ticks (about a second); then the error word is set and the kernel returns.  dc_extra_wait: wait once more at the end,
+// for a phase that nothing completes (for the test of the give-up path).  Both set by ni_delta_chunk_set_wait.
+#define DC_ERR_WAIT 41
+__constant__ long long dc_wait_limit = 2000000000LL;
+__constant__ int dc_extra_wait = 0;
+
+__device__ __forceinline__ uint32_t dc_smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ bool dc_wait(uint64_t* bar, uint32_t parity, int* error) {
+    const uint32_t addr = dc_smem_addr(bar);
+    long long start = 0;
+    for (int iter = 0;; ++iter) {
+        uint32_t done;
+        asm volatile(
+            "{\n.reg .pred p;\n"
+            "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+            "selp.b32 %0, 1, 0, p;\n}\n"
+            : "=r"(done) : "r"(addr), "r"(parity) : "memory");
+        if (done) return true;
+        if ((iter & 1023) == 1023) {
+            const long long now = clock64();
+            if (start == 0) start = now;
+            if (now - start > dc_wait_limit) {
+                atomicExch(error, DC_ERR_WAIT);
+                return false;
+            }
+        }
+    }
+}
+__device__ __forceinline__ void dc_bulk_copy(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+                 ::"r"(dc_smem_addr(dst)), "l"(src), "r"(bytes), "r"(dc_smem_addr(bar)) : "memory");
+}
+
 template <int DP> __host__ __device__ constexpr int dc_stage_bytes() {
     return 6 * DC_C * (DP + DC_PAD) * 2 + 2 * DC_C * DC_BS * 2 + DP * 4 + DC_C * DC_VS * 4;
 }
@@ -315,7 +350,7 @@ template <int DP>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, float* __restrict__ state, long long state_stride,
                         const int* __restrict__ cu_q, const int* __restrict__ slots, int H, int D, int V,
-                        float* __restrict__ out) {
+                        float* __restrict__ out, int* __restrict__ error) {
     constexpr int RS = DP + DC_PAD;                  // row stride of the operand planes
     constexpr int FIXED = dc_stage_bytes<DP>() - DC_C * DC_VS * 4;      // of a stage: everything but the slice of U0
     extern __shared__ __align__(16) unsigned char dc_raw[];
@@ -333,19 +368,25 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
     __nv_bfloat16* u_lo = u_hi + DC_C * DC_SS;
     float* S = state + (size_t)slots[seq] * state_stride + (size_t)h * D * V;
 
-    auto fetch = [&](int c) {                        // the operands of chunk c into their stage, as they lie in the buffer
-        const unsigned char* rec = rec0 + (size_t)c * rec_step + 16 * tid;
-        unsigned char* st = dc_raw + (c % DC_STAGES) * dc_stage_bytes<DP>() + 16 * tid;
-#pragma unroll
-        for (int i = 0; i < (FIXED + 16 * DC_THREADS - 1) / (16 * DC_THREADS); ++i)
-            if ((i + 1) * 16 * DC_THREADS <= FIXED || 16 * tid + i * 16 * DC_THREADS < FIXED)
-                lt_cp_async16(st + i * 16 * DC_THREADS, rec + i * 16 * DC_THREADS);
-        if (tid < DC_C * DC_VS / 4) lt_cp_async16(st + FIXED, rec + lay.u_off() + (size_t)blockIdx.x * DC_C * DC_VS * 4);
-    };
-    for (int c = 0; c < DC_STAGES - 1; ++c) {
-        if (c < n_chunks) fetch(c);
-        lt_cp_async_commit();                        // one group per chunk, empty or not
+    __shared__ __align__(8) uint64_t full[DC_STAGES];
+    if (tid == 0) {
+        for (int i = 0; i < DC_STAGES; ++i)
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;\n" ::"r"(dc_smem_addr(&full[i])) : "memory");
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
     }
+    __syncthreads();
+    auto fetch = [&](int c) {                        // one thread: the operands of chunk c into their stage, as they lie in the buffer
+        const unsigned char* rec = rec0 + (size_t)c * rec_step;
+        unsigned char* st = dc_raw + (c % DC_STAGES) * dc_stage_bytes<DP>();
+        uint64_t* bar = &full[c % DC_STAGES];
+        constexpr int SLICE = DC_C * DC_VS * 4;
+        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(dc_smem_addr(bar)), "r"(FIXED + SLICE) : "memory");
+        dc_bulk_copy(st, rec, FIXED, bar);
+        dc_bulk_copy(st + FIXED, rec + lay.u_off() + (size_t)blockIdx.x * SLICE, SLICE, bar);
+    };
+    if (tid == 0)
+        for (int c = 0; c < DC_STAGES - 1 && c < n_chunks; ++c) fetch(c);
     // this warp's 16 rows of S; two column tiles of 8
     const bool owns = warp < DP / 16;
     float s[2][4];
@@ -373,10 +414,14 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
     const int mi = lane >> 3, lr = lane & 7;
     const int rt = warp & 3, ct = warp >> 2;         // row tile of [W; Q] (0, 1: W), column tile
     for (int c = 0; c < n_chunks; ++c) {
-        lt_cp_async_wait<DC_STAGES - 2>();
-        __syncthreads();                             // chunk c's operands and the planes of S are there; the stage of c - 1 is free
-        if (c + DC_STAGES - 1 < n_chunks) fetch(c + DC_STAGES - 1);
-        lt_cp_async_commit();
+        const bool arrived = dc_wait(&full[c % DC_STAGES], (uint32_t)(c / DC_STAGES) & 1u, error);
+        if (!__syncthreads_and(arrived)) {           // given up: the copies that are still under way end before the block does
+            if (tid == 0)
+                for (int k = c; k < min(c + DC_STAGES - 1, n_chunks); ++k) dc_wait(&full[k % DC_STAGES], (uint32_t)(k / DC_STAGES) & 1u, error);
+            return;
+        }
+        // chunk c's operands and the planes of S are there; the stage of c - 1 is free
+        if (tid == 0 && c + DC_STAGES - 1 < n_chunks) fetch(c + DC_STAGES - 1);
         const unsigned char* st = dc_raw + (c % DC_STAGES) * dc_stage_bytes<DP>();
         const __nv_bfloat16* planes = reinterpret_cast<const __nv_bfloat16*>(st);
         const __nv_bfloat16* b_hi = planes + 6 * DC_C * RS;
@@ -487,6 +532,14 @@ delta_chunk_scan_kernel(const unsigned char* __restrict__ buf, DcLayout lay, flo
             const int row = 16 * warp + g + 8 * (e >> 1), col = v0 + 8 * j + 2 * t + (e & 1);
             if (row < D && col < V) S[(size_t)row * V + col] = s[j][e];
         }
+    if (dc_extra_wait) dc_wait(&full[0], (uint32_t)((n_chunks + DC_STAGES - 1) / DC_STAGES) & 1u, error);
+}
+
+NI_EXPORT int ni_delta_chunk_set_wait(long long ticks, int extra_wait) {
+    if (ticks <= 0) ticks = 2000000000LL;
+    cudaError_t e = cudaMemcpyToSymbol(dc_wait_limit, &ticks, sizeof(ticks));
+    if (e == cudaSuccess) e = cudaMemcpyToSymbol(dc_extra_wait, &extra_wait, sizeof(extra_wait));
+    return e == cudaSuccess ? NI_OK : (int)e;
 }
 
 // Bytes of the buffer that ni_delta_chunk_recurrence needs.
@@ -498,7 +551,8 @@ NI_EXPORT long long ni_delta_chunk_buffer_bytes(int n_tokens, int n_seqs, int H,
 NI_EXPORT int ni_delta_chunk_max_dim() { return 128; }
 
 template <int DP, int TAPS>
-static int dc_launch(const DcInput& in, float* state, int n_seqs, int max_q_len, void* buf, float* out, cudaStream_t stream) {
+static int dc_launch(const DcInput& in, float* state, int n_seqs, int max_q_len, void* buf, float* out, int* error,
+                     cudaStream_t stream) {
     const DcLayout lay{DP, (in.V + DC_VS - 1) / DC_VS * DC_VS};
     const size_t smem_p = (size_t)(3 * DC_C * DP + 2 * DC_C * DC_AS + DC_C * lay.VP) * sizeof(float), smem_s = dc_scan_smem<DP>();
     static size_t configured = 0;
@@ -514,20 +568,22 @@ static int dc_launch(const DcInput& in, float* state, int n_seqs, int max_q_len,
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     delta_chunk_scan_kernel<DP><<<grid_s, DC_THREADS, smem_s, stream>>>((const unsigned char*)buf, lay, state, in.state_stride,
-                                                                        in.cu_q, in.slots, in.H, in.D, in.V, out);
+                                                                        in.cu_q, in.slots, in.H, in.D, in.V, out, error);
     NI_RETURN_LAUNCH_STATUS();
 }
 
 // The rule over a step's prompt portions, from the projection (see DcInput) to the read-outs, out FP32 [T, H V]: the state
 // [H, D, V] at the start of a request's row moves on; the convolution history behind it is read (ni_delta_gated_norm, which
-// must follow, writes the new one).  max_q_len: the most tokens a request brings.  buf: 16-byte aligned,
+// must follow, writes the new one).  error: a device int, zero on entry; non-zero afterwards if a wait inside the kernel ran
+// out.  max_q_len: the most tokens a request brings.  buf: 16-byte aligned,
 // ni_delta_chunk_buffer_bytes long.
 NI_EXPORT int ni_delta_chunk_recurrence(const void* proj, int ld, int b_off, const float* conv_w, const float* a_log,
                                         const float* dt_bias, const float* z, int ld_z, float* state, long long state_stride,
                                         const int* cu_q, const int* slots, int n_tokens, int n_seqs, int max_q_len, int G, int H,
-                                        int D, int V, int taps, void* buf, long long buf_bytes, float* out, cudaStream_t stream) {
+                                        int D, int V, int taps, void* buf, long long buf_bytes, float* out, int* error,
+                                        cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return NI_OK;
-    if (G <= 0 || H <= 0 || D <= 0 || V <= 0 || taps <= 0 || H % G || ld_z < H * D || max_q_len <= 0 || buf == nullptr ||
+    if (G <= 0 || H <= 0 || D <= 0 || V <= 0 || taps <= 0 || H % G || ld_z < H * D || max_q_len <= 0 || buf == nullptr || error == nullptr ||
         (reinterpret_cast<size_t>(buf) & 15) || buf_bytes < ni_delta_chunk_buffer_bytes(n_tokens, n_seqs, H, D, V) || b_off < 0 ||
         ld < b_off + H || ld < 2 * G * D + H * V || state_stride < (long long)H * D * V + (long long)(taps - 1) * (2 * G * D + H * V))
         return NI_ERR_BAD_ARGUMENT;
@@ -536,8 +592,8 @@ NI_EXPORT int ni_delta_chunk_recurrence(const void* proj, int ld, int b_off, con
                         ld, b_off, ld_z, G, H, D, V, taps};
     const bool four = taps == 4 && (reinterpret_cast<size_t>(conv_w) & 15) == 0;
 #define GO(DP)                                                                                    \
-    return four ? dc_launch<DP, 4>(in, state, n_seqs, max_q_len, buf, out, stream)                \
-                : dc_launch<DP, 0>(in, state, n_seqs, max_q_len, buf, out, stream)
+    return four ? dc_launch<DP, 4>(in, state, n_seqs, max_q_len, buf, out, error, stream)         \
+                : dc_launch<DP, 0>(in, state, n_seqs, max_q_len, buf, out, error, stream)
     if (D <= 32) GO(32);
     if (D <= 64) GO(64);
     GO(128);

@@ -99,7 +99,8 @@ _SIGNATURES = {
         "ni_delta_gated_norm": [_P, _P, _I, _I, _P, _F, _F, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _LL, _P, _P, _P],
     },
     "delta_chunk": {
-        "ni_delta_chunk_recurrence": [_P, _I, _I, _P, _P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _P],
+        "ni_delta_chunk_recurrence": [_P, _I, _I, _P, _P, _P, _P, _I, _P, _LL, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _LL, _P, _P, _P],
+        "ni_delta_chunk_set_wait": [_LL, _I],
         "ni_delta_chunk_max_dim": [],
     },
     "latent": {
@@ -633,8 +634,8 @@ def delta_chunk_recurrence(proj, col0, b_col, conv_w, a_log, dt_bias, z, state, 
         _dev(proj, "proj", torch.bfloat16) + 2 * col0, proj.shape[1], b_col - col0, _dev(conv_w, "conv_w", f32),
         _dev(a_log, "a_log", f32), _dev(dt_bias, "dt_bias", f32), _dev(z, "z", f32), z.shape[1], _dev(state, "state", f32),
         state.shape[1], _dev(cu_q, "cu_q", torch.int32), _dev(slots, "slots", torch.int32), n, n_seqs, int(max_q_len), n_q_heads_kv,
-        n_heads, dim, vdim, taps, _dev(buf, "buf"), buf.numel() * buf.element_size(), _dev(out, "out", f32), _stream()),
-        "delta_chunk_recurrence")
+        n_heads, dim, vdim, taps, _dev(buf, "buf"), buf.numel() * buf.element_size(), _dev(out, "out", f32),
+        _error_word(proj.device).data_ptr(), _stream()), "delta_chunk_recurrence")
 
 
 DELTA_TOKEN_MAX_DIM = 128      # the largest key and value sizes whose state a block of the token kernel holds in registers
@@ -1532,6 +1533,7 @@ DEVICE_ERROR_CODES = {
     31: "fused decode step (decode_fused): a grid barrier was not reached by every block in time",
     32: "fused decode step (decode_fused): the weight loader gave up waiting for a free stage",
     33: "fused decode step (decode_fused): a consumer gave up waiting for its weights",
+    41: "delta rule in chunks (delta_chunk): the scan gave up waiting for a chunk's operands",
 }
 
 
@@ -1569,7 +1571,7 @@ def check_device_errors(device=None) -> None:
 
 _WAIT_SETTERS = {"gemm_tc": "ni_gemm_tc_set_wait", "gemm_tc2": "ni_gemm_tc2_set_wait",
                  "gemm_swap_tc": "ni_gemm_swap_tc_set_wait",
-                 "attention_prefill_tc": "ni_attention_prefill_tc_set_wait"}
+                 "attention_prefill_tc": "ni_attention_prefill_tc_set_wait", "delta_chunk": "ni_delta_chunk_set_wait"}
 
 
 def set_wait_limit(module: str, ticks: int = 0, extra_wait: bool = False) -> None:

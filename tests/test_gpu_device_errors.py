@@ -2,7 +2,7 @@
 the record, and the next launch is an ordinary one.
 
 The waits of the tcgen05 kernels (on mbarriers, between the loader, the MMA issuer and the
-epilogue or softmax warps) are bounded in clock ticks.  For these tests the limit is set to about
+epilogue or softmax warps) and of the chunked delta rule (for its bulk copies) are bounded in clock ticks.  For these tests the limit is set to about
 a millisecond and the kernels are told to wait once more at their end, for a phase that nothing
 completes: the wait runs out by itself.  Nothing traps, faults or spins without a bound.
 """
@@ -59,13 +59,37 @@ def _attention(ops):
     return out, want
 
 
-CODES = {"gemm_tc": 3, "gemm_tc2": 3, "gemm_swap_tc": 23, "attention_prefill_tc": 13}
+def _delta_chunks(ops):
+    """One request of 70 tokens through the chunked delta rule; returns (read-outs, those of the kernels that go token by
+    token)."""
+    H, D, V, n = 2, 32, 16, 70
+    C = 2 * H * D + H * V
+    proj, z = _randn(n, C + 8, seed=6), _randn(n, H * D, seed=7).float()
+    conv_w, a_log, dt_bias = (torch.ones(*shape, device=DEV) * x for shape, x in (((C, 2), 0.5), ((H,), 0.0), ((H * D,), -2.0)))
+    i32 = dict(dtype=torch.int32, device=DEV)
+    cu, slots = torch.tensor([0, n], **i32), torch.zeros(1, **i32)
+    outs = []
+    for chunks in (True, False):
+        state, out = torch.zeros(1, H * D * V + C, device=DEV), torch.zeros(n, H * V, device=DEV)
+        if chunks:
+            buf = torch.empty(ops.delta_chunk_buffer_bytes(n, 1, H, D, V) // 4, device=DEV)
+            ops.delta_chunk_recurrence(proj, 0, C, conv_w, a_log, dt_bias, z, state, cu, slots, 1, n, H, H, D, V, 2, buf, out)
+        else:
+            qkv, gates, zz = torch.empty(n, C, device=DEV), torch.empty(n, H, 2, device=DEV), z.clone()
+            ops.delta_prepare(proj, conv_w, a_log, dt_bias, state, torch.zeros(n, **i32), cu, slots, 1, H, H, D, V, 2, qkv, gates, b_col=C, z=zz)
+            ops.delta_recurrence(qkv, gates, state, cu, slots, 1, H, H, D, V, out, z=zz)
+        outs.append(out)
+    return outs[0], outs[1].cpu()
+
+
+CODES = {"delta_chunk": 41, "gemm_tc": 3, "gemm_tc2": 3, "gemm_swap_tc": 23, "attention_prefill_tc": 13}
 
 
 @pytest.mark.parametrize("module", sorted(CODES))
 def test_a_wait_that_runs_out_is_recorded_and_the_kernel_returns(module):
     from nanoinfer_b200.kernels import ops
-    run = (lambda: _attention(ops)) if module == "attention_prefill_tc" else (lambda: _product(ops, module))
+    run = {"attention_prefill_tc": lambda: _attention(ops), "delta_chunk": lambda: _delta_chunks(ops)}.get(
+        module, lambda: _product(ops, module))
     run()                                     # loads the library; an ordinary launch leaves no record
     torch.cuda.synchronize()
     ops.check_device_errors()
