@@ -8,7 +8,7 @@ The norms are RMS norms whose weight is stored around zero (the gain is 1 + w). 
                       then every head of q and k divided by its own root mean square; causal; a softmax with one added
                       to its denominator; keys and values may differ in size;
   "latent_attention"  attention over one compressed vector per token plus one rotated key part that all heads share
-                      (adjacent pairs rotated); a token sees itself and the ``mask.size`` - 1 tokens before it;
+                      (adjacent pairs rotated); a window of ``mask.size`` tokens, the newest included;
   "parallel"          two mixers that read the same input, their outputs added with a scale each: on the left
                       grouped-query attention with an RMS norm over the WHOLE query and key projections, linearly
                       scaled rotary frequencies, a mask of chunks of ``mask.size`` positions and a sigmoid gate per

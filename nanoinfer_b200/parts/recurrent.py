@@ -230,7 +230,7 @@ class GatedDeltaRule(Part):
 
 class LightningAttention(Part):
     """Lightning attention: linear attention with a fixed decay per head.  Per head, with a matrix state S
-    [head_dim, value_dim] in FP32 that starts at zero and is carried from token to token for each request:
+    [head_dim, value_dim] in FP32, zero before a request's first token:
 
         q = silu(W_q x), k = silu(W_k x)  (head_dim entries), v = silu(W_v x)  (value_dim entries)
         S <- decay_head * S + k v^T;   o = S^T q                           (no other scale)
